@@ -1,7 +1,8 @@
 """Device arrays behind the cache manager's pages and state slots.
 
 Per cache number (a run item's `cache`): K and V arrays [pages, kv_heads, page_size, head_dim]
-(V with its own width where a mixer asks for one) in the engine's storage dtype (the reference's layout, src/memory/page_atten.zig:2,
+(V with its own width where a mixer asks for one; where it asks for a number per token beside them, one float32
+array [pages, page_size] more) in the engine's storage dtype (the reference's layout, src/memory/page_atten.zig:2,
 src/backend/cuda/attention/attention.cu:12), and/or one state array [slots, *shape].  Cache
 numbers that share a group share its page ids; each keeps its own arrays.
 """
@@ -37,7 +38,7 @@ def bytes_per_page(kv_requests: Dict[int, KVRequest], group_index: Dict[int, int
                    dtype: torch.dtype) -> int:
     """Bytes one page id of `group` occupies over all cache numbers of that group."""
     elem = torch.empty((), dtype=dtype).element_size()
-    return sum(r.num_kv_heads * page_size * (r.head_dim + r.value_dim) * elem
+    return sum(r.num_kv_heads * page_size * (r.head_dim + r.value_dim) * elem + (4 * page_size if r.token_scales else 0)
                for c, r in kv_requests.items() if group_index[c] == group)
 
 
@@ -48,11 +49,14 @@ class CacheStorage:
         self.page_size = page_size
         self.group_index = group_index
         self.kv: Dict[int, Tuple[torch.Tensor, torch.Tensor]] = {}
+        self.scales: Dict[int, torch.Tensor] = {}
         self.state: Dict[int, torch.Tensor] = {}
         for c, r in kv_requests.items():
             shape = (pages_per_group[group_index[c]], r.num_kv_heads, page_size)
             self.kv[c] = (torch.zeros(shape + (r.head_dim,), dtype=dtype, device=device),
                           torch.zeros(shape + (r.value_dim,), dtype=dtype, device=device) if r.values else None)
+            if r.token_scales:
+                self.scales[c] = torch.zeros((shape[0], page_size), dtype=torch.float32, device=device)
         for c, r in state_requests.items():
             self.state[c] = torch.zeros((num_state_slots, *r.shape), dtype=r.dtype, device=device)
 
@@ -61,7 +65,7 @@ class CacheStorage:
             return LayerCache(page_size=self.page_size, writes=writes)
         k, v = self.kv.get(cache_id, (None, None))
         return LayerCache(k=k, v=v, group=self.group_index.get(cache_id, 0), page_size=self.page_size,
-                          writes=writes, state=self.state.get(cache_id))
+                          writes=writes, state=self.state.get(cache_id), k_scale=self.scales.get(cache_id))
 
     def reset_state(self, slots: Sequence[int]) -> None:
         """Zero the state of slots that were just handed to new requests."""
@@ -73,4 +77,4 @@ class CacheStorage:
 
     def bytes_held(self) -> int:
         n = sum(t.numel() * t.element_size() for kv in self.kv.values() for t in kv if t is not None)
-        return n + sum(t.numel() * t.element_size() for t in self.state.values())
+        return n + sum(t.numel() * t.element_size() for table in (self.state, self.scales) for t in table.values())

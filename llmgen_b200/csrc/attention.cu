@@ -28,7 +28,9 @@
 // one number per head, applied as the row is written; before the gate a head's row may be turned back in pairs (m, m + vd / 2) by minus
 // its query's position (values that were cached turned by theirs);
 // a mask in blocks of `chunk` positions counted from the sequence's start: a query sees the keys at or before it that lie
-// in its own block, floor(k / chunk) = floor(q / chunk) (with key parts, the visible keys of a single token are what is split).
+// in its own block, floor(k / chunk) = floor(q / chunk) (with key parts, the visible keys of a single token are what is split);
+// entries that are key and value at once (`k_scale`: a factor on the scores per cached token, [pages, page_size]; there is no value
+// array, and the tile of keys in shared memory serves both products).
 #define LLMK_MODULE_NAME "attention"
 #include "common.cuh"
 
@@ -54,6 +56,7 @@ struct AttnParams {
     const float* sink_values;  // with `sink`: the sink's score per query head [nq]; null: 0 for every head
     const float* turn_cos;     // [positions, vd / 2] (with turn_sin; vd 64 or 128): every head's row is turned back in pairs
     const float* turn_sin;     // (m, m + vd / 2) by minus its query's position before the gate; null: rows leave as they are
+    const float* k_scale;      // non-null: keys are values too; a cached token's factor on its scores
     int gate_heads;            // 1: the gate is one number per head, [tokens, nq]
     long long q_stride, o_stride, gate_stride;
     int max_blocks, nq, nkv, hd, vd, page_size, window, num_parts, part_size, bq, gc, chunks, sink, chunk;
@@ -68,7 +71,9 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
     const int hd = p.hd, vd = p.vd;
     float* Qs = smem;                       // [MAX_ROWS][hd], pre-multiplied by scale
     float* Ks = Qs + MAX_ROWS * hd;         // [KT][hd + 1]
-    float* Vs = Ks + KT * (hd + 1);         // [KT][vd]
+    const bool shared_kv = p.k_scale != nullptr;
+    float* Vs = shared_kv ? Ks : Ks + KT * (hd + 1);         // [KT][vd] (or the keys' own rows)
+    const int vld = shared_kv ? hd + 1 : vd;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int s = p.tile_seq[blockIdx.x];
     if (s < 0) return;                      // padding of a tile list of fixed length
@@ -132,7 +137,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
         for (int j = 0; j < HDL; ++j) acc[i][j] = 0.f;
 
     constexpr int VN = Vec16<T>::N;
-    const int vecs = hd / VN, vvecs = vd / VN;
+    const int vecs = hd / VN, vvecs = shared_kv ? 0 : vd / VN;
     const bool vec_rows = hd % VN == 0 && vd % VN == 0;      // 16-byte reads of the cache's rows; else value by value
     for (int t0 = k_beg; t0 < k_end; t0 += KT) {
         __syncthreads();  // previous tile consumed (and Qs written, first time)
@@ -158,8 +163,9 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
                 for (int i = 0; i < VN; ++i) dst[i] = f[i];
             }
         } else {
-            for (int idx = threadIdx.x; idx < KT * (hd + vd); idx += blockDim.x) {
-                const int key = idx / (hd + vd), d = idx % (hd + vd);
+            const int wide = hd + (shared_kv ? 0 : vd);
+            for (int idx = threadIdx.x; idx < KT * wide; idx += blockDim.x) {
+                const int key = idx / wide, d = idx % wide;
                 const int kpos = t0 + key;
                 float f = 0.f;
                 if (kpos < k_end) {
@@ -173,6 +179,9 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
         }
         __syncthreads();
         if (!valid[0] && !valid[1]) continue;
+        float key_scale = 1.f;
+        if (shared_kv && t0 + lane < k_end)
+            key_scale = p.k_scale[(size_t)bt[(t0 + lane) / p.page_size] * p.page_size + (t0 + lane) % p.page_size];
         // scores of key `lane` for both rows
         float sc[2] = {0.f, 0.f};
         {
@@ -195,6 +204,10 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
                 sc[1] = fmaf(b.x, k0, sc[1]); sc[1] = fmaf(b.y, k1, sc[1]);
                 sc[1] = fmaf(b.z, k2, sc[1]); sc[1] = fmaf(b.w, k3, sc[1]);
             }
+        }
+        if (shared_kv) {
+            sc[0] *= key_scale;
+            sc[1] *= key_scale;
         }
         if (p.softcap > 0.f) {
             sc[0] = p.softcap * tanhf(sc[0] / p.softcap);
@@ -225,7 +238,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
         for (int k = 0; k < kmax; ++k) {
             const float p0 = __shfl_sync(0xffffffffu, pr[0], k);
             const float p1 = __shfl_sync(0xffffffffu, pr[1], k);
-            const float* vr = Vs + k * vd;
+            const float* vr = Vs + k * vld;
 #pragma unroll
             for (int j = 0; j < HDL; ++j) {
                 const int d = lane + 32 * j;
@@ -392,12 +405,14 @@ LLMK_EXPORT int llmk_paged_attention(void* out, long long o_stride, const void* 
                                      int page_size, int window, float scale, int num_parts, int part_size,
                                      void* scratch, int vd, float softcap, int sink, const float* sink_values, const void* gate,
                                      long long gate_stride, int chunk, int gate_heads, const float* turn_cos, const float* turn_sin,
-                                     const int* positions, int dtype, void* stream) {
+                                     const int* positions, const float* k_scale, int dtype, void* stream) {
     if (n_tiles <= 0 || n_tokens <= 0) return LLMK_OK;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0) LLMK_FAIL("paged_attention: %d query heads are not a multiple of %d kv heads", nq, nkv);
     if (hd <= 0 || hd > 512) LLMK_FAIL("paged_attention: head_dim %d must be positive, at most 512", hd);
     if (vd <= 0) vd = hd;
     if (vd > 512) LLMK_FAIL("paged_attention: value width %d must be at most 512", vd);
+    if (k_scale && vd != hd) LLMK_FAIL("paged_attention: keys that are values have one width (%d, %d)", hd, vd);
+    if (!k_scale && !vcache) LLMK_FAIL("paged_attention: no values");
     if (softcap < 0.f) LLMK_FAIL("paged_attention: softcap %g", (double)softcap);
     if (page_size <= 0) LLMK_FAIL("paged_attention: page_size %d", page_size);
     if (chunk < 0) LLMK_FAIL("paged_attention: blocks of %d positions", chunk);
@@ -409,7 +424,7 @@ LLMK_EXPORT int llmk_paged_attention(void* out, long long o_stride, const void* 
     p.gc = G < MAX_ROWS ? G : MAX_ROWS;
     p.bq = MAX_ROWS / p.gc;
     p.chunks = ceil_div(G, p.gc);
-    p.q = q; p.kcache = kcache; p.vcache = vcache; p.out = out;
+    p.q = q; p.kcache = kcache; p.vcache = vcache; p.out = out; p.k_scale = k_scale;
     p.block_tables = block_tables; p.ctx_len = ctx_len; p.cu_q = cu_q; p.tile_seq = tile_seq; p.tile_q0 = tile_q0;
     p.q_stride = q_stride; p.o_stride = o_stride; p.max_blocks = max_blocks;
     p.nq = nq; p.nkv = nkv; p.hd = hd; p.vd = vd; p.page_size = page_size; p.window = window;
@@ -418,7 +433,7 @@ LLMK_EXPORT int llmk_paged_attention(void* out, long long o_stride, const void* 
     p.num_parts = num_parts; p.part_size = part_size; p.scale = scale;
     p.part_o = (float*)scratch;
     p.part_ml = num_parts > 1 ? (float*)scratch + (size_t)n_tokens * nq * num_parts * vd : nullptr;
-    const size_t smem = ((size_t)MAX_ROWS * hd + (size_t)KT * (hd + 1) + (size_t)KT * vd) * sizeof(float);
+    const size_t smem = ((size_t)MAX_ROWS * hd + (size_t)KT * (hd + 1) + (k_scale ? 0 : (size_t)KT * vd)) * sizeof(float);
     dim3 grid(n_tiles, nkv * p.chunks, num_parts);
     cudaStream_t s = (cudaStream_t)stream;
     int rc;

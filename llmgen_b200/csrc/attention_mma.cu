@@ -12,6 +12,8 @@
 // Block = 64 queries of one sequence x one query head, four warps of 16 rows; keys in tiles of 64 through shared
 // memory: 16-byte `cp.async` copies out of the pages into two buffers, the next tile on its way while this one is used.  Semantics as in csrc/attention.cu (which takes float32, single tokens in
 // parts, and every size this kernel refuses): query j of a portion sits at position ctx - q_len + j.
+// Entries that are key and value at once (SHARED: `k_scale`, a factor on the scores per cached token; no value array): a tile of
+// keys is copied once and serves both products, its tokens' factors beside it.
 // Taken: key width and value width 64 or 128 each.
 #define LLMK_MODULE_NAME "attention_mma"
 #include "common.cuh"
@@ -31,6 +33,7 @@ struct Params {
     const float* sink_values;     // with `sink`: the sink's score per query head [nq]; null: 0
     const float* turn_cos;        // [positions, VD / 2] (with turn_sin): every head's row is turned back in pairs (m, m + VD / 2) by minus
     const float* turn_sin;        // its query's position before the gate; null: rows leave as they are
+    const float* k_scale;         // SHARED: [pages, page_size]
     int gate_heads;               // 1: the gate is one number per head, [tokens, nq]
     const int* block_tables;
     const int* ctx_len;
@@ -59,6 +62,10 @@ __device__ __forceinline__ void cp_async16(void* smem_dst, const void* src) {
     const uint32_t d = (uint32_t)__cvta_generic_to_shared(smem_dst);
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
 }
+__device__ __forceinline__ void cp_async4(void* smem_dst, const void* src) {
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(smem_dst);
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
+}
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 // tanh(x) = 1 - 2 / (1 + e^(2x)): an absolute error of a few 1e-7, which is what a score needs (it is an exponent)
 __device__ __forceinline__ float tanh_abs(float x) { return 1.0f - __fdividef(2.0f, 1.0f + exp2f(x * 2.8853900817779268f)); }
@@ -74,13 +81,15 @@ __device__ __forceinline__ void split3(float x, float& a, float& b, float& c) {
     c = __bfloat162float(__float2bfloat16_rn(r - b));
 }
 
-template <int HD, int VD>
+template <int HD, int VD, bool SHARED>
 __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
+    static_assert(!SHARED || HD == VD, "keys that are values have one width");
     constexpr int QLD = HD + 8, VLD = VD + 8;      // rows 16 bytes longer: the eight rows of an ldmatrix fall on different banks
     extern __shared__ __align__(16) uint8_t smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);      // [BM][QLD]
     bf16* Kbuf = Qs + BM * QLD;                         // 2 x [BN][QLD]
-    bf16* Vbuf = Kbuf + 2 * BN * QLD;                   // 2 x [BN][VLD]
+    bf16* Vbuf = SHARED ? Kbuf : Kbuf + 2 * BN * QLD;   // 2 x [BN][VLD] (SHARED: the keys' own rows)
+    float* Sbuf = reinterpret_cast<float*>(Kbuf + 2 * BN * QLD);      // SHARED: 2 x [BN] factors
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int g = lane >> 2, tq = lane & 3;
     const int s = p.tile_seq[blockIdx.x];
@@ -125,7 +134,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
     const float inv_cap = p.softcap > 0.f ? 1.0f / p.softcap : 0.f;
     constexpr float LOG2E = 1.4426950408889634f;
 
-    constexpr int VECS = HD / 8 + VD / 8;
+    constexpr int VECS = HD / 8 + (SHARED ? 0 : VD / 8);
     auto load_tile = [&](int t0, int buf) {
         bf16* Kd = Kbuf + buf * BN * QLD;
         bf16* Vd = Vbuf + buf * BN * VLD;
@@ -140,6 +149,14 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
                 cp_async16(dst, v < HD / 8 ? p.kcache + row * HD + v * 8 : p.vcache + row * VD + (v - HD / 8) * 8);
             } else {
                 *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+            }
+        }
+        if constexpr (SHARED) {
+            for (int key = threadIdx.x; key < BN; key += WARPS * 32) {
+                const int kpos = t0 + key;
+                const int page = kpos < k_end ? bt[kpos / p.page_size] : -1;
+                if (page >= 0) cp_async4(Sbuf + buf * BN + key, p.k_scale + (size_t)page * p.page_size + kpos % p.page_size);
+                else Sbuf[buf * BN + key] = 0.f;
             }
         }
     };
@@ -176,6 +193,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
                 const int r = e >> 1;
                 const int kpos = t0 + n * 8 + 2 * tq + (e & 1);
                 float v = sc[n][e] * p.scale;
+                if constexpr (SHARED) v *= Sbuf[turn * BN + n * 8 + 2 * tq + (e & 1)];
                 if (p.softcap > 0.f) v = p.softcap * tanh_abs(v * inv_cap);
                 const bool vis = kpos <= qpos[r] && kpos < k_end && (p.window <= 0 || kpos > qpos[r] - p.window) && kpos >= kmin[r];
                 v = vis ? v : -INFINITY;
@@ -284,16 +302,16 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
     }
 }
 
-template <int HD, int VD>
+template <int HD, int VD, bool SHARED = false>
 int launch(const Params& p, dim3 grid, cudaStream_t s) {
-    const size_t smem = ((size_t)(BM + 2 * BN) * (HD + 8) + (size_t)2 * BN * (VD + 8)) * sizeof(bf16);
+    const size_t smem = ((size_t)(BM + 2 * BN) * (HD + 8) + (SHARED ? 0 : (size_t)2 * BN * (VD + 8))) * sizeof(bf16) + (SHARED ? 2 * BN * sizeof(float) : 0);
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_mma_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_mma_kernel<HD, VD, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) LLMK_FAIL("attention_mma: cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
         configured = true;
     }
-    LLMK_CHECK_LAUNCH_RC("attention_mma", llmk_launch(attention_mma_kernel<HD, VD>, grid, dim3(WARPS * 32), smem, s, true, p));
+    LLMK_CHECK_LAUNCH_RC("attention_mma", llmk_launch(attention_mma_kernel<HD, VD, SHARED>, grid, dim3(WARPS * 32), smem, s, true, p));
     return LLMK_OK;
 }
 
@@ -313,7 +331,7 @@ LLMK_EXPORT int llmk_attention_mma(void* out, long long o_stride, const void* q,
                                    const int* tile_seq, const int* tile_q0, int n_tiles, int nq, int nkv, int hd, int vd,
                                    int page_size, int window, float scale, float softcap, int sink, const float* sink_values, const void* gate,
                                    long long gate_stride, int chunk, int gate_heads, const float* turn_cos, const float* turn_sin,
-                                   void* stream) {
+                                   const float* k_scale, void* stream) {
     if (n_tiles <= 0) return LLMK_OK;
     if (llmk_attention_mma_tile_queries(nq, nkv, hd, vd) == 0)
         LLMK_FAIL("attention_mma: not taken (heads %d/%d, key width %d and value width %d must be 64 or 128)", nq, nkv, hd, vd);
@@ -321,15 +339,18 @@ LLMK_EXPORT int llmk_attention_mma(void* out, long long o_stride, const void* q,
         (reinterpret_cast<uintptr_t>(out) & 3) != 0 || page_size <= 0)
         LLMK_FAIL("attention_mma: q and the cache must start on 16-byte boundaries, q's row stride a multiple of 8");
     if (nq > 65535) LLMK_FAIL("attention_mma: grid too large");
+    if (k_scale && hd != vd) LLMK_FAIL("attention_mma: keys that are values have one width (%d, %d)", hd, vd);
+    if (!k_scale && !vcache) LLMK_FAIL("attention_mma: no values");
     Params p;
     p.q = (const bf16*)q; p.kcache = (const bf16*)kcache; p.vcache = (const bf16*)vcache; p.out = (bf16*)out;
     p.gate = (const bf16*)gate; p.sink_values = sink_values; p.gate_heads = gate_heads ? 1 : 0;
     p.turn_cos = (turn_cos && turn_sin) ? turn_cos : nullptr; p.turn_sin = turn_sin; p.block_tables = block_tables; p.ctx_len = ctx_len; p.cu_q = cu_q;
     p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.q_stride = q_stride; p.o_stride = o_stride; p.gate_stride = gate_stride;
     p.max_blocks = max_blocks; p.nq = nq; p.nkv = nkv; p.page_size = page_size; p.window = window; p.sink = sink ? 1 : 0; p.chunk = chunk > 0 ? chunk : 0;
-    p.scale = scale; p.softcap = softcap;
+    p.scale = scale; p.softcap = softcap; p.k_scale = k_scale;
     dim3 grid(n_tiles, nq);
     cudaStream_t s = (cudaStream_t)stream;
+    if (k_scale) return hd == 64 ? launch<64, 64, true>(p, grid, s) : launch<128, 128, true>(p, grid, s);
     if (hd == 64 && vd == 64) return launch<64, 64>(p, grid, s);
     if (hd == 64) return launch<64, 128>(p, grid, s);
     if (vd == 64) return launch<128, 64>(p, grid, s);

@@ -648,6 +648,116 @@ LLMK_EXPORT int llmk_attn_prep_rows(const float* x, long long ld, void* q_out, l
     return LLMK_OK;
 }
 
+// Attention whose values are its projected keys: a token's entry is stored once, as projected, and what the key's norm does to it
+// is one number beside it.  With q = x[0 : nQ] + b and k = x[nQ : nQ + nK] + b of a token's packed row, rq and rk the inverse root
+// mean squares of the two whole rows:
+//   cache[slot, g, :]  = k of key head g                        (storage dtype; keys and values of the attention)
+//   k_scale[slot]      = rk                                     (float32; multiplies the token's scores)
+//   q_out[t, h, :]     = q rq * gains[h, :] * temperature       (gains: q's times those of the key head that h reads, folded at load)
+// temperature = 1 + coef ln(floor((position + 1) / every) + 1), or 1 with coef 0.  The packed row is an array of T or float32
+// slices of a product.  A block per token; the row passes through shared memory, V values a thread at a time.
+template <typename T>
+__device__ __forceinline__ float packed_sum(const void* x, size_t at, int splits, long long split_stride) {
+    if (splits == 0) return to_float(static_cast<const T*>(x)[at]);
+    const float* p = static_cast<const float*>(x) + at;
+    float acc = p[0];
+    for (int s = 1; s < splits; ++s) acc += p[(size_t)s * split_stride];
+    return acc;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) attn_prep_shared_rows_kernel(const void* __restrict__ x, long long ld, int splits, long long split_stride,
+                                                                    const float* __restrict__ bias, T* __restrict__ q_out, long long q_stride,
+                                                                    T* __restrict__ cache, float* __restrict__ k_scale,
+                                                                    const int* __restrict__ positions, const int* __restrict__ slots,
+                                                                    const float* __restrict__ gains, int nq, int nk, int nkv_cache, int hd,
+                                                                    int page_size, float eps, float coef, float every) {
+    extern __shared__ __align__(16) float prow[];     // nQ + nK floats, 33 scratch
+    const int nQ = nq * hd, nK = nk * hd, n = nQ + nK;
+    float* scratch = prow + n;
+    const size_t t = blockIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t base = t * ld;
+    float ssq = 0.f, ssk = 0.f;
+    const bool vec = sizeof(T) == 2 && splits == 0 && (nQ & 7) == 0 && (nK & 7) == 0 && (ld & 7) == 0 && aligned16(x);
+    if (vec) {
+        for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+            Vec16<bf16> raw;
+            raw.raw = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(x) + base + i);
+            float v[8];
+            raw.unpack(v);
+            float ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                if (bias) v[e] += bias[i + e];
+                ss = fmaf(v[e], v[e], ss);
+            }
+            *reinterpret_cast<float4*>(prow + i) = make_float4(v[0], v[1], v[2], v[3]);
+            *reinterpret_cast<float4*>(prow + i + 4) = make_float4(v[4], v[5], v[6], v[7]);
+            if (i < nQ) ssq += ss; else ssk += ss;
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) {
+            const float v = packed_sum<T>(x, base + i, splits, split_stride) + (bias ? bias[i] : 0.f);
+            prow[i] = v;
+            if (i < nQ) ssq = fmaf(v, v, ssq); else ssk = fmaf(v, v, ssk);
+        }
+    }
+    ssq = block_sum(ssq, scratch);
+    ssk = nK > 0 ? block_sum(ssk, scratch) : 0.f;       // block_sum also orders the row in shared memory
+    const int pos = positions[t];
+    float rq = 1.0f / sqrtf(ssq / (float)nQ + eps);
+    if (coef != 0.f) rq *= 1.0f + coef * logf(floorf((float)(pos + 1) / every) + 1.0f);
+    T* qo = q_out + t * q_stride;
+    if (vec && (q_stride & 7) == 0 && aligned16(q_out)) {
+        for (int i = threadIdx.x * 8; i < nQ; i += blockDim.x * 8) {
+            float v[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = prow[i + e] * rq * gains[i + e];
+            Vec16<bf16> raw;
+            raw.pack(v);
+            *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(qo) + i) = raw.raw;
+        }
+    } else {
+        for (int i = threadIdx.x; i < nQ; i += blockDim.x) qo[i] = from_float<T>(prow[i] * rq * gains[i]);
+    }
+    const int slot = slots ? slots[t] : -1;
+    if (slot < 0 || nK == 0) return;
+    const int page = slot / page_size, off = slot % page_size;
+    for (int i = threadIdx.x; i < nK; i += blockDim.x) {
+        const int g = i / hd, d = i % hd;
+        cache[(((size_t)page * nkv_cache + g) * page_size + off) * hd + d] = from_float<T>(prow[nQ + i]);
+    }
+    if (threadIdx.x == 0) k_scale[slot] = 1.0f / sqrtf(ssk / (float)nK + eps);
+}
+
+LLMK_EXPORT int llmk_attn_prep_shared_rows(const void* x, long long ld, int splits, long long split_stride, const float* bias, void* q_out,
+                                           long long q_stride, void* cache, float* k_scale, const int* positions, const int* slots,
+                                           const float* gains, int n_tokens, int nq, int nk, int nkv_cache, int hd, int page_size, float eps,
+                                           float coef, float every, int dtype, void* stream) {
+    if (n_tokens <= 0) return LLMK_OK;
+    if (nq <= 0 || nk < 0 || hd <= 0 || !x || !q_out || !gains || !positions) LLMK_FAIL("attn_prep_shared_rows: bad arguments (nq %d, nk %d, hd %d)", nq, nk, hd);
+    if (nk > 0 && (!cache || !k_scale || page_size <= 0 || nkv_cache < nk)) LLMK_FAIL("attn_prep_shared_rows: bad cache geometry page_size=%d kv heads=%d", page_size, nkv_cache);
+    if (coef != 0.f && !(every > 0.f)) LLMK_FAIL("attn_prep_shared_rows: a temperature every %g positions", (double)every);
+    const size_t smem = ((size_t)(nq + nk) * hd + 33) * sizeof(float);
+    if (smem > 200 * 1024) LLMK_FAIL("attn_prep_shared_rows: a row of %d values does not fit shared memory", (nq + nk) * hd);
+    cudaStream_t s = (cudaStream_t)stream;
+    cudaError_t e;
+    if (dtype == LLMK_F32) {
+        if (smem > 48 * 1024) cudaFuncSetAttribute(attn_prep_shared_rows_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        e = llmk_launch(attn_prep_shared_rows_kernel<float>, dim3(n_tokens), dim3(256), smem, s, true, x, ld, splits, split_stride, bias, (float*)q_out,
+                        q_stride, (float*)cache, k_scale, positions, slots, gains, nq, nk, nkv_cache, hd, page_size, eps, coef, every);
+    } else if (dtype == LLMK_BF16) {
+        if (smem > 48 * 1024) cudaFuncSetAttribute(attn_prep_shared_rows_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        e = llmk_launch(attn_prep_shared_rows_kernel<bf16>, dim3(n_tokens), dim3(256), smem, s, true, x, ld, splits, split_stride, bias, (bf16*)q_out,
+                        q_stride, (bf16*)cache, k_scale, positions, slots, gains, nq, nk, nkv_cache, hd, page_size, eps, coef, every);
+    } else
+        LLMK_FAIL("attn_prep_shared_rows: unknown dtype %d", dtype);
+    LLMK_CHECK_LAUNCH_RC("attn_prep_shared_rows", e);
+    return LLMK_OK;
+}
+
 // The attention's rows on their way to the output projection: each head's vd values turned back in pairs (m, m + vd / 2) by
 // minus the position's angles (vcos / vsin [max_positions, vd / 2]; none: as they are), then multiplied by sigmoid(gate[t, h]),
 // one number per head (gate rows `gate_stride` apart; none: no gate).  In place; a thread per pair.

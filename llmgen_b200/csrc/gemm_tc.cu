@@ -66,7 +66,14 @@ __device__ __forceinline__ float silu(float g) { return __fdividef(g, 1.0f + __e
 // costs what silu costs.  (A selector passed at launch was built first: with it two cases of the replay tests of another
 // architecture failed when the whole suite ran, though not alone; as a template parameter it leaves those kernels as
 // they were.)
-enum { GATE_NONE = 0, GATE_SILU = 1, GATE_GELU_TANH = 2 };
+// ACT_RELU2 (grouped products only) is no gate: the epilogue leaves relu(c)^2, as many columns as W has rows.
+enum { GATE_NONE = 0, GATE_SILU = 1, GATE_GELU_TANH = 2, ACT_RELU2 = 3 };
+constexpr bool is_glu(int act) { return act == GATE_SILU || act == GATE_GELU_TANH; }
+template <int ACT>
+__device__ __forceinline__ float plain_act(float c) {
+    if constexpr (ACT == ACT_RELU2) return fmaxf(c, 0.f) * fmaxf(c, 0.f);
+    else return c;
+}
 template <int ACT>
 __device__ __forceinline__ float gate_act(float g) {
     if constexpr (ACT == GATE_GELU_TANH) return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
@@ -90,13 +97,14 @@ __device__ __forceinline__ float gate_act(float g) {
 // commits arrive on the `empty` and `acc_full` barriers of both blocks; the epilogue warps of both
 // release an accumulator set on rank 0's `acc_empty`.  Each block reads its own 128 rows of the
 // accumulator out of its own tensor memory.
-template <typename TC, int BN, int STAGES, int GATED, int MB, bool PAIR = false, int KS = 1>
+template <typename TC, int BN, int STAGES, int ACT, int MB, bool PAIR = false, int KS = 1>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                const __grid_constant__ CUtensorMap map_c, int store_by_tma, int splits,
                TC* __restrict__ C, int M, int N, int K, long long ldc, int* error_flag,
                const int* __restrict__ tile_group) {
     static_assert(!PAIR || MB == 1, "a pair of blocks takes one block of rows each");
+    constexpr bool GATED = is_glu(ACT);
     using L = Smem<BN, STAGES, MB, PAIR, KS>;
     constexpr int ROWS = (PAIR ? 2 : MB) * BM;                     // rows of a tile
     constexpr int ACC_SETS = 2 * MB * BN <= 512 ? 2 : 1;
@@ -338,7 +346,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                             if constexpr (GATED) {
                                 float o[16];
 #pragma unroll
-                                for (int i = 0; i < 16; ++i) o[i] = gate_act<GATED>(__uint_as_float(r[i])) * __uint_as_float(r[16 + i]);
+                                for (int i = 0; i < 16; ++i) o[i] = gate_act<ACT>(__uint_as_float(r[i])) * __uint_as_float(r[16 + i]);
 #pragma unroll
                                 for (int q = 0; q < 2; ++q) {
                                     Vec16<bf16> v;
@@ -351,7 +359,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 for (int q = 0; q < 4; ++q) {
                                     float f[8];
 #pragma unroll
-                                    for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(r[8 * q + j]);
+                                    for (int j = 0; j < 8; ++j) f[j] = plain_act<ACT>(__uint_as_float(r[8 * q + j]));
                                     Vec16<bf16> v;
                                     v.pack(f);
                                     const int chunk = 4 * h + q;
@@ -427,7 +435,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     const int j0 = (n0 + c0) / 2;
                     float o[16];
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) o[i] = gate_act<GATED>(__uint_as_float(r[i])) * __uint_as_float(r[16 + i]);
+                    for (int i = 0; i < 16; ++i) o[i] = gate_act<ACT>(__uint_as_float(r[i])) * __uint_as_float(r[16 + i]);
                     TC* dst = C + (size_t)row * ldc + j0;
                     if (vec_ok && j0 + 16 <= n_out) {
                         if constexpr (sizeof(TC) == 2) {
@@ -453,7 +461,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                             for (int i = 0; i < 4; ++i) {
                                 float f[8];
 #pragma unroll
-                                for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(r[8 * i + j]);
+                                for (int j = 0; j < 8; ++j) f[j] = plain_act<ACT>(__uint_as_float(r[8 * i + j]));
                                 Vec16<bf16> v;
                                 v.pack(f);
                                 reinterpret_cast<uint4*>(dst)[i] = v.raw;
@@ -467,7 +475,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         }
                     } else {
                         for (int i = 0; i < 32; ++i)
-                            if (n0 + c0 + i < N) dst[i] = from_float<TC>(__uint_as_float(r[i]));
+                            if (n0 + c0 + i < N) dst[i] = from_float<TC>(plain_act<ACT>(__uint_as_float(r[i])));
                     }
                 }
             }
@@ -549,11 +557,13 @@ bool get_slice_map(CUtensorMap* out, const void* base, uint64_t rows, uint64_t c
     return true;
 }
 
-template <typename TC, int BN, int STAGES, int GATED, int MB, bool PAIR = false, int KS = 1>
+template <typename TC, int BN, int STAGES, int ACT, int MB, bool PAIR = false, int KS = 1>
 int launch(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int M, int N, int K, long long ldc,
            int* error_flag, int pdl, cudaStream_t s, int splits = 1, const int* tile_group = nullptr) {
+    static_assert(ACT != ACT_RELU2 || sizeof(TC) == 2, "the squared relu is built for bfloat16 results");
+    constexpr bool GATED = is_glu(ACT);
     using L = Smem<BN, STAGES, MB, PAIR, KS>;
-    auto kernel = gemm_tc_kernel<TC, BN, STAGES, GATED, MB, PAIR, KS>;
+    auto kernel = gemm_tc_kernel<TC, BN, STAGES, ACT, MB, PAIR, KS>;
     static bool configured = false;   // per instantiation
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
@@ -685,8 +695,9 @@ LLMK_EXPORT int llmk_gemm_tc_sliced(float* C, const void* A, const void* W, int 
 // [128 i, 128 i + 128); -1: a tile of padding, skipped), W stacks the groups' matrices ([groups * N, K]) and
 // C[m, :] = A[m, :] * W[group of m's tile]^T.  The list of groups lives on the device, so the launch has the same
 // shape whatever the groups' sizes are (a mixture of experts whose rows were sorted by expert on the device).
+// relu2 != 0 (bfloat16 results): C = relu(.)^2 of that, applied in the epilogue.
 LLMK_EXPORT int llmk_gemm_tc_grouped(void* C, const void* A, const void* W, int M, int N, int K, long long lda, long long ldw,
-                                     long long ldc, int groups, const int* tile_group, int out_dtype, int* error_flag, int pdl,
+                                     long long ldc, int groups, const int* tile_group, int relu2, int out_dtype, int* error_flag, int pdl,
                                      void* stream) {
     if (M <= 0 || N <= 0 || groups <= 0) return LLMK_OK;
     if (!llmk_gemm_tc_usable(A, W, M, N, K, lda, ldw))
@@ -698,6 +709,12 @@ LLMK_EXPORT int llmk_gemm_tc_grouped(void* C, const void* A, const void* W, int 
     if (!get_map(&ma, A, M, K, lda, BM) || !get_map(&mw, W, (uint64_t)groups * N, K, ldw, bn))
         LLMK_FAIL("gemm_tc_grouped: cuTensorMapEncodeTiled failed (M=%d N=%d K=%d groups=%d)", M, N, K, groups);
     cudaStream_t s = (cudaStream_t)stream;
+    if (relu2) {
+        if (out_dtype != LLMK_BF16) LLMK_FAIL("gemm_tc_grouped: the squared relu is built for bfloat16 results");
+        if (bn == 256) return launch<bf16, 256, 4, ACT_RELU2, 1>(ma, mw, C, M, N, K, ldc, error_flag, pdl, s, 1, tile_group);
+        if (bn == 128) return launch<bf16, 128, STAGES_128, ACT_RELU2, 1, false, KS_128>(ma, mw, C, M, N, K, ldc, error_flag, pdl, s, 1, tile_group);
+        return launch<bf16, 64, STAGES_64, ACT_RELU2, 1>(ma, mw, C, M, N, K, ldc, error_flag, pdl, s, 1, tile_group);
+    }
     if (out_dtype == LLMK_BF16) {
         if (bn == 256) return launch<bf16, 256, 4, false, 1>(ma, mw, C, M, N, K, ldc, error_flag, pdl, s, 1, tile_group);
         if (bn == 128) return launch<bf16, 128, STAGES_128, false, 1, false, KS_128>(ma, mw, C, M, N, K, ldc, error_flag, pdl, s, 1, tile_group);

@@ -9,6 +9,9 @@
 // so the attention itself is one shared "kv head" of width rank + rot whose values are the first `rank` entries of
 // the same cached vector.  Four kernels:
 //
+// (A layer may project its queries straight from the stream, without a latent; read entries that another layer cached, making
+// none; and see the last `window` positions only.)
+//
 //   latent_prep      per token: cq = rmsnorm(dq~) * gain (the query's latent, for the product that follows);
 //                    c and the rotated kr written to the token's place in the paged cache
 //   latent_absorb    qa[t, h] = [Wuk_h^T qn | rotate(qr)]                      float32 [tokens, heads, rank + rot]
@@ -35,6 +38,30 @@ __device__ __forceinline__ void rotate_into(float* dst, const float* src, int ro
     dst[b] = v * c + u * s;
 }
 
+// A token's cached vector z = [rmsnorm(c~) * gain | rotate(kr)] from its projected row [c~ | kr], by the whole block.
+// `sm`: 33 + 2 rot floats of shared memory.
+template <typename T>
+__device__ __forceinline__ void latent_entry(T* __restrict__ z, const T* __restrict__ src, int rank, int rot, const float* __restrict__ gain,
+                                             float eps, int pos, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                             int pairing, float* sm) {
+    float* scratch = sm;
+    float* kr_in = sm + 33;
+    float* kr_out = kr_in + rot;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < rank; i += blockDim.x) {
+        const float v = to_float(src[i]);
+        ss += v * v;
+    }
+    for (int i = threadIdx.x; i < rot; i += blockDim.x) kr_in[i] = to_float(src[rank + i]);
+    ss = block_sum(ss, scratch);         // also orders kr_in
+    const float rinv = 1.0f / sqrtf(ss / (float)rank + eps);
+    for (int i = threadIdx.x; i < rank; i += blockDim.x) z[i] = from_float<T>(to_float(src[i]) * rinv * gain[i]);
+    for (int i = threadIdx.x; i < rot / 2; i += blockDim.x)
+        rotate_into(kr_out, kr_in, rot, pairing, cos_t + (size_t)pos * (rot / 2), sin_t + (size_t)pos * (rot / 2), i);
+    __syncthreads();
+    for (int i = threadIdx.x; i < rot; i += blockDim.x) z[rank + i] = from_float<T>(kr_out[i]);
+}
+
 // ---------------------------------------------------------------------------------------------- prep
 // One block per token.  `dq` [q_rank] and `dkv` [rank + rot] are read from the packed projection row.
 template <typename T>
@@ -43,10 +70,8 @@ __global__ void latent_prep_kernel(const T* __restrict__ packed, long long ld, i
                                    T* __restrict__ cq_out, T* __restrict__ cache, const int* __restrict__ positions,
                                    const int* __restrict__ slots, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                                    int pairing) {
-    extern __shared__ float sm[];   // rot floats in, rot floats out, 33 scratch
-    float* kr_in = sm;
-    float* kr_out = sm + rot;
-    float* scratch = sm + 2 * rot;
+    extern __shared__ float sm[];   // 33 scratch, rot floats in, rot floats out
+    float* scratch = sm;
     const size_t t = blockIdx.x;
     pdl_launch_dependents();
     pdl_wait();
@@ -64,21 +89,7 @@ __global__ void latent_prep_kernel(const T* __restrict__ packed, long long ld, i
     }
     const int slot = slots ? slots[t] : -1;
     if (slot < 0 || !cache) return;      // a row that belongs to no sequence, or a pass that stores nothing
-    T* z = cache + (size_t)slot * (rank + rot);
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-        const float v = to_float(row[dkv_off + i]);
-        ss += v * v;
-    }
-    for (int i = threadIdx.x; i < rot; i += blockDim.x) kr_in[i] = to_float(row[dkv_off + rank + i]);
-    ss = block_sum(ss, scratch);         // also orders kr_in
-    const float rinv = 1.0f / sqrtf(ss / (float)rank + eps);
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) z[i] = from_float<T>(to_float(row[dkv_off + i]) * rinv * kv_gain[i]);
-    const int pos = positions[t];
-    for (int i = threadIdx.x; i < rot / 2; i += blockDim.x)
-        rotate_into(kr_out, kr_in, rot, pairing, cos_t + (size_t)pos * (rot / 2), sin_t + (size_t)pos * (rot / 2), i);
-    __syncthreads();
-    for (int i = threadIdx.x; i < rot; i += blockDim.x) z[rank + i] = from_float<T>(kr_out[i]);
+    latent_entry<T>(cache + (size_t)slot * (rank + rot), row + dkv_off, rank, rot, kv_gain, eps, positions[t], cos_t, sin_t, pairing, sm);
 }
 
 LLMK_EXPORT int llmk_latent_prep(const void* packed, long long ld, int dq_off, int dkv_off, int q_rank, int rank, int rot,
@@ -86,6 +97,7 @@ LLMK_EXPORT int llmk_latent_prep(const void* packed, long long ld, int dq_off, i
                                  const int* positions, const int* slots, const float* cos_t, const float* sin_t, int pairing,
                                  int n_tokens, int dtype, void* stream) {
     if (n_tokens <= 0) return LLMK_OK;
+    if (!cache && (!cq_out || q_rank <= 0)) return LLMK_OK;
     if (rank <= 0 || rot < 0 || rot % 2 != 0) LLMK_FAIL("latent_prep: bad sizes (rank %d, rot %d)", rank, rot);
     if (pairing != LLMK_PAIR_INTERLEAVED && pairing != LLMK_PAIR_HALF_SPLIT) LLMK_FAIL("latent_prep: unknown rotary pairing %d", pairing);
     const size_t smem = ((size_t)2 * rot + 33) * sizeof(float);
@@ -105,14 +117,24 @@ LLMK_EXPORT int llmk_latent_prep(const void* packed, long long ld, int dq_off, i
 
 // -------------------------------------------------------------------------------------------- absorb
 // Block (tile of TT tokens, head).  q [tokens, heads * (dim + rot)] of T; wuk [heads * dim, rank] of T (as stored:
-// row h * dim + d is key dimension d of head h); qa float32 [tokens, heads, rank + rot].
+// row h * dim + d is key dimension d of head h); qa float32 [tokens, heads, rank + rot].  With `cache` the launch has blocks of
+// one more "head", which write the tokens' cached vectors (projected rows at `dkv`, `ldq` apart).
 constexpr int LT_TT = 16;
+
+struct LatentEntries {
+    const void* dkv;            // [tokens, rank + rot] of T, rows as far apart as q's
+    const float* gain;
+    void* cache;                // null: no entries are written
+    const int* slots;
+    float eps;
+};
 
 template <typename T>
 __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ wuk,
                                                             float* __restrict__ qa, const int* __restrict__ positions,
                                                             const float* __restrict__ cos_t, const float* __restrict__ sin_t,
-                                                            int n_tokens, int heads, int dim, int rot, int rank, int pairing) {
+                                                            int n_tokens, int heads, int dim, int rot, int rank, int pairing,
+                                                            LatentEntries en) {
     extern __shared__ float sm[];   // [TT][dim] unrotated parts, [TT][rot] rotated parts in, [TT][rot] out
     float* qn = sm;
     float* qr = qn + LT_TT * dim;
@@ -121,6 +143,17 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict_
     const int n = min(LT_TT, n_tokens - t0);
     pdl_launch_dependents();
     pdl_wait();
+    if (h == heads) {
+        for (int i = blockIdx.z; i < n; i += gridDim.z) {
+            const size_t t = (size_t)(t0 + i);
+            const int slot = en.slots[t];
+            if (slot < 0) continue;         // uniform over the block
+            __syncthreads();                // the token before is done with the shared memory
+            latent_entry<T>(static_cast<T*>(en.cache) + (size_t)slot * (rank + rot), static_cast<const T*>(en.dkv) + t * ldq, rank, rot, en.gain,
+                            en.eps, positions[t], cos_t, sin_t, pairing, sm);
+        }
+        return;
+    }
     const int hd = dim + rot;
     for (int idx = threadIdx.x; idx < LT_TT * hd; idx += blockDim.x) {
         const int i = idx / hd, d = idx % hd;
@@ -172,25 +205,84 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict_
 
 LLMK_EXPORT int llmk_latent_absorb(float* qa, const void* q, long long ldq, const void* wuk, const int* positions,
                                    const float* cos_t, const float* sin_t, int n_tokens, int heads, int dim, int rot, int rank,
-                                   int pairing, int dtype, void* stream) {
+                                   int pairing, const void* dkv, const float* kv_gain, float eps, void* cache, const int* slots,
+                                   int dtype, void* stream) {
     if (n_tokens <= 0) return LLMK_OK;
-    if (heads <= 0 || heads > 65535 || dim < 0 || rot < 0 || rot % 2 != 0 || rank <= 0) LLMK_FAIL("latent_absorb: bad sizes");
+    if (cache && (!dkv || !kv_gain || !slots)) LLMK_FAIL("latent_absorb: cached vectors come from projected rows, gains and slots");
+    if (heads <= 0 || heads > 65534 || dim < 0 || rot < 0 || rot % 2 != 0 || rank <= 0) LLMK_FAIL("latent_absorb: bad sizes");
     if (pairing != LLMK_PAIR_INTERLEAVED && pairing != LLMK_PAIR_HALF_SPLIT) LLMK_FAIL("latent_absorb: unknown rotary pairing %d", pairing);
-    const size_t smem = (size_t)LT_TT * (dim + 2 * rot) * sizeof(float);
-    dim3 grid(ceil_div(n_tokens, LT_TT), heads, ceil_div(rank, 128));
+    size_t smem = (size_t)LT_TT * (dim + 2 * rot) * sizeof(float);
+    if (smem < (33 + 2 * (size_t)rot) * sizeof(float)) smem = (33 + 2 * (size_t)rot) * sizeof(float);
+    dim3 grid(ceil_div(n_tokens, LT_TT), heads + (cache ? 1 : 0), ceil_div(rank, 128));
+    LatentEntries en;
+    en.dkv = dkv; en.gain = kv_gain; en.cache = cache; en.slots = slots; en.eps = eps;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
     if (dtype == LLMK_F32) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(latent_absorb_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         e = llmk_launch(latent_absorb_kernel<float>, grid, dim3(128), smem, s, true, (const float*)q, ldq, (const float*)wuk, qa, positions,
-                        cos_t, sin_t, n_tokens, heads, dim, rot, rank, pairing);
+                        cos_t, sin_t, n_tokens, heads, dim, rot, rank, pairing, en);
     } else if (dtype == LLMK_BF16) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(latent_absorb_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         e = llmk_launch(latent_absorb_kernel<bf16>, grid, dim3(128), smem, s, true, (const bf16*)q, ldq, (const bf16*)wuk, qa, positions,
-                        cos_t, sin_t, n_tokens, heads, dim, rot, rank, pairing);
+                        cos_t, sin_t, n_tokens, heads, dim, rot, rank, pairing, en);
     } else
         LLMK_FAIL("latent_absorb: unknown dtype %d", dtype);
     LLMK_CHECK_LAUNCH_RC("latent_absorb", e);
+    return LLMK_OK;
+}
+
+// --------------------------------------------------------------------------------------------- split
+// For whole portions in bfloat16, queries projected straight from the stream: the heads' unrotated parts go head-major to
+// qn [heads, t_pad, dim] (the operand of the grouped product with Wuk, whose result is columns [0, rank) of qa_hm), their rotated
+// parts turned to columns [rank, rank + rot) of qa_hm [heads, t_pad, rank + rot], and, with `cache`, the token's cached vector to
+// its slot.  One block per token.
+__global__ void __launch_bounds__(256) latent_split_kernel(const bf16* __restrict__ packed, long long ld, bf16* __restrict__ qn,
+                                                           bf16* __restrict__ qa_hm, const int* __restrict__ positions,
+                                                           const float* __restrict__ cos_t, const float* __restrict__ sin_t, int heads,
+                                                           int dim, int rot, int rank, int t_pad, int pairing, int dkv_off, LatentEntries en) {
+    extern __shared__ float sm[];
+    const size_t t = blockIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    const bf16* row = packed + t * ld;
+    const int hd = dim + rot, half = rot / 2, pos = positions[t];
+    const int vecs = dim / 8;                // dim, rot, rank and the row stride are multiples of 8
+    for (int idx = threadIdx.x; idx < heads * vecs; idx += blockDim.x) {
+        const int h = idx / vecs, v = idx % vecs;
+        *reinterpret_cast<uint4*>(qn + ((size_t)h * t_pad + t) * dim + v * 8) = *reinterpret_cast<const uint4*>(row + (size_t)h * hd + v * 8);
+    }
+    for (int idx = threadIdx.x; idx < heads * half; idx += blockDim.x) {
+        const int h = idx / half, i = idx % half;
+        const bf16* src = row + (size_t)h * hd + dim;
+        bf16* dst = qa_hm + ((size_t)h * t_pad + t) * (rank + rot) + rank;
+        const int a = pairing == LLMK_PAIR_INTERLEAVED ? 2 * i : i;
+        const int b = pairing == LLMK_PAIR_INTERLEAVED ? 2 * i + 1 : i + half;
+        const float u = to_float(src[a]), w = to_float(src[b]), c = cos_t[(size_t)pos * half + i], s = sin_t[(size_t)pos * half + i];
+        dst[a] = __float2bfloat16_rn(u * c - w * s);
+        dst[b] = __float2bfloat16_rn(w * c + u * s);
+    }
+    if (!en.cache) return;
+    const int slot = en.slots[t];
+    if (slot < 0) return;
+    latent_entry<bf16>(static_cast<bf16*>(en.cache) + (size_t)slot * (rank + rot), row + dkv_off, rank, rot, en.gain, en.eps, pos, cos_t, sin_t,
+                       pairing, sm);
+}
+
+LLMK_EXPORT int llmk_latent_split(const void* packed, long long ld, void* qn, void* qa_hm, const int* positions, const float* cos_t,
+                                  const float* sin_t, int n_tokens, int heads, int dim, int rot, int rank, int t_pad, int pairing, int dkv_off,
+                                  const float* kv_gain, float eps, void* cache, const int* slots, void* stream) {
+    if (n_tokens <= 0) return LLMK_OK;
+    if (heads <= 0 || dim <= 0 || dim % 8 != 0 || rot < 0 || rot % 8 != 0 || rank <= 0 || rank % 8 != 0 || ld % 8 != 0 || t_pad < n_tokens)
+        LLMK_FAIL("latent_split: widths %d, %d, %d and the row stride must be multiples of 8", dim, rot, rank);
+    if (!host_aligned16(packed) || !host_aligned16(qn) || !host_aligned16(qa_hm)) LLMK_FAIL("latent_split: rows must start on 16-byte boundaries");
+    if (pairing != LLMK_PAIR_INTERLEAVED && pairing != LLMK_PAIR_HALF_SPLIT) LLMK_FAIL("latent_split: unknown rotary pairing %d", pairing);
+    if (cache && (!kv_gain || !slots)) LLMK_FAIL("latent_split: cached vectors need gains and slots");
+    LatentEntries en;
+    en.dkv = nullptr; en.gain = kv_gain; en.cache = cache; en.slots = slots; en.eps = eps;
+    LLMK_CHECK_LAUNCH_RC("latent_split", llmk_launch(latent_split_kernel, dim3(n_tokens), dim3(256), (33 + 2 * (size_t)rot) * sizeof(float),
+                                                     (cudaStream_t)stream, true, (const bf16*)packed, ld, (bf16*)qn, (bf16*)qa_hm, positions, cos_t,
+                                                     sin_t, heads, dim, rot, rank, t_pad, pairing, dkv_off, en));
     return LLMK_OK;
 }
 
@@ -252,9 +344,27 @@ struct LatentAttnParams {
     const int* tile_q0;
     float* part_o;
     float* part_ml;
+    const bf16* qa_hm;         // or, if set (tensor-core form): the queries as bfloat16 [heads, tq_pad, za] in place of `qa`
+    int tq_pad;
+    int window;                // > 0: a query sees the last `window` positions up to its own
     int max_blocks, heads, rank, za, page_size, num_parts, bq, gc, chunks;
     float scale;
 };
+
+// The keys [k_beg, k_end) of this block: what its tile's queries can see, or its part of that.  Without a window the parts cut
+// the sequence's whole context, under one the tile's visible keys.
+__device__ __forceinline__ void latent_key_range(const LatentAttnParams& p, int first_pos, int nq_tile, int ctx, int part, int kt, int& k_beg,
+                                                 int& k_end) {
+    k_end = first_pos + nq_tile;
+    k_beg = p.window > 0 ? max(0, first_pos - p.window + 1) : 0;
+    if (p.num_parts > 1) {
+        const int base = k_beg;
+        const int seen = p.window > 0 ? k_end - k_beg : ctx;
+        const int part_size = ceil_div(ceil_div(max(seen, 1), p.num_parts), kt) * kt;
+        k_beg = base + part * part_size;
+        k_end = min(k_end, base + (part + 1) * part_size);
+    }
+}
 
 template <typename T, int RL>
 __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_kernel(LatentAttnParams p) {
@@ -277,12 +387,7 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_kernel(LatentA
     const bool padding = ctx < q_len || nq_tile <= 0;
     const int first_pos = ctx - q_len + q0;
     int k_beg = 0, k_end = 0;
-    if (!padding) k_end = first_pos + nq_tile;
-    if (p.num_parts > 1) {
-        const int part_size = ceil_div(ceil_div(max(ctx, 1), p.num_parts), LT_KT) * LT_KT;
-        k_beg = max(k_beg, part * part_size);
-        k_end = min(k_end, (part + 1) * part_size);
-    }
+    if (!padding) latent_key_range(p, first_pos, nq_tile, ctx, part, LT_KT, k_beg, k_end);
     const T* zc = static_cast<const T*>(p.cache);
     const int* bt = p.block_tables + (size_t)s * p.max_blocks;
     const int rows = p.bq * p.gc;
@@ -403,7 +508,7 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_kernel(LatentA
 #pragma unroll
         for (int i = 0; i < LT_R; ++i) {
             const int qpos = first_pos + qi_of[i];
-            const bool ok = valid[i] && kpos < k_end && kpos <= qpos;
+            const bool ok = valid[i] && kpos < k_end && kpos <= qpos && (p.window <= 0 || kpos > qpos - p.window);
             const float sv = ok ? sc[i] : -INFINITY;
             const float tmax = warp_max(sv);
             const float m_new = fmaxf(m[i], tmax);
@@ -528,12 +633,7 @@ __global__ void __launch_bounds__(256) latent_attention_mma_kernel(LatentAttnPar
     const bool padding = ctx < q_len || nq_tile <= 0;
     const int first_pos = ctx - q_len + q0;
     int k_beg = 0, k_end = 0;
-    if (!padding) k_end = first_pos + nq_tile;
-    if (p.num_parts > 1) {
-        const int part_size = ceil_div(ceil_div(max(ctx, 1), p.num_parts), MT_KT) * MT_KT;
-        k_beg = max(k_beg, part * part_size);
-        k_end = min(k_end, (part + 1) * part_size);
-    }
+    if (!padding) latent_key_range(p, first_pos, nq_tile, ctx, part, MT_KT, k_beg, k_end);
     const int rows = p.bq * p.gc;
     if (p.num_parts > 1 && k_beg >= k_end) {
         for (int r = threadIdx.x; r < rows; r += blockDim.x) {
@@ -552,6 +652,12 @@ __global__ void __launch_bounds__(256) latent_attention_mma_kernel(LatentAttnPar
     for (int r = warp; r < LT_ROWS; r += LT_WARPS) {
         const int qi = r / p.gc, hh = chunk * p.gc + r % p.gc;
         const bool live = r < rows && qi < nq_tile && hh < p.heads;
+        if (p.qa_hm) {
+            const bf16* src = p.qa_hm + ((size_t)(live ? hh : 0) * p.tq_pad + (size_t)(q_beg + q0 + (live ? qi : 0))) * za;
+            for (int d = lane * 8; d < za; d += 256)
+                *reinterpret_cast<uint4*>(Qs + r * zp + d) = live ? *reinterpret_cast<const uint4*>(src + d) : make_uint4(0u, 0u, 0u, 0u);
+            continue;
+        }
         const float* src = p.qa + ((size_t)(q_beg + q0 + (live ? qi : 0)) * p.heads + (live ? hh : 0)) * za;
         for (int d = lane * 2; d < za; d += 64) {
             float2 v = make_float2(0.f, 0.f);
@@ -656,7 +762,7 @@ __global__ void __launch_bounds__(256) latent_attention_mma_kernel(LatentAttnPar
                     for (int e = 0; e < 2; ++e) {
                         const int col = 16 * t + 8 * h + (lane & 3) * 2 + e;
                         const int kpos = t0 + col;
-                        const bool ok = valid[i] && kpos < k_end && kpos <= qpos[i];
+                        const bool ok = valid[i] && kpos < k_end && kpos <= qpos[i] && (p.window <= 0 || kpos > qpos[i] - p.window);
                         const float sv = ok ? Ss[(rg * 16 + (lane >> 2) + 8 * i) * 33 + col] : -INFINITY;
                         pv[i][t][h][e] = sv;
                         tmax[i] = fmaxf(tmax[i], sv);
@@ -858,11 +964,12 @@ LLMK_EXPORT int llmk_latent_attention_on_tensor_cores(int rank, int rot, int dty
     return dtype == LLMK_BF16 && g_latent_mma && (rank + rot) % 16 == 0 && rank % 64 == 0 && rank <= 512;
 }
 
+// qa_hm (optional, tensor-core form only): the queries as bfloat16 [heads, tq_pad, rank + rot] in place of float32 `qa`.
 // out_hm (optional, tensor-core form only): the result as bfloat16 [heads, t_pad, rank] instead of float32 in `out`.
 LLMK_EXPORT int llmk_latent_attention(float* out, const float* qa, const void* cache, const int* block_tables, int max_blocks,
                                       const int* ctx_len, const int* cu_q, const int* tile_seq, const int* tile_q0, int n_tiles,
-                                      int n_tokens, int heads, int rank, int rot, int page_size, float scale, int num_parts,
-                                      float* scratch, void* out_hm, int t_pad, int dtype, void* stream) {
+                                      int n_tokens, int heads, int rank, int rot, int page_size, float scale, int window, int num_parts,
+                                      float* scratch, void* out_hm, int t_pad, const void* qa_hm, int tq_pad, int dtype, void* stream) {
     if (n_tiles <= 0 || n_tokens <= 0) return LLMK_OK;
     if (heads <= 0 || rank <= 0 || rank > 512 || rot < 0) LLMK_FAIL("latent_attention: bad sizes (heads %d, rank %d, rot %d)", heads, rank, rot);
     if (page_size <= 0) LLMK_FAIL("latent_attention: page_size %d", page_size);
@@ -878,12 +985,17 @@ LLMK_EXPORT int llmk_latent_attention(float* out, const float* qa, const void* c
     p.part_ml = num_parts > 1 ? scratch + (size_t)n_tokens * heads * num_parts * rank : nullptr;
     p.out_hm = static_cast<bf16*>(out_hm);
     p.t_pad = t_pad;
+    p.qa_hm = static_cast<const bf16*>(qa_hm);
+    p.tq_pad = tq_pad;
+    p.window = window > 0 ? window : 0;
     const size_t smem = ((size_t)LT_ROWS * ((p.za + 3) & ~3) + (size_t)LT_KT * (p.za + 1)) * sizeof(float);
     if (smem > 220 * 1024) LLMK_FAIL("latent_attention: cached vectors of %d values do not fit shared memory", p.za);
     dim3 grid(n_tiles, p.chunks, num_parts);
     cudaStream_t s = (cudaStream_t)stream;
     int rc;
     const bool mma = llmk_latent_attention_on_tensor_cores(rank, rot, dtype) && host_aligned16(cache) && ((uintptr_t)qa & 7) == 0;
+    if (qa_hm && (!mma || tq_pad < n_tokens || !host_aligned16(qa_hm))) LLMK_FAIL("latent_attention: head-major queries need the tensor-core form and room for %d tokens", n_tokens);
+    if (!qa_hm && !qa) LLMK_FAIL("latent_attention: no queries");
     if (out_hm && (!mma || t_pad < n_tokens)) LLMK_FAIL("latent_attention: a head-major result needs the tensor-core form and room for %d tokens", n_tokens);
     if (mma) {
         const size_t smem_mma = ((size_t)(LT_ROWS + MT_KT) * (p.za + 8)) * sizeof(bf16) + (size_t)LT_ROWS * 33 * sizeof(float);

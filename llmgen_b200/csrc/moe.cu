@@ -3,7 +3,8 @@
 //
 //   moe_route     per token: z = Wr h (+ b) (float32), s = sigmoid(z) or softmax(z), the `top` largest s choose experts;
 //                 slot t * top + c holds (expert, weight); or the `top` largest z choose and the weights are the softmax
-//                 over the chosen z alone
+//                 over the chosen z alone.  A correction per expert may be added to s for the choice (not for the weights), and
+//                 the weights may be multiplied by a constant
 //   moe_plan      one block: slots grouped by expert, cut into tiles of TT rows of one expert each; the list of tiles
 //                 has a fixed length (slots / TT + experts), padded with expert -1
 //   moe_experts   grid (tiles, column blocks): first product of a tile's rows with its expert's matrices and the
@@ -16,7 +17,7 @@
 //
 // The weight multiplies the expert's input (mode "input") or its output (mode "output").
 // Gated activation: g' = min(g, L), u' = clamp(u, -L, L), y = g' sigmoid(alpha g') (u' + 1)   (L <= 0: no clamp),
-// or the plain gated unit y = g sigmoid(g) u.
+// or the plain gated unit y = g sigmoid(g) u, or without a gate y = relu(u)^2.
 #define LLMK_MODULE_NAME "moe"
 #include "common.cuh"
 
@@ -33,10 +34,12 @@ template <typename T>
 __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict__ wr,
                                                         const float* __restrict__ bias, int* __restrict__ slot_expert,
                                                         float* __restrict__ slot_weight, int K, int E, int top, int scoring,
-                                                        int renorm) {
-    extern __shared__ float sm[];   // [K] the row in float32, [E] scores
+                                                        int renorm, const float* __restrict__ choice_bias, float weight_scale,
+                                                        float sum_eps) {
+    extern __shared__ float sm[];   // [K] the row in float32, [E] scores, [E] what chooses (with `choice_bias`)
     float* xs = sm;
     float* s = sm + K;
+    float* by = choice_bias ? s + E : s;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     const size_t t = blockIdx.x;
     pdl_launch_dependents();
@@ -75,6 +78,8 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h,
     } else {
         for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
     }
+    if (choice_bias)
+        for (int e = lane; e < E; e += 32) by[e] = s[e] + choice_bias[e];
     __syncwarp();
     float total = 0.f;
     for (int c = 0; c < top; ++c) {
@@ -82,7 +87,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h,
         float best = -INFINITY;
         int arg = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
-            const float v = s[e];
+            const float v = by[e];
             if (v > best) { best = v; arg = e; }
         }
         for (int o = 16; o > 0; o >>= 1) {
@@ -91,11 +96,12 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h,
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
         if (arg >= E) { arg = c < E ? c : 0; best = 0.f; }     // nothing comparable was left: a padded row's garbage
+        else if (choice_bias) best = s[arg];                   // the correction chooses, the score weighs
         total += best;
         if (lane == 0) {
             slot_expert[t * top + c] = arg;
             slot_weight[t * top + c] = best;
-            s[arg] = -INFINITY;
+            by[arg] = -INFINITY;
         }
         __syncwarp();
     }
@@ -105,20 +111,25 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h,
             const float mx = slot_weight[t * top];
             float sum = 0.f;
             for (int c = 0; c < top; ++c) sum += expf(slot_weight[t * top + c] - mx);
-            for (int c = 0; c < top; ++c) slot_weight[t * top + c] = expf(slot_weight[t * top + c] - mx) / sum;
+            for (int c = 0; c < top; ++c) slot_weight[t * top + c] = expf(slot_weight[t * top + c] - mx) / sum * weight_scale;
         }
         return;
     }
-    if (renorm && lane == 0)
-        for (int c = 0; c < top; ++c) slot_weight[t * top + c] /= total;
+    if (lane == 0 && (renorm || weight_scale != 1.f))
+        for (int c = 0; c < top; ++c) {
+            const float w = slot_weight[t * top + c];
+            slot_weight[t * top + c] = (renorm ? w / (total + sum_eps) : w) * weight_scale;
+        }
 }
 
 LLMK_EXPORT int llmk_moe_route(const void* h, long long ldh, const float* wr, const float* bias, int* slot_expert, float* slot_weight,
-                               int n_tokens, int K, int E, int top, int scoring, int renorm, int dtype, void* stream) {
+                               int n_tokens, int K, int E, int top, int scoring, int renorm, const float* choice_bias,
+                               float weight_scale, float sum_eps, int dtype, void* stream) {
     if (n_tokens <= 0) return LLMK_OK;
     if (E <= 0 || top <= 0 || top > E || K <= 0) LLMK_FAIL("moe_route: bad sizes (experts %d, top %d, width %d)", E, top, K);
     if (scoring < 0 || scoring > 2) LLMK_FAIL("moe_route: unknown scoring %d", scoring);
-    const size_t smem = ((size_t)K + E) * sizeof(float);
+    if (choice_bias && scoring == 2) LLMK_FAIL("moe_route: a correction of the scores needs scores (scoring %d)", scoring);
+    const size_t smem = ((size_t)K + 2 * E) * sizeof(float);
     if (smem > 200 * 1024) LLMK_FAIL("moe_route: a row of %d values and %d experts do not fit shared memory", K, E);
     const int threads = E >= 8 ? 256 : 32 * E;
     cudaStream_t s = (cudaStream_t)stream;
@@ -126,11 +137,11 @@ LLMK_EXPORT int llmk_moe_route(const void* h, long long ldh, const float* wr, co
     if (dtype == LLMK_F32) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         e = llmk_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(threads), smem, s, true, (const float*)h, ldh, wr, bias, slot_expert,
-                        slot_weight, K, E, top, scoring, renorm);
+                        slot_weight, K, E, top, scoring, renorm, choice_bias, weight_scale, sum_eps);
     } else if (dtype == LLMK_BF16) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         e = llmk_launch(moe_route_kernel<bf16>, dim3(n_tokens), dim3(threads), smem, s, true, (const bf16*)h, ldh, wr, bias, slot_expert,
-                        slot_weight, K, E, top, scoring, renorm);
+                        slot_weight, K, E, top, scoring, renorm, choice_bias, weight_scale, sum_eps);
     } else
         LLMK_FAIL("moe_route: unknown dtype %d", dtype);
     LLMK_CHECK_LAUNCH_RC("moe_route", e);
@@ -274,7 +285,8 @@ __global__ void __launch_bounds__(128) moe_experts_kernel(float* __restrict__ ou
     }
     __syncthreads();
     const T* wa = w0 + ((size_t)e * N + (col < N ? col : 0)) * K;
-    const T* wb = FIRST ? w1 + ((size_t)e * N + (col < N ? col : 0)) * K : nullptr;
+    const bool gated = FIRST && plain != 2;
+    const T* wb = gated ? w1 + ((size_t)e * N + (col < N ? col : 0)) * K : nullptr;
     float acc0[MOE_TT], acc1[FIRST ? MOE_TT : 1];
 #pragma unroll
     for (int i = 0; i < MOE_TT; ++i) acc0[i] = 0.f;
@@ -302,7 +314,7 @@ __global__ void __launch_bounds__(128) moe_experts_kernel(float* __restrict__ ou
                 const float a = to_float(wa[k0 + k]);
 #pragma unroll
                 for (int i = 0; i < MOE_TT; ++i) acc0[i] = fmaf(xs[i][k], a, acc0[i]);
-                if (FIRST) {
+                if (FIRST && gated) {
                     const float b = to_float(wb[k0 + k]);
 #pragma unroll
                     for (int i = 0; i < MOE_TT; ++i) acc1[i] = fmaf(xs[i][k], b, acc1[i]);
@@ -317,7 +329,9 @@ __global__ void __launch_bounds__(128) moe_experts_kernel(float* __restrict__ ou
         float v;
         if (FIRST) {
             float g = acc0[i], u = acc1[i];
-            if (plain) {
+            if (plain == 2) {
+                v = fmaxf(g, 0.f) * fmaxf(g, 0.f);
+            } else if (plain) {
                 v = g / (1.0f + expf(-g)) * u;
             } else {
                 if (limit > 0.f) {
@@ -333,7 +347,7 @@ __global__ void __launch_bounds__(128) moe_experts_kernel(float* __restrict__ ou
     }
 }
 
-// plain != 0: the gated unit is silu(g) u (alpha and limit unused).
+// plain 1: the gated unit is silu(g) u; 2: no gate, relu(u)^2 with w0 = up and no w1 (alpha and limit unused).
 // first != 0: in = h [tokens, width] of the storage dtype, w0 / w1 = gate / up [E, ff, width], out = y [slots, ff]; the rows
 //             are multiplied by their weights when weight_on_input.
 // first == 0: in = y [slots, ff] float32, w0 = down [E, width, ff], out [slots, width]; multiplied by the weights
@@ -343,6 +357,7 @@ LLMK_EXPORT int llmk_moe_experts(float* out, const void* in, long long ld_in, co
                                  int n_slots, int E, int top, int K, int N, int first, int weight_on_input, float alpha, float limit,
                                  int plain, int dtype, void* stream) {
     if (n_slots <= 0) return LLMK_OK;
+    if (first && plain != 2 && !w1) LLMK_FAIL("moe_experts: a gated unit needs two matrices");
     dim3 grid(llmk_moe_max_tiles(n_slots, E, 0), ceil_div(N, 128));
     cudaStream_t s = (cudaStream_t)stream;
     const int scale_rows = first ? (weight_on_input ? 1 : 0) : (weight_on_input ? 0 : 1);

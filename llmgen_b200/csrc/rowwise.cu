@@ -5,6 +5,9 @@
 //                   for the products that read the residual itself; y may be a weighted sum of two products
 //                   (a y + b y2), and the copy may be the next sublayer's normed input, rmsnorm(resid) * w_next,
 //                   for layers that norm a sublayer's input as well as its output
+//   parallel_add    layers whose two sublayers run side by side: resid[r, :] += a . y1[r, :] + b . y2[r, :] with gain vectors a
+//                   and b, and the next layer's normed input, rmsnorm(resid) * w, in the same pass; y2 may be the rows of a routed
+//                   feed-forward before their sum
 //   scaled_sum      out (float32) = a y + b y2, for consumers that take one array
 //   cast_rows       out = (T) in, float32 in
 //   act_rows        relu(x)^2, tanh(x), gelu_tanh(x), the clamped gated unit  g' s(alpha g') (u' + 1)  with g' = min(g, L), u' = clamp(u, -L, L),
@@ -104,6 +107,189 @@ LLMK_EXPORT int llmk_norm_add2(float* resid, const void* y, const float* w, void
 LLMK_EXPORT int llmk_norm_add(float* resid, const void* y, const float* w, void* copy, int n_rows, int H, float eps,
                               int splits, long long split_stride, int dtype, void* stream) {
     return llmk_norm_add2(resid, y, w, copy, n_rows, H, eps, splits, split_stride, nullptr, 0, 0, 1.f, 0.f, nullptr, 0.f, dtype, stream);
+}
+
+// ------------------------------------------------------------------------------------------------ two sublayers side by side
+// resid[r, i] += ga[i] * y1[r, i] + gb[i] * y2[r, i]; normed[r, :] = rmsnorm(resid[r, :]) * w (w null: not asked for).  y1, y2 are
+// arrays of T or float32 slices; or y2 is `routed`: float32 rows of a routed feed-forward, of which token r takes
+// pos_of_slot[r * top + k] times slot_weight[r * top + k], k < top in order (a weight already applied: slot_weight null).
+// Either sublayer may be absent (null); a gain vector that is null counts as ones.  A block per row, V values a thread at a time.
+struct ParallelAdd {
+    float* resid;
+    const void* y1;
+    const void* y2;
+    const float* routed;
+    const int* pos_of_slot;
+    const float* slot_weight;
+    const float* ga;
+    const float* gb;
+    const float* w;
+    void* normed;
+    long long stride1, stride2;
+    int splits1, splits2, top, H;
+    float eps;
+};
+
+template <typename T, int V>
+__device__ __forceinline__ void load_sum_vec(float (&v)[V], const void* y, size_t at, int splits, long long split_stride) {
+    if constexpr (V == 1) {
+        v[0] = load_sum<T>(y, at, splits, split_stride);
+    } else if (splits == 0) {
+        if constexpr (sizeof(T) == 2) {
+            const uint2 raw = *reinterpret_cast<const uint2*>(static_cast<const T*>(y) + at);
+            const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+            const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+            v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+        } else {
+            const float4 f = *reinterpret_cast<const float4*>(static_cast<const float*>(y) + at);
+            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+        }
+    } else {
+        const float* p = static_cast<const float*>(y) + at;
+        float4 acc = *reinterpret_cast<const float4*>(p);
+#pragma unroll 4
+        for (int s = 1; s < splits; ++s) {
+            const float4 f = *reinterpret_cast<const float4*>(p + (size_t)s * split_stride);
+            acc.x += f.x; acc.y += f.y; acc.z += f.z; acc.w += f.w;
+        }
+        v[0] = acc.x; v[1] = acc.y; v[2] = acc.z; v[3] = acc.w;
+    }
+}
+
+template <int V>
+__device__ __forceinline__ void load_f32_vec(float (&v)[V], const float* p) {
+    if constexpr (V == 1) {
+        v[0] = p[0];
+    } else {
+        const float4 f = *reinterpret_cast<const float4*>(p);
+        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(512) parallel_add_kernel(ParallelAdd p) {
+    extern __shared__ __align__(16) float prow[];  // H floats + 33 scratch, then the row's slots: top positions, top weights
+    const int H = p.H;
+    float* scratch = prow + ((H + 3) & ~3);
+    int* pos = reinterpret_cast<int*>(scratch + 36);
+    float* wgt = reinterpret_cast<float*>(pos + p.top);
+    const size_t r = blockIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (p.routed) {
+        for (int k = threadIdx.x; k < p.top; k += blockDim.x) {
+            pos[k] = p.pos_of_slot[r * p.top + k];
+            wgt[k] = p.slot_weight ? p.slot_weight[r * p.top + k] : 1.f;
+        }
+        __syncthreads();
+    }
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+        float x[V], v[V], g[V];
+        load_f32_vec<V>(x, p.resid + r * H + i);
+        float add[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) add[e] = 0.f;
+        if (p.y1) {
+            load_sum_vec<T, V>(v, p.y1, r * H + i, p.splits1, p.stride1);
+            if (p.ga) {
+                load_f32_vec<V>(g, p.ga + i);
+#pragma unroll
+                for (int e = 0; e < V; ++e) add[e] = g[e] * v[e];
+            } else {
+#pragma unroll
+                for (int e = 0; e < V; ++e) add[e] = v[e];
+            }
+        }
+        if (p.y2 || p.routed) {
+            if (p.routed) {
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] = 0.f;
+                for (int k = 0; k < p.top; ++k) {
+                    if (pos[k] < 0) continue;
+                    float row[V];
+                    load_f32_vec<V>(row, p.routed + (size_t)pos[k] * H + i);
+#pragma unroll
+                    for (int e = 0; e < V; ++e) v[e] += wgt[k] * row[e];
+                }
+            } else {
+                load_sum_vec<T, V>(v, p.y2, r * H + i, p.splits2, p.stride2);
+            }
+            if (p.gb) {
+                load_f32_vec<V>(g, p.gb + i);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] *= g[e];
+            }
+#pragma unroll
+            for (int e = 0; e < V; ++e) add[e] += v[e];
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            x[e] += add[e];
+            ss = fmaf(x[e], x[e], ss);
+        }
+        if constexpr (V == 1) {
+            p.resid[r * H + i] = x[0];
+            prow[i] = x[0];
+        } else {
+            const float4 f = make_float4(x[0], x[1], x[2], x[3]);
+            *reinterpret_cast<float4*>(p.resid + r * H + i) = f;
+            *reinterpret_cast<float4*>(prow + i) = f;
+        }
+    }
+    if (!p.w) return;
+    ss = block_sum(ss, scratch);
+    const float rinv = 1.0f / sqrtf(ss / (float)H + p.eps);
+    T* out = static_cast<T*>(p.normed) + r * H;
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {       // every thread its own values again
+        float x[V], g[V];
+        load_f32_vec<V>(x, prow + i);
+        load_f32_vec<V>(g, p.w + i);
+        if constexpr (V == 1) {
+            out[i] = from_float<T>(x[0] * rinv * g[0]);
+        } else if constexpr (sizeof(T) == 2) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(x[0] * rinv * g[0], x[1] * rinv * g[1]);
+            const __nv_bfloat162 hi = __floats2bfloat162_rn(x[2] * rinv * g[2], x[3] * rinv * g[3]);
+            *reinterpret_cast<uint2*>(out + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        } else {
+            *reinterpret_cast<float4*>(out + i) = make_float4(x[0] * rinv * g[0], x[1] * rinv * g[1], x[2] * rinv * g[2], x[3] * rinv * g[3]);
+        }
+    }
+}
+
+// `pdl` 0: a plain launch (behind an event of another stream).
+LLMK_EXPORT int llmk_parallel_add(float* resid, const void* y1, int splits1, long long stride1, const void* y2, int splits2, long long stride2,
+                                  const float* routed, const int* pos_of_slot, const float* slot_weight, int top, const float* ga,
+                                  const float* gb, const float* w, float eps, void* normed, int n_rows, int H, int pdl, int dtype,
+                                  void* stream) {
+    if (n_rows <= 0) return LLMK_OK;
+    if (H <= 0 || !resid || (!y1 && !y2 && !routed)) LLMK_FAIL("parallel_add: bad arguments (H %d)", H);
+    if (routed && (y2 || !pos_of_slot || top <= 0 || top > 1024)) LLMK_FAIL("parallel_add: routed rows come with their slots, in place of the second result");
+    if (w && !normed) LLMK_FAIL("parallel_add: the next norm's output needs a place");
+    ParallelAdd p;
+    p.resid = resid; p.y1 = y1; p.y2 = y2; p.routed = routed; p.pos_of_slot = pos_of_slot; p.slot_weight = slot_weight;
+    p.ga = ga; p.gb = gb; p.w = w; p.normed = normed; p.stride1 = stride1; p.stride2 = stride2;
+    p.splits1 = splits1; p.splits2 = splits2; p.top = routed ? top : 0; p.H = H; p.eps = eps;
+    const size_t smem = ((size_t)((H + 3) & ~3) + 36 + 2 * (size_t)p.top) * sizeof(float);
+    if (smem > 200 * 1024) LLMK_FAIL("parallel_add: a row of %d values does not fit shared memory", H);
+    // four values a thread at a time where every row starts on 16 bytes (8 of bfloat16)
+    const bool vec = H % 4 == 0 && stride1 % 4 == 0 && stride2 % 4 == 0 && host_aligned16(resid) && (!y1 || host_aligned16(y1)) &&
+                     (!y2 || host_aligned16(y2)) && (!routed || host_aligned16(routed)) && (!ga || host_aligned16(ga)) &&
+                     (!gb || host_aligned16(gb)) && (!w || host_aligned16(w)) && (!normed || host_aligned16(normed));
+    const int per = vec ? H / 4 : H;
+    const int threads = per > 256 ? 512 : per > 128 ? 256 : per > 64 ? 128 : 64;
+    cudaStream_t s = (cudaStream_t)stream;
+    cudaError_t e;
+#define PARALLEL_ADD_LAUNCH(TYPE, V)                                                                                                   do {                                                                                                                                   if (smem > 48 * 1024) cudaFuncSetAttribute(parallel_add_kernel<TYPE, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         e = llmk_launch(parallel_add_kernel<TYPE, V>, dim3(n_rows), dim3(threads), smem, s, pdl != 0, p);                              } while (0)
+    if (dtype == LLMK_F32) {
+        if (vec) PARALLEL_ADD_LAUNCH(float, 4); else PARALLEL_ADD_LAUNCH(float, 1);
+    } else if (dtype == LLMK_BF16) {
+        if (vec) PARALLEL_ADD_LAUNCH(bf16, 4); else PARALLEL_ADD_LAUNCH(bf16, 1);
+    } else
+        LLMK_FAIL("parallel_add: unknown dtype %d", dtype);
+#undef PARALLEL_ADD_LAUNCH
+    LLMK_CHECK_LAUNCH_RC("parallel_add", e);
+    return LLMK_OK;
 }
 
 // out[i] (float32) = a * y[i] + b * y2[i]; y and y2 arrays of T or float32 slices.

@@ -124,9 +124,12 @@ class Executor:
             for table, req in ((kv_requests, kv), (state_requests, st)):
                 if req is None:
                     continue
-                if item.cache in table and table[item.cache] != req:
+                held = table.get(item.cache, req)
+                # items that share a cache may look back to different depths: its pages serve the deepest view
+                both = held.shared_with(req) if table is kv_requests else (req if held == req else None)
+                if both is None:
                     raise StepError(f"run items sharing cache {item.cache} ask for different geometries")
-                table[item.cache] = req
+                table[item.cache] = both
         self.kv_requests, self.state_requests = kv_requests, state_requests
         self.group_specs, self.group_index = plan_groups(kv_requests)
         pages = self._pages_per_group()

@@ -539,6 +539,14 @@ def _check_sinks(who: str, sink: bool, sink_values: Optional[torch.Tensor], nq: 
         raise KernelError(f"{who}: the sinks' scores are one float32 per query head, with `sink` set")
 
 
+def _check_k_scale(who: str, k_scale: Optional[torch.Tensor], kcache: torch.Tensor, vcache: Optional[torch.Tensor]) -> None:
+    if (k_scale is None) != (vcache is not None):
+        raise KernelError(f"{who}: values are an array of their own, or the keys with a factor per token on their scores")
+    if k_scale is not None and (k_scale.dtype != torch.float32 or not k_scale.is_contiguous()
+                                or k_scale.numel() != kcache.shape[0] * kcache.shape[2]):
+        raise KernelError(f"{who}: the factors on the scores are float32 [pages, page_size]")
+
+
 ATTENTION_TURN_WIDTHS = (64, 128)    # value widths whose rows the attention kernels turn back themselves
 
 
@@ -560,15 +568,19 @@ def paged_attention(out: torch.Tensor, q: torch.Tensor, q_stride: int, kcache: t
                     hd: int, page_size: int, window: int, scale: float, num_parts: int = 1, part_size: int = 0,
                     scratch: Optional[torch.Tensor] = None, vd: int = 0, softcap: float = 0.0, sink: bool = False,
                     gate: Optional[torch.Tensor] = None, chunk: int = 0, sink_values: Optional[torch.Tensor] = None,
-                    gate_per_head: bool = False, turn_back: Optional[tuple] = None, positions: Optional[torch.Tensor] = None) -> None:
+                    gate_per_head: bool = False, turn_back: Optional[tuple] = None, positions: Optional[torch.Tensor] = None,
+                    k_scale: Optional[torch.Tensor] = None) -> None:
     """out[t, nq*vd] = causal GQA of q[t] over the paged cache (see csrc/attention.cu).  `vd`: the values' width where
     it differs from `hd`; `softcap` > 0 bounds the scores by softcap * tanh(s / softcap); `sink` adds exp(0) to the
     softmax's denominator (exp(sink_values[head]) with `sink_values`, float32 [nq]); `gate` [tokens, nq*vd] (storage dtype): the result is multiplied by sigmoid(gate)
     (`gate_per_head`: [tokens, nq], one number per head); `turn_back` = (cos, sin) float32 [positions, vd / 2] with `positions` (the
     tokens' positions): each head's row is turned back in pairs (m, m + vd / 2) by minus its position before the gate (value widths
     `ATTENTION_TURN_WIDTHS`); `chunk` > 0:
-    a query sees the keys at or before it inside its own block of that many positions, counted from the sequence's start."""
+    a query sees the keys at or before it inside its own block of that many positions, counted from the sequence's start.
+    `k_scale` (float32 [pages, page_size], `vcache` None): the cached keys are the values too, and a token's scores are
+    multiplied by its entry of `k_scale`."""
     lib = build.load("attention")
+    _check_k_scale("paged_attention", k_scale, kcache, vcache)
     if gate is not None and gate.dtype != q.dtype:
         raise KernelError("paged_attention: the gate has the storage dtype")
     _check_sinks("paged_attention", sink, sink_values, nq)
@@ -584,7 +596,7 @@ def paged_attention(out: torch.Tensor, q: torch.Tensor, q_stride: int, kcache: t
                                          c_int(window), c_float(scale), c_int(num_parts), c_int(part_size),
                                          _ptr(scratch), c_int(vd), c_float(softcap), c_int(1 if sink else 0), _ptr(sink_values),
                                          _ptr(gate), c_longlong(_row_stride(gate) if gate is not None else 0), c_int(chunk),
-                                         c_int(1 if gate_per_head else 0), _ptr(tcos), _ptr(tsin), _ptr(positions),
+                                         c_int(1 if gate_per_head else 0), _ptr(tcos), _ptr(tsin), _ptr(positions), _ptr(k_scale),
                                          c_int(dtype_code(q.dtype)), _stream()),
            2 if num_parts > 1 else 1)
 
@@ -598,20 +610,22 @@ def attention_mma(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcac
                   max_blocks: int, ctx_len: torch.Tensor, cu_q: torch.Tensor, tile_seq: torch.Tensor, tile_q0: torch.Tensor,
                   n_tiles: int, nq: int, nkv: int, hd: int, vd: int, page_size: int, window: int, scale: float,
                   softcap: float = 0.0, sink: bool = False, gate: Optional[torch.Tensor] = None, chunk: int = 0,
-                  sink_values: Optional[torch.Tensor] = None, gate_per_head: bool = False, turn_back: Optional[tuple] = None) -> None:
+                  sink_values: Optional[torch.Tensor] = None, gate_per_head: bool = False, turn_back: Optional[tuple] = None,
+                  k_scale: Optional[torch.Tensor] = None) -> None:
     """Prompt portions in bfloat16 with 32-bit softmax weights on the tensor cores (csrc/attention_mma.cu): the same
     result as `paged_attention` with these options, tiles of `attention_mma_tile_queries` queries."""
     lib = build.load("attention_mma")
     if q.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or kcache.dtype != torch.bfloat16 or (gate is not None and gate.dtype != torch.bfloat16):
         raise KernelError("attention_mma: bfloat16 only")
     _check_sinks("attention_mma", sink, sink_values, nq)
+    _check_k_scale("attention_mma", k_scale, kcache, vcache)
     tcos, tsin = _check_turn("attention_mma", turn_back, ctx_len, vd, gate, gate_per_head, nq)
     _check(lib, lib.llmk_attention_mma(_ptr(out), c_longlong(_row_stride(out)), _ptr(q), c_longlong(_row_stride(q)), _ptr(kcache),
                                        _ptr(vcache), _ptr(block_tables), c_int(max_blocks), _ptr(ctx_len), _ptr(cu_q), _ptr(tile_seq),
                                        _ptr(tile_q0), c_int(n_tiles), c_int(nq), c_int(nkv), c_int(hd), c_int(vd), c_int(page_size),
                                        c_int(window), c_float(scale), c_float(softcap), c_int(1 if sink else 0), _ptr(sink_values),
                                        _ptr(gate), c_longlong(_row_stride(gate) if gate is not None else 0), c_int(chunk),
-                                       c_int(1 if gate_per_head else 0), _ptr(tcos), _ptr(tsin), _stream()))
+                                       c_int(1 if gate_per_head else 0), _ptr(tcos), _ptr(tsin), _ptr(k_scale), _stream()))
 
 
 def attention_decode_set_cluster_merge(on: bool) -> None:
@@ -802,6 +816,61 @@ def scaled_sum(out: torch.Tensor, pair: WeightedPair, dtype: torch.dtype) -> Par
     return Partials(out)
 
 
+class RoutedRows:
+    """The result of a routed feed-forward before its rows are added up: token t is the sum over its `top` slots, in order, of
+    rows[pos_of_slot[t * top + k]] (float32) times slot_weight[t * top + k] (None: the weight was applied before).  `parallel_add`
+    takes it as it is; `sum` adds it up for consumers that take one array."""
+
+    def __init__(self, rows: torch.Tensor, pos_of_slot: torch.Tensor, slot_weight: Optional[torch.Tensor], top: int):
+        if rows.dtype != torch.float32 or not rows.is_contiguous() or pos_of_slot.dtype != torch.int32 \
+                or (slot_weight is not None and slot_weight.dtype != torch.float32):
+            raise KernelError("routed rows are contiguous float32, their places int32, their weights float32")
+        self.rows, self.pos_of_slot, self.slot_weight, self.top = rows, pos_of_slot, slot_weight, top
+
+    @property
+    def n_tokens(self) -> int:
+        return self.pos_of_slot.numel() // self.top
+
+    def sum(self, out: torch.Tensor) -> Partials:
+        """out (float32 [1, n, H], contiguous) = the tokens' sums; returned as a one-slice `Partials`."""
+        moe_combine(out[0], self.rows, self.pos_of_slot, None, self.top, slot_weight=self.slot_weight)
+        return Partials(out)
+
+
+def parallel_add(resid: torch.Tensor, first, first_gain: Optional[torch.Tensor], second, second_gain: Optional[torch.Tensor],
+                 dtype: torch.dtype, next_gain: Optional[torch.Tensor] = None, eps: float = 0.0,
+                 normed: Optional[torch.Tensor] = None, pdl: bool = True) -> None:
+    """resid (float32 [n, H]) += first_gain * first + second_gain * second (gains float32 [H], None: ones); with `next_gain`,
+    normed (storage dtype) = rmsnorm(resid) * next_gain.  `first` is an array of the storage dtype or a `Partials`; `second` one
+    of these, a `RoutedRows`, or None.  `pdl=False`: not launched as a programmatic dependent (behind an event of another stream)."""
+    lib = build.load("rowwise")
+    n, H = resid.shape
+    if resid.dtype != torch.float32 or not resid.is_contiguous():
+        raise KernelError("parallel_add: the residual is contiguous float32")
+    for g in (first_gain, second_gain, next_gain):
+        if g is not None and (g.dtype != torch.float32 or g.numel() != H or not g.is_contiguous()):
+            raise KernelError("parallel_add: gains are contiguous float32 [H]")
+    if next_gain is not None and (normed is None or normed.dtype != dtype or tuple(normed.shape) != (n, H) or not normed.is_contiguous()):
+        raise KernelError("parallel_add: the next norm's output needs a place [n, H] of the storage dtype")
+    src, splits, stride = _delta_args(first, dtype)
+    if (first.rows if isinstance(first, Partials) else first.shape[0]) != n or (first.cols if isinstance(first, Partials) else first.shape[1]) != H:
+        raise KernelError("parallel_add: shapes do not fit")
+    src2, splits2, stride2, routed = None, 0, 0, None
+    if isinstance(second, RoutedRows):
+        routed = second
+        if routed.n_tokens != n or routed.rows.shape[1] != H:
+            raise KernelError("parallel_add: shapes do not fit")
+    elif second is not None:
+        src2, splits2, stride2 = _delta_args(second, dtype)
+        if (second.rows if isinstance(second, Partials) else second.shape[0]) != n or (second.cols if isinstance(second, Partials) else second.shape[1]) != H:
+            raise KernelError("parallel_add: shapes do not fit")
+    _check(lib, lib.llmk_parallel_add(_ptr(resid), _ptr(src), c_int(splits), c_longlong(stride), _ptr(src2), c_int(splits2), c_longlong(stride2),
+                                      _ptr(routed.rows if routed else None), _ptr(routed.pos_of_slot if routed else None),
+                                      _ptr(routed.slot_weight if routed else None), c_int(routed.top if routed else 0), _ptr(first_gain),
+                                      _ptr(second_gain), _ptr(next_gain), c_float(eps), _ptr(normed), c_int(n), c_int(H), c_int(1 if pdl else 0),
+                                      c_int(dtype_code(dtype)), _stream()))
+
+
 def cast_rows(out: torch.Tensor, src: torch.Tensor) -> None:
     """out (storage dtype, contiguous) = src (float32, contiguous), element by element."""
     lib = build.load("rowwise")
@@ -953,6 +1022,35 @@ def attn_prep_rows(x: torch.Tensor, q_out: torch.Tensor, kcache: Optional[torch.
                                         _ptr(vcache), _ptr(positions), _ptr(slots), _ptr(cos), _ptr(sin), _ptr(vcos), _ptr(vsin),
                                         _ptr(q_gain), _ptr(k_gain), c_int(n), c_int(nq), c_int(nk), c_int(nkv_cache), c_int(hd), c_int(vd),
                                         c_int(rot), c_int(page_size), c_float(eps), c_int(dtype_code(q_out.dtype)), _stream()))
+
+
+def attn_prep_shared_rows(x, bias: Optional[torch.Tensor], q_out: torch.Tensor, cache: Optional[torch.Tensor], k_scale: Optional[torch.Tensor],
+                          positions: torch.Tensor, slots: Optional[torch.Tensor], gains: torch.Tensor, nq: int, nk: int, hd: int,
+                          page_size: int, eps: float, coef: float = 0.0, every: float = 1.0) -> None:
+    """x = [q | k] of each token (an array of the storage dtype or a `Partials`), + `bias` (float32 over the packed columns): the
+    projected keys go to the paged `cache` as they are, the inverse root mean square of a token's row of them to `k_scale`
+    (float32 [pages, page_size]), and the query, divided by the root mean square of its row, times `gains` (float32 [nq hd]) and
+    1 + coef ln(floor((position + 1) / every) + 1), to `q_out` (csrc/attn_prep.cu)."""
+    lib = build.load("attn_prep")
+    n = q_out.shape[0]
+    if isinstance(x, Partials):
+        src, splits, stride, ld, cols, rows = x.tensor, x.splits, x.split_stride, x.cols, x.cols, x.rows
+    else:
+        src, splits, stride, ld, cols, rows = x, 0, 0, _row_stride(x), x.shape[1], x.shape[0]
+        if x.dtype != q_out.dtype:
+            raise KernelError("attn_prep_shared_rows: rows of the storage dtype or float32 slices")
+    if rows != n or cols < (nq + nk) * hd or q_out.shape[1] < nq * hd or gains.dtype != torch.float32 or gains.numel() != nq * hd \
+            or (bias is not None and (bias.dtype != torch.float32 or bias.numel() < (nq + nk) * hd)):
+        raise KernelError("attn_prep_shared_rows: shapes do not fit")
+    if nk > 0:
+        if cache is None or cache.dtype != q_out.dtype:
+            raise KernelError("attn_prep_shared_rows: the cache has the storage dtype")
+        _check_k_scale("attn_prep_shared_rows", k_scale, cache, None)
+    _check(lib, lib.llmk_attn_prep_shared_rows(_ptr(src), c_longlong(ld), c_int(splits), c_longlong(stride), _ptr(bias), _ptr(q_out),
+                                               c_longlong(_row_stride(q_out)), _ptr(cache), _ptr(k_scale), _ptr(positions), _ptr(slots),
+                                               _ptr(gains), c_int(n), c_int(nq), c_int(nk), c_int(cache.shape[1] if nk > 0 else 0), c_int(hd),
+                                               c_int(page_size), c_float(eps), c_float(coef), c_float(every), c_int(dtype_code(q_out.dtype)),
+                                               _stream()))
 
 
 def unrotate_gate(o: torch.Tensor, gate: Optional[torch.Tensor], positions: torch.Tensor, vcos: Optional[torch.Tensor],
@@ -1231,15 +1329,42 @@ def latent_prep(packed: torch.Tensor, dq_off: int, dkv_off: int, q_rank: int, ra
 
 
 def latent_absorb(qa: torch.Tensor, q: torch.Tensor, wuk: torch.Tensor, positions: torch.Tensor, cos: Optional[torch.Tensor],
-                  sin: Optional[torch.Tensor], heads: int, dim: int, rot: int, rank: int, pairing: str) -> None:
-    """qa float32 [n, heads, rank + rot] = [Wuk_h^T q_unrotated | rotate(q_rotated)] of q [n, heads * (dim + rot)]."""
+                  sin: Optional[torch.Tensor], heads: int, dim: int, rot: int, rank: int, pairing: str,
+                  dkv: Optional[torch.Tensor] = None, kv_gain: Optional[torch.Tensor] = None, eps: float = 0.0,
+                  cache: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None) -> None:
+    """qa float32 [n, heads, rank + rot] = [Wuk_h^T q_unrotated | rotate(q_rotated)] of q [n, >= heads * (dim + rot)].  With `cache`
+    the same launch writes the tokens' cached vectors, [rmsnorm(c) * kv_gain | rotate(kr)] of `dkv` [n, rank + rot] (a view of
+    the rows q is a view of), at `slots`."""
     lib = build.load("latent_attention")
     n = q.shape[0]
     if qa.dtype != torch.float32 or not qa.is_contiguous() or qa.numel() != n * heads * (rank + rot) or wuk.dtype != q.dtype:
         raise KernelError("latent_absorb: shapes or dtypes do not fit")
+    if cache is not None and (dkv is None or dkv.dtype != q.dtype or cache.dtype != q.dtype or _row_stride(dkv) != _row_stride(q)
+                              or dkv.shape[1] < rank + rot or kv_gain is None or kv_gain.dtype != torch.float32):
+        raise KernelError("latent_absorb: the cached vectors come from rows as far apart as the queries'")
     _check(lib, lib.llmk_latent_absorb(_ptr(qa), _ptr(q), c_longlong(_row_stride(q)), _ptr(wuk), _ptr(positions), _ptr(cos), _ptr(sin),
                                        c_int(n), c_int(heads), c_int(dim), c_int(rot), c_int(rank), c_int(pairing_code(pairing)),
+                                       _ptr(dkv), _ptr(kv_gain), c_float(eps), _ptr(cache), _ptr(slots),
                                        c_int(dtype_code(q.dtype)), _stream()))
+
+
+def latent_split(packed: torch.Tensor, dkv_off: int, qn: torch.Tensor, qa_hm: torch.Tensor, positions: torch.Tensor,
+                 cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], heads: int, dim: int, rot: int, rank: int, pairing: str,
+                 kv_gain: Optional[torch.Tensor] = None, eps: float = 0.0, cache: Optional[torch.Tensor] = None,
+                 slots: Optional[torch.Tensor] = None) -> None:
+    """packed bfloat16 [n, >= heads * (dim + rot)]: the heads' unrotated parts to qn [heads, t_pad, dim], their turned rotated
+    parts to columns [rank, rank + rot) of qa_hm [heads, t_pad, rank + rot], and, with `cache`, the tokens' cached vectors
+    [rmsnorm(c) * kv_gain | rotate(kr)] (columns `dkv_off` on) to their slots."""
+    lib = build.load("latent_attention")
+    n = packed.shape[0]
+    t_pad = qn.shape[1]
+    if packed.dtype != torch.bfloat16 or tuple(qn.shape) != (heads, t_pad, dim) or tuple(qa_hm.shape) != (heads, t_pad, rank + rot) \
+            or not qn.is_contiguous() or not qa_hm.is_contiguous() or qn.dtype != torch.bfloat16 or qa_hm.dtype != torch.bfloat16 \
+            or packed.shape[1] < (dkv_off + rank + rot if cache is not None else heads * (dim + rot)):
+        raise KernelError("latent_split: shapes or dtypes do not fit")
+    _check(lib, lib.llmk_latent_split(_ptr(packed), c_longlong(_row_stride(packed)), _ptr(qn), _ptr(qa_hm), _ptr(positions), _ptr(cos), _ptr(sin),
+                                      c_int(n), c_int(heads), c_int(dim), c_int(rot), c_int(rank), c_int(t_pad), c_int(pairing_code(pairing)),
+                                      c_int(dkv_off), _ptr(kv_gain), c_float(eps), _ptr(cache), _ptr(slots), _stream()))
 
 
 def latent_rotate(qa: torch.Tensor, positions: torch.Tensor, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], heads: int,
@@ -1272,13 +1397,16 @@ def latent_attention_on_tensor_cores(dtype: torch.dtype, rank: int, rot: int) ->
     return bool(build.load("latent_attention").llmk_latent_attention_on_tensor_cores(c_int(rank), c_int(rot), c_int(dtype_code(dtype))))
 
 
-def latent_attention(out: Optional[torch.Tensor], qa: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, max_blocks: int,
+def latent_attention(out: Optional[torch.Tensor], qa: Optional[torch.Tensor], cache: torch.Tensor, block_tables: torch.Tensor, max_blocks: int,
                      ctx_len: torch.Tensor, cu_q: torch.Tensor, tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tokens: int,
                      heads: int, rank: int, rot: int, page_size: int, scale: float, parts: int = 1,
-                     scratch: Optional[torch.Tensor] = None, out_head_major: Optional[torch.Tensor] = None) -> None:
+                     scratch: Optional[torch.Tensor] = None, out_head_major: Optional[torch.Tensor] = None, window: int = 0,
+                     q_head_major: Optional[torch.Tensor] = None) -> None:
     """out float32 [n, heads, rank] = causal softmax attention of qa over the cached vectors (one shared kv head whose
     values are the first `rank` entries of the cached vector).  With `out_head_major` (bfloat16 [heads, t_pad, rank]; the
-    tensor-core form only) the result goes there instead, rounded, for the grouped product that follows."""
+    tensor-core form only) the result goes there instead, rounded, for the grouped product that follows.  `q_head_major`
+    (bfloat16 [heads, t_pad, rank + rot]; the tensor-core form only): the queries, in place of float32 `qa`.  `window` > 0: a
+    query sees the last `window` positions up to its own."""
     lib = build.load("latent_attention")
     t_pad = 0
     if out_head_major is not None:
@@ -1288,14 +1416,21 @@ def latent_attention(out: Optional[torch.Tensor], qa: torch.Tensor, cache: torch
         t_pad = out_head_major.shape[1]
     elif out is None or out.dtype != torch.float32:
         raise KernelError("latent_attention: outputs are float32")
-    if qa.dtype != torch.float32:
+    tq_pad = 0
+    if q_head_major is not None:
+        if q_head_major.dtype != torch.bfloat16 or q_head_major.dim() != 3 or q_head_major.shape[0] != heads \
+                or q_head_major.shape[2] != rank + rot or not q_head_major.is_contiguous():
+            raise KernelError("latent_attention: head-major queries are contiguous bfloat16 [heads, t_pad, rank + rot]")
+        tq_pad = q_head_major.shape[1]
+    elif qa is None or qa.dtype != torch.float32:
         raise KernelError("latent_attention: queries are float32")
     if parts > 1 and (scratch is None or scratch.numel() < latent_attention_scratch_floats(n_tokens, heads, rank, parts)):
         raise KernelError("latent_attention: scratch too small")
     _check(lib, lib.llmk_latent_attention(_ptr(out), _ptr(qa), _ptr(cache), _ptr(block_tables), c_int(max_blocks), _ptr(ctx_len),
                                           _ptr(cu_q), _ptr(tile_seq), _ptr(tile_q0), c_int(tile_seq.numel()), c_int(n_tokens),
-                                          c_int(heads), c_int(rank), c_int(rot), c_int(page_size), c_float(scale), c_int(parts),
-                                          _ptr(scratch), _ptr(out_head_major), c_int(t_pad), c_int(dtype_code(cache.dtype)), _stream()),
+                                          c_int(heads), c_int(rank), c_int(rot), c_int(page_size), c_float(scale), c_int(window), c_int(parts),
+                                          _ptr(scratch), _ptr(out_head_major), c_int(t_pad), _ptr(q_head_major), c_int(tq_pad),
+                                          c_int(dtype_code(cache.dtype)), _stream()),
            2 if parts > 1 else 1)
 
 
@@ -1334,17 +1469,20 @@ def moe_max_tiles(n_slots: int, experts: int, tile: int = 0) -> int:
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, slot_expert: torch.Tensor, slot_weight: torch.Tensor, top: int,
-              scoring: str = "sigmoid", renormalize: bool = False, bias: Optional[torch.Tensor] = None) -> None:
+              scoring: str = "sigmoid", renormalize: bool = False, bias: Optional[torch.Tensor] = None,
+              choice_bias: Optional[torch.Tensor] = None, weight_scale: float = 1.0, sum_eps: float = 0.0) -> None:
     """Per row of h [n, K]: scores of router (float32 [E, K]) h (+ `bias`, float32 [E]), the `top` largest choose; slot
-    n * top + c receives (expert, score)."""
+    n * top + c receives (expert, score).  `choice_bias` (float32 [E]) is added to the scores for the choice alone;
+    `renormalize`: the weights are divided by the chosen scores' sum + `sum_eps`; they are then multiplied by `weight_scale`."""
     lib = build.load("moe")
     n, K = h.shape
     E = router.shape[0]
     if router.dtype != torch.float32 or slot_expert.dtype != torch.int32 or slot_weight.dtype != torch.float32 \
-            or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != E)):
+            or any(b is not None and (b.dtype != torch.float32 or b.numel() != E) for b in (bias, choice_bias)):
         raise KernelError("moe_route: router, bias and weights float32, experts int32")
     _check(lib, lib.llmk_moe_route(_ptr(h), c_longlong(_row_stride(h)), _ptr(router), _ptr(bias), _ptr(slot_expert), _ptr(slot_weight), c_int(n),
                                    c_int(K), c_int(E), c_int(top), c_int(ROUTER_SCORINGS[scoring]), c_int(1 if renormalize else 0),
+                                   _ptr(choice_bias), c_float(weight_scale), c_float(sum_eps),
                                    c_int(dtype_code(h.dtype)), _stream()))
 
 
@@ -1370,10 +1508,11 @@ def moe_gather(out: torch.Tensor, h: torch.Tensor, order: torch.Tensor, slot_wei
                                     c_int(K), c_int(1 if scale_rows else 0), c_int(dtype_code(out.dtype)), _stream()))
 
 
-def gemm_tc_grouped(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, real_rows: int = 0) -> None:
+def gemm_tc_grouped(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, real_rows: int = 0,
+                    activation: Optional[str] = None) -> None:
     """out[m] = a[m] @ w[g]^T where g = tile_group[m // 128] (int32 on the device; -1: the tile is skipped): a [M, K] with
     M a multiple of 128, w [groups, N, K] contiguous, both bfloat16; out [M, N] bfloat16 or float32 (csrc/gemm_tc.cu).
-    `real_rows`: how many rows hold data (for the profiler's count of the work; the kernel does not read it)."""
+    `activation` "relu2": relu(.)^2 of the product, in the epilogue (bfloat16 results).  `real_rows`: how many rows hold data (for the profiler's count of the work; the kernel does not read it)."""
     lib = build.load("gemm_tc")
     M, K = a.shape
     G, N, Kw = w.shape
@@ -1381,17 +1520,19 @@ def gemm_tc_grouped(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, tile_gr
         raise KernelError(f"gemm_tc_grouped: a{list(a.shape)} w{list(w.shape)} out{list(out.shape)} do not fit")
     if tile_group.dtype != torch.int32 or tile_group.numel() < M // MOE_GROUPED_TILE:
         raise KernelError("gemm_tc_grouped: one int32 group per tile of 128 rows")
+    if activation not in (None, "relu2"):
+        raise KernelError(f"gemm_tc_grouped: activation {activation!r} is not built")
     _check(lib, lib.llmk_gemm_tc_grouped(_ptr(out), _ptr(a), _ptr(w), c_int(M), c_int(N), c_int(K), c_longlong(_row_stride(a)),
                                          c_longlong(K), c_longlong(_row_stride(out)), c_int(G), _ptr(tile_group),
-                                         c_int(dtype_code(out.dtype)), _ptr(tc_error_flag(a.device)), c_int(1), _stream()))
+                                         c_int(1 if activation == "relu2" else 0), c_int(dtype_code(out.dtype)), _ptr(tc_error_flag(a.device)), c_int(1), _stream()))
 
 
 def moe_experts(out: torch.Tensor, x: torch.Tensor, w0: torch.Tensor, w1: Optional[torch.Tensor], order: torch.Tensor,
                 slot_weight: torch.Tensor, tile_expert: torch.Tensor, tile_start: torch.Tensor, tile_rows: torch.Tensor,
                 n_slots: int, top: int, first: bool, weight_on_input: bool, alpha: float = 1.0, limit: float = 0.0,
-                plain: bool = False) -> None:
+                plain: bool = False, relu2: bool = False) -> None:
     """first: out float32 [slots, ff] = gated activation of the rows' products with w0 = gate, w1 = up [E, ff, K]
-    (`plain`: silu(gate) * up instead of the clamped unit);
+    (`plain`: silu(gate) * up instead of the clamped unit; `relu2`: relu(.)^2 of the product with w0 = up, no w1);
     else out float32 [slots, K] = rows of x (float32 [slots, ff]) times w0 = down [E, K, ff]."""
     lib = build.load("moe")
     E, N, K = w0.shape
@@ -1400,7 +1541,7 @@ def moe_experts(out: torch.Tensor, x: torch.Tensor, w0: torch.Tensor, w1: Option
     _check(lib, lib.llmk_moe_experts(_ptr(out), _ptr(x), c_longlong(_row_stride(x)), _ptr(w0), _ptr(w1), _ptr(order), _ptr(slot_weight),
                                      _ptr(tile_expert), _ptr(tile_start), _ptr(tile_rows), c_int(n_slots), c_int(E), c_int(top),
                                      c_int(K), c_int(N), c_int(1 if first else 0), c_int(1 if weight_on_input else 0), c_float(alpha),
-                                     c_float(limit), c_int(1 if plain else 0), c_int(dtype_code(w0.dtype)), _stream()))
+                                     c_float(limit), c_int(2 if relu2 else 1 if plain else 0), c_int(dtype_code(w0.dtype)), _stream()))
 
 
 def moe_combine(out: torch.Tensor, rows: torch.Tensor, pos_of_slot: torch.Tensor, shared_out: Optional[torch.Tensor], top: int,

@@ -60,7 +60,12 @@ class GQAAttention(Mixer):
     are applied inside the attention kernels that take the steps of a layer that has any of them: in bfloat16 portions of
     prompts run on the tensor cores with float32 softmax weights (csrc/attention_mma.cu), single decoded tokens (their
     keys in parts), float32 and other sizes on the general kernel (csrc/attention.cu); the output projection's bias is
-    added to its result (or to the first of its slices)."""
+    added to its result (or to the first of its slices).
+
+    Values that are the projected keys (`values_from_keys`): a token's entry is cached once, as projected, and the inverse root
+    mean square of its row of keys beside it as one float32 (`KVRequest.token_scales`).  The key's norm is then a factor on the
+    token's scores and gains folded into the query's, so half the bytes are stored and read, and a tile of keys in shared memory
+    serves both products."""
 
     # what `prepare_step` adds depends on the lengths of the step's portions only, not on their
     # positions or requests: the engine may keep it across decode steps of one batch size
@@ -74,8 +79,10 @@ class GQAAttention(Mixer):
     def weight_decls(spec: AttentionSpec):
         qd, kd = spec.num_heads * spec.head_dim, spec.num_kv_heads * spec.head_dim
         vd, od = spec.num_kv_heads * spec.value_dim, spec.num_heads * spec.value_dim
-        decls = [WeightDecl(spec.q_proj, (qd, spec.hidden_size)), WeightDecl(spec.k_proj, (kd, spec.hidden_size)),
-                 WeightDecl(spec.v_proj, (vd, spec.hidden_size)), WeightDecl(spec.o_proj, (spec.hidden_size, od))]
+        decls = [WeightDecl(spec.q_proj, (qd, spec.hidden_size)), WeightDecl(spec.k_proj, (kd, spec.hidden_size))]
+        if not spec.values_from_keys:
+            decls.append(WeightDecl(spec.v_proj, (vd, spec.hidden_size)))
+        decls.append(WeightDecl(spec.o_proj, (spec.hidden_size, od)))
         for name, width in ((spec.q_bias, qd), (spec.k_bias, kd), (spec.v_bias, vd), (spec.o_bias, spec.hidden_size)):
             if name:
                 decls.append(WeightDecl(name, (width,), VECTOR))
@@ -101,13 +108,13 @@ class GQAAttention(Mixer):
         """True for a layer that only the general kernels take (see the class's last paragraph)."""
         return bool(spec.q_bias or spec.k_bias or spec.v_bias or spec.o_bias or spec.gate_proj or spec.sink or spec.softcap > 0
                     or spec.value_dim != spec.head_dim or spec.chunk or spec.unit_norm_eps is not None
-                    or spec.conv is not None or spec.row_norms or spec.rotate_values or spec.sink_scores or spec.gate_per_head
+                    or spec.conv is not None or spec.values_from_keys or spec.query_temperature is not None or spec.row_norms or spec.rotate_values or spec.sink_scores or spec.gate_per_head
                     or (spec.position is not None and getattr(spec.position, "pairing", "half") != "half"))
 
     def __init__(self, spec: AttentionSpec, weights, dtype, device):
         if spec.num_heads % spec.num_kv_heads != 0:
             raise ValueError(f"attention: {spec.num_heads} heads are not a multiple of {spec.num_kv_heads} kv heads")
-        if spec.head_dim % 2 != 0 or spec.head_dim > 512:
+        if (spec.head_dim % 2 != 0 and spec.position is not None) or spec.head_dim > 512:
             raise ValueError(f"attention: head_dim {spec.head_dim} must be even, at most 512")
         for n, heads in ((spec.q_norm, spec.num_heads), (spec.k_norm, spec.num_kv_heads)):
             if n is not None and spec.row_norms:
@@ -122,7 +129,7 @@ class GQAAttention(Mixer):
             raise ValueError(f"attention: the values' width {self.vd} must be at most 512")
         self.is_varied = self.varied(spec)
         # packed on the device: each matrix goes up through the loader's pinned stage as the file holds it
-        names = [spec.q_proj, spec.k_proj, spec.v_proj] + ([spec.gate_proj] if spec.gate_proj else [])
+        names = [spec.q_proj, spec.k_proj] + ([] if spec.values_from_keys else [spec.v_proj]) + ([spec.gate_proj] if spec.gate_proj else [])
         self.w_qkv = torch.cat([weights.device_tensor(n, dtype, device, keep=False) for n in names], dim=0).contiguous()
         self.w_q = self.w_qkv[: self.nq * self.hd]
         self.gate_off = (self.nq + self.nkv) * self.hd + self.nkv * self.vd if spec.gate_proj else -1
@@ -130,7 +137,7 @@ class GQAAttention(Mixer):
         self.w_q_gate = (torch.cat([self.w_q, self.w_qkv[self.gate_off:]], dim=0).contiguous() if spec.gate_proj else self.w_q)
         self.bias = None
         if spec.q_bias or spec.k_bias or spec.v_bias:
-            widths = (self.nq * self.hd, self.nkv * self.hd, self.nkv * self.vd)
+            widths = (self.nq * self.hd, self.nkv * self.hd, 0 if spec.values_from_keys else self.nkv * self.vd)
             self.bias = torch.cat([weights.device_tensor(n, dtype, device, keep=False) if n else
                                    torch.zeros(w, dtype=torch.float32, device=device)
                                    for n, w in zip((spec.q_bias, spec.k_bias, spec.v_bias), widths)]).contiguous()
@@ -173,7 +180,16 @@ class GQAAttention(Mixer):
                 raise ValueError("attention: rotated values are turned in half-split pairs by plain frequencies")
             self.value_position = build_position(RopeSpec(rotary_dim=self.vd, theta=spec.position.theta,
                                                           max_positions=spec.position.max_positions), weights, dtype, device)
-        if spec.row_norms and (spec.q_bias or spec.k_bias or spec.v_bias or spec.softcap > 0 or spec.chunk or spec.unit_norm_eps is not None
+        self.folded_gains = None
+        if spec.values_from_keys or spec.query_temperature is not None:
+            if not (spec.values_from_keys and spec.row_norms and spec.q_norm and spec.k_norm) or spec.position is not None or spec.conv is not None \
+                    or self.vd != self.hd or spec.v_bias or spec.gate_proj or spec.rotate_values:
+                raise ValueError("attention: values that are the keys (and a query temperature) come with norms over whole projections, and "
+                                 "without a position encoding, a convolution, a gate or a width of their own")
+            # the keys' gains act on the query: q . (k g) = (q g) . k, per key head that a query head reads
+            per_head = self.k_gain.view(self.nkv, 1, self.hd).expand(self.nkv, self.nq // self.nkv, self.hd)
+            self.folded_gains = (self.q_gain.view(self.nkv, -1, self.hd) * per_head).reshape(-1).contiguous()
+        elif spec.row_norms and (spec.q_bias or spec.k_bias or spec.v_bias or spec.softcap > 0 or spec.chunk or spec.unit_norm_eps is not None
                                or self.pairing != "half"):
             raise ValueError("attention: norms over whole projections exclude biases, a bound, a mask in blocks and other pairings")
         if (spec.sink_scores or spec.gate_per_head) and not spec.row_norms:
@@ -196,8 +212,9 @@ class GQAAttention(Mixer):
         # a mask in blocks of `chunk` positions never looks further back than chunk - 1 keys: its pages are a
         # window group's, given back as the blocks pass
         held = self.window or self.chunk
+        shared = self.spec.values_from_keys
         return KVRequest(WINDOW if held else FULL, held, self.nkv, self.hd,
-                         v_head_dim=self.vd if self.vd != self.hd else 0)
+                         v_head_dim=self.vd if self.vd != self.hd else 0, values=not shared, token_scales=shared)
 
     def state_request(self):
         # the convolution's last taps - 1 inputs over the channels of q, k and v side by side, oldest first
@@ -325,6 +342,8 @@ class GQAAttention(Mixer):
         """A layer with biases, another value width, a bound on the scores, a sink or a gate: the packed projection as
         an array (the gate's columns are read from it as they are), the general preparation and attention kernels."""
         T, ws = ctx.n_tokens, ctx.workspace
+        if self.spec.values_from_keys:
+            return self._forward_shared(ctx, x, cache, group)
         if self.row_norms:
             return self._forward_row_norms(ctx, x, cache, group, cos, sin, rot)
         w = self.w_qkv if cache.writes else self.w_q_gate
@@ -423,6 +442,40 @@ class GQAAttention(Mixer):
                                 positions=ctx.positions)
         if not inside:
             ops.unrotate_gate(o, gate if per_head else None, ctx.positions, vcos, vsin, nq, vd)
+        out = linear_sliced(ws, "mixer_out", o, self.w_o, self.dtype)
+        if self.o_bias is not None:
+            ops.add_bias(out, self.o_bias)
+        return out
+
+    def _forward_shared(self, ctx, x, cache, group):
+        """A layer whose values are its projected keys: the packed projection [q | k] (or its slices) -> one kernel for the biases,
+        both norms, the query's temperature and the write of the tokens' entries -> attention over entries that serve as keys
+        and values."""
+        T, ws, spec = ctx.n_tokens, ctx.workspace, self.spec
+        if not cache.writes:
+            raise ValueError("attention: a layer whose values are its keys writes its own cache")
+        nq, nk, hd = self.nq, self.nkv, self.hd
+        packed = linear_sliced(ws, "attn_qk", x, self.w_qkv, self.dtype)
+        q = ws.buffer("attn_q", T, nq * hd, self.dtype)
+        coef, every = spec.query_temperature if spec.query_temperature is not None else (0.0, 1.0)
+        ops.attn_prep_shared_rows(packed, self.bias, q, cache.k, cache.k_scale, ctx.positions, group.slots, self.folded_gains, nq, nk, hd,
+                                  cache.page_size, self.norm_eps, float(coef), float(every))
+        o = ws.buffer("attn_o", T, nq * hd, self.dtype)
+        mma_bq = 0 if ctx.pure_decode else self.mma_tile_queries()
+        if mma_bq and ctx.has_array(f"attention_tiles_bq{mma_bq}_seq"):
+            tile_seq = ctx.array(f"attention_tiles_bq{mma_bq}_seq")
+            ops.attention_mma(o, q, cache.k, None, group.block_tables, group.max_blocks, ctx.ctx_len, ctx.cu_q, tile_seq,
+                              ctx.array(f"attention_tiles_bq{mma_bq}_q0"), tile_seq.numel(), nq, nk, hd, hd, cache.page_size, self.window,
+                              float(spec.scale), softcap=self.softcap, sink=self.sink, sink_values=self.sink_scores, chunk=self.chunk,
+                              k_scale=cache.k_scale)
+        else:
+            tile_seq = ctx.array(self.tiles_name + "_seq")
+            parts, part_size = self._split(ctx)
+            scratch = ws.flat("attn_split", ops.attention_scratch_floats(T, nq, hd, parts), torch.float32) if parts > 1 else None
+            ops.paged_attention(o, q, q.stride(0), cache.k, None, group.block_tables, group.max_blocks, ctx.ctx_len, ctx.cu_q, tile_seq,
+                                ctx.array(self.tiles_name + "_q0"), tile_seq.numel(), T, nq, nk, hd, cache.page_size, self.window,
+                                float(spec.scale), parts, part_size, scratch, softcap=self.softcap, sink=self.sink, chunk=self.chunk,
+                                sink_values=self.sink_scores, k_scale=cache.k_scale)
         out = linear_sliced(ws, "mixer_out", o, self.w_o, self.dtype)
         if self.o_bias is not None:
             ops.add_bias(out, self.o_bias)

@@ -56,7 +56,7 @@ Block:
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Optional, Tuple
 
 import torch
@@ -71,12 +71,22 @@ class KVRequest:
     head_dim: int
     v_head_dim: int = 0      # width of a value where it differs from a key's (0: the same)
     values: bool = True      # False: one array per token only (a mixer that reads keys and values out of one entry)
+    token_scales: bool = False   # one float32 beside every cached token (`LayerCache.k_scale`)
 
     @property
     def value_dim(self) -> int:
         if not self.values:
             return 0
         return self.v_head_dim or self.head_dim
+
+    def shared_with(self, other: "KVRequest") -> Optional["KVRequest"]:
+        """What a cache that serves both requests has to offer: one geometry, and the pages of the wider view (every key, or the
+        larger window).  None: the geometries differ."""
+        if replace(self, group_kind=other.group_kind, window=other.window) != other:
+            return None
+        if self.group_kind != other.group_kind:
+            return self if not self.window else other
+        return self if self.window >= other.window else other
 
 
 @dataclass(frozen=True)
@@ -95,6 +105,7 @@ class LayerCache:
     page_size: int = 0
     writes: bool = True                     # False: read what another run item wrote
     state: Optional[torch.Tensor] = None    # [slots, *shape]
+    k_scale: Optional[torch.Tensor] = None  # float32 [pages, page_size] (KVRequest.token_scales)
 
 
 class Part:

@@ -8,7 +8,7 @@ from .registry import (build_feed_forward, build_mixer, build_norm, feed_forward
                        register_block)
 from ..kernels import ops
 from .parallel import finish_pair
-from .spec import INIT_EYE_PLUS_NORMAL, INIT_ONE_PLUS_NORMAL, VECTOR, MultiStreamBlockSpec, PostNormBlockSpec, PreNormBlockSpec, SandwichBlockSpec, WeightDecl
+from .spec import INIT_EYE_PLUS_NORMAL, INIT_ONE_PLUS_NORMAL, VECTOR, MultiStreamBlockSpec, ParallelBlockSpec, PostNormBlockSpec, PreNormBlockSpec, SandwichBlockSpec, WeightDecl
 
 
 class PreNormBlock(Part):
@@ -292,7 +292,68 @@ class MultiStreamBlock(Part):
         return None
 
 
+class ParallelBlock(Part):
+    """x <- x + a mixer(h) + b ffn(h), h = norm(x): the mixer and the feed-forward read one normed stream and join it together.
+
+    One kernel (`parallel_add`) ends a layer: it adds both results to the residual, each times its gain vector (the mixer's an
+    array or float32 slices, a routed feed-forward's still the rows of its experts), and writes the next layer's normed input in
+    the same pass (when the run list's next item is a block of this kind: the model names it in `ctx.next_block`).  A block whose
+    input nobody prepared norms it itself, which also finishes a sum the block before left open.  It hands on nothing to add."""
+
+    @staticmethod
+    def weight_decls(spec: ParallelBlockSpec):
+        H = spec.mixer_norm.dim
+        decls = norm_class(spec.mixer_norm).weight_decls(spec.mixer_norm) + mixer_class(spec.mixer).weight_decls(spec.mixer)
+        if spec.ffn is not None:
+            decls += feed_forward_class(spec.ffn).weight_decls(spec.ffn)
+        gains = (spec.mixer_gain, spec.ffn_gain if spec.ffn is not None else None)
+        return decls + [WeightDecl(g, (H,), VECTOR, INIT_ONE_PLUS_NORMAL) for g in gains if g]
+
+    @staticmethod
+    def kernel_modules(spec: ParallelBlockSpec):
+        mods = ("rowwise", "elementwise") + tuple(mixer_class(spec.mixer).kernel_modules(spec.mixer))
+        if spec.ffn is not None:
+            mods += tuple(feed_forward_class(spec.ffn).kernel_modules(spec.ffn))
+        return mods
+
+    def __init__(self, spec: ParallelBlockSpec, weights, dtype, device):
+        if spec.mixer_norm.kind != "rmsnorm" or spec.mixer_norm.weight_offset != 0.0:
+            raise ValueError("parallel block: its norm is a plain RMSNorm")
+        self.spec, self.dtype = spec, dtype
+        self.mixer_norm = build_norm(spec.mixer_norm, weights, dtype, device)
+        self.mixer = build_mixer(spec.mixer, weights, dtype, device)
+        self.ffn = build_feed_forward(spec.ffn, weights, dtype, device) if spec.ffn is not None else None
+        gain = lambda name: weights.device_tensor(name, dtype, device).contiguous() if name else None
+        self.mixer_gain, self.ffn_gain = gain(spec.mixer_gain), gain(spec.ffn_gain) if spec.ffn is not None else None
+        # a routed feed-forward hands over its experts' rows, which `parallel_add` weighs and adds up
+        self.takes_rows = spec.ffn is not None and getattr(spec.ffn, "kind", None) == "routed_mlp"
+
+    def workspace_bytes(self, tokens: int) -> int:
+        elem = 2 if self.dtype == torch.bfloat16 else 4
+        own = tokens * self.spec.mixer_norm.dim * elem
+        asks = [getattr(p, "workspace_bytes", None) for p in (self.mixer, self.ffn) if p is not None]
+        return own + sum(f(tokens) for f in asks if f is not None)        # both results are held at once
+
+    def forward(self, ctx, resid: torch.Tensor, delta, cache: LayerCache):
+        T, H = resid.shape
+        normed = ctx.workspace.buffer("block_normed", T, H, self.dtype)
+        if delta is not None or getattr(ctx, "normed_for", None) is not self:
+            self.mixer_norm.add_norm(resid, finish_pair(ctx, delta, self.dtype) if delta is not None else None, normed)
+        ctx.normed_for = None
+        follower = getattr(ctx, "next_block", None)
+        follow = follower.mixer_norm if isinstance(follower, ParallelBlock) else None
+        out = None
+        if self.ffn is not None:
+            out = self.ffn.forward(ctx, normed, combine=False) if self.takes_rows else self.ffn.forward(ctx, normed)
+        mixed = finish_pair(ctx, self.mixer.forward(ctx, normed, cache), self.dtype)
+        ops.parallel_add(resid, mixed, self.mixer_gain, out, self.ffn_gain, self.dtype, next_gain=follow.weight if follow is not None else None,
+                         eps=follow.eps if follow is not None else 0.0, normed=normed if follow is not None else None)
+        ctx.normed_for = follower if follow is not None else None
+        return None
+
+
 register_block("prenorm", PreNormBlock)
+register_block("parallel_block", ParallelBlock)
 register_block("multi_stream", MultiStreamBlock)
 register_block("sandwich", SandwichBlock)
 register_block("postnorm", PostNormBlock)

@@ -7,7 +7,7 @@ from ..kernels import ops
 from .base import FeedForward
 from .linear import GEMM_MODULES, linear, linear_sliced
 from .registry import register_feed_forward
-from .spec import VECTOR, ClampedExpertSpec, DenseMLPSpec, GatedExpertSpec, GatedMLPSpec, RoutedMLPSpec, WeightDecl
+from .spec import VECTOR, ClampedExpertSpec, DenseMLPSpec, GatedExpertSpec, GatedMLPSpec, PlainExpertSpec, RoutedMLPSpec, WeightDecl
 
 
 class DenseMLP(FeedForward):
@@ -45,6 +45,10 @@ class DenseMLP(FeedForward):
 
 def _expert_form(e):
     """(activation of `act_rows`, alpha, limit, plain gated unit?) of an expert's spec."""
+    if isinstance(e, PlainExpertSpec):
+        if e.activation != "relu2":
+            raise ValueError(f"routed feed-forward: expert activation {e.activation!r} is not supported")
+        return "relu2", 1.0, 0.0, False
     if isinstance(e, GatedExpertSpec):
         if e.activation != "silu":
             raise ValueError(f"routed feed-forward: expert activation {e.activation!r} is not supported")
@@ -53,8 +57,8 @@ def _expert_form(e):
 
 
 def _expert_decls(e, hidden: int):
-    return [WeightDecl(e.gate_proj, (e.intermediate_size, hidden)), WeightDecl(e.up_proj, (e.intermediate_size, hidden)),
-            WeightDecl(e.down_proj, (hidden, e.intermediate_size))]
+    gate = [] if isinstance(e, PlainExpertSpec) else [WeightDecl(e.gate_proj, (e.intermediate_size, hidden))]
+    return gate + [WeightDecl(e.up_proj, (e.intermediate_size, hidden)), WeightDecl(e.down_proj, (hidden, e.intermediate_size))]
 
 
 class RoutedMLP(FeedForward):
@@ -69,8 +73,11 @@ class RoutedMLP(FeedForward):
       bfloat16   tiles of 128 rows, every expert's rows starting on a tile: `moe_gather` copies the rows (times their
                  weights, where the weight is on the expert's input; else `moe_combine` applies it) into that order, and the grouped tensor-core product (`gemm_tc_grouped`: TMA, tcgen05.mma,
                  the expert of each tile read from the device) runs gate/up of all experts in one launch, the clamped
-                 gated activation follows row-wise, and a second grouped launch runs down
+                 gated activation follows row-wise (experts without a gate: relu squared in the product's epilogue), and a
+                 second grouped launch runs down
       float32    (and operands TMA refuses) tiles of 16 rows through `moe_experts`, float32 sums on the CUDA cores
+
+    A caller that adds the experts' rows up itself (`forward(..., combine=False)`) gets them as an `ops.RoutedRows`.
 
     The shared expert is two of the framework's own products with the same activation between them; a plain
     silu-gated one is the dense gated feed-forward's first half (`GatedMLP.hidden`: the activation in the product's
@@ -83,6 +90,8 @@ class RoutedMLP(FeedForward):
         decls = [WeightDecl(spec.router, (len(spec.experts), spec.hidden_size))]
         if spec.router_bias:
             decls.append(WeightDecl(spec.router_bias, (len(spec.experts),), VECTOR))
+        if spec.choice_bias:
+            decls.append(WeightDecl(spec.choice_bias, (len(spec.experts),), VECTOR))
         for e in spec.experts:
             decls += _expert_decls(e, spec.hidden_size)
         if spec.shared is not None:
@@ -106,16 +115,20 @@ class RoutedMLP(FeedForward):
         self.E, self.top, self.F = len(spec.experts), spec.top_k, first.intermediate_size
         self.router = weights.device_tensor(spec.router, torch.float32, device)      # routing is float32 in both dtypes
         self.router_bias = weights.device_tensor(spec.router_bias, dtype, device).contiguous() if spec.router_bias else None
+        self.choice_bias = weights.device_tensor(spec.choice_bias, dtype, device).contiguous() if spec.choice_bias else None
         self.act, self.alpha, self.limit, self.plain = _expert_form(first)
+        self.gateless = isinstance(first, PlainExpertSpec)
+        if isinstance(spec.shared, PlainExpertSpec):
+            raise ValueError("routed feed-forward: a shared expert without a gate is not supported")
         self.shared_form = _expert_form(spec.shared) if spec.shared is not None else None
         stack = lambda names: torch.stack([weights.device_tensor(n, dtype, device, keep=False) for n in names]).contiguous()
-        self.w_gate = stack([e.gate_proj for e in spec.experts])     # [E, F, H]
+        self.w_gate = None if self.gateless else stack([e.gate_proj for e in spec.experts])     # [E, F, H]
         self.w_up = stack([e.up_proj for e in spec.experts])         # [E, F, H]
         self.w_down = stack([e.down_proj for e in spec.experts])     # [E, H, F]
         # the tensor-core path reads gate and up as one matrix per expert, [E, 2F, H]: gate rows, then up rows
         H = spec.hidden_size
         self.grouped = dtype == torch.bfloat16 and H % 8 == 0 and self.F % 8 == 0
-        if self.grouped:
+        if self.grouped and not self.gateless:
             self.w_gate_up = torch.cat([self.w_gate, self.w_up], dim=1).contiguous()
             self.w_gate = self.w_up = None
         self.shared_gate_up = self.shared_down = self.shared_mlp = None
@@ -139,7 +152,7 @@ class RoutedMLP(FeedForward):
         rows = slots + ops.MOE_GROUPED_TILE * min(self.E, slots) if self.grouped else slots
         return rows * (3 * self.F + 2 * H) * 4 + tokens * H * 4 + shared + 16 * (rows + self.E) + 2 * ops.SLICED_PRODUCT_BYTES
 
-    def forward(self, ctx, x):
+    def forward(self, ctx, x, combine: bool = True):
         T, H = x.shape
         ws = ctx.workspace
         spec, top = self.spec, self.top
@@ -151,24 +164,33 @@ class RoutedMLP(FeedForward):
         slot_expert, pos_of_slot, order = ints[:n_slots], ints[n_slots:2 * n_slots], ints[2 * n_slots:2 * n_slots + n_rows]
         tile_expert, tile_start, tile_rows = (ints[2 * n_slots + n_rows + i * tiles:2 * n_slots + n_rows + (i + 1) * tiles] for i in range(3))
         slot_weight = ws.flat("moe_weights", n_slots, torch.float32)
-        ops.moe_route(x, self.router, slot_expert, slot_weight, top, spec.scoring, spec.renormalize, bias=self.router_bias)
+        ops.moe_route(x, self.router, slot_expert, slot_weight, top, spec.scoring, spec.renormalize, bias=self.router_bias,
+                      choice_bias=self.choice_bias, weight_scale=float(spec.weight_scale), sum_eps=float(spec.sum_eps))
         ops.moe_plan(slot_expert, n_slots, self.E, order, pos_of_slot, tile_expert, tile_start, tile_rows, tile=tile, padded=self.grouped)
         cap = (ws.default_rows * top // 128 + self.E) * 128 if self.grouped else ws.default_rows * top
         rows = ws.buffer("moe_rows", n_rows, H, torch.float32, capacity_rows=cap)
         if self.grouped:
             xs = ws.buffer("moe_in", n_rows, H, self.dtype, capacity_rows=cap)
             ops.moe_gather(xs, x, order, slot_weight, top, scale_rows=spec.weight_on_input)
-            gate_up = ws.buffer("moe_gate_up", n_rows, 2 * self.F, self.dtype, capacity_rows=cap)
-            ops.gemm_tc_grouped(gate_up, xs, self.w_gate_up, tile_expert, real_rows=n_slots)
             y = ws.buffer("moe_act", n_rows, self.F, self.dtype, capacity_rows=cap)
-            ops.act_rows(y, gate_up, self.act, alpha=self.alpha, limit=self.limit)
+            if self.gateless:
+                ops.gemm_tc_grouped(y, xs, self.w_up, tile_expert, real_rows=n_slots, activation="relu2")
+            else:
+                gate_up = ws.buffer("moe_gate_up", n_rows, 2 * self.F, self.dtype, capacity_rows=cap)
+                ops.gemm_tc_grouped(gate_up, xs, self.w_gate_up, tile_expert, real_rows=n_slots)
+                ops.act_rows(y, gate_up, self.act, alpha=self.alpha, limit=self.limit)
             ops.gemm_tc_grouped(rows, y, self.w_down, tile_expert, real_rows=n_slots)
         else:
             y = ws.buffer("moe_act", n_rows, self.F, torch.float32, capacity_rows=cap)
-            ops.moe_experts(y, x, self.w_gate, self.w_up, order, slot_weight, tile_expert, tile_start, tile_rows, n_slots, top,
-                            first=True, weight_on_input=spec.weight_on_input, alpha=self.alpha, limit=self.limit, plain=self.plain)
+            first = (self.w_up, None) if self.gateless else (self.w_gate, self.w_up)
+            ops.moe_experts(y, x, *first, order, slot_weight, tile_expert, tile_start, tile_rows, n_slots, top, first=True,
+                            weight_on_input=spec.weight_on_input, alpha=self.alpha, limit=self.limit, plain=self.plain, relu2=self.gateless)
             ops.moe_experts(rows, y, self.w_down, None, order, slot_weight, tile_expert, tile_start, tile_rows, n_slots, top,
                             first=False, weight_on_input=spec.weight_on_input)
+        # the grouped products leave an expert's plain output: a weight on the output is applied as the rows are added
+        late_weight = slot_weight if self.grouped and not spec.weight_on_input else None
+        if not combine and spec.shared is None:
+            return ops.RoutedRows(rows, pos_of_slot, late_weight, top)
         shared_out = None
         if self.shared_mlp is not None:
             shared_out = linear(self.shared_mlp.hidden(ctx, x), self.shared_mlp.w_down, ws.buffer("moe_shared_out", T, H, self.dtype))
@@ -179,9 +201,7 @@ class RoutedMLP(FeedForward):
             ops.act_rows(act, gate_up, self.shared_form[0], alpha=self.shared_form[1], limit=self.shared_form[2])
             shared_out = linear(act, self.shared_down, ws.buffer("moe_shared_out", T, H, self.dtype))
         out = ws.flat("moe_out", T * H, torch.float32).view(1, T, H)
-        # the grouped products leave an expert's plain output: a weight on the output is applied as the rows are added
-        ops.moe_combine(out[0], rows, pos_of_slot, shared_out, top,
-                        slot_weight=slot_weight if self.grouped and not spec.weight_on_input else None)
+        ops.moe_combine(out[0], rows, pos_of_slot, shared_out, top, slot_weight=late_weight)
         return ops.Partials(out)
 
 

@@ -67,6 +67,11 @@ class RopeSpec:
     # l = 2 pi / f, f stays where l < original / high, becomes f / factor where l > original / low, and between the two
     # (1 - s) f / factor + s f with s = (original / l - low) / (high - low).  None: the plain frequencies.
     scaling: Optional[Tuple[float, float, float, float]] = None
+    # Frequencies scaled by the pair's place (YaRN), (factor, original, fast, slow): with
+    # place(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(place(fast)), 0) and
+    # hi = min(ceil(place(slow)), rotary_dim - 1), pair i turns at f_i (1 - r) + (f_i / factor) r, r = clamp((i - lo) / max(hi - lo, 0.001), 0, 1);
+    # cos and sin are multiplied by 0.1 ln(factor) + 1.
+    yarn: Optional[Tuple[float, float, float, float]] = None
     kind: str = "rope"
 
 
@@ -128,6 +133,12 @@ class AttentionSpec:
     rotate_values: bool = False
     sink_scores: Optional[str] = None
     gate_per_head: bool = False
+    # `values_from_keys`: there is no `v_proj`; a token's values are its projected keys (bias included) before their norm.  The
+    # cache then holds the projected keys once, and the inverse root mean square of each token's row of them beside.
+    # `query_temperature` (coef, every): the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
+    # Both come with `row_norms`, without a position encoding.
+    values_from_keys: bool = False
+    query_temperature: Optional[Tuple[float, float]] = None
     kind: str = "attention"
 
     @property
@@ -163,11 +174,14 @@ class LinearAttentionSpec:
 class LatentAttentionSpec:
     """Causal softmax attention whose keys and values are expanded from a cached latent vector per token.
 
-    Queries through a latent of their own: cq = norm(x Wdq^T), q = cq Wuq^T, per head [nope_dim | rope_dim].
+    Queries through a latent of their own: cq = norm(x Wdq^T), q = cq Wuq^T, per head [nope_dim | rope_dim]; or straight
+    from the stream, q = x Wq^T (`q_proj`; then `q_rank` is 0 and there is no `dq_proj`, `uq_proj`, `q_norm`).
     x Wdkv^T has kv_rank + rope_dim values: the first kv_rank, normed, are the latent c; the last rope_dim are one
     rotated key part shared by all heads.  Head h: key [Wuk_h c | rotated part], value Wuv_h c (value_dim);
     score = (q . key) * scale.  The heads side by side are multiplied by sigmoid(x Wg^T) (`gate_proj`, optional) and
     projected by Wo.  Only [c | rotated part] is cached (one shared entry of kv_rank + rope_dim values per token).
+    Without `dkv_proj` (and `kv_norm`) the layer makes no entries: its run items read another layer's (`writes_cache=False`).
+    `window`: a query sees the last `window` positions up to its own (None: all of them).
     """
     hidden_size: int
     num_heads: int
@@ -177,16 +191,18 @@ class LatentAttentionSpec:
     q_rank: int
     kv_rank: int
     scale: float
-    dq_proj: str
-    uq_proj: str
-    dkv_proj: str
+    dq_proj: Optional[str]
+    uq_proj: Optional[str]
+    dkv_proj: Optional[str]
     uk_proj: str
     uv_proj: str
     o_proj: str
-    q_norm: RMSNormSpec
-    kv_norm: RMSNormSpec
+    q_norm: Optional[RMSNormSpec]
+    kv_norm: Optional[RMSNormSpec]
     position: Optional[RopeSpec] = None
     gate_proj: Optional[str] = None
+    q_proj: Optional[str] = None
+    window: Optional[int] = None
     # fold Wuk into the query's up-projection when the model is loaded (one product straight into the latent space
     # instead of a product and a per-head product); False keeps the two matrices apart
     absorb_at_load: bool = True
@@ -446,12 +462,23 @@ class GatedExpertSpec:
 
 
 @dataclass(frozen=True)
+class PlainExpertSpec:
+    """One small feed-forward without a gate: act(x Wup^T) Wdown^T, act = relu(.)^2; no biases."""
+    intermediate_size: int
+    up_proj: str
+    down_proj: str
+    activation: str = "relu2"
+
+
+@dataclass(frozen=True)
 class RoutedMLPSpec:
     """Mixture of experts: router scores s = sigmoid(x Wr^T + b) (or softmax) in float32, the `top_k` largest choose
     experts, their scores are the weights (renormalised over the chosen ones if `renormalize`); with scoring
     "softmax_top" the logits themselves choose and the weights are the softmax over the chosen logits alone.  The weight
     multiplies the expert's input (`weight_on_input`) or its output.  An optional shared expert runs for every token and
-    is added.  Experts are `ClampedExpertSpec` or `GatedExpertSpec`, all routed ones of one kind and size."""
+    is added.  Experts are `ClampedExpertSpec`, `GatedExpertSpec` or `PlainExpertSpec`, all routed ones of one kind and size.
+    `choice_bias`: name of a vector per expert added to the scores for the choice alone, not for the weights.  The weights
+    are multiplied by `weight_scale`; renormalised ones are divided by the chosen scores' sum + `sum_eps`."""
     hidden_size: int
     router: str
     experts: Tuple[object, ...]
@@ -461,6 +488,9 @@ class RoutedMLPSpec:
     renormalize: bool = False
     weight_on_input: bool = True
     router_bias: Optional[str] = None
+    choice_bias: Optional[str] = None
+    weight_scale: float = 1.0
+    sum_eps: float = 0.0
     kind: str = "routed_mlp"
 
 
@@ -517,6 +547,18 @@ class SandwichBlockSpec:
     ffn: Optional[object] = None
     ffn_out_norm: Optional[object] = None
     kind: str = "sandwich"
+
+
+@dataclass(frozen=True)
+class ParallelBlockSpec:
+    """x <- x + a mixer(h) + b ffn(h) with h = norm(x): both sublayers read one normed stream and join it together, each
+    multiplied element by element by a gain vector (`mixer_gain`, `ffn_gain`: tensor names; None: as it is).  `ffn` may be None."""
+    mixer_norm: object
+    mixer: object
+    ffn: Optional[object] = None
+    mixer_gain: Optional[str] = None
+    ffn_gain: Optional[str] = None
+    kind: str = "parallel_block"
 
 
 @dataclass(frozen=True)
