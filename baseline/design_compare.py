@@ -1,13 +1,15 @@
-"""`bench.py --designs`: Derupel (or, with `--designs-family sarulix`, `fonuvik` or `nasozen`, that design) beside Qwen3 at equal
-layer sizes, random weights, one B200; `--designs-beside` names another design to stand beside it (Nasozen stands beside
-Fonuvik, the closest model, unless told otherwise).
+"""`bench.py --designs`: Derupel (or, with `--designs-family sarulix`, `fonuvik`, `nasozen` or `zuvasun`, that design) beside Qwen3 at
+equal layer sizes, random weights, one B200; `--designs-beside` names another design to stand beside it (Nasozen stands beside
+Fonuvik and Zuvasun beside Derupel, the closest models, unless told otherwise).
 
 For each size two models are built: a Derupel whose layers alternate its two mixers and its two feed-forwards (a Sarulix
 whose four layers are a recurrent unit, the delta rule, attention and a recurrent unit again, each with a feed-forward,
 entered once through its loop's mixing step; a Fonuvik whose layers alternate the parallel mixer and the token-shift
 mixer, each with a routed feed-forward whose chosen and shared experts together are as wide as the dense one; a Nasozen of
 four residual streams whose layers are the parallel mixer, the generalized delta rule, the parallel mixer and the matrix
-memory under a running maximum, three with a routed feed-forward and one with a dense one), and the
+memory under a running maximum, three with a routed feed-forward and one with a dense one; a Zuvasun whose layers are attention
+over every key, latent attention under a window, latent attention that reads the entries of the layer before it, and attention
+again, each with a routed feed-forward beside it), and the
 Qwen3 of the same width, depth, feed-forward width and vocabulary.
 Measured for both:
 
@@ -91,9 +93,25 @@ def nasozen_config(s: dict) -> dict:
             "layers": layers, "max_positions": CONTEXT}
 
 
-FAMILIES = {"derupel": derupel_config, "sarulix": sarulix_config, "fonuvik": fonuvik_config, "nasozen": nasozen_config}
+def zuvasun_config(s: dict) -> dict:
+    heads, hd = s["heads"], s["hd"]
+    routed = {"kind": "moe", "router": {"experts": s["experts"], "top": s["top"], "scale": 2.0}, "expert": {"ff": s["expert_ff"]}}
+    att = {"heads": heads, "kv_heads": max(1, heads // 2), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "q_temp": {"coef": 0.1, "every": 1024}}
+    latent = {"heads": heads, "dim": hd, "rot_dim": s["rot"], "vdim": hd, "kv_rank": s["kv_rank"], "scale": (hd + s["rot"]) ** -0.5,
+              "mask": {"size": 1024}, "rot": {"base": 10000.0, "dims": s["rot"],
+                                              "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    layers = []
+    for i in range(s["layers"]):
+        kind = "attention" if i % 4 in (0, 3) else "latent_attention"
+        mixer = att if kind == "attention" else latent if i % 4 == 1 else dict(latent, kv_from=i - 1)
+        layers.append({"type": kind, "mixer": mixer, "mlp": routed})
+    return {"architecture": "Zuvasun", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "layers": layers, "max_positions": CONTEXT}
+
+
+FAMILIES = {"derupel": derupel_config, "sarulix": sarulix_config, "fonuvik": fonuvik_config, "nasozen": nasozen_config,
+            "zuvasun": zuvasun_config}
 # the design that stands beside a family's where it is not Qwen3: the framework's closest model
-BESIDE = {"nasozen": "fonuvik"}
+BESIDE = {"nasozen": "fonuvik", "zuvasun": "derupel"}
 
 
 def qwen3_config(s: dict) -> dict:

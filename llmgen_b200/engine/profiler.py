@@ -133,6 +133,7 @@ class AttentionTerm:
     q_dim: int                  # query heads x head size
     kv_dim: int                 # key/value heads x head size
     window: int                 # 0: every key
+    stores: bool = True         # False: the item reads what another one cached
 
 
 @dataclass(frozen=True)
@@ -160,12 +161,14 @@ class ModelCost:
             if kind == "attention":
                 q_dim, kv_dim = mixer.num_heads * mixer.head_dim, mixer.num_kv_heads * mixer.head_dim
                 v_dim, o_dim = mixer.num_kv_heads * mixer.value_dim, mixer.num_heads * mixer.value_dim
+                if getattr(mixer, "values_from_keys", False):
+                    v_dim = 0                               # one entry is key and value
                 n_mm += mixer.hidden_size * (q_dim + o_dim)
                 if writes_cache:                            # an item that reads another's cache projects no k, v
                     n_mm += mixer.hidden_size * (kv_dim + v_dim)
                 if mixer.gate_proj:
                     n_mm += mixer.hidden_size * (mixer.num_heads if getattr(mixer, "gate_per_head", False) else o_dim)
-                terms.append(AttentionTerm((q_dim + o_dim) // 2, (kv_dim + v_dim) // 2, int(mixer.window or 0)))
+                terms.append(AttentionTerm((q_dim + o_dim) // 2, (kv_dim + v_dim) // 2, int(mixer.window or 0), writes_cache))
             elif kind == "linear_attention":
                 kd, vd = mixer.num_heads * mixer.key_dim, mixer.num_heads * mixer.value_dim
                 n_mm += mixer.hidden_size * (2 * kd + (3 if mixer.gate_proj else 2) * vd)
@@ -173,13 +176,16 @@ class ModelCost:
                 state_bytes += 4 * mixer.num_heads * mixer.key_dim * mixer.value_dim
             elif kind == "latent_attention":
                 n, za = mixer.num_heads, mixer.kv_rank + mixer.rope_dim
-                n_mm += mixer.hidden_size * (mixer.q_rank + za + (2 if mixer.gate_proj else 1) * n * mixer.value_dim)
-                if getattr(mixer, "absorb_at_load", False):     # the query goes straight into the latent space
+                entries = za if getattr(mixer, "dkv_proj", None) else 0
+                n_mm += mixer.hidden_size * (mixer.q_rank + entries + (2 if mixer.gate_proj else 1) * n * mixer.value_dim)
+                if getattr(mixer, "q_proj", None):              # queries straight from the stream
+                    n_mm += mixer.hidden_size * n * (mixer.nope_dim + mixer.rope_dim) + n * mixer.kv_rank * (mixer.nope_dim + mixer.value_dim)
+                elif getattr(mixer, "absorb_at_load", False):     # the query goes straight into the latent space
                     n_mm += mixer.q_rank * n * za + n * mixer.kv_rank * mixer.value_dim
                 else:
                     n_mm += mixer.q_rank * n * (mixer.nope_dim + mixer.rope_dim) + n * mixer.kv_rank * (mixer.nope_dim + mixer.value_dim)
                 # one shared entry of kv_rank + rope_dim values per token; per key and head 2 (za + kv_rank) flops
-                terms.append(AttentionTerm(n * (za + mixer.kv_rank) // 2, (za + 1) // 2, 0))
+                terms.append(AttentionTerm(n * (za + mixer.kv_rank) // 2, (za + 1) // 2, int(getattr(mixer, "window", None) or 0), writes_cache))
             elif kind == "parallel":
                 return all([count(b, writes_cache) for b in mixer.branches])
             elif kind == "min_gru":
@@ -211,7 +217,8 @@ class ModelCost:
                 n_mm += 2 * ffn.hidden_size * ffn.intermediate_size
             elif getattr(ffn, "kind", None) == "routed_mlp":
                 # what one token uses: the router, its chosen experts and the shared one
-                n_mm += ffn.hidden_size * (len(ffn.experts) + 3 * ffn.top_k * ffn.experts[0].intermediate_size)
+                matrices = 3 if getattr(ffn.experts[0], "gate_proj", None) else 2
+                n_mm += ffn.hidden_size * (len(ffn.experts) + matrices * ffn.top_k * ffn.experts[0].intermediate_size)
                 if ffn.shared is not None:
                     n_mm += 3 * ffn.hidden_size * ffn.shared.intermediate_size
             elif ffn is not None:
@@ -230,7 +237,7 @@ class ModelCost:
         return below * first_ctx + below * (below - 1) // 2 + (n - below) * window
 
     def kv_bytes_per_token(self) -> int:
-        return sum(2 * t.kv_dim * self.kv_elem for t in self.attention)
+        return sum(2 * t.kv_dim * self.kv_elem for t in self.attention if t.stores)
 
     def prefill_flops(self, p: int, logits_rows: int = 1) -> int:
         """A prompt of p tokens under the causal mask, the output projection on `logits_rows` rows
@@ -327,9 +334,10 @@ def _cost_attention(a, info: PassInfo) -> Tuple[int, int]:
     elem = a["kcache"].element_size()
     tokens = sum(info.q_lens)
     vd = int(a.get("vd") or 0) or hd                       # values of their own width
+    entry = hd if a.get("k_scale") is not None else hd + vd    # one entry that is key and value
     block = int(a.get("chunk") or 0)                       # a mask in blocks: only the own block's keys are seen and read
     flops = 2 * nq * (hd + vd) * (info.visible_keys_in_blocks(block) if block else info.visible_keys(window))
-    bytes_ = nkv * (hd + vd) * elem * (info.keys_read_in_blocks(block) if block else info.keys_read(window)) + tokens * nq * (hd + vd) * elem
+    bytes_ = nkv * entry * elem * (info.keys_read_in_blocks(block) if block else info.keys_read(window)) + tokens * nq * (hd + vd) * elem
     packed = a.get("packed")
     if packed is not None:                                 # the kernel also reads the projection and stores k, v
         bytes_ += _nbytes(packed) + 2 * tokens * int(a.get("nk") or 0) * hd * elem
@@ -465,14 +473,38 @@ def _cost_scaled_sum(a, info: PassInfo) -> Tuple[int, int]:
 def _cost_latent_attention(a, info: PassInfo) -> Tuple[int, int]:
     heads, rank, rot = int(a["heads"]), int(a["rank"]), int(a["rot"])
     tokens = sum(info.q_lens)
-    flops = 2 * heads * (2 * rank + rot) * info.visible_keys(0)
-    bytes_ = (rank + rot) * a["cache"].element_size() * info.keys_read(0) + tokens * heads * (2 * rank + rot) * 4
+    window = int(a.get("window") or 0)
+    flops = 2 * heads * (2 * rank + rot) * info.visible_keys(window)
+    q_elem = 2 if a.get("q_head_major") is not None else 4
+    o_elem = 2 if a.get("out_head_major") is not None else 4
+    bytes_ = (rank + rot) * a["cache"].element_size() * info.keys_read(window) + tokens * heads * ((rank + rot) * q_elem + rank * o_elem)
     return flops, bytes_
 
 
 def _cost_latent_absorb(a, info: PassInfo) -> Tuple[int, int]:
-    n = int(a["q"].shape[0])
-    return 2 * n * int(a["heads"]) * int(a["dim"]) * int(a["rank"]), _nbytes(a["q"]) + _nbytes(a["qa"]) + _nbytes(a["wuk"])
+    n, heads, dim, rank, rot = int(a["q"].shape[0]), int(a["heads"]), int(a["dim"]), int(a["rank"]), int(a["rot"])
+    elem = a["q"].element_size()
+    entries = 2 * n * (rank + rot) * elem if a.get("cache") is not None else 0
+    return 2 * n * heads * dim * rank, n * heads * (dim + rot) * elem + _nbytes(a["qa"]) + _nbytes(a["wuk"]) + entries
+
+
+def _cost_latent_query_split(a, info: PassInfo) -> Tuple[int, int]:
+    n, heads, dim, rank, rot = int(a["packed"].shape[0]), int(a["heads"]), int(a["dim"]), int(a["rank"]), int(a["rot"])
+    moved = heads * (dim + rot) + (rank + rot if a.get("cache") is not None else 0)
+    return 3 * n * heads * rot, 2 * n * moved * a["packed"].element_size() + n * rot * 4
+
+
+def _cost_attn_prep_shared_rows(a, info: PassInfo) -> Tuple[int, int]:
+    q = a["q_out"]
+    n, nq, nk, hd = int(q.shape[0]), int(a["nq"]), int(a["nk"]), int(a["hd"])
+    return 5 * n * (nq + nk) * hd, _nbytes(a["x"]) + n * (nq + nk) * hd * q.element_size()
+
+
+def _cost_parallel_add(a, info: PassInfo) -> Tuple[int, int]:
+    resid, second = a["resid"], a.get("second")
+    routed = getattr(second, "pos_of_slot", None)
+    read = routed.numel() * int(resid.shape[1]) * 4 if routed is not None else _nbytes(second)     # the chosen experts' rows
+    return 9 * resid.numel(), 2 * _nbytes(resid) + _nbytes(a["first"]) + read + _nbytes(a.get("normed"))
 
 
 def _cost_latent_expand(a, info: PassInfo) -> Tuple[int, int]:
@@ -532,6 +564,7 @@ OP_COSTS: Dict[str, Callable] = {
     "stream_step": _cost_stream_step, "stream_spread": _cost_in_place, "attn_prep_rows": _cost_attn_prep_rows,
     "unrotate_gate": _cost_in_place, "min_gru": _cost_min_gru, "mlstm_gates": _cost_mlstm_gates,
     "delta_rule_prep": _cost_delta_rule_prep, "memory_scan": _cost_memory_scan,
+    "attn_prep_shared_rows": _cost_attn_prep_shared_rows, "latent_split": _cost_latent_query_split, "parallel_add": _cost_parallel_add,
 }
 
 

@@ -32,13 +32,15 @@ def _layer_body(spec, item) -> str:
     parts = []
     if getattr(mixer, "kind", None) == "attention":
         reach = f"window {mixer.window}" if mixer.window else "all keys"
-        parts.append(f"attention {mixer.num_heads}/{mixer.num_kv_heads} heads x {mixer.head_dim}, {reach}")
+        parts.append(f"attention {mixer.num_heads}/{mixer.num_kv_heads} heads x {mixer.head_dim}, {reach}"
+                     + (", the keys are the values" if mixer.values_from_keys else ""))
     elif getattr(mixer, "kind", None) == "linear_attention":
         parts.append(f"linear attention {mixer.num_heads} heads x {mixer.key_dim}/{mixer.value_dim}, a decay per head, "
                      f"state {_size(4 * mixer.num_heads * mixer.key_dim * mixer.value_dim)} a request")
     elif getattr(mixer, "kind", None) == "latent_attention":
         parts.append(f"latent attention {mixer.num_heads} heads x {mixer.nope_dim}+{mixer.rope_dim}/{mixer.value_dim}, "
-                     f"latents {mixer.q_rank}/{mixer.kv_rank}, {mixer.kv_rank + mixer.rope_dim} cached values a token")
+                     + (f"latents {mixer.q_rank}/{mixer.kv_rank}, " if mixer.q_rank else f"latent {mixer.kv_rank}, ")
+                     + (f"window {mixer.window}, " if mixer.window else "") + f"{mixer.kv_rank + mixer.rope_dim} cached values a token")
     elif mixer is not None:
         parts.append(f"mixer '{getattr(mixer, 'kind', '?')}'")
     if getattr(ffn, "kind", None) == "gated_mlp":

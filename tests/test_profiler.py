@@ -292,7 +292,10 @@ def test_every_listed_binding_exists_with_the_operands_its_cost_reads():
              pf._cost_attn_prep_rows: [("x",), ("q_out",), ("nq",), ("nk",), ("hd",), ("vd",), ("rot",)],
              pf._cost_memory_scan: [("heads",), ("dim",), ("vdim",), ("form",), ("r",), ("aux",), ("dots",), ("out",)],
              pf._cost_min_gru: [("out",), ("zxg",)], pf._cost_delta_rule_prep: [("r",), ("heads",), ("dim",), ("aux",), ("dots",)],
-             pf._cost_mlstm_gates: [("q",), ("heads",), ("dim",), ("gates",)]}
+             pf._cost_mlstm_gates: [("q",), ("heads",), ("dim",), ("gates",)],
+             pf._cost_attn_prep_shared_rows: [("x",), ("q_out",), ("nq",), ("nk",), ("hd",)],
+             pf._cost_latent_query_split: [("packed",), ("heads",), ("dim",), ("rank",), ("rot",), ("cache",)],
+             pf._cost_parallel_add: [("resid",), ("first",), ("second",), ("normed",)]}
     for name, cost in pf.OP_COSTS.items():
         params = inspect.signature(getattr(ops, name)).parameters
         for alternatives in needs[cost]:
