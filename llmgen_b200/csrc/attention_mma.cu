@@ -15,6 +15,11 @@
 // Entries that are key and value at once (SHARED: `k_scale`, a factor on the scores per cached token; no value array): a tile of
 // keys is copied once and serves both products, its tokens' factors beside it.
 // Taken: key width and value width 64 or 128 each.
+//
+// `attention_mma_parts` is the same arithmetic for steps of single tokens: the rows of a block are the query heads of one key head
+// (up to 16), its keys one part of what the token sees; four warps take 16 keys each of a tile of 64, with a softmax of their own
+// that is merged at the end, and the blocks of one (token, key head) are a cluster that merges the parts through each other's
+// shared memory, in part order.  No gate and no turn back there.
 #define LLMK_MODULE_NAME "attention_mma"
 #include "common.cuh"
 
@@ -66,6 +71,8 @@ __device__ __forceinline__ void cp_async4(void* smem_dst, const void* src) {
     const uint32_t d = (uint32_t)__cvta_generic_to_shared(smem_dst);
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
 }
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_wait_but_one() { asm volatile("cp.async.wait_group 1;" ::: "memory"); }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 // tanh(x) = 1 - 2 / (1 + e^(2x)): an absolute error of a few 1e-7, which is what a score needs (it is an exponent)
 __device__ __forceinline__ float tanh_abs(float x) { return 1.0f - __fdividef(2.0f, 1.0f + exp2f(x * 2.8853900817779268f)); }
@@ -315,6 +322,263 @@ int launch(const Params& p, dim3 grid, cudaStream_t s) {
     return LLMK_OK;
 }
 
+// ------------------------------------------------------------------------------------- single tokens, keys in parts
+constexpr int PROWS = 16;
+
+template <int HD, int VD, bool SHARED>
+struct PartsSmem {
+    static constexpr int QLD = HD + 8, VLD = VD + 8, OLD = VD + 4;
+    static constexpr size_t Q = (size_t)PROWS * QLD * sizeof(bf16);
+    static constexpr size_t KV = ((size_t)2 * BN * QLD + (SHARED ? 0 : (size_t)2 * BN * VLD)) * sizeof(bf16);
+    static constexpr size_t FACTORS = SHARED ? 2 * BN * sizeof(float) : 0;
+    static constexpr size_t OUT = ((size_t)PROWS * OLD + 2 * PROWS + 2 * WARPS * PROWS) * sizeof(float);
+    static constexpr size_t TOTAL = Q + KV + FACTORS + OUT;
+};
+
+template <int HD, int VD, bool SHARED>
+__global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params p, int gc, int chunks, int parts) {
+    using L = PartsSmem<HD, VD, SHARED>;
+    constexpr int QLD = L::QLD, VLD = SHARED ? L::QLD : L::VLD, OLD = L::OLD;
+    static_assert(!SHARED || HD == VD, "keys that are values have one width");
+    extern __shared__ __align__(16) uint8_t smem_raw[];
+    bf16* Qs = reinterpret_cast<bf16*>(smem_raw);
+    bf16* Kbuf = Qs + PROWS * QLD;
+    bf16* Vbuf = SHARED ? Kbuf : Kbuf + 2 * BN * QLD;
+    float* Sbuf = reinterpret_cast<float*>(smem_raw + L::Q + L::KV);
+    float* Os = reinterpret_cast<float*>(smem_raw + L::Q + L::KV + L::FACTORS);      // [PROWS][OLD]
+    float* Ml = Os + PROWS * OLD;                                                    // [PROWS] maxima, [PROWS] sums
+    float* Wm = Ml + 2 * PROWS;                                                      // [WARPS][PROWS]
+    float* Wl = Wm + WARPS * PROWS;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int g = lane >> 2, tq = lane & 3;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int s = blockIdx.x, part = blockIdx.z;
+    const int G = p.nq / p.nkv;
+    const int kvh = blockIdx.y / chunks, chunk = blockIdx.y % chunks;
+    const int heads = min(gc, G - chunk * gc);                  // rows of this block
+    const int head0 = kvh * G + chunk * gc;
+    const int q_beg = p.cu_q[s], q_len = p.cu_q[s + 1] - q_beg, ctx = p.ctx_len[s];
+    const bool live = q_len == 1 && ctx >= 1;
+    const int qpos = ctx - 1;
+    int k_beg = 0, k_end = 0;
+    if (live) {
+        int first = p.window > 0 ? max(0, qpos - p.window + 1) : 0;
+        if (p.chunk > 0) first = max(first, qpos / p.chunk * p.chunk);
+        const int size = ceil_div(ceil_div(qpos + 1 - first, parts), BN) * BN;       // whole tiles a part
+        k_beg = first + part * size;
+        k_end = min(qpos + 1, k_beg + size);
+    }
+    const int* bt = p.block_tables + (size_t)s * p.max_blocks;
+
+    constexpr int VECS = HD / 8 + (SHARED ? 0 : VD / 8);
+    auto load_tile = [&](int t0, int buf) {
+        bf16* Kd = Kbuf + buf * BN * QLD;
+        bf16* Vd = Vbuf + buf * BN * VLD;
+#pragma unroll 4
+        for (int idx = threadIdx.x; idx < BN * VECS; idx += WARPS * 32) {
+            const int key = idx / VECS, v = idx % VECS;
+            const int kpos = t0 + key;
+            bf16* dst = v < HD / 8 ? Kd + key * QLD + v * 8 : Vd + key * VLD + (v - HD / 8) * 8;
+            const int page = kpos < k_end ? bt[kpos / p.page_size] : -1;
+            if (page >= 0) {
+                const size_t row = ((size_t)page * p.nkv + kvh) * p.page_size + kpos % p.page_size;
+                cp_async16(dst, v < HD / 8 ? p.kcache + row * HD + v * 8 : p.vcache + row * VD + (v - HD / 8) * 8);
+            } else {
+                *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+            }
+        }
+        if constexpr (SHARED) {
+            for (int key = threadIdx.x; key < BN; key += WARPS * 32) {
+                const int kpos = t0 + key;
+                const int page = kpos < k_end ? bt[kpos / p.page_size] : -1;
+                if (page >= 0) cp_async4(Sbuf + buf * BN + key, p.k_scale + (size_t)page * p.page_size + kpos % p.page_size);
+                else Sbuf[buf * BN + key] = 0.f;
+            }
+        }
+        cp_async_commit();
+    };
+    if (k_beg < k_end) load_tile(k_beg, 0);
+    for (int idx = threadIdx.x; idx < PROWS * (HD / 8); idx += blockDim.x) {
+        const int r = idx / (HD / 8), v = idx % (HD / 8);
+        uint4 val = make_uint4(0, 0, 0, 0);
+        if (live && r < heads) val = *reinterpret_cast<const uint4*>(p.q + (size_t)q_beg * p.q_stride + (size_t)(head0 + r) * HD + v * 8);
+        *reinterpret_cast<uint4*>(Qs + r * QLD + v * 8) = val;
+    }
+    __syncthreads();
+    uint32_t qf[HD / 16][4];
+#pragma unroll
+    for (int j = 0; j < HD / 16; ++j) ldmatrix_x4(qf[j], Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * QLD + j * 16 + (lane >> 4) * 8);
+
+    float o[VD / 8][4];
+#pragma unroll
+    for (int n = 0; n < VD / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    const float inv_cap = p.softcap > 0.f ? 1.0f / p.softcap : 0.f;
+    constexpr float LOG2E = 1.4426950408889634f;
+    int turn = 0;
+    for (int t0 = k_beg; t0 < k_end; t0 += BN, turn ^= 1) {
+        // the other buffer's readers are done (the barrier at the end of the turn before), so the next tile may be asked for
+        if (t0 + BN < k_end) { load_tile(t0 + BN, turn ^ 1); cp_async_wait_but_one(); }
+        else cp_async_wait_all();
+        __syncthreads();
+        const int kw = warp * 16;                               // this warp's keys of the tile
+        if (t0 + kw < k_end) {
+            const bf16* Ks = Kbuf + turn * BN * QLD + kw * QLD;
+            const bf16* Vs = Vbuf + turn * BN * VLD + kw * VLD;
+            float sc[2][4];
+#pragma unroll
+            for (int n = 0; n < 2; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+#pragma unroll
+            for (int j = 0; j < HD / 16; ++j) {
+                uint32_t kb[4];
+                ldmatrix_x4(kb, Ks + ((lane >> 4) * 8 + (lane & 7)) * QLD + j * 16 + ((lane >> 3) & 1) * 8);
+                mma_bf16(sc[0], qf[j], kb[0], kb[1]);
+                mma_bf16(sc[1], qf[j], kb[2], kb[3]);
+            }
+            float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int r = e >> 1, key = kw + n * 8 + 2 * tq + (e & 1);
+                    float v = sc[n][e] * p.scale;
+                    if constexpr (SHARED) v *= Sbuf[turn * BN + key];
+                    if (p.softcap > 0.f) v = p.softcap * tanh_abs(v * inv_cap);
+                    v = t0 + key < k_end ? v : -INFINITY;
+                    sc[n][e] = v;
+                    mx[r] = fmaxf(mx[r], v);
+                }
+            }
+            float alpha[2];
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+                const float m_new = fmaxf(m[r], mx[r]);
+                alpha[r] = (m[r] == -INFINITY) ? 0.f : exp2f((m[r] - m_new) * LOG2E);
+                m[r] = m_new;
+                l[r] *= alpha[r];
+            }
+#pragma unroll
+            for (int n = 0; n < VD / 8; ++n) {
+                o[n][0] *= alpha[0]; o[n][1] *= alpha[0];
+                o[n][2] *= alpha[1]; o[n][3] *= alpha[1];
+            }
+            uint32_t pa[3][4];
+#pragma unroll
+            for (int q4 = 0; q4 < 4; ++q4) {
+                const int n = q4 >> 1, e = (q4 & 1) * 2, r = e >> 1;
+                const float p0 = (sc[n][e] == -INFINITY) ? 0.f : exp2f((sc[n][e] - m[r]) * LOG2E);
+                const float p1 = (sc[n][e + 1] == -INFINITY) ? 0.f : exp2f((sc[n][e + 1] - m[r]) * LOG2E);
+                l[r] += p0 + p1;
+                float a0, b0, c0, a1, b1, c1;
+                split3(p0, a0, b0, c0);
+                split3(p1, a1, b1, c1);
+                pa[0][q4] = pack2(a0, a1);
+                pa[1][q4] = pack2(b0, b1);
+                pa[2][q4] = pack2(c0, c1);
+            }
+#pragma unroll
+            for (int n2 = 0; n2 < VD / 16; ++n2) {
+                uint32_t vb[4];
+                ldmatrix_x4_trans(vb, Vs + (((lane >> 3) & 1) * 8 + (lane & 7)) * VLD + n2 * 16 + (lane >> 4) * 8);
+#pragma unroll
+                for (int term = 2; term >= 0; --term) {
+                    mma_bf16(o[2 * n2], pa[term], vb[0], vb[1]);
+                    mma_bf16(o[2 * n2 + 1], pa[term], vb[2], vb[3]);
+                }
+            }
+        }
+        __syncthreads();          // this tile is consumed by every warp
+    }
+    // the warps' sums: one maximum per row over the block, the warps add up in their order
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+        if (tq == 0) {
+            Wm[warp * PROWS + g + 8 * r] = m[r];
+            Wl[warp * PROWS + g + 8 * r] = l[r];
+        }
+    }
+    __syncthreads();
+    float fac[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        float M = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < WARPS; ++w) M = fmaxf(M, Wm[w * PROWS + g + 8 * r]);
+        fac[r] = (m[r] == -INFINITY) ? 0.f : exp2f((m[r] - M) * LOG2E);
+    }
+    for (int w = 0; w < WARPS; ++w) {
+        if (warp == w) {
+#pragma unroll
+            for (int n = 0; n < VD / 8; ++n) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    float* dst = Os + (g + 8 * (e >> 1)) * OLD + n * 8 + 2 * tq + (e & 1);
+                    const float v = o[n][e] * fac[e >> 1];
+                    *dst = w == 0 ? v : *dst + v;
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (threadIdx.x < PROWS) {
+        float M = -INFINITY, sum = 0.f;
+        for (int w = 0; w < WARPS; ++w) M = fmaxf(M, Wm[w * PROWS + threadIdx.x]);
+        for (int w = 0; w < WARPS; ++w) {
+            const float mw = Wm[w * PROWS + threadIdx.x];
+            if (mw != -INFINITY) sum += exp2f((mw - M) * LOG2E) * Wl[w * PROWS + threadIdx.x];
+        }
+        Ml[threadIdx.x] = M;
+        Ml[PROWS + threadIdx.x] = sum;
+    }
+    // the parts of this (token, key head) merge through each other's shared memory; every block finishes a share of the values
+    cluster_sync_all();
+    if (q_len == 1) {
+        const uint32_t os = (uint32_t)__cvta_generic_to_shared(Os), ml = (uint32_t)__cvta_generic_to_shared(Ml);
+        for (int idx = part * (WARPS * 32) + threadIdx.x; idx < heads * VD; idx += parts * (WARPS * 32)) {
+            const int r = idx / VD, d = idx % VD;
+            float M = -INFINITY;
+            for (int pt = 0; pt < parts; ++pt) M = fmaxf(M, cluster_ld_f32(cluster_map_shared(ml + r * 4, pt)));
+            float den = 0.f, v = 0.f;
+            if (M > -INFINITY) {
+                const float z = (p.sink && p.sink_values) ? p.sink_values[head0 + r] : 0.f;
+                if (p.sink) M = fmaxf(M, z);
+                for (int pt = 0; pt < parts; ++pt) {
+                    const float mp = cluster_ld_f32(cluster_map_shared(ml + r * 4, pt));
+                    if (mp == -INFINITY) continue;
+                    const float w = exp2f((mp - M) * LOG2E);
+                    den = fmaf(w, cluster_ld_f32(cluster_map_shared(ml + (PROWS + r) * 4, pt)), den);
+                    v = fmaf(w, cluster_ld_f32(cluster_map_shared(os + (r * OLD + d) * 4, pt)), v);
+                }
+                if (p.sink) den += expf(z - M);
+            }
+            p.out[(size_t)q_beg * p.o_stride + (size_t)(head0 + r) * VD + d] = __float2bfloat16_rn(den > 0.f ? v / den : 0.f);
+        }
+    }
+    cluster_sync_all();           // nobody leaves while its shared memory is read
+}
+
+template <int HD, int VD, bool SHARED>
+int launch_parts(const Params& p, int n_seqs, int parts, cudaStream_t s) {
+    const int G = p.nq / p.nkv;
+    const int gc = G < PROWS ? G : PROWS;
+    const int chunks = (G + gc - 1) / gc;
+    constexpr size_t smem = PartsSmem<HD, VD, SHARED>::TOTAL;
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(attention_mma_parts_kernel<HD, VD, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) LLMK_FAIL("attention_mma_parts: cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
+        configured = true;
+    }
+    LLMK_CHECK_LAUNCH_RC("attention_mma_parts", llmk_launch_clusters(attention_mma_parts_kernel<HD, VD, SHARED>, dim3(n_seqs, p.nkv * chunks, parts),
+                                                                     dim3(WARPS * 32), smem, s, true, dim3(1, 1, parts), p, gc, chunks, parts));
+    return LLMK_OK;
+}
+
 }  // namespace
 
 // Queries per tile (0: the kernel does not take these sizes).
@@ -355,4 +619,32 @@ LLMK_EXPORT int llmk_attention_mma(void* out, long long o_stride, const void* q,
     if (hd == 64) return launch<64, 128>(p, grid, s);
     if (vd == 64) return launch<128, 64>(p, grid, s);
     return launch<128, 128>(p, grid, s);
+}
+
+// Steps of single tokens: sequence s < n_seqs owns the one query row cu_q[s] (or none), its visible keys are cut into `parts` (1 to 8)
+// parts that merge inside a cluster.  Everything else as above; no gate, no turn back.
+LLMK_EXPORT int llmk_attention_mma_parts(void* out, long long o_stride, const void* q, long long q_stride, const void* kcache,
+                                         const void* vcache, const int* block_tables, int max_blocks, const int* ctx_len, const int* cu_q,
+                                         int n_seqs, int nq, int nkv, int hd, int vd, int page_size, int window, float scale, float softcap,
+                                         int sink, const float* sink_values, int chunk, const float* k_scale, int parts, void* stream) {
+    if (n_seqs <= 0) return LLMK_OK;
+    if (llmk_attention_mma_tile_queries(nq, nkv, hd, vd) == 0)
+        LLMK_FAIL("attention_mma_parts: not taken (heads %d/%d, key width %d and value width %d must be 64 or 128)", nq, nkv, hd, vd);
+    if (parts < 1 || parts > 8) LLMK_FAIL("attention_mma_parts: %d parts (1 to 8)", parts);
+    if (k_scale && hd != vd) LLMK_FAIL("attention_mma_parts: keys that are values have one width (%d, %d)", hd, vd);
+    if (!k_scale && !vcache) LLMK_FAIL("attention_mma_parts: no values");
+    if (q_stride % 8 != 0 || !host_aligned16(q) || !host_aligned16(kcache) || !host_aligned16(vcache) || page_size <= 0)
+        LLMK_FAIL("attention_mma_parts: q and the cache must start on 16-byte boundaries, q's row stride a multiple of 8");
+    if ((long long)nkv * ceil_div(nq / nkv, PROWS) > 65535) LLMK_FAIL("attention_mma_parts: grid too large");
+    Params p = {};
+    p.q = (const bf16*)q; p.kcache = (const bf16*)kcache; p.vcache = (const bf16*)vcache; p.out = (bf16*)out;
+    p.sink_values = sink_values; p.k_scale = k_scale; p.block_tables = block_tables; p.ctx_len = ctx_len; p.cu_q = cu_q;
+    p.q_stride = q_stride; p.o_stride = o_stride; p.max_blocks = max_blocks; p.nq = nq; p.nkv = nkv; p.page_size = page_size;
+    p.window = window; p.sink = sink ? 1 : 0; p.chunk = chunk > 0 ? chunk : 0; p.scale = scale; p.softcap = softcap;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (k_scale) return hd == 64 ? launch_parts<64, 64, true>(p, n_seqs, parts, s) : launch_parts<128, 128, true>(p, n_seqs, parts, s);
+    if (hd == 64 && vd == 64) return launch_parts<64, 64, false>(p, n_seqs, parts, s);
+    if (hd == 64) return launch_parts<64, 128, false>(p, n_seqs, parts, s);
+    if (vd == 64) return launch_parts<128, 64, false>(p, n_seqs, parts, s);
+    return launch_parts<128, 128, false>(p, n_seqs, parts, s);
 }

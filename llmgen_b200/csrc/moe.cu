@@ -27,123 +27,152 @@ constexpr int MOE_TT = 16;      // rows per tile
 constexpr int MOE_KC = 256;     // input values per pass through shared memory
 
 // ---------------------------------------------------------------------------------------------- route
-// One block per token: the warps share the experts (a warp per dot product, float32 sums in a fixed order), warp 0 then
-// scores and picks.  scoring 0: sigmoid, 1: softmax over all experts, 2: the logits themselves choose, and the weights
+// The warps share the experts (a warp per dot product, float32 sums in a fixed order), then a warp scores and picks for a
+// token.  scoring 0: sigmoid, 1: softmax over all experts, 2: the logits themselves choose, and the weights
 // are the softmax over the chosen logits.
-template <typename T>
-__global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict__ wr,
+// TOK tokens per block: a prompt's rows share what a block reads of the router; steps of a few tokens take a token a block
+// with a warp per expert.
+template <typename T, int TOK>
+__global__ void __launch_bounds__(TOK > 1 ? 256 : 1024) moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict__ wr,
                                                         const float* __restrict__ bias, int* __restrict__ slot_expert,
-                                                        float* __restrict__ slot_weight, int K, int E, int top, int scoring,
+                                                        float* __restrict__ slot_weight, int n_tokens, int K, int E, int top, int scoring,
                                                         int renorm, const float* __restrict__ choice_bias, float weight_scale,
                                                         float sum_eps) {
-    extern __shared__ float sm[];   // [K] the row in float32, [E] scores, [E] what chooses (with `choice_bias`)
+    extern __shared__ float sm[];   // [TOK][K] the rows in float32, [TOK][E] scores, [TOK][E] what chooses (with `choice_bias`)
     float* xs = sm;
-    float* s = sm + K;
-    float* by = choice_bias ? s + E : s;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-    const size_t t = blockIdx.x;
+    const int t0 = blockIdx.x * TOK, n = min(TOK, n_tokens - t0);
     pdl_launch_dependents();
     pdl_wait();
-    const T* x = h + t * ldh;
-    for (int k = threadIdx.x; k < K; k += blockDim.x) xs[k] = to_float(x[k]);
+    for (int idx = threadIdx.x; idx < TOK * K; idx += blockDim.x) {
+        const int i = idx / K, k = idx - i * K;
+        xs[idx] = i < n ? to_float(h[(size_t)(t0 + i) * ldh + k]) : 0.f;
+    }
     __syncthreads();
     const bool vec = (K & 3) == 0;
     for (int e = warp; e < E; e += nwarps) {
         const float* w = wr + (size_t)e * K;
-        float acc = 0.f;
+        float acc[TOK];
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) acc[i] = 0.f;
         if (vec) {
+#pragma unroll 4
             for (int k = lane * 4; k < K; k += 128) {
-                const float4 a = *reinterpret_cast<const float4*>(xs + k);
                 const float4 b = __ldg(reinterpret_cast<const float4*>(w + k));
-                acc = fmaf(a.x, b.x, acc); acc = fmaf(a.y, b.y, acc); acc = fmaf(a.z, b.z, acc); acc = fmaf(a.w, b.w, acc);
+#pragma unroll
+                for (int i = 0; i < TOK; ++i) {
+                    const float4 a = *reinterpret_cast<const float4*>(xs + i * K + k);
+                    acc[i] = fmaf(a.x, b.x, acc[i]); acc[i] = fmaf(a.y, b.y, acc[i]); acc[i] = fmaf(a.z, b.z, acc[i]); acc[i] = fmaf(a.w, b.w, acc[i]);
+                }
             }
         } else {
-            for (int k = lane; k < K; k += 32) acc = fmaf(xs[k], w[k], acc);
+            for (int k = lane; k < K; k += 32) {
+                const float b = w[k];
+#pragma unroll
+                for (int i = 0; i < TOK; ++i) acc[i] = fmaf(xs[i * K + k], b, acc[i]);
+            }
         }
-        acc = warp_sum(acc);
-        if (lane == 0) s[e] = acc + (bias ? bias[e] : 0.f);
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) {
+            acc[i] = warp_sum(acc[i]);
+            if (lane == 0) sm[TOK * K + i * E + e] = acc[i] + (bias ? bias[e] : 0.f);
+        }
     }
     __syncthreads();
-    if (warp != 0) return;
-    if (scoring == 2) {
-        // the logits choose
-    } else if (scoring == 1) {
-        float mx = -INFINITY;
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, s[e]);
-        mx = warp_max(mx);
-        float sum = 0.f;
-        for (int e = lane; e < E; e += 32) sum += expf(s[e] - mx);
-        sum = warp_sum(sum);
-        for (int e = lane; e < E; e += 32) s[e] = expf(s[e] - mx) / sum;
-    } else {
-        for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
-    }
-    if (choice_bias)
-        for (int e = lane; e < E; e += 32) by[e] = s[e] + choice_bias[e];
-    __syncwarp();
-    float total = 0.f;
-    for (int c = 0; c < top; ++c) {
-        // the largest remaining score; ties and values that compare with nothing (NaN) go to the smallest index
-        float best = -INFINITY;
-        int arg = 0x7fffffff;
-        for (int e = lane; e < E; e += 32) {
-            const float v = by[e];
-            if (v > best) { best = v; arg = e; }
-        }
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-            if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-        }
-        if (arg >= E) { arg = c < E ? c : 0; best = 0.f; }     // nothing comparable was left: a padded row's garbage
-        else if (choice_bias) best = s[arg];                   // the correction chooses, the score weighs
-        total += best;
-        if (lane == 0) {
-            slot_expert[t * top + c] = arg;
-            slot_weight[t * top + c] = best;
-            by[arg] = -INFINITY;
-        }
-        __syncwarp();
-    }
-    if (scoring == 2) {
-        // softmax over the chosen logits; the first chosen is the largest
-        if (lane == 0) {
-            const float mx = slot_weight[t * top];
+    for (int i = warp; i < n; i += nwarps) {        // a warp scores and picks for a token
+        const size_t t = t0 + i;
+        float* s = sm + TOK * K + i * E;
+        float* by = choice_bias ? s + TOK * E : s;
+        if (scoring == 2) {
+            // the logits choose
+        } else if (scoring == 1) {
+            float mx = -INFINITY;
+            for (int e = lane; e < E; e += 32) mx = fmaxf(mx, s[e]);
+            mx = warp_max(mx);
             float sum = 0.f;
-            for (int c = 0; c < top; ++c) sum += expf(slot_weight[t * top + c] - mx);
-            for (int c = 0; c < top; ++c) slot_weight[t * top + c] = expf(slot_weight[t * top + c] - mx) / sum * weight_scale;
+            for (int e = lane; e < E; e += 32) sum += expf(s[e] - mx);
+            sum = warp_sum(sum);
+            for (int e = lane; e < E; e += 32) s[e] = expf(s[e] - mx) / sum;
+        } else {
+            for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
         }
-        return;
-    }
-    if (lane == 0 && (renorm || weight_scale != 1.f))
+        if (choice_bias)
+            for (int e = lane; e < E; e += 32) by[e] = s[e] + choice_bias[e];
+        __syncwarp();
+        float total = 0.f;
         for (int c = 0; c < top; ++c) {
-            const float w = slot_weight[t * top + c];
-            slot_weight[t * top + c] = (renorm ? w / (total + sum_eps) : w) * weight_scale;
+            // the largest remaining score; ties and values that compare with nothing (NaN) go to the smallest index
+            float best = -INFINITY;
+            int arg = 0x7fffffff;
+            for (int e = lane; e < E; e += 32) {
+                const float v = by[e];
+                if (v > best) { best = v; arg = e; }
+            }
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+                if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+            }
+            if (arg >= E) { arg = c < E ? c : 0; best = 0.f; }     // nothing comparable was left: a padded row's garbage
+            else if (choice_bias) best = s[arg];                   // the correction chooses, the score weighs
+            total += best;
+            if (lane == 0) {
+                slot_expert[t * top + c] = arg;
+                slot_weight[t * top + c] = best;
+                by[arg] = -INFINITY;
+            }
+            __syncwarp();
         }
+        if (scoring == 2) {
+            // softmax over the chosen logits; the first chosen is the largest
+            if (lane == 0) {
+                const float mx = slot_weight[t * top];
+                float sum = 0.f;
+                for (int c = 0; c < top; ++c) sum += expf(slot_weight[t * top + c] - mx);
+                for (int c = 0; c < top; ++c) slot_weight[t * top + c] = expf(slot_weight[t * top + c] - mx) / sum * weight_scale;
+            }
+            continue;
+        }
+        if (lane == 0 && (renorm || weight_scale != 1.f))
+            for (int c = 0; c < top; ++c) {
+                const float w = slot_weight[t * top + c];
+                slot_weight[t * top + c] = (renorm ? w / (total + sum_eps) : w) * weight_scale;
+            }
+    }
 }
 
+// `pdl` 0: a plain launch (behind an event of another stream).
 LLMK_EXPORT int llmk_moe_route(const void* h, long long ldh, const float* wr, const float* bias, int* slot_expert, float* slot_weight,
                                int n_tokens, int K, int E, int top, int scoring, int renorm, const float* choice_bias,
-                               float weight_scale, float sum_eps, int dtype, void* stream) {
+                               float weight_scale, float sum_eps, int pdl, int dtype, void* stream) {
     if (n_tokens <= 0) return LLMK_OK;
     if (E <= 0 || top <= 0 || top > E || K <= 0) LLMK_FAIL("moe_route: bad sizes (experts %d, top %d, width %d)", E, top, K);
     if (scoring < 0 || scoring > 2) LLMK_FAIL("moe_route: unknown scoring %d", scoring);
     if (choice_bias && scoring == 2) LLMK_FAIL("moe_route: a correction of the scores needs scores (scoring %d)", scoring);
-    const size_t smem = ((size_t)K + 2 * E) * sizeof(float);
+    // four tokens a block where there are blocks for every SM all the same and their rows fit
+    constexpr int MANY = 4;
+    const size_t one = ((size_t)K + 2 * E) * sizeof(float);
+    const bool many = n_tokens >= 2 * MANY * device_sm_count() / 2 && MANY * one <= 96 * 1024;
+    const size_t smem = many ? MANY * one : one;
     if (smem > 200 * 1024) LLMK_FAIL("moe_route: a row of %d values and %d experts do not fit shared memory", K, E);
-    const int threads = E >= 8 ? 256 : 32 * E;
+    const int most = many ? 8 : n_tokens <= device_sm_count() ? 32 : 8;
+    const int threads = 32 * (E < most ? E : most);
+    const dim3 grid(many ? ceil_div(n_tokens, MANY) : n_tokens);
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
+#define MOE_ROUTE_LAUNCH(TYPE, TOK)                                                                                                      \
+    do {                                                                                                                                 \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<TYPE, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        e = llmk_launch(moe_route_kernel<TYPE, TOK>, grid, dim3(threads), smem, s, pdl != 0, (const TYPE*)h, ldh, wr, bias, slot_expert,  \
+                        slot_weight, n_tokens, K, E, top, scoring, renorm, choice_bias, weight_scale, sum_eps);                          \
+    } while (0)
     if (dtype == LLMK_F32) {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        e = llmk_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(threads), smem, s, true, (const float*)h, ldh, wr, bias, slot_expert,
-                        slot_weight, K, E, top, scoring, renorm, choice_bias, weight_scale, sum_eps);
+        if (many) MOE_ROUTE_LAUNCH(float, MANY); else MOE_ROUTE_LAUNCH(float, 1);
     } else if (dtype == LLMK_BF16) {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        e = llmk_launch(moe_route_kernel<bf16>, dim3(n_tokens), dim3(threads), smem, s, true, (const bf16*)h, ldh, wr, bias, slot_expert,
-                        slot_weight, K, E, top, scoring, renorm, choice_bias, weight_scale, sum_eps);
+        if (many) MOE_ROUTE_LAUNCH(bf16, MANY); else MOE_ROUTE_LAUNCH(bf16, 1);
     } else
         LLMK_FAIL("moe_route: unknown dtype %d", dtype);
+#undef MOE_ROUTE_LAUNCH
     LLMK_CHECK_LAUNCH_RC("moe_route", e);
     return LLMK_OK;
 }
@@ -224,7 +253,8 @@ LLMK_EXPORT int llmk_moe_plan(const int* slot_expert, int n_slots, int E, int ti
 }
 
 // --------------------------------------------------------------------------------------------- gather
-// xs[pos, :] = (T)(weight * h[token of order[pos], :]) for the rows a padded plan filled; rows of padding are zeroed.
+// xs[pos, :] = (T)(weight * h[token of order[pos], :]) for the rows a padded plan filled; rows of padding stay as they are: the
+// products that follow compute them like any other and nobody reads the result.
 template <typename T>
 __global__ void moe_gather_kernel(T* __restrict__ xs, const T* __restrict__ h, long long ldh, const int* __restrict__ order,
                                   const float* __restrict__ slot_weight, int top, int K, int scale_rows) {
@@ -233,10 +263,7 @@ __global__ void moe_gather_kernel(T* __restrict__ xs, const T* __restrict__ h, l
     pdl_wait();
     const int slot = order[pos];
     T* dst = xs + pos * K;
-    if (slot < 0) {
-        for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = from_float<T>(0.f);
-        return;
-    }
+    if (slot < 0) return;
     const float w = scale_rows ? slot_weight[slot] : 1.f;
     const T* src = h + (size_t)(slot / top) * ldh;
     for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = from_float<T>(to_float(src[k]) * w);

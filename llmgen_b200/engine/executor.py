@@ -509,6 +509,7 @@ class Executor:
         if self.profiler is not None:
             self.profiler.begin_pass([e.start for e in entries], [len(e.tokens) for e in entries])
         ctx, want_rows, temps, keys, n_want = self._build_meta(entries, pad_to=pad_to)
+        ctx.serial = self.profiler is not None
         ctx.fixed_shapes = pad_to > 0      # the launch shapes a captured graph of this step would have
         resid, delta = self.model.hidden_states(ctx, self.layer_caches)
         return self._finish_pass(entries, ctx, resid, delta, want_rows, temps, keys, n_want, sample, return_logits)

@@ -49,6 +49,8 @@ class DecoderModel:
         for item in spec.run_order:
             if not 0 <= item.layer < len(self.layers):
                 raise ValueError(f"run list names layer {item.layer}, the model has {len(self.layers)}")
+        # for blocks whose two sublayers run side by side
+        self.side_stream = torch.cuda.Stream(device=device) if any(getattr(l, "takes_rows", False) for l in self.layers) else None
         self.bad_token_flag = ops.bad_token_flag(device)      # read by the engine with every step's results
 
     # -- what the engine needs to size caches and limits
@@ -102,6 +104,7 @@ class DecoderModel:
             ops.widen(x0, resid)
         delta = None
         ctx.normed_for = None
+        ctx.side_stream = None if ctx.serial else self.side_stream
         stream = resid
         n_streams = int(getattr(self.spec, "residual_streams", 0) or 0)
         if n_streams > 0:

@@ -557,7 +557,7 @@ OP_COSTS: Dict[str, Callable] = {
     "embed_rows": _cost_embed, "add_rmsnorm": _cost_norm, "silu_mul": _cost_all_operands, "widen": _cost_all_operands,
     "attn_prep": _cost_attn_prep, "gemm_simt": _cost_product, "gemv_bf16": _cost_product, "gemm_tc": _cost_product,
     "gemm_skinny": _cost_product, "gemm_rows8": _cost_product, "gemm_rows8_gated": _cost_product, "paged_attention": _cost_attention, "attention_decode": _cost_attention,
-    "attention_tc": _cost_attention, "attention_mma": _cost_attention, "sample": _cost_all_operands,
+    "attention_tc": _cost_attention, "attention_mma": _cost_attention, "attention_mma_parts": _cost_attention, "sample": _cost_all_operands,
     "short_conv": _cost_short_conv, "rglru": _cost_rglru, "delta_scan": _cost_delta_scan, "add_bias": _cost_all_operands,
     "concat_stream": _cost_all_operands, "logit_cap": _cost_all_operands,
     "decay_scan": _cost_decay_scan, "token_shift_mix": _cost_token_shift, "scaled_sum": _cost_scaled_sum,

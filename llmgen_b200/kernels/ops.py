@@ -628,6 +628,28 @@ def attention_mma(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcac
                                        c_int(1 if gate_per_head else 0), _ptr(tcos), _ptr(tsin), _ptr(k_scale), _stream()))
 
 
+ATTENTION_MMA_MAX_PARTS = 8
+
+
+def attention_mma_parts(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: Optional[torch.Tensor], block_tables: torch.Tensor,
+                        max_blocks: int, ctx_len: torch.Tensor, cu_q: torch.Tensor, n_seqs: int, nq: int, nkv: int, hd: int, vd: int,
+                        page_size: int, window: int, scale: float, parts: int, softcap: float = 0.0, sink: bool = False, chunk: int = 0,
+                        sink_values: Optional[torch.Tensor] = None, k_scale: Optional[torch.Tensor] = None) -> None:
+    """Single tokens in bfloat16 with 32-bit softmax weights on the tensor cores (csrc/attention_mma.cu): row cu_q[s] of q for every
+    sequence that has one, its visible keys in `parts` parts (at most `ATTENTION_MMA_MAX_PARTS`) merged inside a cluster; the widths
+    that `attention_mma_tile_queries` takes."""
+    lib = build.load("attention_mma")
+    if q.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or kcache.dtype != torch.bfloat16:
+        raise KernelError("attention_mma_parts: bfloat16 only")
+    _check_sinks("attention_mma_parts", sink, sink_values, nq)
+    _check_k_scale("attention_mma_parts", k_scale, kcache, vcache)
+    _check(lib, lib.llmk_attention_mma_parts(_ptr(out), c_longlong(_row_stride(out)), _ptr(q), c_longlong(_row_stride(q)), _ptr(kcache),
+                                             _ptr(vcache), _ptr(block_tables), c_int(max_blocks), _ptr(ctx_len), _ptr(cu_q), c_int(n_seqs),
+                                             c_int(nq), c_int(nkv), c_int(hd), c_int(vd), c_int(page_size), c_int(window), c_float(scale),
+                                             c_float(softcap), c_int(1 if sink else 0), _ptr(sink_values), c_int(chunk), _ptr(k_scale),
+                                             c_int(parts), _stream()))
+
+
 def attention_decode_set_cluster_merge(on: bool) -> None:
     """Whether `attention_decode` merges up to 8 key parts through the shared memory of a thread-block
     cluster (the default) or through global memory and a ticket (for measurements and tests)."""
@@ -1470,7 +1492,7 @@ def moe_max_tiles(n_slots: int, experts: int, tile: int = 0) -> int:
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, slot_expert: torch.Tensor, slot_weight: torch.Tensor, top: int,
               scoring: str = "sigmoid", renormalize: bool = False, bias: Optional[torch.Tensor] = None,
-              choice_bias: Optional[torch.Tensor] = None, weight_scale: float = 1.0, sum_eps: float = 0.0) -> None:
+              choice_bias: Optional[torch.Tensor] = None, weight_scale: float = 1.0, sum_eps: float = 0.0, pdl: bool = True) -> None:
     """Per row of h [n, K]: scores of router (float32 [E, K]) h (+ `bias`, float32 [E]), the `top` largest choose; slot
     n * top + c receives (expert, score).  `choice_bias` (float32 [E]) is added to the scores for the choice alone;
     `renormalize`: the weights are divided by the chosen scores' sum + `sum_eps`; they are then multiplied by `weight_scale`."""
@@ -1482,7 +1504,7 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, slot_expert: torch.Tensor, 
         raise KernelError("moe_route: router, bias and weights float32, experts int32")
     _check(lib, lib.llmk_moe_route(_ptr(h), c_longlong(_row_stride(h)), _ptr(router), _ptr(bias), _ptr(slot_expert), _ptr(slot_weight), c_int(n),
                                    c_int(K), c_int(E), c_int(top), c_int(ROUTER_SCORINGS[scoring]), c_int(1 if renormalize else 0),
-                                   _ptr(choice_bias), c_float(weight_scale), c_float(sum_eps),
+                                   _ptr(choice_bias), c_float(weight_scale), c_float(sum_eps), c_int(1 if pdl else 0),
                                    c_int(dtype_code(h.dtype)), _stream()))
 
 
@@ -1499,7 +1521,7 @@ def moe_plan(slot_expert: torch.Tensor, n_slots: int, experts: int, order: torch
 
 
 def moe_gather(out: torch.Tensor, h: torch.Tensor, order: torch.Tensor, slot_weight: torch.Tensor, top: int, scale_rows: bool) -> None:
-    """out[pos] = h[order[pos] // top] (times the slot's weight if `scale_rows`), zeros where order[pos] < 0."""
+    """out[pos] = h[order[pos] // top] (times the slot's weight if `scale_rows`); rows where order[pos] < 0 are left as they are."""
     lib = build.load("moe")
     n, K = out.shape
     if out.dtype != h.dtype or not out.is_contiguous() or order.numel() < n:

@@ -468,6 +468,12 @@ class GQAAttention(Mixer):
                               ctx.array(f"attention_tiles_bq{mma_bq}_q0"), tile_seq.numel(), nq, nk, hd, hd, cache.page_size, self.window,
                               float(spec.scale), softcap=self.softcap, sink=self.sink, sink_values=self.sink_scores, chunk=self.chunk,
                               k_scale=cache.k_scale)
+        elif ctx.pure_decode and self.mma_tile_queries():
+            # single tokens in bfloat16: the parts of a token's keys are the blocks of a cluster
+            parts = min(self._split(ctx)[0], ops.ATTENTION_MMA_MAX_PARTS)
+            ops.attention_mma_parts(o, q, cache.k, None, group.block_tables, group.max_blocks, ctx.ctx_len, ctx.cu_q, ctx.n_seqs, nq, nk, hd, hd,
+                                    cache.page_size, self.window, float(spec.scale), parts, softcap=self.softcap, sink=self.sink,
+                                    chunk=self.chunk, sink_values=self.sink_scores, k_scale=cache.k_scale)
         else:
             tile_seq = ctx.array(self.tiles_name + "_seq")
             parts, part_size = self._split(ctx)

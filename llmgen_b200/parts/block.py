@@ -298,7 +298,11 @@ class ParallelBlock(Part):
     One kernel (`parallel_add`) ends a layer: it adds both results to the residual, each times its gain vector (the mixer's an
     array or float32 slices, a routed feed-forward's still the rows of its experts), and writes the next layer's normed input in
     the same pass (when the run list's next item is a block of this kind: the model names it in `ctx.next_block`).  A block whose
-    input nobody prepared norms it itself, which also finishes a sum the block before left open.  It hands on nothing to add."""
+    input nobody prepared norms it itself, which also finishes a sum the block before left open.  It hands on nothing to add.
+
+    The two sublayers do not wait for each other: a routed feed-forward runs on the model's side stream (`ctx.side_stream`)
+    beside the mixer, forked behind the kernel that wrote the normed input and joined before the sum; in a captured step these are
+    branches of the graph.  The first kernel behind the fork and the one behind the join are plain launches."""
 
     @staticmethod
     def weight_decls(spec: ParallelBlockSpec):
@@ -327,6 +331,7 @@ class ParallelBlock(Part):
         self.mixer_gain, self.ffn_gain = gain(spec.mixer_gain), gain(spec.ffn_gain) if spec.ffn is not None else None
         # a routed feed-forward hands over its experts' rows, which `parallel_add` weighs and adds up
         self.takes_rows = spec.ffn is not None and getattr(spec.ffn, "kind", None) == "routed_mlp"
+        self.forked, self.joined = torch.cuda.Event(), torch.cuda.Event()
 
     def workspace_bytes(self, tokens: int) -> int:
         elem = 2 if self.dtype == torch.bfloat16 else 4
@@ -342,12 +347,22 @@ class ParallelBlock(Part):
         ctx.normed_for = None
         follower = getattr(ctx, "next_block", None)
         follow = follower.mixer_norm if isinstance(follower, ParallelBlock) else None
-        out = None
-        if self.ffn is not None:
+        out, side = None, getattr(ctx, "side_stream", None) if self.takes_rows else None
+        if side is not None:
+            main = torch.cuda.current_stream()
+            self.forked.record(main)
+            side.wait_event(self.forked)
+            with torch.cuda.stream(side):
+                out = self.ffn.forward(ctx, normed, combine=False, pdl=False)
+                self.joined.record(side)
+        elif self.ffn is not None:
             out = self.ffn.forward(ctx, normed, combine=False) if self.takes_rows else self.ffn.forward(ctx, normed)
         mixed = finish_pair(ctx, self.mixer.forward(ctx, normed, cache), self.dtype)
+        if side is not None:
+            main.wait_event(self.joined)
         ops.parallel_add(resid, mixed, self.mixer_gain, out, self.ffn_gain, self.dtype, next_gain=follow.weight if follow is not None else None,
-                         eps=follow.eps if follow is not None else 0.0, normed=normed if follow is not None else None)
+                         eps=follow.eps if follow is not None else 0.0, normed=normed if follow is not None else None,
+                         pdl=side is None)
         ctx.normed_for = follower if follow is not None else None
         return None
 

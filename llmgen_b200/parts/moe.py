@@ -77,7 +77,8 @@ class RoutedMLP(FeedForward):
                  second grouped launch runs down
       float32    (and operands TMA refuses) tiles of 16 rows through `moe_experts`, float32 sums on the CUDA cores
 
-    A caller that adds the experts' rows up itself (`forward(..., combine=False)`) gets them as an `ops.RoutedRows`.
+    A caller that adds the experts' rows up itself (`forward(..., combine=False)`) gets them as an `ops.RoutedRows`; one that has
+    just changed streams says `pdl=False`, and the first launch is a plain one.
 
     The shared expert is two of the framework's own products with the same activation between them; a plain
     silu-gated one is the dense gated feed-forward's first half (`GatedMLP.hidden`: the activation in the product's
@@ -152,7 +153,7 @@ class RoutedMLP(FeedForward):
         rows = slots + ops.MOE_GROUPED_TILE * min(self.E, slots) if self.grouped else slots
         return rows * (3 * self.F + 2 * H) * 4 + tokens * H * 4 + shared + 16 * (rows + self.E) + 2 * ops.SLICED_PRODUCT_BYTES
 
-    def forward(self, ctx, x, combine: bool = True):
+    def forward(self, ctx, x, combine: bool = True, pdl: bool = True):
         T, H = x.shape
         ws = ctx.workspace
         spec, top = self.spec, self.top
@@ -165,7 +166,7 @@ class RoutedMLP(FeedForward):
         tile_expert, tile_start, tile_rows = (ints[2 * n_slots + n_rows + i * tiles:2 * n_slots + n_rows + (i + 1) * tiles] for i in range(3))
         slot_weight = ws.flat("moe_weights", n_slots, torch.float32)
         ops.moe_route(x, self.router, slot_expert, slot_weight, top, spec.scoring, spec.renormalize, bias=self.router_bias,
-                      choice_bias=self.choice_bias, weight_scale=float(spec.weight_scale), sum_eps=float(spec.sum_eps))
+                      choice_bias=self.choice_bias, weight_scale=float(spec.weight_scale), sum_eps=float(spec.sum_eps), pdl=pdl)
         ops.moe_plan(slot_expert, n_slots, self.E, order, pos_of_slot, tile_expert, tile_start, tile_rows, tile=tile, padded=self.grouped)
         cap = (ws.default_rows * top // 128 + self.E) * 128 if self.grouped else ws.default_rows * top
         rows = ws.buffer("moe_rows", n_rows, H, torch.float32, capacity_rows=cap)

@@ -169,6 +169,62 @@ def test_tensor_core_attention_over_entries_that_are_key_and_value(nq, nkv, hd, 
     close(out, want, 1e-2)
 
 
+@pytest.mark.parametrize("shared", [True, False])
+@pytest.mark.parametrize("nq,nkv,hd,vd,page", [(6, 3, 64, 64, 16), (2, 1, 128, 128, 32), (4, 4, 128, 128, 16), (20, 1, 64, 64, 16), (4, 2, 64, 128, 16),
+                                               (6, 2, 128, 64, 16)])
+def test_single_tokens_on_the_tensor_cores_with_their_keys_in_a_cluster_of_parts(nq, nkv, hd, vd, page, shared):
+    """Sequences of 1 to 300 keys in one step, one without a token and one of padding, parts beyond the keys there are; windows,
+    blocks of positions, a bound on the scores and sinks; entries that are key and value, or two arrays."""
+    from llmgen_b200.kernels import ops
+    if shared and hd != vd:
+        pytest.skip("keys that are values have one width")
+    scale, lens = 0.25, [300, 1, 64, 65, 0, 130]
+    seqs = [entries(max(n, 1), nkv, hd, page, torch.bfloat16, 5 + 2 * i) for i, n in enumerate(lens)]
+    values = [rnd((max(n, 1), nkv, vd), 40 + i, 1.0, torch.bfloat16) for i, n in enumerate(lens)]
+    sizes = [s[2].shape[0] for s in seqs]
+    base = [sum(sizes[:i]) for i in range(len(sizes))]
+    kc, ks = torch.cat([s[2] for s in seqs]), torch.cat([s[3] for s in seqs])
+    vc = torch.zeros(kc.shape[0], nkv, page, vd, dtype=torch.bfloat16, device=DEV)
+    most = max(s[4].numel() for s in seqs)
+    bt = torch.full((len(lens), most), -1, dtype=torch.int32, device=DEV)
+    for i, s in enumerate(seqs):
+        bt[i, :s[4].numel()] = s[4] + base[i]
+        for j in range(values[i].shape[0]):
+            vc[int(bt[i, j // page]), :, j % page] = values[i][j].to(DEV)
+    cu = [0, 1, 2, 3, 4, 5, 6]
+    q = rnd((6, nq * hd), 6, 1.0, torch.bfloat16)
+    sinks = rnd((nq,), 7, 2.0)
+    forms = [dict(), dict(window=70), dict(chunk=96, softcap=3.0), dict(sink=True), dict(sink=True, sink_values=sinks.to(DEV), window=33)]
+    for form in forms:
+        window, chunk, cap = form.get("window", 0), form.get("chunk", 0), form.get("softcap", 0.0)
+        want = torch.zeros(6, nq, vd, dtype=torch.float64)
+        for i, n in enumerate(lens):
+            if n == 0:
+                continue
+            first = max(0, n - window) if window else (n - 1) // chunk * chunk if chunk else 0
+            for h in range(nq):
+                g = h // (nq // nkv)
+                sc = seqs[i][0][first:n, g] @ q[i, h * hd:(h + 1) * hd].double() * scale
+                if shared:
+                    sc = sc * seqs[i][1][first:n]
+                if cap:
+                    sc = cap * torch.tanh(sc / cap)
+                e = torch.exp(sc - sc.max())
+                sink = math.exp((float(sinks[h]) if "sink_values" in form else 0.0) - float(sc.max())) if form.get("sink") else 0.0
+                v = seqs[i][0][first:n, g] if shared else values[i][first:n, g].double()
+                want[i, h] = (e / (e.sum() + sink)) @ v
+        for parts in (1, 3, 8):
+            out = torch.full((6, nq * vd), 5.0, dtype=torch.bfloat16, device=DEV)
+            ops.attention_mma_parts(out, q.to(DEV), kc, None if shared else vc, bt, most, ints(lens), ints(cu), 6, nq, nkv, hd, vd, page, window, scale,
+                                    parts, softcap=cap, sink=form.get("sink", False), chunk=chunk, sink_values=form.get("sink_values"),
+                                    k_scale=ks if shared else None)
+            for i, n in enumerate(lens):
+                if n:
+                    close(out[i], want[i].reshape(-1), 1e-2)
+                else:
+                    assert float(out[i].float().abs().max()) == 0.0
+
+
 def test_values_and_factors_exclude_each_other():
     from llmgen_b200.kernels import ops
     k, factor, kc, ks, bt = entries(16, 1, 64, 16, torch.bfloat16, 5)
