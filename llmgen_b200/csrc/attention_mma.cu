@@ -4,7 +4,7 @@
 //
 //   S = Q K^T      Q and K are the cache's bfloat16 values, every product exact, sums float32
 //   scores         s * scale, then (softcap > 0) softcap * tanh(s / softcap), the causal (and window, or block) mask, the row's
-//                  running maximum and sum, the weights exp(s - m): float32, `tanhf` and `exp2f` at full precision
+//                  running maximum and sum, the weights exp(s - m): float32 (powers of two of scores times log2(e))
 //   O += P V       a float32 weight enters as THREE bfloat16 terms p = p1 + p2 + p3 (24 bits of mantissa), so every
 //                  product with a bfloat16 value is what float32 arithmetic would give; three MMAs a step
 //   finish         the sink (one more term exp(0) in the denominator), the division, the output gate sigmoid(g)
@@ -80,16 +80,22 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&v);
 }
-// x = a + b + c with a, b, c bfloat16: the three most significant pieces of a float32
-__device__ __forceinline__ void split3(float x, float& a, float& b, float& c) {
-    a = __bfloat162float(__float2bfloat16_rn(x));
-    const float r = x - a;
-    b = __bfloat162float(__float2bfloat16_rn(r));
-    c = __bfloat162float(__float2bfloat16_rn(r - b));
+// 2^x (the hardware's approximation: 2 ulp; results below the smallest normal number are zero)
+__device__ __forceinline__ float pow2(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+// two float32 as three pairs of bfloat16: x = w1 + w2 + w3, the most significant pieces first
+__device__ __forceinline__ void split3(float x0, float x1, uint32_t& w1, uint32_t& w2, uint32_t& w3) {
+    w1 = pack2(x0, x1);
+    const float r0 = x0 - __uint_as_float(w1 << 16), r1 = x1 - __uint_as_float(w1 & 0xffff0000u);
+    w2 = pack2(r0, r1);
+    w3 = pack2(r0 - __uint_as_float(w2 << 16), r1 - __uint_as_float(w2 & 0xffff0000u));
 }
 
 template <int HD, int VD, bool SHARED>
-__global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
+__global__ void __launch_bounds__(WARPS * 32, SHARED || VD == 64 ? 3 : 2) attention_mma_kernel(Params p) {
     static_assert(!SHARED || HD == VD, "keys that are values have one width");
     constexpr int QLD = HD + 8, VLD = VD + 8;      // rows 16 bytes longer: the eight rows of an ldmatrix fall on different banks
     extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -138,8 +144,9 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     const int qpos[2] = {first_pos + warp * 16 + g, first_pos + warp * 16 + g + 8};
     const int kmin[2] = {p.chunk > 0 ? qpos[0] / p.chunk * p.chunk : 0, p.chunk > 0 ? qpos[1] / p.chunk * p.chunk : 0};
-    const float inv_cap = p.softcap > 0.f ? 1.0f / p.softcap : 0.f;
     constexpr float LOG2E = 1.4426950408889634f;
+    // the bound on the scores, as they are: cap2 tanh(s2 / cap2) with s2 = s log2(e), cap2 = cap log2(e)
+    const float scale2 = p.scale * LOG2E, cap2 = p.softcap * LOG2E, inv_cap2 = p.softcap > 0.f ? 1.0f / cap2 : 0.f;
 
     constexpr int VECS = HD / 8 + (SHARED ? 0 : VD / 8);
     auto load_tile = [&](int t0, int buf) {
@@ -191,46 +198,69 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
                 mma_bf16(sc[2 * n2 + 1], qf[j], kb[2], kb[3]);
             }
         }
-        // scores, mask, the rows' maxima
+        // scores as powers of two, s log2(e), and the rows' maxima; the mask where a tile is not wholly visible to these rows
+        const bool whole = t0 + BN - 1 <= first_pos + warp * 16 && t0 + BN <= k_end && (p.window <= 0 || t0 > first_pos + warp * 16 + 15 - p.window) &&
+                           t0 >= kmin[1];
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int n = 0; n < BN / 8; ++n) {
+            float2 f = make_float2(scale2, scale2);
+            if constexpr (SHARED) {
+                const float2 ks = *reinterpret_cast<const float2*>(Sbuf + turn * BN + n * 8 + 2 * tq);
+                f.x *= ks.x;
+                f.y *= ks.y;
+            }
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int r = e >> 1;
-                const int kpos = t0 + n * 8 + 2 * tq + (e & 1);
-                float v = sc[n][e] * p.scale;
-                if constexpr (SHARED) v *= Sbuf[turn * BN + n * 8 + 2 * tq + (e & 1)];
-                if (p.softcap > 0.f) v = p.softcap * tanh_abs(v * inv_cap);
-                const bool vis = kpos <= qpos[r] && kpos < k_end && (p.window <= 0 || kpos > qpos[r] - p.window) && kpos >= kmin[r];
-                v = vis ? v : -INFINITY;
-                sc[n][e] = v;
-                mx[r] = fmaxf(mx[r], v);
+            for (int e = 0; e < 4; ++e) sc[n][e] *= (e & 1) ? f.y : f.x;
+        }
+        if (p.softcap > 0.f) {
+#pragma unroll
+            for (int n = 0; n < BN / 8; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) sc[n][e] = cap2 * tanh_abs(sc[n][e] * inv_cap2);
+        }
+        if (!whole) {
+#pragma unroll
+            for (int n = 0; n < BN / 8; ++n) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int r = e >> 1;
+                    const int kpos = t0 + n * 8 + 2 * tq + (e & 1);
+                    const bool vis = kpos <= qpos[r] && kpos < k_end && (p.window <= 0 || kpos > qpos[r] - p.window) && kpos >= kmin[r];
+                    sc[n][e] = vis ? sc[n][e] : -INFINITY;
+                }
             }
         }
-        float alpha[2];
+#pragma unroll
+        for (int n = 0; n < BN / 8; ++n) {
+            mx[0] = fmaxf(mx[0], fmaxf(sc[n][0], sc[n][1]));
+            mx[1] = fmaxf(mx[1], fmaxf(sc[n][2], sc[n][3]));
+        }
+        float alpha[2], base[2];
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
             mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
             mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
             const float m_new = fmaxf(m[r], mx[r]);
-            alpha[r] = (m[r] == -INFINITY) ? 0.f : exp2f((m[r] - m_new) * LOG2E);
+            base[r] = m_new > -INFINITY ? m_new : 0.f;        // a row that has seen nothing: every weight 2^-inf
+            alpha[r] = pow2(m[r] - base[r]);
             m[r] = m_new;
             l[r] *= alpha[r];
         }
+        if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
 #pragma unroll
-        for (int n = 0; n < VD / 8; ++n) {
-            o[n][0] *= alpha[0]; o[n][1] *= alpha[0];
-            o[n][2] *= alpha[1]; o[n][3] *= alpha[1];
+            for (int n = 0; n < VD / 8; ++n) {
+                o[n][0] *= alpha[0]; o[n][1] *= alpha[0];
+                o[n][2] *= alpha[1]; o[n][3] *= alpha[1];
+            }
         }
 #pragma unroll
         for (int n = 0; n < BN / 8; ++n) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int r = e >> 1;
-                const float pv = (sc[n][e] == -INFINITY) ? 0.f : exp2f((sc[n][e] - m[r]) * LOG2E);
+                const float pv = pow2(sc[n][e] - base[e >> 1]);
                 sc[n][e] = pv;
-                l[r] += pv;
+                l[e >> 1] += pv;
             }
         }
         // O += P V, sixteen keys a step, the weights in three bfloat16 terms
@@ -240,21 +270,23 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
 #pragma unroll
             for (int q4 = 0; q4 < 4; ++q4) {
                 const int n = 2 * j + (q4 >> 1), e = (q4 & 1) * 2;
-                float a0, b0, c0, a1, b1, c1;
-                split3(sc[n][e], a0, b0, c0);
-                split3(sc[n][e + 1], a1, b1, c1);
-                pa[0][q4] = pack2(a0, a1);
-                pa[1][q4] = pack2(b0, b1);
-                pa[2][q4] = pack2(c0, c1);
+                split3(sc[n][e], sc[n][e + 1], pa[0][q4], pa[1][q4], pa[2][q4]);
             }
+            // four steps of 16 columns at a time, a term over all of them before the next: consecutive products on one
+            // accumulator would wait for each other
 #pragma unroll
-            for (int n2 = 0; n2 < VD / 16; ++n2) {
-                uint32_t vb[4];
-                ldmatrix_x4_trans(vb, Vs + (j * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * VLD + n2 * 16 + (lane >> 4) * 8);
+            for (int n4 = 0; n4 < VD / 16; n4 += 4) {
+                uint32_t vb[4][4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+                    ldmatrix_x4_trans(vb[u], Vs + (j * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * VLD + (n4 + u) * 16 + (lane >> 4) * 8);
 #pragma unroll
                 for (int term = 2; term >= 0; --term) {          // smallest terms first
-                    mma_bf16(o[2 * n2], pa[term], vb[0], vb[1]);
-                    mma_bf16(o[2 * n2 + 1], pa[term], vb[2], vb[3]);
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        mma_bf16(o[2 * (n4 + u)], pa[term], vb[u][0], vb[u][1]);
+                        mma_bf16(o[2 * (n4 + u) + 1], pa[term], vb[u][2], vb[u][3]);
+                    }
                 }
             }
         }
@@ -272,8 +304,9 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_kernel(Params p) {
         float inv = l[r] > 0.f ? 1.0f / l[r] : 0.f;
         if (p.sink && l[r] > 0.f) {
             const float z = p.sink_values ? p.sink_values[head] : 0.f;
-            const float M = fmaxf(m[r], z);
-            const float w = expf(m[r] - M);
+            const float mr = m[r] * 0.6931471805599453f;          // as a power of e
+            const float M = fmaxf(mr, z);
+            const float w = expf(mr - M);
             inv = w / (l[r] * w + expf(z - M));
         }
         const size_t tok = (size_t)(q_beg + q0 + row);
@@ -324,15 +357,18 @@ int launch(const Params& p, dim3 grid, cudaStream_t s) {
 
 // ------------------------------------------------------------------------------------- single tokens, keys in parts
 constexpr int PROWS = 16;
+constexpr int PSTAGES = 3;           // tiles of keys on their way
+constexpr int PPAGES = 512;          // page ids of a part that are looked up once, in front of the first tile (longer parts: as they go)
 
 template <int HD, int VD, bool SHARED>
 struct PartsSmem {
     static constexpr int QLD = HD + 8, VLD = VD + 8, OLD = VD + 4;
     static constexpr size_t Q = (size_t)PROWS * QLD * sizeof(bf16);
-    static constexpr size_t KV = ((size_t)2 * BN * QLD + (SHARED ? 0 : (size_t)2 * BN * VLD)) * sizeof(bf16);
-    static constexpr size_t FACTORS = SHARED ? 2 * BN * sizeof(float) : 0;
-    static constexpr size_t OUT = ((size_t)PROWS * OLD + 2 * PROWS + 2 * WARPS * PROWS) * sizeof(float);
-    static constexpr size_t TOTAL = Q + KV + FACTORS + OUT;
+    static constexpr size_t KV = ((size_t)PSTAGES * BN * QLD + (SHARED ? 0 : (size_t)PSTAGES * BN * VLD)) * sizeof(bf16);
+    static constexpr size_t FACTORS = SHARED ? PSTAGES * BN * sizeof(float) : 0;
+    static constexpr size_t OUT = ((size_t)PROWS * OLD + 2 * PROWS + 2 * WARPS * PROWS + 3 * 8 * PROWS) * sizeof(float);
+    static constexpr size_t PAGES = PPAGES * sizeof(int);
+    static constexpr size_t TOTAL = Q + KV + FACTORS + OUT + PAGES;
 };
 
 template <int HD, int VD, bool SHARED>
@@ -343,12 +379,15 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
     extern __shared__ __align__(16) uint8_t smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);
     bf16* Kbuf = Qs + PROWS * QLD;
-    bf16* Vbuf = SHARED ? Kbuf : Kbuf + 2 * BN * QLD;
+    bf16* Vbuf = SHARED ? Kbuf : Kbuf + PSTAGES * BN * QLD;
     float* Sbuf = reinterpret_cast<float*>(smem_raw + L::Q + L::KV);
     float* Os = reinterpret_cast<float*>(smem_raw + L::Q + L::KV + L::FACTORS);      // [PROWS][OLD]
     float* Ml = Os + PROWS * OLD;                                                    // [PROWS] maxima, [PROWS] sums
     float* Wm = Ml + 2 * PROWS;                                                      // [WARPS][PROWS]
     float* Wl = Wm + WARPS * PROWS;
+    float* Rm = Wl + WARPS * PROWS;                                                  // [8 parts][2 PROWS] the parts' maxima and sums
+    float* Rw = Rm + 8 * 2 * PROWS;                                                  // [8 parts][PROWS] their weights
+    int* pages = reinterpret_cast<int*>(smem_raw + L::Q + L::KV + L::FACTORS + L::OUT);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int g = lane >> 2, tq = lane & 3;
     pdl_launch_dependents();
@@ -370,6 +409,13 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
         k_end = min(qpos + 1, k_beg + size);
     }
     const int* bt = p.block_tables + (size_t)s * p.max_blocks;
+    const int page0 = k_beg / p.page_size;
+    const int n_pages = k_beg < k_end ? (k_end - 1) / p.page_size - page0 + 1 : 0;
+    const bool staged = n_pages <= PPAGES;
+    if (staged) {
+        for (int i = threadIdx.x; i < n_pages; i += WARPS * 32) pages[i] = bt[page0 + i];
+        __syncthreads();
+    }
 
     constexpr int VECS = HD / 8 + (SHARED ? 0 : VD / 8);
     auto load_tile = [&](int t0, int buf) {
@@ -380,25 +426,30 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
             const int key = idx / VECS, v = idx % VECS;
             const int kpos = t0 + key;
             bf16* dst = v < HD / 8 ? Kd + key * QLD + v * 8 : Vd + key * VLD + (v - HD / 8) * 8;
-            const int page = kpos < k_end ? bt[kpos / p.page_size] : -1;
+            const int at = kpos / p.page_size;
+            const int page = kpos < k_end ? (staged ? pages[at - page0] : bt[at]) : -1;
             if (page >= 0) {
-                const size_t row = ((size_t)page * p.nkv + kvh) * p.page_size + kpos % p.page_size;
+                const int off = kpos - at * p.page_size;
+                const size_t row = ((size_t)page * p.nkv + kvh) * p.page_size + off;
                 cp_async16(dst, v < HD / 8 ? p.kcache + row * HD + v * 8 : p.vcache + row * VD + (v - HD / 8) * 8);
+                if constexpr (SHARED) {
+                    if (v == 0) cp_async4(Sbuf + buf * BN + key, p.k_scale + (size_t)page * p.page_size + off);
+                }
             } else {
                 *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
-            }
-        }
-        if constexpr (SHARED) {
-            for (int key = threadIdx.x; key < BN; key += WARPS * 32) {
-                const int kpos = t0 + key;
-                const int page = kpos < k_end ? bt[kpos / p.page_size] : -1;
-                if (page >= 0) cp_async4(Sbuf + buf * BN + key, p.k_scale + (size_t)page * p.page_size + kpos % p.page_size);
-                else Sbuf[buf * BN + key] = 0.f;
+                if constexpr (SHARED) {
+                    if (v == 0) Sbuf[buf * BN + key] = 0.f;
+                }
             }
         }
         cp_async_commit();
     };
-    if (k_beg < k_end) load_tile(k_beg, 0);
+    // every turn asks for the tile two ahead; a group is committed for every turn, also where there is no tile left
+#pragma unroll
+    for (int i = 0; i < PSTAGES - 1; ++i) {
+        if (k_beg + i * BN < k_end) load_tile(k_beg + i * BN, i);
+        else cp_async_commit();
+    }
     for (int idx = threadIdx.x; idx < PROWS * (HD / 8); idx += blockDim.x) {
         const int r = idx / (HD / 8), v = idx % (HD / 8);
         uint4 val = make_uint4(0, 0, 0, 0);
@@ -414,14 +465,15 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
 #pragma unroll
     for (int n = 0; n < VD / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-    const float inv_cap = p.softcap > 0.f ? 1.0f / p.softcap : 0.f;
     constexpr float LOG2E = 1.4426950408889634f;
+    const float scale2 = p.scale * LOG2E, cap2 = p.softcap * LOG2E, inv_cap2 = p.softcap > 0.f ? 1.0f / cap2 : 0.f;
     int turn = 0;
-    for (int t0 = k_beg; t0 < k_end; t0 += BN, turn ^= 1) {
-        // the other buffer's readers are done (the barrier at the end of the turn before), so the next tile may be asked for
-        if (t0 + BN < k_end) { load_tile(t0 + BN, turn ^ 1); cp_async_wait_but_one(); }
-        else cp_async_wait_all();
-        __syncthreads();
+    for (int t0 = k_beg; t0 < k_end; t0 += BN, turn = turn + 1 == PSTAGES ? 0 : turn + 1) {
+        cp_async_wait_but_one();  // this tile has arrived (the one after it may still be on its way) ...
+        __syncthreads();          // ... for every thread, and the buffer of the tile before is free
+        const int ahead = t0 + (PSTAGES - 1) * BN;
+        if (ahead < k_end) load_tile(ahead, turn == 0 ? PSTAGES - 1 : turn - 1);
+        else cp_async_commit();
         const int kw = warp * 16;                               // this warp's keys of the tile
         if (t0 + kw < k_end) {
             const bf16* Ks = Kbuf + turn * BN * QLD + kw * QLD;
@@ -441,56 +493,57 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
             for (int n = 0; n < 2; ++n) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const int r = e >> 1, key = kw + n * 8 + 2 * tq + (e & 1);
-                    float v = sc[n][e] * p.scale;
+                    const int key = kw + n * 8 + 2 * tq + (e & 1);
+                    float v = sc[n][e] * scale2;
                     if constexpr (SHARED) v *= Sbuf[turn * BN + key];
-                    if (p.softcap > 0.f) v = p.softcap * tanh_abs(v * inv_cap);
+                    if (p.softcap > 0.f) v = cap2 * tanh_abs(v * inv_cap2);
                     v = t0 + key < k_end ? v : -INFINITY;
                     sc[n][e] = v;
-                    mx[r] = fmaxf(mx[r], v);
+                    mx[e >> 1] = fmaxf(mx[e >> 1], v);
                 }
             }
-            float alpha[2];
+            float alpha[2], base[2];
 #pragma unroll
             for (int r = 0; r < 2; ++r) {
                 mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
                 mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
                 const float m_new = fmaxf(m[r], mx[r]);
-                alpha[r] = (m[r] == -INFINITY) ? 0.f : exp2f((m[r] - m_new) * LOG2E);
+                base[r] = m_new > -INFINITY ? m_new : 0.f;
+                alpha[r] = pow2(m[r] - base[r]);
                 m[r] = m_new;
                 l[r] *= alpha[r];
             }
+            if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
 #pragma unroll
-            for (int n = 0; n < VD / 8; ++n) {
-                o[n][0] *= alpha[0]; o[n][1] *= alpha[0];
-                o[n][2] *= alpha[1]; o[n][3] *= alpha[1];
+                for (int n = 0; n < VD / 8; ++n) {
+                    o[n][0] *= alpha[0]; o[n][1] *= alpha[0];
+                    o[n][2] *= alpha[1]; o[n][3] *= alpha[1];
+                }
             }
             uint32_t pa[3][4];
 #pragma unroll
             for (int q4 = 0; q4 < 4; ++q4) {
                 const int n = q4 >> 1, e = (q4 & 1) * 2, r = e >> 1;
-                const float p0 = (sc[n][e] == -INFINITY) ? 0.f : exp2f((sc[n][e] - m[r]) * LOG2E);
-                const float p1 = (sc[n][e + 1] == -INFINITY) ? 0.f : exp2f((sc[n][e + 1] - m[r]) * LOG2E);
+                const float p0 = pow2(sc[n][e] - base[r]), p1 = pow2(sc[n][e + 1] - base[r]);
                 l[r] += p0 + p1;
-                float a0, b0, c0, a1, b1, c1;
-                split3(p0, a0, b0, c0);
-                split3(p1, a1, b1, c1);
-                pa[0][q4] = pack2(a0, a1);
-                pa[1][q4] = pack2(b0, b1);
-                pa[2][q4] = pack2(c0, c1);
+                split3(p0, p1, pa[0][q4], pa[1][q4], pa[2][q4]);
             }
 #pragma unroll
-            for (int n2 = 0; n2 < VD / 16; ++n2) {
-                uint32_t vb[4];
-                ldmatrix_x4_trans(vb, Vs + (((lane >> 3) & 1) * 8 + (lane & 7)) * VLD + n2 * 16 + (lane >> 4) * 8);
+            for (int n4 = 0; n4 < VD / 16; n4 += 4) {
+                uint32_t vb[4][4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+                    ldmatrix_x4_trans(vb[u], Vs + (((lane >> 3) & 1) * 8 + (lane & 7)) * VLD + (n4 + u) * 16 + (lane >> 4) * 8);
 #pragma unroll
                 for (int term = 2; term >= 0; --term) {
-                    mma_bf16(o[2 * n2], pa[term], vb[0], vb[1]);
-                    mma_bf16(o[2 * n2 + 1], pa[term], vb[2], vb[3]);
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        mma_bf16(o[2 * (n4 + u)], pa[term], vb[u][0], vb[u][1]);
+                        mma_bf16(o[2 * (n4 + u) + 1], pa[term], vb[u][2], vb[u][3]);
+                    }
                 }
             }
         }
-        __syncthreads();          // this tile is consumed by every warp
     }
     // the warps' sums: one maximum per row over the block, the warps add up in their order
 #pragma unroll
@@ -509,7 +562,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < WARPS; ++w) M = fmaxf(M, Wm[w * PROWS + g + 8 * r]);
-        fac[r] = (m[r] == -INFINITY) ? 0.f : exp2f((m[r] - M) * LOG2E);
+        fac[r] = (m[r] == -INFINITY) ? 0.f : pow2(m[r] - M);
     }
     for (int w = 0; w < WARPS; ++w) {
         if (warp == w) {
@@ -530,33 +583,47 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
         for (int w = 0; w < WARPS; ++w) M = fmaxf(M, Wm[w * PROWS + threadIdx.x]);
         for (int w = 0; w < WARPS; ++w) {
             const float mw = Wm[w * PROWS + threadIdx.x];
-            if (mw != -INFINITY) sum += exp2f((mw - M) * LOG2E) * Wl[w * PROWS + threadIdx.x];
+            if (mw != -INFINITY) sum += pow2(mw - M) * Wl[w * PROWS + threadIdx.x];
         }
         Ml[threadIdx.x] = M;
         Ml[PROWS + threadIdx.x] = sum;
     }
     // the parts of this (token, key head) merge through each other's shared memory; every block finishes a share of the values
     cluster_sync_all();
+    const uint32_t os = (uint32_t)__cvta_generic_to_shared(Os), ml = (uint32_t)__cvta_generic_to_shared(Ml);
+    for (int i = threadIdx.x; i < parts * 2 * PROWS; i += WARPS * 32)
+        Rm[i] = cluster_ld_f32(cluster_map_shared(ml + (i % (2 * PROWS)) * 4, i / (2 * PROWS)));
+    __syncthreads();
+    if (threadIdx.x < PROWS) {
+        // a row's weights of the parts: 2^(m_part - M) over the sum of all of them (the sink among them)
+        const int r = threadIdx.x;
+        float M = -INFINITY;
+        for (int pt = 0; pt < parts; ++pt) M = fmaxf(M, Rm[pt * 2 * PROWS + r]);
+        const bool seen = M > -INFINITY;
+        const float z = (p.sink && p.sink_values && r < heads) ? p.sink_values[head0 + r] * LOG2E : 0.f;
+        if (p.sink && seen) M = fmaxf(M, z);
+        float den = (p.sink && seen) ? pow2(z - M) : 0.f;
+        for (int pt = 0; pt < parts; ++pt) {
+            const float mp = Rm[pt * 2 * PROWS + r];
+            const float w = mp == -INFINITY ? 0.f : pow2(mp - M);
+            Rw[pt * PROWS + r] = w;
+            den = fmaf(w, Rm[pt * 2 * PROWS + PROWS + r], den);
+        }
+        const float inv = den > 0.f ? 1.0f / den : 0.f;
+        for (int pt = 0; pt < parts; ++pt) Rw[pt * PROWS + r] *= inv;
+    }
+    __syncthreads();
     if (q_len == 1) {
-        const uint32_t os = (uint32_t)__cvta_generic_to_shared(Os), ml = (uint32_t)__cvta_generic_to_shared(Ml);
         for (int idx = part * (WARPS * 32) + threadIdx.x; idx < heads * VD; idx += parts * (WARPS * 32)) {
             const int r = idx / VD, d = idx % VD;
-            float M = -INFINITY;
-            for (int pt = 0; pt < parts; ++pt) M = fmaxf(M, cluster_ld_f32(cluster_map_shared(ml + r * 4, pt)));
-            float den = 0.f, v = 0.f;
-            if (M > -INFINITY) {
-                const float z = (p.sink && p.sink_values) ? p.sink_values[head0 + r] : 0.f;
-                if (p.sink) M = fmaxf(M, z);
-                for (int pt = 0; pt < parts; ++pt) {
-                    const float mp = cluster_ld_f32(cluster_map_shared(ml + r * 4, pt));
-                    if (mp == -INFINITY) continue;
-                    const float w = exp2f((mp - M) * LOG2E);
-                    den = fmaf(w, cluster_ld_f32(cluster_map_shared(ml + (PROWS + r) * 4, pt)), den);
-                    v = fmaf(w, cluster_ld_f32(cluster_map_shared(os + (r * OLD + d) * 4, pt)), v);
-                }
-                if (p.sink) den += expf(z - M);
-            }
-            p.out[(size_t)q_beg * p.o_stride + (size_t)(head0 + r) * VD + d] = __float2bfloat16_rn(den > 0.f ? v / den : 0.f);
+            float v[8];
+#pragma unroll
+            for (int pt = 0; pt < 8; ++pt) v[pt] = pt < parts ? cluster_ld_f32(cluster_map_shared(os + (r * OLD + d) * 4, pt)) : 0.f;
+            float sum = 0.f;
+#pragma unroll
+            for (int pt = 0; pt < 8; ++pt)
+                if (pt < parts) sum = fmaf(Rw[pt * PROWS + r], v[pt], sum);
+            p.out[(size_t)q_beg * p.o_stride + (size_t)(head0 + r) * VD + d] = __float2bfloat16_rn(sum);
         }
     }
     cluster_sync_all();           // nobody leaves while its shared memory is read

@@ -666,7 +666,7 @@ __device__ __forceinline__ float packed_sum(const void* x, size_t at, int splits
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) attn_prep_shared_rows_kernel(const void* __restrict__ x, long long ld, int splits, long long split_stride,
+__global__ void __launch_bounds__(512) attn_prep_shared_rows_kernel(const void* __restrict__ x, long long ld, int splits, long long split_stride,
                                                                     const float* __restrict__ bias, T* __restrict__ q_out, long long q_stride,
                                                                     T* __restrict__ cache, float* __restrict__ k_scale,
                                                                     const int* __restrict__ positions, const int* __restrict__ slots,
@@ -695,6 +695,24 @@ __global__ void __launch_bounds__(256) attn_prep_shared_rows_kernel(const void* 
             }
             *reinterpret_cast<float4*>(prow + i) = make_float4(v[0], v[1], v[2], v[3]);
             *reinterpret_cast<float4*>(prow + i + 4) = make_float4(v[4], v[5], v[6], v[7]);
+            if (i < nQ) ssq += ss; else ssk += ss;
+        }
+    } else if (splits > 0 && (nQ & 3) == 0 && (nK & 3) == 0 && (ld & 3) == 0 && (split_stride & 3) == 0 && aligned16(x) && (!bias || aligned16(bias))) {
+        // slices, four values a thread at a time, the loads of four slices in flight together
+        for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+            const float* p = static_cast<const float*>(x) + base + i;
+            float4 v = *reinterpret_cast<const float4*>(p);
+#pragma unroll 4
+            for (int s = 1; s < splits; ++s) {
+                const float4 f = *reinterpret_cast<const float4*>(p + (size_t)s * split_stride);
+                v.x += f.x; v.y += f.y; v.z += f.z; v.w += f.w;
+            }
+            if (bias) {
+                const float4 b = *reinterpret_cast<const float4*>(bias + i);
+                v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+            }
+            *reinterpret_cast<float4*>(prow + i) = v;
+            const float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
             if (i < nQ) ssq += ss; else ssk += ss;
         }
     } else {
@@ -742,15 +760,16 @@ LLMK_EXPORT int llmk_attn_prep_shared_rows(const void* x, long long ld, int spli
     if (coef != 0.f && !(every > 0.f)) LLMK_FAIL("attn_prep_shared_rows: a temperature every %g positions", (double)every);
     const size_t smem = ((size_t)(nq + nk) * hd + 33) * sizeof(float);
     if (smem > 200 * 1024) LLMK_FAIL("attn_prep_shared_rows: a row of %d values does not fit shared memory", (nq + nk) * hd);
+    const int threads = splits > 0 && (nq + nk) * hd >= 2048 ? 512 : 256;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
     if (dtype == LLMK_F32) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(attn_prep_shared_rows_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        e = llmk_launch(attn_prep_shared_rows_kernel<float>, dim3(n_tokens), dim3(256), smem, s, true, x, ld, splits, split_stride, bias, (float*)q_out,
+        e = llmk_launch(attn_prep_shared_rows_kernel<float>, dim3(n_tokens), dim3(threads), smem, s, true, x, ld, splits, split_stride, bias, (float*)q_out,
                         q_stride, (float*)cache, k_scale, positions, slots, gains, nq, nk, nkv_cache, hd, page_size, eps, coef, every);
     } else if (dtype == LLMK_BF16) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(attn_prep_shared_rows_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        e = llmk_launch(attn_prep_shared_rows_kernel<bf16>, dim3(n_tokens), dim3(256), smem, s, true, x, ld, splits, split_stride, bias, (bf16*)q_out,
+        e = llmk_launch(attn_prep_shared_rows_kernel<bf16>, dim3(n_tokens), dim3(threads), smem, s, true, x, ld, splits, split_stride, bias, (bf16*)q_out,
                         q_stride, (bf16*)cache, k_scale, positions, slots, gains, nq, nk, nkv_cache, hd, page_size, eps, coef, every);
     } else
         LLMK_FAIL("attn_prep_shared_rows: unknown dtype %d", dtype);

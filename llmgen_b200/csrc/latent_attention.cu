@@ -129,7 +129,9 @@ struct LatentEntries {
     float eps;
 };
 
-template <typename T>
+// QS: into how many shares of the key dimension a block's threads are cut (128 / QS latent columns a block); steps of a few tokens
+// take 4, so that there are blocks for the SMs, and add the shares up in their order.
+template <typename T, int QS>
 __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ wuk,
                                                             float* __restrict__ qa, const int* __restrict__ positions,
                                                             const float* __restrict__ cos_t, const float* __restrict__ sin_t,
@@ -170,14 +172,17 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict_
     }
     const int za = rank + rot;
     const T* w = wuk + (size_t)h * dim * rank;
-    // this block's slice of the latent's columns: a thread per column, the loads of W eight rows ahead of their use
-    const int r = blockIdx.z * blockDim.x + threadIdx.x;
-    if (r < rank) {
-        float acc[LT_TT];
+    // this block's slice of the latent's columns: a thread per column (and share), the loads of W eight rows ahead of their use
+    constexpr int COLS = 128 / QS;
+    const int r = blockIdx.z * COLS + threadIdx.x % COLS, share = threadIdx.x / COLS;
+    const int d_each = ceil_div(dim, QS);
+    float acc[LT_TT];
 #pragma unroll
-        for (int i = 0; i < LT_TT; ++i) acc[i] = 0.f;
-        int d = 0;
-        for (; d + 8 <= dim; d += 8) {
+    for (int i = 0; i < LT_TT; ++i) acc[i] = 0.f;
+    if (r < rank) {
+        int d = share * d_each;
+        const int d_end = min(dim, d + d_each);
+        for (; d + 8 <= d_end; d += 8) {
             float wv[8];
 #pragma unroll
             for (int u = 0; u < 8; ++u) wv[u] = to_float(w[(size_t)(d + u) * rank + r]);
@@ -186,11 +191,27 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict_
 #pragma unroll
                 for (int i = 0; i < LT_TT; ++i) acc[i] = fmaf(qn[i * dim + d + u], wv[u], acc[i]);
         }
-        for (; d < dim; ++d) {
+        for (; d < d_end; ++d) {
             const float wv = to_float(w[(size_t)d * rank + r]);
 #pragma unroll
             for (int i = 0; i < LT_TT; ++i) acc[i] = fmaf(qn[i * dim + d], wv, acc[i]);
         }
+    }
+    if constexpr (QS > 1) {
+        __shared__ float shares[QS - 1][LT_TT][COLS];
+        if (share > 0) {
+#pragma unroll
+            for (int i = 0; i < LT_TT; ++i) shares[share - 1][i][threadIdx.x % COLS] = acc[i];
+        }
+        __syncthreads();
+        if (share == 0) {
+#pragma unroll
+            for (int q = 0; q < QS - 1; ++q)
+#pragma unroll
+                for (int i = 0; i < LT_TT; ++i) acc[i] += shares[q][i][threadIdx.x];
+        }
+    }
+    if (r < rank && share == 0) {
 #pragma unroll
         for (int i = 0; i < LT_TT; ++i)
             if (i < n) qa[((size_t)(t0 + i) * heads + h) * za + r] = acc[i];
@@ -213,20 +234,24 @@ LLMK_EXPORT int llmk_latent_absorb(float* qa, const void* q, long long ldq, cons
     if (pairing != LLMK_PAIR_INTERLEAVED && pairing != LLMK_PAIR_HALF_SPLIT) LLMK_FAIL("latent_absorb: unknown rotary pairing %d", pairing);
     size_t smem = (size_t)LT_TT * (dim + 2 * rot) * sizeof(float);
     if (smem < (33 + 2 * (size_t)rot) * sizeof(float)) smem = (33 + 2 * (size_t)rot) * sizeof(float);
-    dim3 grid(ceil_div(n_tokens, LT_TT), heads + (cache ? 1 : 0), ceil_div(rank, 128));
+    const bool few = n_tokens <= 4 * LT_TT;
+    dim3 grid(ceil_div(n_tokens, LT_TT), heads + (cache ? 1 : 0), ceil_div(rank, few ? 32 : 128));
     LatentEntries en;
     en.dkv = dkv; en.gain = kv_gain; en.cache = cache; en.slots = slots; en.eps = eps;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
+#define LATENT_ABSORB_LAUNCH(TYPE, QS)                                                                                                    \
+    do {                                                                                                                                  \
+        if (smem > 40 * 1024) cudaFuncSetAttribute(latent_absorb_kernel<TYPE, QS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        e = llmk_launch(latent_absorb_kernel<TYPE, QS>, grid, dim3(128), smem, s, true, (const TYPE*)q, ldq, (const TYPE*)wuk, qa, positions, \
+                        cos_t, sin_t, n_tokens, heads, dim, rot, rank, pairing, en);                                                      \
+    } while (0)
     if (dtype == LLMK_F32) {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(latent_absorb_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        e = llmk_launch(latent_absorb_kernel<float>, grid, dim3(128), smem, s, true, (const float*)q, ldq, (const float*)wuk, qa, positions,
-                        cos_t, sin_t, n_tokens, heads, dim, rot, rank, pairing, en);
+        if (few) LATENT_ABSORB_LAUNCH(float, 4); else LATENT_ABSORB_LAUNCH(float, 1);
     } else if (dtype == LLMK_BF16) {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(latent_absorb_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        e = llmk_launch(latent_absorb_kernel<bf16>, grid, dim3(128), smem, s, true, (const bf16*)q, ldq, (const bf16*)wuk, qa, positions,
-                        cos_t, sin_t, n_tokens, heads, dim, rot, rank, pairing, en);
+        if (few) LATENT_ABSORB_LAUNCH(bf16, 4); else LATENT_ABSORB_LAUNCH(bf16, 1);
     } else
+#undef LATENT_ABSORB_LAUNCH
         LLMK_FAIL("latent_absorb: unknown dtype %d", dtype);
     LLMK_CHECK_LAUNCH_RC("latent_absorb", e);
     return LLMK_OK;
@@ -574,18 +599,19 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_kernel(LatentA
 //   S = Q Z^T          Q rounded to bfloat16 as it enters shared memory, Z as cached; scores float32
 //   O += P Z[:, :rank] the float32 weights P enter as three bfloat16 terms (p = p1 + p2 + p3, 24 bits of mantissa: every
 //                      product p_i z is exact in float32 and the sum is a float32 sum), so the weights are not rounded
-// A block has 8 warps = 2 groups of 16 rows x 4: for the scores a warp takes its group's rows and 8 of the tile's 32
-// keys; the scores pass through shared memory, every warp of a group then does the group's softmax and takes a
-// quarter of the latent's values for the weighted sums.  Rows, tiles, key parts and the merge are those of the
-// kernel above.
+// A block takes 16 RG rows (queries x heads) in RG groups of four warps and walks tiles of 32 cached vectors, which come by
+// `cp.async` into two buffers, the next tile on its way while this one is used.  In a group, per tile:
+//   scores    each warp the group's 16 rows x all 32 keys over a quarter of the vector's steps of 16; the four float32 partial sums
+//             go to shared memory
+//   softmax   each warp four of the rows, a lane a key: the sum of the partials, mask, running maximum and sum; the weights' three
+//             terms go to shared memory
+//   sums      each warp a quarter of the latent's values for all 16 rows
+// with a barrier of the group between them.  Key parts and their merge are those of the kernel above.
 constexpr int MT_KT = 32;
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldmatrix_x2(uint32_t (&r)[2], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
 }
 __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -596,28 +622,44 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t*>(&v);
+__device__ __forceinline__ void cp_async16(void* smem_dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(src) : "memory");
 }
-// p = t1 + t2 + t3 with bfloat16 terms; returns the packed pairs of two neighbouring weights
-__device__ __forceinline__ void split3(float p0, float p1, uint32_t& w1, uint32_t& w2, uint32_t& w3) {
-    const float a0 = __bfloat162float(__float2bfloat16_rn(p0)), a1 = __bfloat162float(__float2bfloat16_rn(p1));
-    const float r0 = p0 - a0, r1 = p1 - a1;
-    const float b0 = __bfloat162float(__float2bfloat16_rn(r0)), b1 = __bfloat162float(__float2bfloat16_rn(r1));
-    w1 = pack_bf16(a0, a1);
-    w2 = pack_bf16(b0, b1);
-    w3 = pack_bf16(r0 - b0, r1 - b1);
+// the largest value of a warp
+__device__ __forceinline__ float redux_max(float v) {
+    float r;
+    asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(r) : "f"(v));
+    return r;
+}
+// 2^x (the hardware's approximation: 2 ulp; results below the smallest normal number are zero)
+__device__ __forceinline__ float pow2(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+__device__ __forceinline__ void group_barrier(int group) {
+    asm volatile("bar.sync %0, 128;" ::"r"(group + 1) : "memory");
 }
 
-template <int NT>       // most tiles of 8 latent values a warp accumulates (rank / 32 of them are used)
-__global__ void __launch_bounds__(256) latent_attention_mma_kernel(LatentAttnParams p) {
+constexpr int MT_SLD = 33;          // row stride of the partial scores (floats)
+constexpr int MT_PLD = 40;          // row stride of the weights' terms (bfloat16): eight rows fall on different banks
+
+static size_t latent_mma_smem(int za, int groups) {
+    return ((size_t)16 * groups + 2 * MT_KT) * (za + 8) * sizeof(bf16) +
+           (size_t)groups * (4 * 16 * MT_SLD * sizeof(float) + 3 * 16 * MT_PLD * sizeof(bf16) + 3 * 16 * sizeof(float));
+}
+
+template <int NT, int RG>       // NT: most tiles of 8 latent values a warp accumulates (rank / 32 of them are used)
+__global__ void __launch_bounds__(128 * RG) latent_attention_mma_kernel(LatentAttnParams p) {
+    constexpr int ROWS = 16 * RG, NWARPS = 4 * RG;
     extern __shared__ __align__(16) unsigned char smem_mma[];
     const int za = p.za, rank = p.rank;
     const int zp = za + 8;                                  // row stride: consecutive rows 16 bytes apart in the banks
-    bf16* Qs = reinterpret_cast<bf16*>(smem_mma);            // [32][zp]
-    bf16* Zs = Qs + LT_ROWS * zp;                            // [32][zp]
-    float* Ss = reinterpret_cast<float*>(Zs + MT_KT * zp);   // [32][33]
+    bf16* Qs = reinterpret_cast<bf16*>(smem_mma);            // [ROWS][zp]
+    bf16* Zb = Qs + ROWS * zp;                               // 2 x [32][zp]
+    float* Sb = reinterpret_cast<float*>(Zb + 2 * MT_KT * zp);      // [RG][4][16][MT_SLD]
+    bf16* Pb = reinterpret_cast<bf16*>(Sb + RG * 4 * 16 * MT_SLD);   // [RG][3][16][MT_PLD]
+    float* Rb = reinterpret_cast<float*>(Pb + RG * 3 * 16 * MT_PLD); // [RG][3][16]: the rows' corrections, maxima, sums
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int rg = warp >> 2, wq = warp & 3;                 // group of 16 rows, quarter
     pdl_launch_dependents();
@@ -648,8 +690,29 @@ __global__ void __launch_bounds__(256) latent_attention_mma_kernel(LatentAttnPar
     }
     const bf16* zc = static_cast<const bf16*>(p.cache);
     const int* bt = p.block_tables + (size_t)s * p.max_blocks;
+    const int vecs = za / 8;
+    // a tile's cached vectors: a warp takes keys warp, warp + NWARPS, ...; the pages of its keys are looked up first
+    auto load_tile = [&](int t0, int buf) {
+        constexpr int PER = MT_KT / NWARPS;
+        bf16* Zd = Zb + buf * MT_KT * zp;
+        const bf16* src[PER];
+#pragma unroll
+        for (int kk = 0; kk < PER; ++kk) {
+            const int kpos = t0 + warp + kk * NWARPS;
+            src[kk] = kpos < k_end ? zc + ((size_t)bt[kpos / p.page_size] * p.page_size + kpos % p.page_size) * za : nullptr;
+        }
+#pragma unroll
+        for (int kk = 0; kk < PER; ++kk) {
+            bf16* dst = Zd + (warp + kk * NWARPS) * zp;
+            for (int vec = lane; vec < vecs; vec += 32) {
+                if (src[kk]) cp_async16(dst + vec * 8, src[kk] + (size_t)vec * 8);
+                else *reinterpret_cast<uint4*>(dst + vec * 8) = make_uint4(0u, 0u, 0u, 0u);
+            }
+        }
+    };
+    if (k_beg < k_end) load_tile(k_beg, 0);
     // the block's queries, rounded to bfloat16
-    for (int r = warp; r < LT_ROWS; r += LT_WARPS) {
+    for (int r = warp; r < ROWS; r += NWARPS) {
         const int qi = r / p.gc, hh = chunk * p.gc + r % p.gc;
         const bool live = r < rows && qi < nq_tile && hh < p.heads;
         if (p.qa_hm) {
@@ -665,18 +728,23 @@ __global__ void __launch_bounds__(256) latent_attention_mma_kernel(LatentAttnPar
             *reinterpret_cast<__nv_bfloat162*>(Qs + r * zp + d) = __floats2bfloat162_rn(v.x, v.y);
         }
     }
-    // this lane's two rows of its group: g and g + 8
-    int qpos[2];
-    bool valid[2];
+    float* Ss = Sb + rg * 4 * 16 * MT_SLD;
+    bf16* Ps = Pb + rg * 3 * 16 * MT_PLD;
+    float* corr_s = Rb + rg * 3 * 16;
+    float* m_s = corr_s + 16;
+    float* l_s = m_s + 16;
+    // the softmax's four rows of this warp
+    int qpos[4];
+    bool valid[4];
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-        const int r = rg * 16 + (lane >> 2) + 8 * i;
+    for (int i = 0; i < 4; ++i) {
+        const int r = rg * 16 + wq * 4 + i;
         const int qi = r / p.gc, hh = chunk * p.gc + r % p.gc;
         valid[i] = r < rows && qi < nq_tile && hh < p.heads && !padding;
         qpos[i] = first_pos + qi;
     }
-    const bool group_live = rg * 16 < rows && (rg * 16) / p.gc < nq_tile;      // uniform over the warp
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    const bool group_live = rg * 16 < rows && (rg * 16) / p.gc < nq_tile;      // uniform over the group
+    float m[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}, l[4] = {0.f, 0.f, 0.f, 0.f};
     float acc[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; ++j)
@@ -684,158 +752,130 @@ __global__ void __launch_bounds__(256) latent_attention_mma_kernel(LatentAttnPar
         for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
     const int nt = rank / 32;                    // tiles of 8 values this warp accumulates
     const int d0 = wq * nt * 8;
-    const int vecs = za / 8;
+    const int steps = za / 16;
+    const float scale2 = p.scale * 1.4426950408889634f;
+    const int seen = p.window > 0 ? p.window : 0x40000000;
     const uint32_t qs_addr = (uint32_t)__cvta_generic_to_shared(Qs);
-    const uint32_t zs_addr = (uint32_t)__cvta_generic_to_shared(Zs);
+    const uint32_t zb_addr = (uint32_t)__cvta_generic_to_shared(Zb);
+    const uint32_t ps_addr = (uint32_t)__cvta_generic_to_shared(Ps);
 
-    for (int t0 = k_beg; t0 < k_end; t0 += MT_KT) {
-        __syncthreads();                         // the tile before is consumed (and Qs written, the first time)
-        // the tile's cached vectors: a warp takes keys warp, warp + 8, ...; the pages of its four keys are looked up
-        // first, then the lanes go across the vectors, the loads of two keys in flight before their stores
+    int turn = 0;
+    for (int t0 = k_beg; t0 < k_end; t0 += MT_KT, turn ^= 1) {
+        asm volatile("cp.async.wait_all;" ::: "memory");
+        __syncthreads();                         // this tile has arrived (and Qs, the first time); the tile before is consumed
+        if (t0 + MT_KT < k_end) load_tile(t0 + MT_KT, turn ^ 1);
+        if (!group_live) continue;
+        const uint32_t zs_addr = zb_addr + (uint32_t)(turn * MT_KT * zp * 2);
         {
-            const bf16* src[MT_KT / LT_WARPS];
-#pragma unroll
-            for (int kk = 0; kk < MT_KT / LT_WARPS; ++kk) {
-                const int kpos = t0 + warp + kk * LT_WARPS;
-                src[kk] = kpos < k_end ? zc + ((size_t)bt[kpos / p.page_size] * p.page_size + kpos % p.page_size) * za : nullptr;
-            }
-#pragma unroll
-            for (int kk = 0; kk < MT_KT / LT_WARPS; kk += 2) {
-                for (int vec = lane; vec < vecs; vec += 32) {
-                    uint4 v0 = make_uint4(0u, 0u, 0u, 0u), v1 = v0;
-                    if (src[kk]) v0 = *reinterpret_cast<const uint4*>(src[kk] + (size_t)vec * 8);
-                    if (src[kk + 1]) v1 = *reinterpret_cast<const uint4*>(src[kk + 1] + (size_t)vec * 8);
-                    *reinterpret_cast<uint4*>(Zs + (warp + kk * LT_WARPS) * zp + vec * 8) = v0;
-                    *reinterpret_cast<uint4*>(Zs + (warp + (kk + 1) * LT_WARPS) * zp + vec * 8) = v1;
-                }
-            }
-        }
-        __syncthreads();
-        // scores of the group's 16 rows with keys 8 wq .. 8 wq + 7
-        if (group_live) {
-            // four accumulators in turn, so that consecutive products do not wait for one another
-            float c4[4][4];
+            float c[4][4];
 #pragma unroll
             for (int u = 0; u < 4; ++u)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) c4[u][e] = 0.f;
+                for (int e = 0; e < 4; ++e) c[u][e] = 0.f;
             const uint32_t a_base = qs_addr + (uint32_t)(((rg * 16 + (lane & 15)) * zp + (lane >> 4) * 8) * 2);
-            const uint32_t b_base = zs_addr + (uint32_t)(((wq * 8 + (lane & 7)) * zp + ((lane >> 3) & 1) * 8) * 2);
-            const int steps = za / 16;
-            int ks = 0;
-            for (; ks + 4 <= steps; ks += 4) {
-#pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    uint32_t a[4], b[2];
-                    ldmatrix_x4(a, a_base + (uint32_t)((ks + u) * 32));
-                    ldmatrix_x2(b, b_base + (uint32_t)((ks + u) * 32));
-                    mma_bf16(c4[u], a, b[0], b[1]);
-                }
-            }
-            for (; ks < steps; ++ks) {
-                uint32_t a[4], b[2];
+            const uint32_t b_base = zs_addr + (uint32_t)((((lane >> 4) * 8 + (lane & 7)) * zp + ((lane >> 3) & 1) * 8) * 2);
+#pragma unroll 3
+            for (int ks = wq; ks < steps; ks += 4) {
+                uint32_t a[4], b0[4], b1[4];
                 ldmatrix_x4(a, a_base + (uint32_t)(ks * 32));
-                ldmatrix_x2(b, b_base + (uint32_t)(ks * 32));
-                mma_bf16(c4[0], a, b[0], b[1]);
+                ldmatrix_x4(b0, b_base + (uint32_t)(ks * 32));
+                ldmatrix_x4(b1, b_base + (uint32_t)(16 * zp * 2 + ks * 32));
+                mma_bf16(c[0], a, b0[0], b0[1]);
+                mma_bf16(c[1], a, b0[2], b0[3]);
+                mma_bf16(c[2], a, b1[0], b1[1]);
+                mma_bf16(c[3], a, b1[2], b1[3]);
             }
-            float c[4];
+            float* srow = Ss + (wq * 16 + (lane >> 2)) * MT_SLD + (lane & 3) * 2;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) c[e] = (c4[0][e] + c4[1][e]) + (c4[2][e] + c4[3][e]);
-            float* srow = Ss + (rg * 16 + (lane >> 2)) * 33 + wq * 8 + (lane & 3) * 2;
-            srow[0] = c[0] * p.scale;
-            srow[1] = c[1] * p.scale;
-            srow[8 * 33] = c[2] * p.scale;
-            srow[8 * 33 + 1] = c[3] * p.scale;
-        }
-        __syncthreads();
-        if (!group_live) continue;
-        // the group's softmax (every warp of the group does it) in the layout of the next product's first operand
-        float pv[2][2][2][2];                    // [row i][step of 16 keys t][half h][e]
-        float tmax[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
-#pragma unroll
-            for (int t = 0; t < 2; ++t)
-#pragma unroll
-                for (int h = 0; h < 2; ++h)
-#pragma unroll
-                    for (int e = 0; e < 2; ++e) {
-                        const int col = 16 * t + 8 * h + (lane & 3) * 2 + e;
-                        const int kpos = t0 + col;
-                        const bool ok = valid[i] && kpos < k_end && kpos <= qpos[i] && (p.window <= 0 || kpos > qpos[i] - p.window);
-                        const float sv = ok ? Ss[(rg * 16 + (lane >> 2) + 8 * i) * 33 + col] : -INFINITY;
-                        pv[i][t][h][e] = sv;
-                        tmax[i] = fmaxf(tmax[i], sv);
-                    }
-        float corr[2];
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 1));
-            tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 2));
-            const float m_new = fmaxf(m[i], tmax[i]);
-            corr[i] = 1.f;
-            float sum = 0.f;
-            if (m_new > -INFINITY) {
-                corr[i] = m[i] > -INFINITY ? expf(m[i] - m_new) : 0.f;
-#pragma unroll
-                for (int t = 0; t < 2; ++t)
-#pragma unroll
-                    for (int h = 0; h < 2; ++h)
-#pragma unroll
-                        for (int e = 0; e < 2; ++e) {
-                            const float sv = pv[i][t][h][e];
-                            const float pe = sv > -INFINITY ? expf(sv - m_new) : 0.f;
-                            pv[i][t][h][e] = pe;
-                            sum += pe;
-                        }
-                m[i] = m_new;
-            } else {
-#pragma unroll
-                for (int t = 0; t < 2; ++t)
-#pragma unroll
-                    for (int h = 0; h < 2; ++h)
-#pragma unroll
-                        for (int e = 0; e < 2; ++e) pv[i][t][h][e] = 0.f;
+            for (int u = 0; u < 4; ++u) {
+                srow[u * 8] = c[u][0];
+                srow[u * 8 + 1] = c[u][1];
+                srow[8 * MT_SLD + u * 8] = c[u][2];
+                srow[8 * MT_SLD + u * 8 + 1] = c[u][3];
             }
-            sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-            sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-            l[i] = l[i] * corr[i] + sum;
+        }
+        group_barrier(rg);
+        // scores, maxima and weights as powers of two: 2^(s log2(e) - m)
+        const int kpos = t0 + lane;
+        float sv[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float* sp = Ss + (wq * 4 + i) * MT_SLD + lane;
+            const bool ok = valid[i] && kpos < k_end && kpos <= qpos[i] && kpos > qpos[i] - seen;
+            const float sum4 = (sp[0] + sp[16 * MT_SLD]) + (sp[32 * MT_SLD] + sp[48 * MT_SLD]);
+            sv[i] = ok ? sum4 * scale2 : -INFINITY;
         }
 #pragma unroll
-        for (int j = 0; j < NT; ++j) {
-            acc[j][0] *= corr[0]; acc[j][1] *= corr[0];
-            acc[j][2] *= corr[1]; acc[j][3] *= corr[1];
+        for (int i = 0; i < 4; ++i) {
+            const int r = wq * 4 + i;
+            const float m_new = fmaxf(m[i], redux_max(sv[i]));
+            const float base = m_new > -INFINITY ? m_new : 0.f;          // a row that has seen nothing: every weight 2^-inf
+            const float corr = pow2(m[i] - base);
+            const float pe = pow2(sv[i] - base);
+            m[i] = m_new;
+            l[i] = l[i] * corr + pe;                                     // this lane's keys; the lanes are added up at the end
+            if (lane == 0) corr_s[r] = corr;
+            // p = t1 + t2 + t3 with bfloat16 terms
+            const bf16 h1 = __float2bfloat16_rn(pe);
+            const float r1 = pe - __bfloat162float(h1);
+            const bf16 h2 = __float2bfloat16_rn(r1);
+            bf16* pr = Ps + r * MT_PLD + lane;
+            pr[0] = h1;
+            pr[16 * MT_PLD] = h2;
+            pr[32 * MT_PLD] = __float2bfloat16_rn(r1 - __bfloat162float(h2));
         }
-        // weights as three bfloat16 terms, per step of 16 keys: a0 (row g, keys 0-7), a1 (row g + 8), a2 (row g, keys 8-15), a3
-        uint32_t pa[2][3][4];
+        group_barrier(rg);
+        const float corr0 = corr_s[lane >> 2], corr1 = corr_s[(lane >> 2) + 8];
+        if (__any_sync(0xffffffffu, corr0 != 1.f || corr1 != 1.f)) {
 #pragma unroll
-        for (int t = 0; t < 2; ++t)
-#pragma unroll
-            for (int h = 0; h < 2; ++h)
-#pragma unroll
-                for (int i = 0; i < 2; ++i)
-                    split3(pv[i][t][h][0], pv[i][t][h][1], pa[t][0][2 * h + i], pa[t][1][2 * h + i], pa[t][2][2 * h + i]);
+            for (int j = 0; j < NT; ++j) {
+                acc[j][0] *= corr0; acc[j][1] *= corr0;
+                acc[j][2] *= corr1; acc[j][3] *= corr1;
+            }
+        }
         // weighted sums over this warp's quarter of the latent's values
+        const uint32_t p_base = ps_addr + (uint32_t)(((lane & 15) * MT_PLD + (lane >> 4) * 8) * 2);
         const uint32_t v_base = zs_addr + (uint32_t)((((lane & 7) + ((lane >> 3) & 1) * 8) * zp + d0 + (lane >> 4) * 8) * 2);
 #pragma unroll
-        for (int jp = 0; jp < NT / 2; ++jp) {
-            if (2 * jp >= nt) break;
+        for (int t = 0; t < 2; ++t) {
+            uint32_t pa[3][4];
 #pragma unroll
-            for (int t = 0; t < 2; ++t) {
-                uint32_t b[4];
-                ldmatrix_x4_trans(b, v_base + (uint32_t)((t * 16 * zp + jp * 16) * 2));
+            for (int term = 0; term < 3; ++term) ldmatrix_x4(pa[term], p_base + (uint32_t)((term * 16 * MT_PLD + t * 16) * 2));
+            // several steps of 16 columns at a time, a term over all of them before the next: consecutive products on one
+            // accumulator would wait for each other
+            constexpr int U = NT >= 4 ? 2 : 1;
+#pragma unroll
+            for (int jp = 0; jp < NT / 2; jp += U) {
+                if (2 * jp >= nt) break;
+                uint32_t b[U][4];
+#pragma unroll
+                for (int u = 0; u < U; ++u) ldmatrix_x4_trans(b[u], v_base + (uint32_t)((t * 16 * zp + min(jp + u, nt / 2 - 1) * 16) * 2));
 #pragma unroll
                 for (int term = 0; term < 3; ++term) {
-                    mma_bf16(acc[2 * jp], pa[t][term], b[0], b[1]);
-                    mma_bf16(acc[2 * jp + 1], pa[t][term], b[2], b[3]);
+#pragma unroll
+                    for (int u = 0; u < U; ++u) {
+                        if (2 * (jp + u) >= nt) break;
+                        mma_bf16(acc[2 * (jp + u)], pa[term], b[u][0], b[u][1]);
+                        mma_bf16(acc[2 * (jp + u) + 1], pa[term], b[u][2], b[u][3]);
+                    }
                 }
             }
         }
     }
     if (!group_live) return;
+    // the rows' maxima and sums, known to the warps of the softmax, for the warps of the values
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        l[i] = warp_sum(l[i]);
+        if (lane == 0) {
+            m_s[wq * 4 + i] = m[i] * 0.6931471805599453f;                // as a power of e
+            l_s[wq * 4 + i] = l[i];
+        }
+    }
+    group_barrier(rg);
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
-        const int r = rg * 16 + (lane >> 2) + 8 * i;
+        const int r16 = (lane >> 2) + 8 * i, r = rg * 16 + r16;
         if (!(r < rows && r / p.gc < max(nq_tile, 0) && chunk * p.gc + r % p.gc < p.heads)) continue;     // nobody's row
         const size_t tokhead = (size_t)(q_beg + q0 + r / p.gc) * p.heads + chunk * p.gc + r % p.gc;
         if (p.num_parts > 1) {
@@ -848,11 +888,11 @@ __global__ void __launch_bounds__(256) latent_attention_mma_kernel(LatentAttnPar
                 p.part_o[row * rank + d + 1] = acc[j][2 * i + 1];
             }
             if (wq == 0 && (lane & 3) == 0) {
-                p.part_ml[row * 2] = m[i];
-                p.part_ml[row * 2 + 1] = l[i];
+                p.part_ml[row * 2] = m_s[r16];
+                p.part_ml[row * 2 + 1] = l_s[r16];
             }
         } else {
-            const float inv = l[i] > 0.f ? 1.0f / l[i] : 0.f;
+            const float inv = l_s[r16] > 0.f ? 1.0f / l_s[r16] : 0.f;
             if (p.out_hm) {
                 bf16* o = p.out_hm + ((size_t)(chunk * p.gc + r % p.gc) * p.t_pad + (size_t)(q_beg + q0 + r / p.gc)) * rank;
 #pragma unroll
@@ -939,24 +979,34 @@ static int dispatch_latent_attention(const LatentAttnParams& p, dim3 grid, size_
     return launch_latent_attention<T, 16>(p, grid, smem, s);
 }
 
-template <int NT>
-static int launch_latent_attention_mma(const LatentAttnParams& p, dim3 grid, size_t smem, cudaStream_t s) {
+template <int NT, int RG>
+static int launch_latent_attention_mma(const LatentAttnParams& p, dim3 grid, cudaStream_t s) {
+    const size_t smem = latent_mma_smem(p.za, RG);
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(latent_attention_mma_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(latent_attention_mma_kernel<NT, RG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) LLMK_FAIL("latent_attention: cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
     }
-    LLMK_CHECK_LAUNCH_RC("latent_attention", llmk_launch(latent_attention_mma_kernel<NT>, grid, dim3(LT_WARPS * 32), smem, s, true, p));
+    LLMK_CHECK_LAUNCH_RC("latent_attention", llmk_launch(latent_attention_mma_kernel<NT, RG>, grid, dim3(128 * RG), smem, s, true, p));
     return LLMK_OK;
+}
+
+template <int RG>
+static int dispatch_latent_attention_mma(const LatentAttnParams& p, dim3 grid, cudaStream_t s) {
+    const int nt = p.rank / 32;
+    return nt <= 2 ? launch_latent_attention_mma<2, RG>(p, grid, s)
+           : nt <= 4 ? launch_latent_attention_mma<4, RG>(p, grid, s)
+           : nt <= 8 ? launch_latent_attention_mma<8, RG>(p, grid, s)
+                     : launch_latent_attention_mma<16, RG>(p, grid, s);
 }
 
 static int g_latent_mma = 1;     // 0: the float32 kernel for bfloat16 caches too (for measurements and tests)
 LLMK_EXPORT void llmk_latent_attention_set_mma(int on) { g_latent_mma = on; }
 
-// Queries per tile for `heads` heads: rows = bq * gc <= 32.
-LLMK_EXPORT int llmk_latent_attention_tile_queries(int heads) {
-    if (heads <= 0) return 0;
-    const int gc = heads < LT_ROWS ? heads : LT_ROWS;
-    return LT_ROWS / gc;
+// Queries per tile of `rows` (16, 32 or 64) rows for `heads` heads: bq * gc <= rows.
+LLMK_EXPORT int llmk_latent_attention_tile_queries(int heads, int rows) {
+    if (heads <= 0 || rows <= 0) return 0;
+    const int gc = heads < rows ? heads : rows;
+    return rows / gc;
 }
 
 // 1 if a bfloat16 cache of these sizes goes through the tensor cores (and may then leave its result head-major).
@@ -964,19 +1014,28 @@ LLMK_EXPORT int llmk_latent_attention_on_tensor_cores(int rank, int rot, int dty
     return dtype == LLMK_BF16 && g_latent_mma && (rank + rot) % 16 == 0 && rank % 64 == 0 && rank <= 512;
 }
 
+// Rows of a block: what the tensor-core form takes best for portions of prompts (single != 0: for single tokens), 32 elsewhere.
+LLMK_EXPORT int llmk_latent_attention_rows(int heads, int rank, int rot, int single, int dtype) {
+    if (!llmk_latent_attention_on_tensor_cores(rank, rot, dtype)) return LT_ROWS;
+    if (single) return heads <= 16 ? 16 : 32;
+    return latent_mma_smem(rank + rot, 4) <= 220 * 1024 ? 64 : 32;
+}
+
+// `rows`: rows of a block, 32 or, in the tensor-core form, 16, 32 or 64 (a tile holds rows / min(heads, rows) queries).
 // qa_hm (optional, tensor-core form only): the queries as bfloat16 [heads, tq_pad, rank + rot] in place of float32 `qa`.
 // out_hm (optional, tensor-core form only): the result as bfloat16 [heads, t_pad, rank] instead of float32 in `out`.
 LLMK_EXPORT int llmk_latent_attention(float* out, const float* qa, const void* cache, const int* block_tables, int max_blocks,
                                       const int* ctx_len, const int* cu_q, const int* tile_seq, const int* tile_q0, int n_tiles,
                                       int n_tokens, int heads, int rank, int rot, int page_size, float scale, int window, int num_parts,
-                                      float* scratch, void* out_hm, int t_pad, const void* qa_hm, int tq_pad, int dtype, void* stream) {
+                                      float* scratch, void* out_hm, int t_pad, const void* qa_hm, int tq_pad, int rows, int dtype, void* stream) {
     if (n_tiles <= 0 || n_tokens <= 0) return LLMK_OK;
     if (heads <= 0 || rank <= 0 || rank > 512 || rot < 0) LLMK_FAIL("latent_attention: bad sizes (heads %d, rank %d, rot %d)", heads, rank, rot);
     if (page_size <= 0) LLMK_FAIL("latent_attention: page_size %d", page_size);
     if (num_parts < 1 || num_parts > 65535 || (num_parts > 1 && !scratch)) LLMK_FAIL("latent_attention: bad split (%d parts)", num_parts);
+    if (rows != 16 && rows != 32 && rows != 64) LLMK_FAIL("latent_attention: blocks of %d rows (16, 32 or 64)", rows);
     LatentAttnParams p;
-    p.gc = heads < LT_ROWS ? heads : LT_ROWS;
-    p.bq = LT_ROWS / p.gc;
+    p.gc = heads < rows ? heads : rows;
+    p.bq = rows / p.gc;
     p.chunks = ceil_div(heads, p.gc);
     p.qa = qa; p.cache = cache; p.out = out; p.block_tables = block_tables; p.ctx_len = ctx_len; p.cu_q = cu_q;
     p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.max_blocks = max_blocks; p.heads = heads; p.rank = rank; p.za = rank + rot;
@@ -996,14 +1055,13 @@ LLMK_EXPORT int llmk_latent_attention(float* out, const float* qa, const void* c
     const bool mma = llmk_latent_attention_on_tensor_cores(rank, rot, dtype) && host_aligned16(cache) && ((uintptr_t)qa & 7) == 0;
     if (qa_hm && (!mma || tq_pad < n_tokens || !host_aligned16(qa_hm))) LLMK_FAIL("latent_attention: head-major queries need the tensor-core form and room for %d tokens", n_tokens);
     if (!qa_hm && !qa) LLMK_FAIL("latent_attention: no queries");
+    if (!mma && rows != LT_ROWS) LLMK_FAIL("latent_attention: blocks of %d rows need the tensor-core form", rows);
     if (out_hm && (!mma || t_pad < n_tokens)) LLMK_FAIL("latent_attention: a head-major result needs the tensor-core form and room for %d tokens", n_tokens);
     if (mma) {
-        const size_t smem_mma = ((size_t)(LT_ROWS + MT_KT) * (p.za + 8)) * sizeof(bf16) + (size_t)LT_ROWS * 33 * sizeof(float);
-        const int nt = rank / 32;
-        rc = nt <= 2 ? launch_latent_attention_mma<2>(p, grid, smem_mma, s)
-             : nt <= 4 ? launch_latent_attention_mma<4>(p, grid, smem_mma, s)
-             : nt <= 8 ? launch_latent_attention_mma<8>(p, grid, smem_mma, s)
-                       : launch_latent_attention_mma<16>(p, grid, smem_mma, s);
+        if (latent_mma_smem(p.za, rows / 16) > 226 * 1024) LLMK_FAIL("latent_attention: %d rows of %d values do not fit shared memory", rows, p.za);
+        rc = rows == 16 ? dispatch_latent_attention_mma<1>(p, grid, s)
+             : rows == 32 ? dispatch_latent_attention_mma<2>(p, grid, s)
+                          : dispatch_latent_attention_mma<4>(p, grid, s);
     } else if (dtype == LLMK_F32)
         rc = dispatch_latent_attention<float>(p, grid, smem, s);
     else if (dtype == LLMK_BF16)

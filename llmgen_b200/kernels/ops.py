@@ -1406,8 +1406,15 @@ def latent_attention_set_mma(on: bool) -> None:
     build.load("latent_attention").llmk_latent_attention_set_mma(c_int(1 if on else 0))
 
 
-def latent_attention_tile_queries(heads: int) -> int:
-    return int(build.load("latent_attention").llmk_latent_attention_tile_queries(c_int(heads)))
+def latent_attention_tile_queries(heads: int, rows: int = 32) -> int:
+    """Queries per tile of `latent_attention` with blocks of `rows` rows."""
+    return int(build.load("latent_attention").llmk_latent_attention_tile_queries(c_int(heads), c_int(rows)))
+
+
+def latent_attention_rows(dtype: torch.dtype, heads: int, rank: int, rot: int, single: bool) -> int:
+    """Rows (queries x heads) of a block that suit portions of prompts (`single`: single tokens) best."""
+    return int(build.load("latent_attention").llmk_latent_attention_rows(c_int(heads), c_int(rank), c_int(rot), c_int(1 if single else 0),
+                                                                         c_int(dtype_code(dtype))))
 
 
 def latent_attention_scratch_floats(n_tokens: int, heads: int, rank: int, parts: int) -> int:
@@ -1423,12 +1430,13 @@ def latent_attention(out: Optional[torch.Tensor], qa: Optional[torch.Tensor], ca
                      ctx_len: torch.Tensor, cu_q: torch.Tensor, tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tokens: int,
                      heads: int, rank: int, rot: int, page_size: int, scale: float, parts: int = 1,
                      scratch: Optional[torch.Tensor] = None, out_head_major: Optional[torch.Tensor] = None, window: int = 0,
-                     q_head_major: Optional[torch.Tensor] = None) -> None:
+                     q_head_major: Optional[torch.Tensor] = None, rows: int = 32) -> None:
     """out float32 [n, heads, rank] = causal softmax attention of qa over the cached vectors (one shared kv head whose
     values are the first `rank` entries of the cached vector).  With `out_head_major` (bfloat16 [heads, t_pad, rank]; the
     tensor-core form only) the result goes there instead, rounded, for the grouped product that follows.  `q_head_major`
     (bfloat16 [heads, t_pad, rank + rot]; the tensor-core form only): the queries, in place of float32 `qa`.  `window` > 0: a
-    query sees the last `window` positions up to its own."""
+    query sees the last `window` positions up to its own.  `rows`: rows of a block (`latent_attention_rows`); the tiles hold
+    `latent_attention_tile_queries(heads, rows)` queries."""
     lib = build.load("latent_attention")
     t_pad = 0
     if out_head_major is not None:
@@ -1452,7 +1460,7 @@ def latent_attention(out: Optional[torch.Tensor], qa: Optional[torch.Tensor], ca
                                           _ptr(cu_q), _ptr(tile_seq), _ptr(tile_q0), c_int(tile_seq.numel()), c_int(n_tokens),
                                           c_int(heads), c_int(rank), c_int(rot), c_int(page_size), c_float(scale), c_int(window), c_int(parts),
                                           _ptr(scratch), _ptr(out_head_major), c_int(t_pad), _ptr(q_head_major), c_int(tq_pad),
-                                          c_int(dtype_code(cache.dtype)), _stream()),
+                                          c_int(rows), c_int(dtype_code(cache.dtype)), _stream()),
            2 if parts > 1 else 1)
 
 

@@ -107,7 +107,9 @@ class LatentAttention(Mixer):
         self.eps = float(spec.kv_norm.eps) if spec.kv_norm is not None else 0.0
         self.position = build_position(spec.position, weights, dtype, device) if spec.position is not None and self.rope else None
         self.pairing = getattr(self.position, "pairing", "half") if self.position is not None else "half"
-        self.bq = ops.latent_attention_tile_queries(self.heads)
+        # rows (queries x heads) of an attention block, and queries per tile, for portions of prompts and for single tokens
+        self.rows, self.rows_single = (ops.latent_attention_rows(dtype, self.heads, self.kv_rank, self.rope, single) for single in (False, True))
+        self.bq, self.bq_single = (ops.latent_attention_tile_queries(self.heads, r) for r in (self.rows, self.rows_single))
         self.sm_count = ops.sm_count(device)
         # bfloat16 caches whose sizes fit leave the attention head-major in bfloat16, and Wuv runs as one grouped tensor-core
         # product over all heads (a group per head); the list of the tiles' heads is made once per padded token count
@@ -126,10 +128,10 @@ class LatentAttention(Mixer):
         return self.position.max_positions if self.position is not None else None
 
     def step_arrays_key(self):
-        return ("attention_tiles", self.bq)
+        return ("attention_tiles", self.bq, self.bq_single)
 
     def prepare_step(self, builder) -> None:
-        add_query_tiles(builder, self.bq)
+        add_query_tiles(builder, self.bq_single if builder.pure_decode else self.bq)
 
     def workspace_bytes(self, tokens: int) -> int:
         elem = 2 if self.dtype == torch.bfloat16 else 4
@@ -141,15 +143,15 @@ class LatentAttention(Mixer):
         return tokens * per_token + ops.SLICED_PRODUCT_BYTES
 
     def _parts(self, ctx) -> int:
-        """Key parts of a step of single tokens: two blocks an SM, at least 128 keys a part (four tiles of the kernel), at
+        """Key parts of a step of single tokens: two blocks an SM, at least 64 keys a part (two tiles of the kernel), at
         most 32 parts; every sequence's own (visible) keys are cut evenly, so the bound of the step's context class decides."""
         if not ctx.pure_decode:
             return 1
-        blocks = max(1, ctx.n_seqs * ((self.heads + 31) // 32))
+        blocks = max(1, ctx.n_seqs * ((self.heads + self.rows_single - 1) // self.rows_single))
         longest = max(ctx.max_ctx_bound, ctx.max_ctx, 1)
         if self.window:
             longest = min(longest, self.window)
-        return max(1, min((2 * self.sm_count) // blocks, longest // 128, 32))
+        return max(1, min((2 * self.sm_count) // blocks, longest // 64, 32))
 
     def _padded(self, ws, T: int):
         """(rows per head of a head-major array of T tokens, rows to make room for): whole tiles of the grouped product."""
@@ -199,14 +201,15 @@ class LatentAttention(Mixer):
         cos, sin = self.position.tables() if self.position is not None else (None, None)
         packed = linear(x, self.w_in, ws.buffer("latent_in", T, self.w_in.shape[0], self.dtype))
         qa, qa_hm = (self._direct_query if self.direct else self._latent_query)(ctx, packed, cache, group, cos, sin)
-        name = f"attention_tiles_bq{self.bq}"
+        bq, rows = (self.bq_single, self.rows_single) if ctx.pure_decode else (self.bq, self.rows)
+        name = f"attention_tiles_bq{bq}"
         parts = self._parts(ctx)
         scratch = None
         if parts > 1:
             scratch = ws.flat("latent_split", ops.latent_attention_scratch_floats(T, n, self.kv_rank, parts), torch.float32)
         gate = packed[:, self.g_off:] if self.spec.gate_proj else None
         y = ws.buffer("latent_y", T, n * self.vd, self.dtype)
-        attend = dict(window=self.window, q_head_major=qa_hm)
+        attend = dict(window=self.window, q_head_major=qa_hm, rows=rows)
         if self.grouped_expand:
             t_pad, cap = self._padded(ws, T)
             oa_hm = ws.buffer("latent_oa_hm", n * t_pad, self.kv_rank, self.dtype, capacity_rows=cap)
