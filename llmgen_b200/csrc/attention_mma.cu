@@ -86,6 +86,9 @@ __device__ __forceinline__ float pow2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
     return r;
 }
+// x / d where d's shift is known (d a power of two), else by division
+__device__ __forceinline__ int quotient(int x, int d, int shift) { return shift >= 0 ? x >> shift : x / d; }
+__device__ __forceinline__ int shift_of(int d) { return (d & (d - 1)) == 0 ? __ffs(d) - 1 : -1; }
 // two float32 as three pairs of bfloat16: x = w1 + w2 + w3, the most significant pieces first
 __device__ __forceinline__ void split3(float x0, float x1, uint32_t& w1, uint32_t& w2, uint32_t& w3) {
     w1 = pack2(x0, x1);
@@ -125,6 +128,7 @@ __global__ void __launch_bounds__(WARPS * 32, SHARED || VD == 64 ? 3 : 2) attent
     int k_beg = p.window > 0 ? max(0, first_pos - p.window + 1) / BN * BN : 0;
     if (p.chunk > 0) k_beg = max(k_beg, first_pos / p.chunk * p.chunk / BN * BN);
     const int* bt = p.block_tables + (size_t)s * p.max_blocks;
+    const int page_shift = shift_of(p.page_size);
 
     for (int idx = threadIdx.x; idx < BM * (HD / 8); idx += blockDim.x) {
         const int r = idx / (HD / 8), v = idx % (HD / 8);
@@ -157,9 +161,10 @@ __global__ void __launch_bounds__(WARPS * 32, SHARED || VD == 64 ? 3 : 2) attent
             const int key = idx / VECS, v = idx % VECS;
             const int kpos = t0 + key;
             bf16* dst = v < HD / 8 ? Kd + key * QLD + v * 8 : Vd + key * VLD + (v - HD / 8) * 8;
-            const int page = kpos < k_end ? bt[kpos / p.page_size] : -1;      // -1 too: a page the window has passed
+            const int at = quotient(kpos, p.page_size, page_shift);
+            const int page = kpos < k_end ? bt[at] : -1;      // -1 too: a page the window has passed
             if (page >= 0) {
-                const size_t row = ((size_t)page * p.nkv + kvh) * p.page_size + kpos % p.page_size;
+                const size_t row = ((size_t)page * p.nkv + kvh) * p.page_size + (kpos - at * p.page_size);
                 cp_async16(dst, v < HD / 8 ? p.kcache + row * HD + v * 8 : p.vcache + row * VD + (v - HD / 8) * 8);
             } else {
                 *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
@@ -168,8 +173,9 @@ __global__ void __launch_bounds__(WARPS * 32, SHARED || VD == 64 ? 3 : 2) attent
         if constexpr (SHARED) {
             for (int key = threadIdx.x; key < BN; key += WARPS * 32) {
                 const int kpos = t0 + key;
-                const int page = kpos < k_end ? bt[kpos / p.page_size] : -1;
-                if (page >= 0) cp_async4(Sbuf + buf * BN + key, p.k_scale + (size_t)page * p.page_size + kpos % p.page_size);
+                const int at = quotient(kpos, p.page_size, page_shift);
+                const int page = kpos < k_end ? bt[at] : -1;
+                if (page >= 0) cp_async4(Sbuf + buf * BN + key, p.k_scale + (size_t)page * p.page_size + (kpos - at * p.page_size));
                 else Sbuf[buf * BN + key] = 0.f;
             }
         }
@@ -409,6 +415,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
         k_end = min(qpos + 1, k_beg + size);
     }
     const int* bt = p.block_tables + (size_t)s * p.max_blocks;
+    const int page_shift = shift_of(p.page_size);
     const int page0 = k_beg / p.page_size;
     const int n_pages = k_beg < k_end ? (k_end - 1) / p.page_size - page0 + 1 : 0;
     const bool staged = n_pages <= PPAGES;
@@ -426,7 +433,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_mma_parts_kernel(Params 
             const int key = idx / VECS, v = idx % VECS;
             const int kpos = t0 + key;
             bf16* dst = v < HD / 8 ? Kd + key * QLD + v * 8 : Vd + key * VLD + (v - HD / 8) * 8;
-            const int at = kpos / p.page_size;
+            const int at = quotient(kpos, p.page_size, page_shift);
             const int page = kpos < k_end ? (staged ? pages[at - page0] : bt[at]) : -1;
             if (page >= 0) {
                 const int off = kpos - at * p.page_size;

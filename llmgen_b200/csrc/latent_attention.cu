@@ -690,6 +690,7 @@ __global__ void __launch_bounds__(128 * RG) latent_attention_mma_kernel(LatentAt
     }
     const bf16* zc = static_cast<const bf16*>(p.cache);
     const int* bt = p.block_tables + (size_t)s * p.max_blocks;
+    const int page_shift = (p.page_size & (p.page_size - 1)) == 0 ? __ffs(p.page_size) - 1 : -1;
     const int vecs = za / 8;
     // a tile's cached vectors: a warp takes keys warp, warp + NWARPS, ...; the pages of its keys are looked up first
     auto load_tile = [&](int t0, int buf) {
@@ -699,7 +700,8 @@ __global__ void __launch_bounds__(128 * RG) latent_attention_mma_kernel(LatentAt
 #pragma unroll
         for (int kk = 0; kk < PER; ++kk) {
             const int kpos = t0 + warp + kk * NWARPS;
-            src[kk] = kpos < k_end ? zc + ((size_t)bt[kpos / p.page_size] * p.page_size + kpos % p.page_size) * za : nullptr;
+            const int at = page_shift >= 0 ? kpos >> page_shift : kpos / p.page_size;
+            src[kk] = kpos < k_end ? zc + ((size_t)bt[at] * p.page_size + (kpos - at * p.page_size)) * za : nullptr;
         }
 #pragma unroll
         for (int kk = 0; kk < PER; ++kk) {
