@@ -169,15 +169,13 @@ def test_tensor_core_attention_over_entries_that_are_key_and_value(nq, nkv, hd, 
     close(out, want, 1e-2)
 
 
-@pytest.mark.parametrize("shared", [True, False])
-@pytest.mark.parametrize("nq,nkv,hd,vd,page", [(6, 3, 64, 64, 16), (2, 1, 128, 128, 32), (4, 4, 128, 128, 16), (20, 1, 64, 64, 16), (4, 2, 64, 128, 16),
-                                               (6, 2, 128, 64, 16)])
+@pytest.mark.parametrize("nq,nkv,hd,vd,page,shared", [
+    (6, 3, 64, 64, 16, True), (2, 1, 128, 128, 32, True), (4, 4, 128, 128, 16, True), (20, 1, 64, 64, 16, True),
+    (6, 3, 64, 64, 48, False), (4, 4, 128, 128, 16, False), (20, 1, 64, 64, 16, False), (4, 2, 64, 128, 16, False), (6, 2, 128, 64, 16, False)])
 def test_single_tokens_on_the_tensor_cores_with_their_keys_in_a_cluster_of_parts(nq, nkv, hd, vd, page, shared):
     """Sequences of 1 to 300 keys in one step, one without a token and one of padding, parts beyond the keys there are; windows,
     blocks of positions, a bound on the scores and sinks; entries that are key and value, or two arrays."""
     from llmgen_b200.kernels import ops
-    if shared and hd != vd:
-        pytest.skip("keys that are values have one width")
     scale, lens = 0.25, [300, 1, 64, 65, 0, 130]
     seqs = [entries(max(n, 1), nkv, hd, page, torch.bfloat16, 5 + 2 * i) for i, n in enumerate(lens)]
     values = [rnd((max(n, 1), nkv, vd), 40 + i, 1.0, torch.bfloat16) for i, n in enumerate(lens)]
