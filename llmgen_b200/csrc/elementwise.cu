@@ -21,7 +21,8 @@ LLMK_DEFINE_LAST_ERROR()
 template <typename T>
 __global__ void embed_rows_kernel(float* __restrict__ out, const T* __restrict__ table,
                                   const int* __restrict__ ids, const int* __restrict__ ids_from,
-                                  const int* __restrict__ sampled, int H, int V, int* bad, float scale) {
+                                  const int* __restrict__ sampled, int H, int V, int* bad, float scale,
+                                  const T* __restrict__ pos_table, const int* __restrict__ positions, int n_pos) {
     const int t = blockIdx.x;
     pdl_launch_dependents();
     pdl_wait();
@@ -31,21 +32,32 @@ __global__ void embed_rows_kernel(float* __restrict__ out, const T* __restrict__
     if (!ok && threadIdx.x == 0 && bad) atomicAdd(bad, 1);
     const T* row = table + (size_t)(ok ? id : 0) * H;
     float* dst = out + (size_t)t * H;
+    if (pos_table) {          // learned positions (a position beyond the table, which the engine's limits exclude, adds nothing)
+        const int p = positions[t];
+        const bool in = p >= 0 && p < n_pos;
+        const T* prow = pos_table + (size_t)(in ? p : 0) * H;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = (ok ? to_float(row[i]) * scale : 0.f) + (in ? to_float(prow[i]) : 0.f);
+        return;
+    }
     for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = ok ? to_float(row[i]) * scale : 0.f;
 }
 
 LLMK_EXPORT int llmk_embed_rows(float* out, const void* table, const int* ids, const int* ids_from, const int* sampled,
-                                int n_tokens, int H, int V, int* bad_flag, int dtype, float scale, void* stream) {
+                                int n_tokens, int H, int V, int* bad_flag, int dtype, float scale, const void* pos_table,
+                                const int* positions, int n_pos, void* stream) {
     if (n_tokens <= 0) return LLMK_OK;
+    if (pos_table && (!positions || n_pos <= 0)) LLMK_FAIL("embed_rows: a table of positions needs the tokens' positions");
     if (H <= 0 || V <= 0) LLMK_FAIL("embed_rows: bad sizes H=%d V=%d", H, V);
     if ((ids_from != nullptr) != (sampled != nullptr)) LLMK_FAIL("embed_rows: ids_from and sampled come together");
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = H >= 1024 ? 256 : 128;
     cudaError_t e;
     if (dtype == LLMK_F32)
-        e = llmk_launch(embed_rows_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, true, out, (const float*)table, ids, ids_from, sampled, H, V, bad_flag, scale);
+        e = llmk_launch(embed_rows_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, true, out, (const float*)table, ids, ids_from, sampled, H, V, bad_flag, scale,
+                        (const float*)pos_table, positions, n_pos);
     else if (dtype == LLMK_BF16)
-        e = llmk_launch(embed_rows_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, true, out, (const bf16*)table, ids, ids_from, sampled, H, V, bad_flag, scale);
+        e = llmk_launch(embed_rows_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, true, out, (const bf16*)table, ids, ids_from, sampled, H, V, bad_flag, scale,
+                        (const bf16*)pos_table, positions, n_pos);
     else
         LLMK_FAIL("embed_rows: unknown dtype %d", dtype);
     LLMK_CHECK_LAUNCH_RC("embed_rows", e);

@@ -4,7 +4,8 @@
 //   moe_route     per token: z = Wr h (+ b) (float32), s = sigmoid(z) or softmax(z), the `top` largest s choose experts;
 //                 slot t * top + c holds (expert, weight); or the `top` largest z choose and the weights are the softmax
 //                 over the chosen z alone.  A correction per expert may be added to s for the choice (not for the weights), and
-//                 the weights may be multiplied by a constant
+//                 the weights may be multiplied by a constant.  The outputs may form groups of neighbours of which only the best
+//                 few (by their largest value that chooses) take part, and one more row of Wr may be a gate sigmoid(z) beside them
 //   moe_plan      one block: slots grouped by expert, cut into tiles of TT rows of one expert each; the list of tiles
 //                 has a fixed length (slots / TT + experts), padded with expert -1
 //   moe_experts   grid (tiles, column blocks): first product of a tile's rows with its expert's matrices and the
@@ -13,7 +14,8 @@
 //   moe_gather    for the tensor-core path: the rows (times their weights) sorted by expert into tiles of 128, every
 //                 expert's rows starting on a tile; the grouped product of csrc/gemm_tc.cu then takes the list of the
 //                 tiles' experts from the device
-//   moe_combine   per token: shared expert's output (if any) + its slots' outputs in slot order
+//   moe_combine   per token: shared expert's output (if any, behind its gate) + its slots' outputs in slot order; a slot whose
+//                 expert lies beyond the real ones adds the token's own row
 //
 // The weight multiplies the expert's input (mode "input") or its output (mode "output").
 // Gated activation: g' = min(g, L), u' = clamp(u, -L, L), y = g' sigmoid(alpha g') (u' + 1)   (L <= 0: no clamp),
@@ -37,8 +39,12 @@ __global__ void __launch_bounds__(TOK > 1 ? 256 : 1024) moe_route_kernel(const T
                                                         const float* __restrict__ bias, int* __restrict__ slot_expert,
                                                         float* __restrict__ slot_weight, int n_tokens, int K, int E, int top, int scoring,
                                                         int renorm, const float* __restrict__ choice_bias, float weight_scale,
-                                                        float sum_eps) {
-    extern __shared__ float sm[];   // [TOK][K] the rows in float32, [TOK][E] scores, [TOK][E] what chooses (with `choice_bias`)
+                                                        float sum_eps, int groups, int keep, float* __restrict__ gate_out) {
+    // [TOK][K] the rows in float32, [TOK][NE] scores (the gate's row last), [TOK][NE] what chooses (with `choice_bias` or
+    // groups), [TOK][groups] the groups' largest
+    extern __shared__ float sm[];
+    const int NE = E + (gate_out ? 1 : 0);
+    const bool apart = choice_bias || groups > 1;
     float* xs = sm;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     const int t0 = blockIdx.x * TOK, n = min(TOK, n_tokens - t0);
@@ -50,7 +56,7 @@ __global__ void __launch_bounds__(TOK > 1 ? 256 : 1024) moe_route_kernel(const T
     }
     __syncthreads();
     const bool vec = (K & 3) == 0;
-    for (int e = warp; e < E; e += nwarps) {
+    for (int e = warp; e < NE; e += nwarps) {
         const float* w = wr + (size_t)e * K;
         float acc[TOK];
 #pragma unroll
@@ -75,14 +81,15 @@ __global__ void __launch_bounds__(TOK > 1 ? 256 : 1024) moe_route_kernel(const T
 #pragma unroll
         for (int i = 0; i < TOK; ++i) {
             acc[i] = warp_sum(acc[i]);
-            if (lane == 0) sm[TOK * K + i * E + e] = acc[i] + (bias ? bias[e] : 0.f);
+            if (lane == 0) sm[TOK * K + i * NE + e] = acc[i] + (bias && e < E ? bias[e] : 0.f);
         }
     }
     __syncthreads();
     for (int i = warp; i < n; i += nwarps) {        // a warp scores and picks for a token
         const size_t t = t0 + i;
-        float* s = sm + TOK * K + i * E;
-        float* by = choice_bias ? s + TOK * E : s;
+        float* s = sm + TOK * K + i * NE;
+        float* by = apart ? s + TOK * NE : s;
+        if (gate_out && lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-s[E]));
         if (scoring == 2) {
             // the logits choose
         } else if (scoring == 1) {
@@ -96,9 +103,26 @@ __global__ void __launch_bounds__(TOK > 1 ? 256 : 1024) moe_route_kernel(const T
         } else {
             for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
         }
-        if (choice_bias)
-            for (int e = lane; e < E; e += 32) by[e] = s[e] + choice_bias[e];
+        if (apart)
+            for (int e = lane; e < E; e += 32) by[e] = s[e] + (choice_bias ? choice_bias[e] : 0.f);
         __syncwarp();
+        if (groups > 1) {
+            const int size = E / groups;
+            float* gm = sm + TOK * K + 2 * TOK * NE + i * groups;
+            for (int g = lane; g < groups; g += 32) {
+                float m = by[g * size];
+                for (int e = 1; e < size; ++e) m = fmaxf(m, by[g * size + e]);
+                gm[g] = m;
+            }
+            __syncwarp();
+            for (int g = lane; g < groups; g += 32) {
+                int before = 0;           // groups that come first: larger, or as large with a smaller index
+                for (int o = 0; o < groups; ++o) before += (gm[o] > gm[g] || (gm[o] == gm[g] && o < g)) ? 1 : 0;
+                if (before >= keep)
+                    for (int e = 0; e < size; ++e) by[g * size + e] = -INFINITY;
+            }
+            __syncwarp();
+        }
         float total = 0.f;
         for (int c = 0; c < top; ++c) {
             // the largest remaining score; ties and values that compare with nothing (NaN) go to the smallest index
@@ -114,7 +138,7 @@ __global__ void __launch_bounds__(TOK > 1 ? 256 : 1024) moe_route_kernel(const T
                 if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
             }
             if (arg >= E) { arg = c < E ? c : 0; best = 0.f; }     // nothing comparable was left: a padded row's garbage
-            else if (choice_bias) best = s[arg];                   // the correction chooses, the score weighs
+            else if (apart) best = s[arg];                   // the correction chooses, the score weighs
             total += best;
             if (lane == 0) {
                 slot_expert[t * top + c] = arg;
@@ -141,22 +165,28 @@ __global__ void __launch_bounds__(TOK > 1 ? 256 : 1024) moe_route_kernel(const T
     }
 }
 
-// `pdl` 0: a plain launch (behind an event of another stream).
+// `pdl` 0: a plain launch (behind an event of another stream).  groups > 1: the E outputs form that many equal groups of which the
+// `keep` best take part.  gate_out [n_tokens] (or null): wr then has one more row, and gate_out receives sigmoid of its product.
 LLMK_EXPORT int llmk_moe_route(const void* h, long long ldh, const float* wr, const float* bias, int* slot_expert, float* slot_weight,
                                int n_tokens, int K, int E, int top, int scoring, int renorm, const float* choice_bias,
-                               float weight_scale, float sum_eps, int pdl, int dtype, void* stream) {
+                               float weight_scale, float sum_eps, int groups, int keep, float* gate_out, int pdl, int dtype,
+                               void* stream) {
     if (n_tokens <= 0) return LLMK_OK;
     if (E <= 0 || top <= 0 || top > E || K <= 0) LLMK_FAIL("moe_route: bad sizes (experts %d, top %d, width %d)", E, top, K);
     if (scoring < 0 || scoring > 2) LLMK_FAIL("moe_route: unknown scoring %d", scoring);
     if (choice_bias && scoring == 2) LLMK_FAIL("moe_route: a correction of the scores needs scores (scoring %d)", scoring);
+    if (groups < 1 || E % groups != 0 || keep < 1 || keep > groups || top > E / groups * keep)
+        LLMK_FAIL("moe_route: %d of %d groups of %d outputs, %d chosen", keep, groups, E, top);
+    if (groups > 1 && scoring == 2) LLMK_FAIL("moe_route: groups need scores (scoring %d)", scoring);
     // four tokens a block where there are blocks for every SM all the same and their rows fit
     constexpr int MANY = 4;
-    const size_t one = ((size_t)K + 2 * E) * sizeof(float);
+    const size_t one = ((size_t)K + 2 * (E + (gate_out ? 1 : 0)) + (groups > 1 ? groups : 0)) * sizeof(float);
     const bool many = n_tokens >= 2 * MANY * device_sm_count() / 2 && MANY * one <= 96 * 1024;
     const size_t smem = many ? MANY * one : one;
     if (smem > 200 * 1024) LLMK_FAIL("moe_route: a row of %d values and %d experts do not fit shared memory", K, E);
     const int most = many ? 8 : n_tokens <= device_sm_count() ? 32 : 8;
-    const int threads = 32 * (E < most ? E : most);
+    const int outputs = E + (gate_out ? 1 : 0);
+    const int threads = 32 * (outputs < most ? outputs : most);
     const dim3 grid(many ? ceil_div(n_tokens, MANY) : n_tokens);
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
@@ -164,7 +194,7 @@ LLMK_EXPORT int llmk_moe_route(const void* h, long long ldh, const float* wr, co
     do {                                                                                                                                 \
         if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<TYPE, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         e = llmk_launch(moe_route_kernel<TYPE, TOK>, grid, dim3(threads), smem, s, pdl != 0, (const TYPE*)h, ldh, wr, bias, slot_expert,  \
-                        slot_weight, n_tokens, K, E, top, scoring, renorm, choice_bias, weight_scale, sum_eps);                          \
+                        slot_weight, n_tokens, K, E, top, scoring, renorm, choice_bias, weight_scale, sum_eps, groups, keep, gate_out);  \
     } while (0)
     if (dtype == LLMK_F32) {
         if (many) MOE_ROUTE_LAUNCH(float, MANY); else MOE_ROUTE_LAUNCH(float, 1);
@@ -410,42 +440,91 @@ LLMK_EXPORT int llmk_moe_experts(float* out, const void* in, long long ld_in, co
 }
 
 // -------------------------------------------------------------------------------------------- combine
-// out[t, c] (float32) = (shared ? shared[t, c] : 0) + sum over the token's slots, in slot order, of rows[pos_of_slot, c]
-// (times the slot's weight where `slot_weight` is given: the weight on an expert's output).
-template <typename T>
-__global__ void moe_combine_kernel(float* __restrict__ out, const float* __restrict__ rows, const int* __restrict__ pos_of_slot,
-                                   const T* __restrict__ shared_out, const float* __restrict__ slot_weight, int n_tokens, int top,
-                                   int H) {
+// out[t, c] (float32) = (shared ? gate[t] * shared[t, c] : 0) + sum over the token's slots, in slot order, of rows[pos_of_slot, c]
+// (times the slot's weight where `slot_weight` is given: the weight on an expert's output).  A slot without a row whose expert is
+// E or more (an output of the router that returns its input) adds its weight times h[t, c].
+struct MoeCombine {
+    float* out;
+    const float* rows;
+    const int* pos_of_slot;
+    const void* shared_out;
+    const float* shared_gate;       // [n_tokens] or null: 1
+    const float* slot_weight;       // on the experts' rows, or null
+    const void* h;                  // identity outputs: the input rows, with slot_expert and their weights; null: none
+    long long ldh;
+    const int* slot_expert;
+    const float* identity_weight;
+    int E, n_tokens, top, H;
+};
+
+template <typename T, int V>
+__global__ void moe_combine_kernel(MoeCombine p) {
     pdl_launch_dependents();
     pdl_wait();
-    const long long total = (long long)n_tokens * H;
+    const int cols = p.H / V;
+    const long long total = (long long)p.n_tokens * cols;
     for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
-        const size_t t = (size_t)(i / H);
-        const int c = (int)(i % H);
-        float v = shared_out ? to_float(shared_out[i]) : 0.f;
-        for (int k = 0; k < top; ++k) {
-            const int pos = pos_of_slot[t * top + k];
-            if (pos >= 0) v += slot_weight ? slot_weight[t * top + k] * rows[(size_t)pos * H + c] : rows[(size_t)pos * H + c];
+        const size_t t = (size_t)(i / cols);
+        const int c = (int)(i % cols) * V;
+        float v[V];
+#pragma unroll
+        for (int u = 0; u < V; ++u) v[u] = 0.f;
+        if (p.shared_out) {
+            const T* sh = static_cast<const T*>(p.shared_out) + t * p.H + c;
+            const float g = p.shared_gate ? p.shared_gate[t] : 1.f;
+#pragma unroll
+            for (int u = 0; u < V; ++u) v[u] = p.shared_gate ? g * to_float(sh[u]) : to_float(sh[u]);
         }
-        out[i] = v;
+        for (int k = 0; k < p.top; ++k) {
+            const size_t slot = t * p.top + k;
+            const int pos = p.pos_of_slot[slot];
+            if (pos >= 0) {
+                const float* row = p.rows + (size_t)pos * p.H + c;
+                const float w = p.slot_weight ? p.slot_weight[slot] : 1.f;
+                float r[V];
+                if (V == 4) {
+                    const float4 q = *reinterpret_cast<const float4*>(row);
+                    r[0] = q.x;
+                    if (V > 1) { r[V > 1 ? 1 : 0] = q.y; r[V > 2 ? 2 : 0] = q.z; r[V > 3 ? 3 : 0] = q.w; }
+                } else {
+                    r[0] = row[0];
+                }
+#pragma unroll
+                for (int u = 0; u < V; ++u) v[u] += p.slot_weight ? w * r[u] : r[u];
+            } else if (p.h && p.slot_expert[slot] >= p.E) {
+                const float w = p.identity_weight[slot];
+                const T* hr = static_cast<const T*>(p.h) + t * p.ldh + c;
+#pragma unroll
+                for (int u = 0; u < V; ++u) v[u] = fmaf(w, to_float(hr[u]), v[u]);
+            }
+        }
+        float* o = p.out + t * p.H + c;
+        if (V == 4) *reinterpret_cast<float4*>(o) = make_float4(v[0], v[V > 1 ? 1 : 0], v[V > 2 ? 2 : 0], v[V > 3 ? 3 : 0]);
+        else o[0] = v[0];
     }
 }
 
-LLMK_EXPORT int llmk_moe_combine(float* out, const float* rows, const int* pos_of_slot, const void* shared_out, const float* slot_weight,
-                                 int n_tokens, int top, int H, int dtype, void* stream) {
-    if (n_tokens <= 0) return LLMK_OK;
-    long long blocks = ((long long)n_tokens * H + 255) / 256;
+template <typename T>
+static cudaError_t launch_combine(const MoeCombine& p, cudaStream_t s) {
+    const bool vec = p.H % 4 == 0 && host_aligned16(p.out) && host_aligned16(p.rows);
+    const long long work = (long long)p.n_tokens * (vec ? p.H / 4 : p.H);
+    long long blocks = (work + 255) / 256;
     if (blocks > device_sm_count() * 16) blocks = device_sm_count() * 16;
+    if (vec) return llmk_launch(moe_combine_kernel<T, 4>, dim3((unsigned)blocks), dim3(256), 0, s, true, p);
+    return llmk_launch(moe_combine_kernel<T, 1>, dim3((unsigned)blocks), dim3(256), 0, s, true, p);
+}
+
+LLMK_EXPORT int llmk_moe_combine(float* out, const float* rows, const int* pos_of_slot, const void* shared_out, const float* shared_gate,
+                                 const float* slot_weight, const void* h, long long ldh, const int* slot_expert, const float* identity_weight,
+                                 int E, int n_tokens, int top, int H, int dtype, void* stream) {
+    if (n_tokens <= 0) return LLMK_OK;
+    if (h && (!slot_expert || !identity_weight)) LLMK_FAIL("moe_combine: identity outputs need the slots' experts and weights");
+    MoeCombine p = {out, rows, pos_of_slot, shared_out, shared_gate, slot_weight, h, ldh, slot_expert, identity_weight, E, n_tokens, top, H};
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
-    if (dtype == LLMK_F32)
-        e = llmk_launch(moe_combine_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, s, true, out, rows, pos_of_slot, (const float*)shared_out,
-                        slot_weight, n_tokens, top, H);
-    else if (dtype == LLMK_BF16)
-        e = llmk_launch(moe_combine_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, s, true, out, rows, pos_of_slot, (const bf16*)shared_out,
-                        slot_weight, n_tokens, top, H);
-    else
-        LLMK_FAIL("moe_combine: unknown dtype %d", dtype);
+    if (dtype == LLMK_F32) e = launch_combine<float>(p, s);
+    else if (dtype == LLMK_BF16) e = launch_combine<bf16>(p, s);
+    else LLMK_FAIL("moe_combine: unknown dtype %d", dtype);
     LLMK_CHECK_LAUNCH_RC("moe_combine", e);
     return LLMK_OK;
 }

@@ -8,6 +8,7 @@
 //   rglru_scan          that recurrence over each sequence's new tokens, times the other branch's gelu
 //   delta_scan          the gated delta rule with a decay per key channel:
 //                       S <- diag(g) S;  d = beta (v - S^T k);  S <- S + k d^T;  o = S^T q
+//   delta_scan_heads    the same with one decay per head, over rows that csrc/head_delta.cu has prepared
 //   token_shift_mix     several blends of every token's row with the row of the token before it, the last row of a
 //                       sequence kept in its state:  m_i[t] = x[t] + (x[t-1] - x[t]) mu_i
 //   decay_scan          linear attention with a decay per key channel, in two orders of a token's steps:
@@ -575,7 +576,7 @@ struct DeltaParams {
     const float* qkv;        // [n_tokens, ld]: q at column 0, k at G * D, v at 2 * G * D, prepared
     long long qkv_ld;
     const float* beta;       // [n_tokens, H + G]: beta of every head, then q . k of every key head
-    const float* decay;      // [n_tokens, H * D]: 1 - g
+    const float* decay;      // [n_tokens, H * D]: 1 - g (null: one decay per head, `beta` is then [n_tokens, 2 H + G]: beta, 1 - g, q . k)
     float* state;            // [slots, state_ld]: S [H][D][E]
     long long state_ld;
     const int* cu_q;
@@ -591,22 +592,24 @@ __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wai
 
 // One chunk's rows into shared memory: q, k, 1 - g as [CHUNK][SL slices][STRIDE] (the padding keeps the slices' 16-byte
 // reads on different banks), v as [CHUNK][COLS], then beta [CHUNK] and q . k [CHUNK].
-template <int DSL, int SL, int WARPS = 4>
+// HEAD: one decay per head: no rows of decays, and 1 - g [CHUNK] behind q . k.
+template <int DSL, int SL, int WARPS = 4, bool HEAD = false>
 struct DeltaShape {
     static constexpr int STRIDE = DSL == 4 ? 12 : DSL + 4;
     static constexpr int ROW = SL * STRIDE;
     static constexpr int COLS = WARPS * (32 / SL);
-    static constexpr int BUF = DELTA_CHUNK * (3 * ROW + COLS) + 2 * DELTA_CHUNK;
+    static constexpr int VS = (HEAD ? 2 : 3) * DELTA_CHUNK * ROW;       // where v begins
+    static constexpr int BUF = VS + DELTA_CHUNK * COLS + (HEAD ? 3 : 2) * DELTA_CHUNK;
 };
 
-template <int DSL, int SL, int WARPS = 4>
+template <int DSL, int SL, int WARPS = 4, bool HEAD = false>
 __device__ __forceinline__ void delta_load_chunk(const DeltaParams& p, float* buf, int t_first, int nc, int h, int kvh, int e0) {
-    using Sh = DeltaShape<DSL, SL, WARPS>;
+    using Sh = DeltaShape<DSL, SL, WARPS, HEAD>;
     constexpr int ROW = Sh::ROW, COLS = Sh::COLS, STRIDE = Sh::STRIDE;
     float* qs = buf;
     float* ks = qs + DELTA_CHUNK * ROW;
     float* gs = ks + DELTA_CHUNK * ROW;
-    float* vs = gs + DELTA_CHUNK * ROW;
+    float* vs = buf + Sh::VS;
     float* bs = vs + DELTA_CHUNK * COLS;
     const int D = p.D, E = p.E, GD = p.G * p.D;
     if (p.vec_ok) {
@@ -617,7 +620,7 @@ __device__ __forceinline__ void delta_load_chunk(const DeltaParams& p, float* bu
             const int at = tt * ROW + (d / DSL) * STRIDE + d % DSL;
             cp_async16(qs + at, p.qkv + t * p.qkv_ld + (size_t)kvh * D + d);
             cp_async16(ks + at, p.qkv + t * p.qkv_ld + GD + (size_t)kvh * D + d);
-            cp_async16(gs + at, p.decay + t * ((size_t)p.H * D) + (size_t)h * D + d);
+            if (!HEAD) cp_async16(gs + at, p.decay + t * ((size_t)p.H * D) + (size_t)h * D + d);
         }
         for (int idx = threadIdx.x; idx < nc * (COLS / 4); idx += WARPS * 32) {
             const int tt = idx / (COLS / 4), cc = (idx % (COLS / 4)) * 4;
@@ -630,7 +633,7 @@ __device__ __forceinline__ void delta_load_chunk(const DeltaParams& p, float* bu
             const int at = tt * ROW + (d / DSL) * STRIDE + d % DSL;
             qs[at] = p.qkv[t * p.qkv_ld + (size_t)kvh * D + d];
             ks[at] = p.qkv[t * p.qkv_ld + GD + (size_t)kvh * D + d];
-            gs[at] = p.decay[t * ((size_t)p.H * D) + (size_t)h * D + d];
+            if (!HEAD) gs[at] = p.decay[t * ((size_t)p.H * D) + (size_t)h * D + d];
         }
         for (int idx = threadIdx.x; idx < nc * COLS; idx += WARPS * 32) {
             const int tt = idx / COLS, cc = idx % COLS;
@@ -638,15 +641,16 @@ __device__ __forceinline__ void delta_load_chunk(const DeltaParams& p, float* bu
         }
     }
     if (threadIdx.x < nc) {
-        const float* row = p.beta + (size_t)(t_first + threadIdx.x) * (p.H + p.G);
+        const float* row = p.beta + (size_t)(t_first + threadIdx.x) * ((HEAD ? 2 : 1) * p.H + p.G);
         bs[threadIdx.x] = row[h];
-        bs[DELTA_CHUNK + threadIdx.x] = row[p.H + kvh];
+        bs[DELTA_CHUNK + threadIdx.x] = row[(HEAD ? 2 : 1) * p.H + kvh];
+        if (HEAD) bs[2 * DELTA_CHUNK + threadIdx.x] = row[p.H + h];
     }
 }
 
-template <int DSL, int SL>
+template <int DSL, int SL, bool HEAD>
 __global__ void __launch_bounds__(DELTA_THREADS) delta_scan_kernel(DeltaParams p) {
-    using Sh = DeltaShape<DSL, SL>;
+    using Sh = DeltaShape<DSL, SL, 4, HEAD>;
     constexpr int ROW = Sh::ROW, COLS = Sh::COLS, STRIDE = Sh::STRIDE, BUF = Sh::BUF;
     extern __shared__ __align__(16) float sm[];
     const int s = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * COLS;
@@ -670,16 +674,16 @@ __global__ void __launch_bounds__(DELTA_THREADS) delta_scan_kernel(DeltaParams p
         S[i] = (st && d < D && e < E) ? st[(size_t)d * E + e] : 0.f;
     }
     __syncthreads();
-    delta_load_chunk<DSL, SL>(p, sm, q_beg, min(DELTA_CHUNK, n), h, kvh, e0);
+    delta_load_chunk<DSL, SL, 4, HEAD>(p, sm, q_beg, min(DELTA_CHUNK, n), h, kvh, e0);
     int turn = 0;
     for (int c0 = 0; c0 < n; c0 += DELTA_CHUNK, turn ^= 1) {
         const int nc = min(DELTA_CHUNK, n - c0);
         cp_async_wait_all();
         __syncthreads();      // this chunk has arrived, and the chunk before is consumed by every warp
         if (c0 + DELTA_CHUNK < n)
-            delta_load_chunk<DSL, SL>(p, sm + (turn ^ 1) * BUF, q_beg + c0 + DELTA_CHUNK, min(DELTA_CHUNK, n - c0 - DELTA_CHUNK), h, kvh, e0);
+            delta_load_chunk<DSL, SL, 4, HEAD>(p, sm + (turn ^ 1) * BUF, q_beg + c0 + DELTA_CHUNK, min(DELTA_CHUNK, n - c0 - DELTA_CHUNK), h, kvh, e0);
         const float* buf = sm + turn * BUF;
-        const float* vs = buf + 3 * DELTA_CHUNK * ROW;
+        const float* vs = buf + Sh::VS;
         const float* bs = vs + DELTA_CHUNK * COLS;
         auto token = [&](int tt) {
             const float4* qr = reinterpret_cast<const float4*>(buf + tt * ROW + slice * STRIDE);
@@ -689,7 +693,10 @@ __global__ void __launch_bounds__(DELTA_THREADS) delta_scan_kernel(DeltaParams p
             float ks4[4] = {0.f, 0.f, 0.f, 0.f}, qs4[4] = {0.f, 0.f, 0.f, 0.f};   // four sums in turn: short chains of dependent adds
 #pragma unroll
             for (int i = 0; i < DSL / 4; ++i) {
-                const float4 g4 = gr[i], k4 = kr[i], q4 = qr[i];
+                float4 g4;
+                if (HEAD) g4.x = g4.y = g4.z = g4.w = bs[2 * DELTA_CHUNK + tt];
+                else g4 = gr[i];
+                const float4 k4 = kr[i], q4 = qr[i];
                 kk[i] = k4;
                 S[4 * i] = fmaf(-g4.x, S[4 * i], S[4 * i]);
                 S[4 * i + 1] = fmaf(-g4.y, S[4 * i + 1], S[4 * i + 1]);
@@ -738,16 +745,16 @@ __global__ void __launch_bounds__(DELTA_THREADS) delta_scan_kernel(DeltaParams p
     }
 }
 
-template <int DSL, int SL>
+template <int DSL, int SL, bool HEAD = false>
 static cudaError_t launch_delta(const DeltaParams& p, int n_seqs, cudaStream_t s) {
-    using Sh = DeltaShape<DSL, SL>;
+    using Sh = DeltaShape<DSL, SL, 4, HEAD>;
     const size_t smem = 2 * (size_t)Sh::BUF * sizeof(float);
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DSL, SL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DSL, SL, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
     dim3 grid(n_seqs, p.H, ceil_div(p.E, Sh::COLS));
-    return llmk_launch(delta_scan_kernel<DSL, SL>, grid, dim3(DELTA_THREADS), smem, s, true, p);
+    return llmk_launch(delta_scan_kernel<DSL, SL, HEAD>, grid, dim3(DELTA_THREADS), smem, s, true, p);
 }
 
 // qkv float32 [n_tokens, >= 2 G D + H E] and decay float32 [n_tokens, H D] are rewritten in place by the preparation;
@@ -783,6 +790,31 @@ LLMK_EXPORT int llmk_delta_scan(float* out, float* qkv, long long qkv_ld, const 
     else if (D <= 128) e = launch_delta<8, 16>(p, n_seqs, s);
     else e = launch_delta<16, 16>(p, n_seqs, s);
     LLMK_CHECK_LAUNCH_RC("delta_scan", e);
+    return LLMK_OK;
+}
+
+// The same walk with one decay per head over rows that are already prepared (csrc/head_delta.cu): qkv float32 with q and k as unit
+// vectors (q scaled), gates float32 [n_tokens, 2 H + G]: beta, 1 - g, q . k of every key head.
+LLMK_EXPORT int llmk_delta_scan_heads(float* out, const float* qkv, long long qkv_ld, const float* gates, float* state, long long state_ld,
+                                      const int* cu_q, const int* state_slots, int n_seqs, int n_tokens, int H, int G, int D, int E,
+                                      void* stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return LLMK_OK;
+    if (H <= 0 || G <= 0 || H % G != 0) LLMK_FAIL("delta_scan_heads: %d heads are not a multiple of %d key heads", H, G);
+    if (D <= 0 || D > 256 || E <= 0) LLMK_FAIL("delta_scan_heads: key width %d (at most 256) or value width %d", D, E);
+    if (!out || !qkv || !gates || !state || !cu_q || !state_slots) LLMK_FAIL("delta_scan_heads: bad arguments");
+    if (H > 65535 || ceil_div(E, 8) > 65535) LLMK_FAIL("delta_scan_heads: grid too large");
+    DeltaParams p;
+    p.out = out; p.qkv = qkv; p.qkv_ld = qkv_ld; p.beta = gates; p.decay = nullptr;
+    p.state = state; p.state_ld = state_ld; p.cu_q = cu_q; p.state_slots = state_slots;
+    p.H = H; p.G = G; p.D = D; p.E = E;
+    p.vec_ok = (D % 4 == 0 && E % 4 == 0 && qkv_ld % 4 == 0 && host_aligned16(qkv)) ? 1 : 0;
+    cudaStream_t s = (cudaStream_t)stream;
+    cudaError_t e;
+    if (D <= 32) e = launch_delta<4, 8, true>(p, n_seqs, s);
+    else if (D <= 64) e = launch_delta<4, 16, true>(p, n_seqs, s);
+    else if (D <= 128) e = launch_delta<8, 16, true>(p, n_seqs, s);
+    else e = launch_delta<16, 16, true>(p, n_seqs, s);
+    LLMK_CHECK_LAUNCH_RC("delta_scan_heads", e);
     return LLMK_OK;
 }
 

@@ -34,6 +34,8 @@ class DecoderModel:
         self.dtype = dtype
         self.device = device
         self.embedding = weights.device_tensor(spec.embedding, dtype, device)
+        # learned positions: a row per position, added to the embedding's rows
+        self.position_table = weights.device_tensor(spec.position_table, dtype, device) if spec.position_table else None
         self.layers = [build_block(ls, weights, dtype, device) for ls in spec.layers]
         # what a run item does to the residual stream before its layer runs (items with equal specs share one object)
         made = {}
@@ -93,7 +95,8 @@ class DecoderModel:
         resid = ctx.workspace.buffer("residual", T, H, torch.float32)
         rows = resid if self.embedding_norm is None else ctx.workspace.buffer("embedding_rows", T, H, torch.float32)
         ops.embed_rows(rows, self.embedding, ctx.ids, self.bad_token_flag, ids_from=ctx.ids_from, sampled=ctx.prev_sampled,
-                       scale=float(self.spec.embedding_scale))
+                       scale=float(self.spec.embedding_scale), position_table=self.position_table,
+                       positions=ctx.positions if self.position_table is not None else None)
         if self.embedding_norm is not None:
             # the table's rows pass a norm before they become the residual stream (float32 in, float32 out)
             self.embedding_norm.add_norm(rows, None, resid)

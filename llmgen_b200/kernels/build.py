@@ -56,6 +56,7 @@ MODULES: Dict[str, List[str]] = {
     "moe": [],
     "recurrent": [],
     "memory_scan": [],
+    "head_delta": [],
     "runtime": [],      # host code only: cache manager, scheduler, step arrays
 }
 

@@ -95,14 +95,19 @@ class Partials:
 
 # ---------------------------------------------------------------------------- elementwise
 def embed_rows(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, bad_flag: Optional[torch.Tensor] = None,
-               ids_from: Optional[torch.Tensor] = None, sampled: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+               ids_from: Optional[torch.Tensor] = None, sampled: Optional[torch.Tensor] = None, scale: float = 1.0,
+               position_table: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None) -> None:
     """out[t] (float32 [n, H]) = table[ids[t]] * scale; ids int32 on the device.  With `ids_from` and
-    `sampled` (int32, device) a row whose ids_from[t] >= 0 takes the id sampled[ids_from[t]]."""
+    `sampled` (int32, device) a row whose ids_from[t] >= 0 takes the id sampled[ids_from[t]].  With `position_table` (of the
+    table's dtype, [positions, H]) its row positions[t] is added, unscaled."""
     lib = build.load("elementwise")
     n, H = out.shape
+    if position_table is not None and (position_table.dtype != table.dtype or position_table.shape[1] != H or positions is None):
+        raise KernelError("embed_rows: the table of positions has the embeddings' dtype and width, and the tokens' positions beside it")
     _check(lib, lib.llmk_embed_rows(_ptr(out), _ptr(table), _ptr(ids), _ptr(ids_from), _ptr(sampled), c_int(n), c_int(H),
                                     c_int(table.shape[0]), _ptr(bad_flag), c_int(dtype_code(table.dtype)), c_float(scale),
-                                    _stream()))
+                                    _ptr(position_table), _ptr(positions),
+                                    c_int(position_table.shape[0] if position_table is not None else 0), _stream()))
 
 
 def logit_cap(logits: torch.Tensor, cap: float, scale: float = 1.0) -> None:
@@ -1243,6 +1248,52 @@ def delta_scan(out: torch.Tensor, qkv: torch.Tensor, beta: torch.Tensor, decay: 
                                     c_int(vdim), c_float(unit_eps), c_float(q_scale), c_int(dtype_code(beta.dtype)), _stream()), 2)
 
 
+def head_delta_prep(qkv: torch.Tensor, gates: torch.Tensor, packed: torch.Tensor, beta_off: int, decay_off: int, taps: torch.Tensor,
+                    dt_bias: torch.Tensor, a_log: torch.Tensor, conv_state: Optional[torch.Tensor], cu_q: torch.Tensor,
+                    state_slots: torch.Tensor, n_seqs: int, heads: int, kv_heads: int, dim: int, vdim: int, unit_eps: float) -> None:
+    """What precedes the gated delta rule with one decay per head (csrc/head_delta.cu).  `packed` [n, ...] (storage dtype, any row
+    stride): the projections of q, k, v at column 0, of beta and of the decays at `beta_off` and `decay_off`.  qkv float32
+    [n, 2 kv_heads dim + heads vdim] = short convolution (`taps` float32 [channels, K]) and silu, q and k as unit vectors per head, q
+    times dim^-1/2; gates float32 [n, 2 heads + kv_heads] = beta, 1 - decay, q . k.  `conv_state` (K > 1): the columns of the state
+    array from the convolution's inputs on, [slots, >= (K - 1) channels], read and left with the last K - 1 inputs."""
+    lib = build.load("head_delta")
+    n, C = qkv.shape
+    K = taps.shape[1]
+    if qkv.dtype != torch.float32 or gates.dtype != torch.float32 or not qkv.is_contiguous() or not gates.is_contiguous() \
+            or C != 2 * kv_heads * dim + heads * vdim or tuple(gates.shape) != (n, 2 * heads + kv_heads) or taps.dtype != torch.float32 \
+            or tuple(taps.shape) != (C, K) or not taps.is_contiguous():
+        raise KernelError("head_delta_prep: shapes or dtypes do not fit")
+    if K > 1 and (conv_state is None or conv_state.dtype != torch.float32 or conv_state.shape[1] < (K - 1) * C):
+        raise KernelError("head_delta_prep: the convolution's state is float32 [slots, (taps - 1) channels]")
+    _check(lib, lib.llmk_head_delta_prep(_ptr(qkv), _ptr(gates), _ptr(packed), c_longlong(_row_stride(packed)), c_int(beta_off), c_int(decay_off),
+                                         _ptr(taps), _ptr(dt_bias), _ptr(a_log), _ptr(conv_state),
+                                         c_longlong(_row_stride(conv_state) if conv_state is not None else 0), _ptr(cu_q), _ptr(state_slots),
+                                         c_int(n_seqs), c_int(n), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(K),
+                                         c_float(unit_eps), c_float(float(dim) ** -0.5), c_int(dtype_code(packed.dtype)), _stream()),
+           2 if K > 1 else 1)
+
+
+def _check_head_delta(who: str, out, qkv, gates, state, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
+    n = out.shape[0]
+    if any(t.dtype != torch.float32 for t in (out, qkv, gates, state)):
+        raise KernelError(f"{who}: out, qkv, gates and state are float32")
+    if not out.is_contiguous() or not qkv.is_contiguous() or not gates.is_contiguous() or out.shape[1] != heads * vdim \
+            or tuple(qkv.shape) != (n, 2 * kv_heads * dim + heads * vdim) or tuple(gates.shape) != (n, 2 * heads + kv_heads) \
+            or state.shape[1] < heads * dim * vdim:
+        raise KernelError(f"{who}: shapes do not fit")
+
+
+def delta_scan_heads(out: torch.Tensor, qkv: torch.Tensor, gates: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor,
+                     state_slots: torch.Tensor, n_seqs: int, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
+    """The gated delta rule with one decay per head, token by token (csrc/recurrent.cu), over what `head_delta_prep` left; state
+    [slots, >= heads dim vdim] float32, out float32 [n, heads vdim]."""
+    lib = build.load("recurrent")
+    _check_head_delta("delta_scan_heads", out, qkv, gates, state, heads, kv_heads, dim, vdim)
+    _check(lib, lib.llmk_delta_scan_heads(_ptr(out), _ptr(qkv), c_longlong(_row_stride(qkv)), _ptr(gates), _ptr(state), c_longlong(_row_stride(state)),
+                                          _ptr(cu_q), _ptr(state_slots), c_int(n_seqs), c_int(out.shape[0]), c_int(heads), c_int(kv_heads),
+                                          c_int(dim), c_int(vdim), _stream()))
+
+
 DECAY_FORMS = {"sigmoid_pow": 0, "exp_exp": 1}
 
 
@@ -1500,19 +1551,25 @@ def moe_max_tiles(n_slots: int, experts: int, tile: int = 0) -> int:
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, slot_expert: torch.Tensor, slot_weight: torch.Tensor, top: int,
               scoring: str = "sigmoid", renormalize: bool = False, bias: Optional[torch.Tensor] = None,
-              choice_bias: Optional[torch.Tensor] = None, weight_scale: float = 1.0, sum_eps: float = 0.0, pdl: bool = True) -> None:
+              choice_bias: Optional[torch.Tensor] = None, weight_scale: float = 1.0, sum_eps: float = 0.0, pdl: bool = True,
+              groups: int = 1, keep_groups: int = 1, gate_out: Optional[torch.Tensor] = None) -> None:
     """Per row of h [n, K]: scores of router (float32 [E, K]) h (+ `bias`, float32 [E]), the `top` largest choose; slot
     n * top + c receives (expert, score).  `choice_bias` (float32 [E]) is added to the scores for the choice alone;
-    `renormalize`: the weights are divided by the chosen scores' sum + `sum_eps`; they are then multiplied by `weight_scale`."""
+    `renormalize`: the weights are divided by the chosen scores' sum + `sum_eps`; they are then multiplied by `weight_scale`.
+    `groups` > 1: the E outputs form that many groups of neighbours, and only those of the `keep_groups` groups with the largest
+    values that choose take part.  `gate_out` (float32 [n]): `router` has one more row, whose product's sigmoid goes there."""
     lib = build.load("moe")
     n, K = h.shape
-    E = router.shape[0]
+    E = router.shape[0] - (1 if gate_out is not None else 0)
+    if gate_out is not None and (gate_out.dtype != torch.float32 or gate_out.numel() < n):
+        raise KernelError("moe_route: the gate is one float32 per token")
     if router.dtype != torch.float32 or slot_expert.dtype != torch.int32 or slot_weight.dtype != torch.float32 \
             or any(b is not None and (b.dtype != torch.float32 or b.numel() != E) for b in (bias, choice_bias)):
         raise KernelError("moe_route: router, bias and weights float32, experts int32")
     _check(lib, lib.llmk_moe_route(_ptr(h), c_longlong(_row_stride(h)), _ptr(router), _ptr(bias), _ptr(slot_expert), _ptr(slot_weight), c_int(n),
                                    c_int(K), c_int(E), c_int(top), c_int(ROUTER_SCORINGS[scoring]), c_int(1 if renormalize else 0),
-                                   _ptr(choice_bias), c_float(weight_scale), c_float(sum_eps), c_int(1 if pdl else 0),
+                                   _ptr(choice_bias), c_float(weight_scale), c_float(sum_eps), c_int(groups), c_int(keep_groups),
+                                   _ptr(gate_out), c_int(1 if pdl else 0),
                                    c_int(dtype_code(h.dtype)), _stream()))
 
 
@@ -1575,11 +1632,17 @@ def moe_experts(out: torch.Tensor, x: torch.Tensor, w0: torch.Tensor, w1: Option
 
 
 def moe_combine(out: torch.Tensor, rows: torch.Tensor, pos_of_slot: torch.Tensor, shared_out: Optional[torch.Tensor], top: int,
-                slot_weight: Optional[torch.Tensor] = None) -> None:
-    """out float32 [n, H] = shared_out (storage dtype, or None) + the token's `top` rows of `rows` (float32 [slots, H]), each
-    times its slot's weight where `slot_weight` (float32 [n * top]) is given."""
+                slot_weight: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None,
+                identity: Optional[tuple] = None) -> None:
+    """out float32 [n, H] = shared_out (storage dtype, or None; times shared_gate, float32 [n], if given) + the token's `top` rows of
+    `rows` (float32 [slots, H]), each times its slot's weight where `slot_weight` (float32 [n * top]) is given.  `identity` =
+    (h, slot_expert, weights, E): a slot without a row whose expert is E or more adds weights[slot] * h[token]."""
     lib = build.load("moe")
     n, H = out.shape
-    dt = shared_out.dtype if shared_out is not None else torch.float32
-    _check(lib, lib.llmk_moe_combine(_ptr(out), _ptr(rows), _ptr(pos_of_slot), _ptr(shared_out), _ptr(slot_weight), c_int(n), c_int(top), c_int(H),
-                                     c_int(dtype_code(dt)), _stream()))
+    h, slot_expert, weights, E = identity if identity is not None else (None, None, None, 0)
+    dt = shared_out.dtype if shared_out is not None else h.dtype if h is not None else torch.float32
+    if h is not None and h.dtype != dt:
+        raise KernelError("moe_combine: the input and the shared expert's output have one dtype")
+    _check(lib, lib.llmk_moe_combine(_ptr(out), _ptr(rows), _ptr(pos_of_slot), _ptr(shared_out), _ptr(shared_gate), _ptr(slot_weight), _ptr(h),
+                                     c_longlong(_row_stride(h) if h is not None else 0), _ptr(slot_expert), _ptr(weights), c_int(E), c_int(n),
+                                     c_int(top), c_int(H), c_int(dtype_code(dt)), _stream()))

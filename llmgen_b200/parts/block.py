@@ -236,8 +236,8 @@ class MultiStreamBlock(Part):
         if not 1 <= S <= ops.MAX_STREAMS:
             raise ValueError(f"multi-stream block: {S} streams (1 to {ops.MAX_STREAMS})")
         for norm in (spec.mixer_norm, spec.ffn_norm if spec.ffn is not None else None):
-            if norm is not None and (norm.kind != "rmsnorm" or norm.weight_offset != 0.0):
-                raise ValueError("multi-stream block: its norms are plain RMSNorms")
+            if norm is not None and norm.kind != "rmsnorm":
+                raise ValueError("multi-stream block: its norms are RMSNorms")
         if S > 1 and (spec.mixer_streams is None or (spec.ffn is not None and spec.ffn_streams is None)):
             raise ValueError("multi-stream block: several streams need coefficients for every sublayer")
         self.spec, self.dtype, self.S = spec, dtype, S
@@ -246,6 +246,11 @@ class MultiStreamBlock(Part):
         self.ffn_norm = build_norm(spec.ffn_norm, weights, dtype, device) if spec.ffn is not None else None
         self.ffn = build_feed_forward(spec.ffn, weights, dtype, device) if spec.ffn is not None else None
         mult = float(spec.residual_mult)
+        # the gains as `stream_step` takes them: a gain stored around zero has its offset added here
+        self.gain1 = self.mixer_norm.weight + self.mixer_norm.offset if self.mixer_norm.offset else self.mixer_norm.weight
+        self.gain2 = None
+        if self.ffn_norm is not None:
+            self.gain2 = self.ffn_norm.weight + self.ffn_norm.offset if self.ffn_norm.offset else self.ffn_norm.weight
 
         def coefficients(c):
             # (read, mult * write, mix); without tensors: one stream read as it is, kept as it is, y added times mult
@@ -273,19 +278,19 @@ class MultiStreamBlock(Part):
         streams = resid.view(T, self.S, H)
         normed = ctx.workspace.buffer("block_normed", T, H, self.dtype)
         if getattr(ctx, "normed_for", None) is not self:
-            ops.stream_step(streams, None, None, None, self.read1, self.mixer_norm.weight, self.mixer_norm.eps, normed, self.dtype)
+            ops.stream_step(streams, None, None, None, self.read1, self.gain1, self.mixer_norm.eps, normed, self.dtype)
         ctx.normed_for = None
         follower = getattr(ctx, "next_block", None)
         follow = follower if isinstance(follower, MultiStreamBlock) and follower.S == self.S else None
         mixed = self.mixer.forward(ctx, normed, cache)
         if self.ffn is not None:
-            ops.stream_step(streams, mixed, self.mix1, self.write1, self.read2, self.ffn_norm.weight, self.ffn_norm.eps, normed, self.dtype)
+            ops.stream_step(streams, mixed, self.mix1, self.write1, self.read2, self.gain2, self.ffn_norm.eps, normed, self.dtype)
             mixed = self.ffn.forward(ctx, normed)
             mix, write = self.mix2, self.write2
         else:
             mix, write = self.mix1, self.write1
         if follow is not None:
-            ops.stream_step(streams, mixed, mix, write, follow.read1, follow.mixer_norm.weight, follow.mixer_norm.eps, normed, self.dtype)
+            ops.stream_step(streams, mixed, mix, write, follow.read1, follow.gain1, follow.mixer_norm.eps, normed, self.dtype)
         else:
             ops.stream_step(streams, mixed, mix, write, None, None, 0.0, None, self.dtype)
         ctx.normed_for = follow

@@ -80,6 +80,10 @@ class RoutedMLP(FeedForward):
     A caller that adds the experts' rows up itself (`forward(..., combine=False)`) gets them as an `ops.RoutedRows`; one that has
     just changed streams says `pdl=False`, and the first launch is a plain one.
 
+    Outputs of the router behind the experts (`identity_outputs`) return the input: the plan gives their slots no row, and
+    `moe_combine` adds the token's own row times the slot's weight.  The shared expert's gate is one more row of the router's
+    product, read by `moe_combine`.
+
     The shared expert is two of the framework's own products with the same activation between them; a plain
     silu-gated one is the dense gated feed-forward's first half (`GatedMLP.hidden`: the activation in the product's
     epilogue) and one more product."""
@@ -88,11 +92,14 @@ class RoutedMLP(FeedForward):
 
     @staticmethod
     def weight_decls(spec: RoutedMLPSpec):
-        decls = [WeightDecl(spec.router, (len(spec.experts), spec.hidden_size))]
+        outputs = len(spec.experts) + spec.identity_outputs
+        decls = [WeightDecl(spec.router, (outputs, spec.hidden_size))]
         if spec.router_bias:
-            decls.append(WeightDecl(spec.router_bias, (len(spec.experts),), VECTOR))
+            decls.append(WeightDecl(spec.router_bias, (outputs,), VECTOR))
         if spec.choice_bias:
-            decls.append(WeightDecl(spec.choice_bias, (len(spec.experts),), VECTOR))
+            decls.append(WeightDecl(spec.choice_bias, (outputs,), VECTOR))
+        if spec.shared_gate:
+            decls.append(WeightDecl(spec.shared_gate, (1, spec.hidden_size)))
         for e in spec.experts:
             decls += _expert_decls(e, spec.hidden_size)
         if spec.shared is not None:
@@ -108,13 +115,21 @@ class RoutedMLP(FeedForward):
         if any((type(e), e.intermediate_size, _expert_form(e)) != (type(first), first.intermediate_size, _expert_form(first))
                for e in spec.experts):
             raise ValueError("routed feed-forward: all routed experts share one kind, size and constants")
-        if not 0 < spec.top_k <= len(spec.experts):
-            raise ValueError(f"routed feed-forward: top {spec.top_k} of {len(spec.experts)} experts")
+        self.outputs = len(spec.experts) + spec.identity_outputs
+        if self.outputs % spec.groups != 0 or not 0 < spec.keep_groups <= spec.groups:
+            raise ValueError(f"routed feed-forward: {spec.keep_groups} of {spec.groups} equal groups of {self.outputs} outputs")
+        if not 0 < spec.top_k <= self.outputs // spec.groups * spec.keep_groups:
+            raise ValueError(f"routed feed-forward: top {spec.top_k} of {self.outputs} outputs ({spec.keep_groups} of {spec.groups} groups)")
+        if spec.shared_gate and spec.shared is None:
+            raise ValueError("routed feed-forward: a gate of a shared expert that is not there")
         if spec.scoring not in ops.ROUTER_SCORINGS:
             raise ValueError(f"routed feed-forward: scoring {spec.scoring!r} is not supported")
         self.spec, self.dtype = spec, dtype
         self.E, self.top, self.F = len(spec.experts), spec.top_k, first.intermediate_size
         self.router = weights.device_tensor(spec.router, torch.float32, device)      # routing is float32 in both dtypes
+        if spec.shared_gate:
+            # the shared expert's gate is one more row of the router's product
+            self.router = torch.cat([self.router, weights.device_tensor(spec.shared_gate, torch.float32, device)], dim=0).contiguous()
         self.router_bias = weights.device_tensor(spec.router_bias, dtype, device).contiguous() if spec.router_bias else None
         self.choice_bias = weights.device_tensor(spec.choice_bias, dtype, device).contiguous() if spec.choice_bias else None
         self.act, self.alpha, self.limit, self.plain = _expert_form(first)
@@ -165,8 +180,10 @@ class RoutedMLP(FeedForward):
         slot_expert, pos_of_slot, order = ints[:n_slots], ints[n_slots:2 * n_slots], ints[2 * n_slots:2 * n_slots + n_rows]
         tile_expert, tile_start, tile_rows = (ints[2 * n_slots + n_rows + i * tiles:2 * n_slots + n_rows + (i + 1) * tiles] for i in range(3))
         slot_weight = ws.flat("moe_weights", n_slots, torch.float32)
+        shared_gate = ws.flat("moe_shared_gate", T, torch.float32) if spec.shared_gate else None
         ops.moe_route(x, self.router, slot_expert, slot_weight, top, spec.scoring, spec.renormalize, bias=self.router_bias,
-                      choice_bias=self.choice_bias, weight_scale=float(spec.weight_scale), sum_eps=float(spec.sum_eps), pdl=pdl)
+                      choice_bias=self.choice_bias, weight_scale=float(spec.weight_scale), sum_eps=float(spec.sum_eps), pdl=pdl,
+                      groups=spec.groups, keep_groups=spec.keep_groups, gate_out=shared_gate)
         ops.moe_plan(slot_expert, n_slots, self.E, order, pos_of_slot, tile_expert, tile_start, tile_rows, tile=tile, padded=self.grouped)
         cap = (ws.default_rows * top // 128 + self.E) * 128 if self.grouped else ws.default_rows * top
         rows = ws.buffer("moe_rows", n_rows, H, torch.float32, capacity_rows=cap)
@@ -190,7 +207,7 @@ class RoutedMLP(FeedForward):
                             first=False, weight_on_input=spec.weight_on_input)
         # the grouped products leave an expert's plain output: a weight on the output is applied as the rows are added
         late_weight = slot_weight if self.grouped and not spec.weight_on_input else None
-        if not combine and spec.shared is None:
+        if not combine and spec.shared is None and not spec.identity_outputs:
             return ops.RoutedRows(rows, pos_of_slot, late_weight, top)
         shared_out = None
         if self.shared_mlp is not None:
@@ -202,7 +219,8 @@ class RoutedMLP(FeedForward):
             ops.act_rows(act, gate_up, self.shared_form[0], alpha=self.shared_form[1], limit=self.shared_form[2])
             shared_out = linear(act, self.shared_down, ws.buffer("moe_shared_out", T, H, self.dtype))
         out = ws.flat("moe_out", T * H, torch.float32).view(1, T, H)
-        ops.moe_combine(out[0], rows, pos_of_slot, shared_out, top, slot_weight=late_weight)
+        identity = (x, slot_expert, slot_weight, self.E) if spec.identity_outputs else None
+        ops.moe_combine(out[0], rows, pos_of_slot, shared_out, top, slot_weight=late_weight, shared_gate=shared_gate, identity=identity)
         return ops.Partials(out)
 
 

@@ -105,6 +105,8 @@ def model_weight_decls(model_spec) -> List[WeightDecl]:
     """Every tensor a whole model reads, in declaration order."""
     _ensure_builtin()
     decls = [WeightDecl(model_spec.embedding, (model_spec.vocab_size, model_spec.hidden_size))]
+    if getattr(model_spec, "position_table", None):
+        decls.append(WeightDecl(model_spec.position_table, (model_spec.max_positions, model_spec.hidden_size)))
     if getattr(model_spec, "embedding_norm", None) is not None:
         decls += norm_class(model_spec.embedding_norm).weight_decls(model_spec.embedding_norm)
     for layer in model_spec.layers:

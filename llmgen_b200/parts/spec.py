@@ -284,6 +284,38 @@ class GatedDeltaSpec:
 
 
 @dataclass(frozen=True)
+class HeadDecayDeltaSpec:
+    """The gated delta rule with one decay per head, state carried from token to token.
+
+    q, k [kv_heads, key_dim] and v [heads, value_dim] as for `GatedDeltaSpec`: projections that pass a short convolution (one spec
+    over the channels of q, k and v side by side) and silu, q and k then unit vectors per head, x / sqrt(sum x^2 + unit_eps), q
+    times key_dim^(-1/2); head h reads q/k head h // (heads / kv_heads).  Per head beta = sigmoid(x Wb^T) and
+    g = exp(-exp(A_log) softplus(x Wa^T + dt_bias)).  S [key_dim, value_dim] float32, zero before the first token:
+    S <- g S;  d = beta (v - S^T k);  S <- S + k d^T;  o = S^T q.  Each head's o passes an RMSNorm over value_dim (`out_norm`, one
+    gain vector for all heads), is multiplied by silu(x Wg^T) and projected by Wo.  State per request: S and the
+    convolution's last taps - 1 inputs."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    key_dim: int
+    value_dim: int
+    conv: ShortConvSpec                  # channels = 2 kv_heads key_dim + heads value_dim
+    conv_weights: Tuple[str, ...]        # the taps of q, k and v, stacked into `conv` when the model is loaded
+    q_proj: str
+    k_proj: str
+    v_proj: str
+    beta_proj: str                       # Wb [heads, hidden]
+    decay_proj: str                      # Wa [heads, hidden]
+    decay_bias: str                      # dt_bias [heads]
+    decay_log: str                       # A_log [heads]
+    gate_proj: str                       # Wg [heads value_dim, hidden]
+    o_proj: str
+    out_norm: RMSNormSpec
+    unit_eps: float = 1e-6
+    kind: str = "head_decay_delta"
+
+
+@dataclass(frozen=True)
 class ChannelDecayAttentionSpec:
     """Linear attention whose state forgets by a decay per head and key channel that the token itself decides.
 
@@ -478,7 +510,11 @@ class RoutedMLPSpec:
     multiplies the expert's input (`weight_on_input`) or its output.  An optional shared expert runs for every token and
     is added.  Experts are `ClampedExpertSpec`, `GatedExpertSpec` or `PlainExpertSpec`, all routed ones of one kind and size.
     `choice_bias`: name of a vector per expert added to the scores for the choice alone, not for the weights.  The weights
-    are multiplied by `weight_scale`; renormalised ones are divided by the chosen scores' sum + `sum_eps`."""
+    are multiplied by `weight_scale`; renormalised ones are divided by the chosen scores' sum + `sum_eps`.
+    `identity_outputs`: the router has that many outputs behind the experts; one that is chosen returns the input itself (times
+    its weight) and has no tensors.  `groups`: the router's outputs form that many equal groups of neighbours, a group's score is
+    the largest (corrected) score in it, and only outputs of the `keep_groups` best groups can be chosen.  `shared_gate`: name of
+    a [1, hidden] tensor; the shared expert's output is multiplied by sigmoid(x Wsg^T), one number per token."""
     hidden_size: int
     router: str
     experts: Tuple[object, ...]
@@ -491,6 +527,10 @@ class RoutedMLPSpec:
     choice_bias: Optional[str] = None
     weight_scale: float = 1.0
     sum_eps: float = 0.0
+    identity_outputs: int = 0
+    groups: int = 1
+    keep_groups: int = 1
+    shared_gate: Optional[str] = None
     kind: str = "routed_mlp"
 
 
@@ -633,6 +673,8 @@ class ModelSpec:
     logit_cap: float = 0.0               # > 0: logits = cap * tanh(logits / cap)
     logit_scale: float = 1.0             # logits are multiplied by this (before the cap)
     embedding_norm: Optional[object] = None   # a norm spec: the embedding's rows pass it before they become the residual
+    # name of a [max_positions, hidden] table: row p is added to the embedding of a token at position p
+    position_table: Optional[str] = None
     # > 0: the layers keep this many residual streams per token (`MultiStreamBlockSpec`): the model hands them a float32
     # [tokens, streams, hidden] array, every stream the embedding's output, and adds the streams up before the final norm
     residual_streams: int = 0
