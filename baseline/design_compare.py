@@ -1,6 +1,6 @@
-"""`bench.py --designs`: Derupel (or, with `--designs-family sarulix`, `fonuvik`, `nasozen` or `zuvasun`, that design) beside Qwen3 at
+"""`bench.py --designs`: Derupel (or, with `--designs-family sarulix`, `fonuvik`, `nasozen`, `zuvasun` or `kugisun`, that design) beside Qwen3 at
 equal layer sizes, random weights, one B200; `--designs-beside` names another design to stand beside it (Nasozen stands beside
-Fonuvik and Zuvasun beside Derupel, the closest models, unless told otherwise).
+Fonuvik, Zuvasun beside Derupel and Kugisun beside Nasozen, the closest models, unless told otherwise).
 
 For each size two models are built: a Derupel whose layers alternate its two mixers and its two feed-forwards (a Sarulix
 whose four layers are a recurrent unit, the delta rule, attention and a recurrent unit again, each with a feed-forward,
@@ -9,7 +9,8 @@ mixer, each with a routed feed-forward whose chosen and shared experts together 
 four residual streams whose layers are the parallel mixer, the generalized delta rule, the parallel mixer and the matrix
 memory under a running maximum, three with a routed feed-forward and one with a dense one; a Zuvasun whose layers are attention
 over every key, latent attention under a window, latent attention that reads the entries of the layer before it, and attention
-again, each with a routed feed-forward beside it), and the
+again, each with a routed feed-forward beside it; a Kugisun of four residual streams whose layers are all attention beside the
+gated delta rule, three with a routed feed-forward and one with a dense one), and the
 Qwen3 of the same width, depth, feed-forward width and vocabulary.
 Measured for both:
 
@@ -108,10 +109,25 @@ def zuvasun_config(s: dict) -> dict:
     return {"architecture": "Zuvasun", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "layers": layers, "max_positions": CONTEXT}
 
 
+def kugisun_config(s: dict) -> dict:
+    heads, hd = s["heads"], s["hd"]
+    routed = {"kind": "moe", "router": {"experts": s["experts"] * 3 // 4, "identity": s["experts"] // 4, "top": s["top"], "scale": 2.0,
+                                        "groups": {"count": 4, "keep": 2}},
+              "expert": {"ff": s["expert_ff"]}, "shared": {"ff": s["expert_ff"]}}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    left = {"heads": heads, "kv_heads": max(1, heads // 2), "dim": hd, "vdim": hd, "scale": hd ** -0.5,
+            "rot": {"base": 500000.0, "dims": hd // 2}}
+    right = {"heads": heads, "kv_heads": max(1, heads // 2), "dim": hd, "vdim": hd, "conv": 4}
+    layers = [{"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.0, "right_scale": 0.5},
+               "mlp": dense if i % 4 == 3 else routed} for i in range(s["layers"])]
+    return {"architecture": "Kugisun", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "streams": 4, "layers": layers,
+            "max_positions": CONTEXT}
+
+
 FAMILIES = {"derupel": derupel_config, "sarulix": sarulix_config, "fonuvik": fonuvik_config, "nasozen": nasozen_config,
-            "zuvasun": zuvasun_config}
+            "zuvasun": zuvasun_config, "kugisun": kugisun_config}
 # the design that stands beside a family's where it is not Qwen3: the framework's closest model
-BESIDE = {"nasozen": "fonuvik", "zuvasun": "derupel"}
+BESIDE = {"nasozen": "fonuvik", "zuvasun": "derupel", "kugisun": "nasozen"}
 
 
 def qwen3_config(s: dict) -> dict:

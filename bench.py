@@ -4,7 +4,7 @@
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl ours|reference]
                     [--shape 0.6b|8b|32b --layers L]      (other layer sizes, beside the default run)
     python bench.py --kernels [--kernels-out FILE.md]     (kernel by kernel beside the reference's own kernels)
-    python bench.py --designs [--designs-family derupel|sarulix|fonuvik|nasozen|zuvasun] [--designs-beside DESIGN] [--designs-out FILE.md]
+    python bench.py --designs [--designs-family derupel|sarulix|fonuvik|nasozen|zuvasun|kugisun] [--designs-beside DESIGN] [--designs-out FILE.md]
                                                           (that design beside Qwen3, or beside the named design, at equal layer sizes)
 
 Prints ONE JSON line.  A "step" is one decode step of `--batch` sequences (default 8) whose
@@ -217,10 +217,10 @@ def main():
                     help="Derupel beside Qwen3 at equal layer sizes: prefill and decode throughput and every kernel's share of the "
                          "measured peaks (baseline/design_compare.py); prints one JSON line of its own")
     ap.add_argument("--designs-size", default="", help="with --designs: only these sizes (comma-separated; default all)")
-    ap.add_argument("--designs-family", default="derupel", choices=["derupel", "sarulix", "fonuvik", "nasozen", "zuvasun"],
+    ap.add_argument("--designs-family", default="derupel", choices=["derupel", "sarulix", "fonuvik", "nasozen", "zuvasun", "kugisun"],
                     help="with --designs: the architecture measured beside Qwen3 (default derupel)")
-    ap.add_argument("--designs-beside", default="", choices=["", "qwen3", "derupel", "sarulix", "fonuvik", "nasozen", "zuvasun"],
-                    help="with --designs: the design that stands beside it (default: Qwen3; for nasozen, fonuvik, and for zuvasun, derupel: the closest models)")
+    ap.add_argument("--designs-beside", default="", choices=["", "qwen3", "derupel", "sarulix", "fonuvik", "nasozen", "zuvasun", "kugisun"],
+                    help="with --designs: the design that stands beside it (default: Qwen3; for nasozen, fonuvik, for zuvasun, derupel, and for kugisun, nasozen: the closest models)")
     ap.add_argument("--designs-out", default="", help="with --designs: also write the tables as markdown to this file")
     args = ap.parse_args()
 

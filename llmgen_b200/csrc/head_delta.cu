@@ -2,7 +2,16 @@
 //
 //   head_delta_prep     from the rows of one packed projection, per token: the short convolution over the channels of q, k and v
 //                       and its silu, q and k as unit vectors (q also times key_dim^-1/2), beta = sigmoid(b),
-//                       1 - g = -expm1(-exp(A_log) softplus(a + dt_bias)), q . k of every key head
+//                       log g = -exp(A_log) softplus(a + dt_bias), q . k of every key head
+//   head_delta_chunks   the recurrence over prompts, chunks of 64 tokens at a time.  Inside a chunk, with L_i = log g_1 + .. + log g_i and
+//                       S the state before it, the writes are the rows of
+//                           U = (I + M)^-1 (diag(beta) V - diag(beta e^L) K S),   M_ij = beta_i e^(L_i - L_j) k_i . k_j  (j < i),
+//                       the outputs  o_i = e^(L_i) S^T q_i + sum_(j <= i) e^(L_i - L_j) (q_i . k_j) u_j,  and the state after the chunk
+//                       e^(L_n) S + sum_j e^(L_n - L_j) k_j u_j^T.  What does not need the state (the two triangular systems' solutions
+//                       W = (I + M)^-1 diag(beta e^L) K and (I + M)^-1 diag(beta) V, the matrix of the read-out) is made for all chunks
+//                       side by side; the walk over the chunks then touches the state once a chunk instead of once a token
+//   head_delta_step     steps of a few tokens (single decoded tokens above all) in one launch: all of the preparation, the
+//                       recurrence, each head's RMSNorm and the gate silu(z)
 //
 // A step's sequences are given as in csrc/recurrent.cu: sequence s owns token rows [cu_q[s], cu_q[s+1]), its state lies in slot
 // state_slots[s] (-1: none), rows beyond cu_q[n_seqs] and sequences without tokens are skipped.  A state row is
@@ -30,7 +39,7 @@ __device__ __forceinline__ float softplusf_(float x) { return x > 20.f ? x : log
 
 struct PrepParams {
     float* qkv;              // [n_tokens, C] prepared: q, k (unit vectors), v
-    float* gates;            // [n_tokens, 2 H + G]: beta, 1 - g, q . k
+    float* gates;            // [n_tokens, 2 H + G]: beta, log g, q . k
     const void* x;           // packed projection [n_tokens, x_ld]: q, k, v at column 0
     long long x_ld;
     int beta_off, decay_off; // columns of b and a in it
@@ -132,7 +141,7 @@ __global__ void __launch_bounds__(256) head_delta_prep_kernel(PrepParams p) {
         const T* row = x + (size_t)(t0 + tt) * p.x_ld;
         float* out = p.gates + (size_t)(t0 + tt) * width;
         out[h] = sigmoidf_(to_float(row[p.beta_off + h]));
-        out[p.H + h] = -expm1f(-expf(p.a_log[h]) * softplusf_(to_float(row[p.decay_off + h]) + p.dt_bias[h]));
+        out[p.H + h] = -expf(p.a_log[h]) * softplusf_(to_float(row[p.decay_off + h]) + p.dt_bias[h]);
     }
 }
 
@@ -198,5 +207,633 @@ LLMK_EXPORT int llmk_head_delta_prep(float* qkv, float* gates, const void* x, lo
     else if (dtype == LLMK_BF16) e = launch_prep<bf16>(p, (cudaStream_t)stream);
     else LLMK_FAIL("head_delta_prep: unknown dtype %d", dtype);
     LLMK_CHECK_LAUNCH_RC("head_delta_prep", e);
+    return LLMK_OK;
+}
+
+// ------------------------------------------------------------------------------------------------ chunks
+// A chunk of a sequence has a place of its own in the scratch: chunk c of sequence s lies at cu_q[s] / CHUNK + s + c.
+constexpr int CHUNK = 64;
+constexpr int CTHREADS = 256;
+
+struct ChunkParams {
+    float* out;              // [n_tokens, H * E]
+    const float* qkv;        // [n_tokens, C]: prepared q, k, v
+    const float* gates;      // [n_tokens, 2 H + G]: beta, log g, q . k
+    float* state;            // [slots, state_ld]: S [H][D][E]
+    long long state_ld;
+    const int* cu_q;
+    const int* state_slots;
+    float* qs;               // [places][G][CHUNK][DP]
+    float* ks;               // [places][G][CHUNK][DP]
+    float* w;                // [places][H][CHUNK][DP]
+    float* uv;               // [places][H][CHUNK][EP]
+    float* p;                // [places][H][CHUNK][CHUNK]
+    float* dec;              // [places][H][2][CHUNK]: e^(L_i), e^(L_n - L_i)
+    int n_seqs, n_tokens, H, G, D, E, EP, vec_ok;
+};
+
+// Everything of one (chunk, head) that does not need the state.
+template <int DP>
+__global__ void __launch_bounds__(CTHREADS, 2) chunk_prep_kernel(ChunkParams p) {
+    constexpr int LD = DP + 4, MLD = CHUNK + 4;
+    extern __shared__ __align__(16) float csm[];
+    float* Ks = csm;                        // [CHUNK][LD]
+    float* Qs = Ks + CHUNK * LD;            // [CHUNK][LD]
+    float* M = Qs + CHUNK * LD;             // [CHUNK][MLD]
+    float* bet = M + CHUNK * MLD;           // [CHUNK]
+    float* L = bet + CHUNK;                 // [CHUNK]
+    const int place = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+    const int kvh = h / (p.H / p.G);
+    const bool writes_qk = h % (p.H / p.G) == 0;
+    pdl_launch_dependents();
+    pdl_wait();
+    // the last sequence whose first chunk lies at or before this place
+    int lo = 0, hi = p.n_seqs;
+    while (hi - lo > 1) {
+        const int mid = (lo + hi) >> 1;
+        if (p.cu_q[mid] / CHUNK + mid <= place) lo = mid; else hi = mid;
+    }
+    const int q_beg = p.cu_q[lo], first = (place - q_beg / CHUNK - lo) * CHUNK;
+    const int n = min(CHUNK, p.cu_q[lo + 1] - q_beg - first);
+    if (n <= 0) return;
+    const int t0 = q_beg + first;
+    const int D = p.D, E = p.E, GD = p.G * D, C = 2 * GD + p.H * E;
+#pragma unroll 4
+    for (int idx = tid; idx < CHUNK * DP / 4; idx += CTHREADS) {
+        const int i = idx / (DP / 4), d = idx % (DP / 4) * 4;
+        float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv;
+        if (i < n && d < D) {
+            const float* row = p.qkv + (size_t)(t0 + i) * C + (size_t)kvh * D + d;
+            if (p.vec_ok) {
+                qv = *reinterpret_cast<const float4*>(row);
+                kv = *reinterpret_cast<const float4*>(row + GD);
+            } else {
+                qv.x = row[0]; kv.x = row[GD];
+                if (d + 1 < D) { qv.y = row[1]; kv.y = row[GD + 1]; }
+                if (d + 2 < D) { qv.z = row[2]; kv.z = row[GD + 2]; }
+                if (d + 3 < D) { qv.w = row[3]; kv.w = row[GD + 3]; }
+            }
+        }
+        *reinterpret_cast<float4*>(Ks + i * LD + d) = kv;
+        *reinterpret_cast<float4*>(Qs + i * LD + d) = qv;
+        if (writes_qk) {
+            const size_t at = ((size_t)(place * p.G + kvh) * CHUNK + i) * DP + d;
+            *reinterpret_cast<float4*>(p.ks + at) = kv;
+            *reinterpret_cast<float4*>(p.qs + at) = qv;
+        }
+    }
+    if (tid < 32) {           // running sums of log g, two rows a lane
+        const float* g0 = p.gates + (size_t)t0 * (2 * p.H + p.G);
+        const int a = 2 * tid, b = a + 1, width = 2 * p.H + p.G;
+        const float la = a < n ? g0[(size_t)a * width + p.H + h] : 0.f, lb = b < n ? g0[(size_t)b * width + p.H + h] : 0.f;
+        bet[a] = a < n ? g0[(size_t)a * width + h] : 0.f;
+        bet[b] = b < n ? g0[(size_t)b * width + h] : 0.f;
+        float sum = la + lb;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float up = __shfl_up_sync(0xffffffffu, sum, o);
+            if (tid >= o) sum += up;
+        }
+        L[a] = sum - lb;
+        L[b] = sum;
+        const float all = __shfl_sync(0xffffffffu, sum, 31);
+        float* dec = p.dec + (size_t)(place * p.H + h) * 2 * CHUNK;
+        dec[a] = expf(sum - lb);
+        dec[b] = expf(sum);
+        dec[CHUNK + a] = expf(all - (sum - lb));
+        dec[CHUNK + b] = expf(all - sum);
+    }
+    __syncthreads();
+    {
+        // k_i . k_j and q_i . k_j, a thread a tile of 4 x 4; tiles above the diagonal are zero
+        const int ti = tid >> 4, tj = tid & 15;
+        float kk[4][4], qk[4][4];
+#pragma unroll
+        for (int a = 0; a < 4; ++a)
+#pragma unroll
+            for (int b = 0; b < 4; ++b) kk[a][b] = qk[a][b] = 0.f;
+        if (tj <= ti) {
+#pragma unroll 2
+            for (int d = 0; d < DP; d += 4) {
+                float4 ka[4], qa[4], kb[4];
+#pragma unroll
+                for (int a = 0; a < 4; ++a) {
+                    ka[a] = *reinterpret_cast<const float4*>(Ks + (ti * 4 + a) * LD + d);
+                    qa[a] = *reinterpret_cast<const float4*>(Qs + (ti * 4 + a) * LD + d);
+                    kb[a] = *reinterpret_cast<const float4*>(Ks + (tj * 4 + a) * LD + d);
+                }
+#pragma unroll
+                for (int a = 0; a < 4; ++a)
+#pragma unroll
+                    for (int b = 0; b < 4; ++b) {
+                        kk[a][b] = fmaf(ka[a].x, kb[b].x, kk[a][b]); qk[a][b] = fmaf(qa[a].x, kb[b].x, qk[a][b]);
+                        kk[a][b] = fmaf(ka[a].y, kb[b].y, kk[a][b]); qk[a][b] = fmaf(qa[a].y, kb[b].y, qk[a][b]);
+                        kk[a][b] = fmaf(ka[a].z, kb[b].z, kk[a][b]); qk[a][b] = fmaf(qa[a].z, kb[b].z, qk[a][b]);
+                        kk[a][b] = fmaf(ka[a].w, kb[b].w, kk[a][b]); qk[a][b] = fmaf(qa[a].w, kb[b].w, qk[a][b]);
+                    }
+            }
+        }
+        float* P = p.p + (size_t)(place * p.H + h) * CHUNK * CHUNK;
+#pragma unroll
+        for (int a = 0; a < 4; ++a) {
+            const int i = ti * 4 + a;
+            float pr[4];
+#pragma unroll
+            for (int b = 0; b < 4; ++b) {
+                const int j = tj * 4 + b;
+                const float e = j <= i ? expf(L[i] - L[j]) : 0.f;
+                pr[b] = e * qk[a][b];
+                M[i * MLD + j] = j < i ? bet[i] * e * kk[a][b] : 0.f;
+            }
+            *reinterpret_cast<float4*>(P + i * CHUNK + tj * 4) = make_float4(pr[0], pr[1], pr[2], pr[3]);
+        }
+    }
+    __syncthreads();
+    // (I + M) x = b, a column a thread: the columns of diag(beta e^L) K, then those of diag(beta) V
+    float* W = p.w + (size_t)(place * p.H + h) * CHUNK * DP;
+    float* U = p.uv + (size_t)(place * p.H + h) * CHUNK * p.EP;
+    for (int c = tid; c < DP + p.EP; c += CTHREADS) {
+        const bool key = c < DP;
+        const int e = c - DP;
+        const float* v = p.qkv + (size_t)t0 * C + 2 * GD + (size_t)h * E + e;
+        float x[CHUNK];
+#pragma unroll
+        for (int i = 0; i < CHUNK; ++i) {
+            if (key) x[i] = bet[i] * expf(L[i]) * Ks[i * LD + c];
+            else x[i] = (i < n && e < E) ? bet[i] * v[(size_t)i * C] : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < CHUNK; ++i) {
+            float part[4] = {x[i], 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int j = 0; j < i; j += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(M + i * MLD + j);
+                part[0] = fmaf(-m.x, x[j], part[0]);
+                if (j + 1 < i) part[1] = fmaf(-m.y, x[j + 1], part[1]);
+                if (j + 2 < i) part[2] = fmaf(-m.z, x[j + 2], part[2]);
+                if (j + 3 < i) part[3] = fmaf(-m.w, x[j + 3], part[3]);
+            }
+            x[i] = (part[0] + part[1]) + (part[2] + part[3]);
+            if (key) W[i * DP + c] = x[i];
+            else U[i * p.EP + e] = x[i];
+        }
+    }
+}
+
+// The sums over LANES neighbouring lanes of N values each, scattered: lane l of the group ends with values [l * N / LANES, ...) in v[0 ..].
+template <int N, int LANES>
+__device__ __forceinline__ void reduce_scatter(float (&v)[N], int lane) {
+    int n = N;
+#pragma unroll
+    for (int bit = LANES / 2; bit > 0; bit >>= 1) {
+        n /= 2;
+        const bool up = (lane & bit) != 0;
+#pragma unroll
+        for (int i = 0; i < N / 2; ++i) {
+            if (i >= n) break;
+            const float send = up ? v[i] : v[i + n];
+            const float keep = up ? v[i + n] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
+        }
+    }
+}
+
+// The walk: block (sequence, head, COLS value columns), the state's columns in shared memory.  A chunk takes three steps:
+//   1  rows of W and of Q times S: a thread has 4 rows, all columns, and one of 8 slices of the key channels; warps 0 .. 3 hold W's rows
+//      and leave U, warps 4 .. 7 hold Q's
+//   2  S <- e^(L_n) S + K^T (U scaled): a thread has 4 key channels, all columns, and one slice of the chunk's tokens
+//   3  (warps 4 .. 7) the outputs: e^(L_i) times the rows of step 1 + P U
+// Operands of W, Q, K and P are used by one thread each and go from global memory straight into registers, asked for a step ahead.
+template <int DP, int COLS>
+__global__ void __launch_bounds__(CTHREADS) chunk_scan_kernel(ChunkParams p) {
+    constexpr int KR = DP / 32;                    // runs of four key channels a thread has in step 1
+    constexpr int TS = CTHREADS / (DP / 4);        // slices of tokens in step 2
+    constexpr int TR = CHUNK / TS;                 // tokens of one
+    constexpr int SQ = 4 * COLS + 4;               // four rows of S side by side, padded: slices read different banks
+    constexpr int UL = COLS + 4;                   // a row of U
+    constexpr int NV = 4 * COLS;                   // outputs of a thread before the slices are summed up
+    __shared__ __align__(16) float S[DP / 4 * SQ];
+    __shared__ __align__(16) float U[2][CHUNK / 4 * SQ];   // as the outputs read it (four rows side by side), two chunks in turn
+    __shared__ __align__(16) float Ud[CHUNK * UL];         // times e^(L_n - L_j)
+    const int s = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * COLS, tid = threadIdx.x;
+    const int lane = tid & 31, warp = tid >> 5;
+    const int kvh = h / (p.H / p.G);
+    const int ks = lane & 7, rt = warp * 4 + (lane >> 3);  // slice of key channels, row tile (0 .. 15: W, 16 .. 31: Q)
+    const bool reads_out = rt >= 16;
+    const int row0 = (reads_out ? rt - 16 : rt) * 4;
+    const int ts = tid & (TS - 1), d0 = tid / TS * 4;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int q_beg = p.cu_q[s], n = p.cu_q[s + 1] - q_beg;
+    if (n <= 0) return;
+    const int slot = p.state_slots[s], D = p.D, E = p.E;
+    float* st = slot >= 0 ? p.state + (size_t)slot * p.state_ld + (size_t)h * D * E : nullptr;
+    for (int idx = tid; idx < DP * COLS; idx += CTHREADS) {
+        const int d = idx / COLS, c = idx % COLS;
+        S[(d >> 2) * SQ + (d & 3) * COLS + c] = (st && d < D && e0 + c < E) ? st[(size_t)d * E + e0 + c] : 0.f;
+    }
+    const int place0 = q_beg / CHUNK + s, chunks = ceil_div(n, CHUNK);
+    float4 a4[4][KR], k4[TR], p4[4][2];
+    auto load_rows = [&](int c) {
+        const size_t place = place0 + c;
+        const float* src = reads_out ? p.qs + ((place * p.G + kvh) * CHUNK + row0) * DP : p.w + ((place * p.H + h) * CHUNK + row0) * DP;
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+#pragma unroll
+            for (int i = 0; i < KR; ++i) a4[r][i] = *reinterpret_cast<const float4*>(src + r * DP + i * 32 + ks * 4);
+    };
+    auto load_keys = [&](int c) {
+        const float* src = p.ks + ((size_t)(place0 + c) * p.G + kvh) * CHUNK * DP + d0;
+#pragma unroll
+        for (int j = 0; j < TR; ++j) k4[j] = *reinterpret_cast<const float4*>(src + (j * TS + ts) * DP);
+    };
+    load_rows(0);
+    load_keys(0);
+    __syncthreads();
+    for (int c = 0; c < chunks; ++c) {
+        const size_t ph = (size_t)(place0 + c) * p.H + h;
+        const float* dec = p.dec + ph * 2 * CHUNK;
+        float v[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) v[i] = 0.f;
+#pragma unroll
+        for (int i = 0; i < KR; ++i) {
+            const float* sr = S + (i * 8 + ks) * SQ;
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+                float4 sv[COLS / 4];
+#pragma unroll
+                for (int u = 0; u < COLS / 4; ++u) sv[u] = *reinterpret_cast<const float4*>(sr + q * COLS + 4 * u);
+#pragma unroll
+                for (int r = 0; r < 4; ++r) {
+                    const float w = q == 0 ? a4[r][i].x : q == 1 ? a4[r][i].y : q == 2 ? a4[r][i].z : a4[r][i].w;
+#pragma unroll
+                    for (int u = 0; u < COLS / 4; ++u) {
+                        v[r * COLS + 4 * u] = fmaf(w, sv[u].x, v[r * COLS + 4 * u]);
+                        v[r * COLS + 4 * u + 1] = fmaf(w, sv[u].y, v[r * COLS + 4 * u + 1]);
+                        v[r * COLS + 4 * u + 2] = fmaf(w, sv[u].z, v[r * COLS + 4 * u + 2]);
+                        v[r * COLS + 4 * u + 3] = fmaf(w, sv[u].w, v[r * COLS + 4 * u + 3]);
+                    }
+                }
+            }
+        }
+        // what the slices add up to: this lane keeps NV / 8 values of one row
+        constexpr int KEEP = NV / 8;
+        const int at = ks * KEEP, row = row0 + at / COLS, col = at % COLS;
+        float4 uv[KEEP / 4];
+        if (!reads_out) {
+#pragma unroll
+            for (int u = 0; u < KEEP / 4; ++u) uv[u] = *reinterpret_cast<const float4*>(p.uv + (ph * CHUNK + row) * p.EP + e0 + col + 4 * u);
+        }
+        const float scale = reads_out ? dec[row] : dec[CHUNK + row], keep = dec[CHUNK - 1];
+        reduce_scatter<NV, 8>(v, ks);
+        float* ur = U[c & 1];
+        if (!reads_out) {
+#pragma unroll
+            for (int u = 0; u < KEEP / 4; ++u) {
+                const float4 x = make_float4(uv[u].x - v[4 * u], uv[u].y - v[4 * u + 1], uv[u].z - v[4 * u + 2], uv[u].w - v[4 * u + 3]);
+                *reinterpret_cast<float4*>(ur + (row >> 2) * SQ + (row & 3) * COLS + col + 4 * u) = x;
+                *reinterpret_cast<float4*>(Ud + row * UL + col + 4 * u) = make_float4(scale * x.x, scale * x.y, scale * x.z, scale * x.w);
+            }
+        }
+        float o[KEEP];
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i) o[i] = scale * v[i];
+        __syncthreads();                     // U is there, and S has been read
+        if (c + 1 < chunks) load_rows(c + 1);
+        if (reads_out) {
+            const float* src = p.p + (ph * CHUNK + row0) * CHUNK;
+#pragma unroll
+            for (int r = 0; r < 4; ++r)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) p4[r][i] = *reinterpret_cast<const float4*>(src + r * CHUNK + i * 32 + ks * 4);
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i) v[i] = 0.f;
+#pragma unroll
+        for (int j = 0; j < TR; ++j) {
+            float4 u4[COLS / 4];
+#pragma unroll
+            for (int u = 0; u < COLS / 4; ++u) u4[u] = *reinterpret_cast<const float4*>(Ud + (j * TS + ts) * UL + 4 * u);
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {
+                const float k = r == 0 ? k4[j].x : r == 1 ? k4[j].y : r == 2 ? k4[j].z : k4[j].w;
+#pragma unroll
+                for (int u = 0; u < COLS / 4; ++u) {
+                    v[r * COLS + 4 * u] = fmaf(k, u4[u].x, v[r * COLS + 4 * u]);
+                    v[r * COLS + 4 * u + 1] = fmaf(k, u4[u].y, v[r * COLS + 4 * u + 1]);
+                    v[r * COLS + 4 * u + 2] = fmaf(k, u4[u].z, v[r * COLS + 4 * u + 2]);
+                    v[r * COLS + 4 * u + 3] = fmaf(k, u4[u].w, v[r * COLS + 4 * u + 3]);
+                }
+            }
+        }
+        if (c + 1 < chunks) load_keys(c + 1);
+        reduce_scatter<NV, TS>(v, ts);
+        {
+            constexpr int KEEP2 = NV / TS;
+            float* sr = S + (d0 >> 2) * SQ + ts * KEEP2;
+            if (KEEP2 % 4 == 0) {
+#pragma unroll
+                for (int u = 0; u < KEEP2 / 4; ++u) {
+                    float4 x = *reinterpret_cast<float4*>(sr + 4 * u);
+                    x.x = fmaf(keep, x.x, v[4 * u]);
+                    x.y = fmaf(keep, x.y, v[4 * u + 1]);
+                    x.z = fmaf(keep, x.z, v[4 * u + 2]);
+                    x.w = fmaf(keep, x.w, v[4 * u + 3]);
+                    *reinterpret_cast<float4*>(sr + 4 * u) = x;
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < KEEP2; ++i) sr[i] = fmaf(keep, sr[i], v[i]);
+            }
+        }
+        __syncthreads();                     // S is the state after the chunk
+        if (reads_out) {
+#pragma unroll
+            for (int i = 0; i < NV; ++i) v[i] = 0.f;
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    const float* uj = ur + (i * 8 + ks) * SQ + q * COLS;
+                    float4 u4[COLS / 4];
+#pragma unroll
+                    for (int u = 0; u < COLS / 4; ++u) u4[u] = *reinterpret_cast<const float4*>(uj + 4 * u);
+#pragma unroll
+                    for (int r = 0; r < 4; ++r) {
+                        const float w = q == 0 ? p4[r][i].x : q == 1 ? p4[r][i].y : q == 2 ? p4[r][i].z : p4[r][i].w;
+#pragma unroll
+                        for (int u = 0; u < COLS / 4; ++u) {
+                            v[r * COLS + 4 * u] = fmaf(w, u4[u].x, v[r * COLS + 4 * u]);
+                            v[r * COLS + 4 * u + 1] = fmaf(w, u4[u].y, v[r * COLS + 4 * u + 1]);
+                            v[r * COLS + 4 * u + 2] = fmaf(w, u4[u].z, v[r * COLS + 4 * u + 2]);
+                            v[r * COLS + 4 * u + 3] = fmaf(w, u4[u].w, v[r * COLS + 4 * u + 3]);
+                        }
+                    }
+                }
+            }
+            reduce_scatter<NV, 8>(v, ks);
+            if (c * CHUNK + row < n) {
+                float* dst = p.out + (size_t)(q_beg + c * CHUNK + row) * ((size_t)p.H * E) + (size_t)h * E + e0 + col;
+#pragma unroll
+                for (int i = 0; i < KEEP; ++i)
+                    if (e0 + col + i < E) dst[i] = o[i] + v[i];
+            }
+        }
+    }
+    if (st) {
+        for (int idx = tid; idx < DP * COLS; idx += CTHREADS) {
+            const int d = idx / COLS, c = idx % COLS;
+            if (d < D && e0 + c < E) st[(size_t)d * E + e0 + c] = S[(d >> 2) * SQ + (d & 3) * COLS + c];
+        }
+    }
+}
+
+static int chunk_width(int D) { return D <= 32 ? 32 : D <= 64 ? 64 : 128; }
+static int chunk_places(int n_tokens, int n_seqs) { return n_tokens / CHUNK + std::min(n_seqs, n_tokens); }
+
+// Floats of scratch for a step of n_tokens rows in n_seqs sequences; 0: the kernels do not take these sizes.
+LLMK_EXPORT long long llmk_head_delta_chunk_floats(int n_tokens, int n_seqs, int H, int G, int D, int E) {
+    if (n_tokens <= 0 || n_seqs <= 0 || D <= 0 || D > 128 || E <= 0 || H <= 0 || G <= 0) return 0;
+    const long long dp = chunk_width(D), ep = ceil_div(E, 16) * 16;
+    return (long long)chunk_places(n_tokens, n_seqs) * CHUNK * (2 * G * dp + H * (dp + ep + CHUNK + 2));
+}
+
+template <int DP>
+static cudaError_t launch_chunks(const ChunkParams& p, int places, cudaStream_t s) {
+    const size_t smem = ((size_t)2 * CHUNK * (DP + 4) + CHUNK * (CHUNK + 4) + 2 * CHUNK) * sizeof(float);
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(chunk_prep_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return e;
+        configured = true;
+    }
+    cudaError_t e = llmk_launch(chunk_prep_kernel<DP>, dim3(places, p.H), dim3(CTHREADS), smem, s, true, p);
+    if (e != cudaSuccess) return e;
+    // sixteen columns a block where eight would not fit the SMs side by side
+    if (p.H * ceil_div(p.E, 8) <= device_sm_count())
+        return llmk_launch(chunk_scan_kernel<DP, 8>, dim3(p.n_seqs, p.H, ceil_div(p.E, 8)), dim3(CTHREADS), 0, s, true, p);
+    return llmk_launch(chunk_scan_kernel<DP, 16>, dim3(p.n_seqs, p.H, ceil_div(p.E, 16)), dim3(CTHREADS), 0, s, true, p);
+}
+
+// scratch: llmk_head_delta_chunk_floats(...) floats on a 16-byte boundary.  qkv and gates as `head_delta_prep` leaves them.
+LLMK_EXPORT int llmk_head_delta_chunks(float* out, const float* qkv, const float* gates, float* state, long long state_ld, const int* cu_q,
+                                       const int* state_slots, float* scratch, int n_seqs, int n_tokens, int H, int G, int D, int E,
+                                       void* stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return LLMK_OK;
+    if (H <= 0 || G <= 0 || H % G != 0) LLMK_FAIL("head_delta_chunks: %d heads are not a multiple of %d key heads", H, G);
+    if (llmk_head_delta_chunk_floats(n_tokens, n_seqs, H, G, D, E) == 0) LLMK_FAIL("head_delta_chunks: key width %d (at most 128), value width %d", D, E);
+    if (!out || !qkv || !gates || !state || !cu_q || !state_slots || !scratch || !host_aligned16(scratch)) LLMK_FAIL("head_delta_chunks: bad arguments");
+    if (H > 65535 || ceil_div(E, 8) > 65535) LLMK_FAIL("head_delta_chunks: grid too large");
+    const int places = chunk_places(n_tokens, n_seqs);
+    const long long dp = chunk_width(D), ep = ceil_div(E, 16) * 16, rows = (long long)places * CHUNK;
+    ChunkParams p;
+    p.out = out; p.qkv = qkv; p.gates = gates; p.state = state; p.state_ld = state_ld; p.cu_q = cu_q; p.state_slots = state_slots;
+    p.qs = scratch;
+    p.ks = p.qs + rows * G * dp;
+    p.w = p.ks + rows * G * dp;
+    p.uv = p.w + rows * H * dp;
+    p.p = p.uv + rows * H * ep;
+    p.dec = p.p + rows * H * CHUNK;
+    p.n_seqs = n_seqs; p.n_tokens = n_tokens; p.H = H; p.G = G; p.D = D; p.E = E; p.EP = (int)ep;
+    p.vec_ok = (D % 4 == 0 && (2 * G * D + H * E) % 4 == 0 && host_aligned16(qkv)) ? 1 : 0;
+    cudaStream_t s = (cudaStream_t)stream;
+    cudaError_t e = dp == 32 ? launch_chunks<32>(p, places, s) : dp == 64 ? launch_chunks<64>(p, places, s) : launch_chunks<128>(p, places, s);
+    LLMK_CHECK_LAUNCH_RC("head_delta_chunks", e);
+    return LLMK_OK;
+}
+
+// ------------------------------------------------------------------------------------------------ a few tokens
+// Block (head, sequence), the heads of one key head a cluster: they all read the key head's history of the convolution, and only then
+// does the first of them write it anew.  The state stays in registers: thread (e, slice) holds column e's rows slice, slice + NS, ...
+constexpr int STHREADS = 512;
+
+struct StepParams {
+    void* y;                 // [n_tokens, y_ld], head h at column h * E
+    long long y_ld;
+    PrepParams prep;         // x, its columns, taps, gates' constants, state (of the convolution), sequences, sizes; qkv and gates unused
+    int gate_off;            // column of the output gate in x
+    const float* norm_gain;  // [E]
+    float norm_eps;
+    float* state;            // [slots, state_ld]: S [H][D][E]
+    int EP;                  // E rounded up to a power of two, 32 at least
+};
+
+template <typename T, int NR>
+__global__ void __launch_bounds__(STHREADS) head_delta_step_kernel(StepParams sp) {
+    extern __shared__ float ssm[];
+    const PrepParams& p = sp.prep;
+    const int D = p.D, E = p.E, K = p.K, GD = p.G * D, C = 2 * GD + p.H * E, Ch = 2 * D + E, EP = sp.EP, NS = STHREADS / EP;
+    float* hist = ssm;                        // [K - 1][Ch]
+    float* row = hist + (K - 1) * Ch;         // [Ch] after the convolution
+    float* red = row + Ch;                    // [2][STHREADS]
+    float* scal = red + 2 * STHREADS;         // fq, fk, dot, beta, 1 - g, the norm's warp sums [8]
+    const int h = blockIdx.x, s = blockIdx.y, R = p.H / p.G, kvh = h / R;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int e = tid & (EP - 1), sl = tid / EP;
+    const T* x = static_cast<const T*>(p.x);
+    pdl_launch_dependents();
+    pdl_wait();
+    const int q_beg = p.cu_q[s], n = p.cu_q[s + 1] - q_beg;
+    if (n <= 0) return;                       // the whole cluster
+    const int slot = p.state_slots[s];
+    float* st = slot >= 0 ? sp.state + (size_t)slot * p.state_ld + (size_t)h * D * E + e : nullptr;
+    float* cst = slot >= 0 && K > 1 ? p.state + (size_t)slot * p.state_ld : nullptr;
+    float S[NR];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        const int d = sl + i * NS;
+        S[i] = (st && d < D && e < E) ? st[(size_t)d * E] : 0.f;
+    }
+    auto channel = [&](int c) { return c < D ? kvh * D + c : c < 2 * D ? GD + kvh * D + c - D : 2 * GD + h * E + c - 2 * D; };
+    for (int idx = tid; idx < (K - 1) * Ch; idx += STHREADS) hist[idx] = cst ? cst[(size_t)(idx / Ch) * C + channel(idx % Ch)] : 0.f;
+    if (R > 1) cluster_sync_all();
+    else __syncthreads();
+    for (int j = 0; j < n; ++j) {
+        const T* xr = x + (size_t)(q_beg + j) * p.x_ld;
+        const float gate = (sl == 0 && e < E) ? to_float(xr[sp.gate_off + h * E + e]) : 0.f;
+        for (int c = tid; c < Ch; c += STHREADS) {
+            const int gc = channel(c);
+            const float v = to_float(xr[gc]);
+            float acc = 0.f;
+            for (int i = 0; i < K - 1; ++i) {
+                acc = fmaf(p.taps[(size_t)gc * K + i], hist[i * Ch + c], acc);
+                hist[i * Ch + c] = i + 1 < K - 1 ? hist[(i + 1) * Ch + c] : v;
+            }
+            acc = fmaf(p.taps[(size_t)gc * K + K - 1], v, acc);
+            row[c] = acc / (1.0f + expf(-acc));
+        }
+        __syncthreads();
+        if (warp == 0) {
+            float sq = 0.f, sk = 0.f, qk = 0.f;
+            for (int d = lane; d < D; d += 32) {
+                const float qv = row[d], kv = row[D + d];
+                sq = fmaf(qv, qv, sq);
+                sk = fmaf(kv, kv, sk);
+                qk = fmaf(qv, kv, qk);
+            }
+            sq = warp_sum(sq);
+            sk = warp_sum(sk);
+            qk = warp_sum(qk);
+            if (lane == 0) {
+                const float fq = p.q_scale / sqrtf(sq + p.unit_eps), fk = 1.0f / sqrtf(sk + p.unit_eps);
+                scal[0] = fq;
+                scal[1] = fk;
+                scal[2] = fq * fk * qk;
+            }
+        } else if (warp == 1 && lane == 0) {
+            scal[3] = sigmoidf_(to_float(xr[p.beta_off + h]));
+            scal[4] = -expm1f(-expf(p.a_log[h]) * softplusf_(to_float(xr[p.decay_off + h]) + p.dt_bias[h]));
+        }
+        __syncthreads();
+        const float fq = scal[0], fk = scal[1], dot = scal[2], beta = scal[3], lost = scal[4];
+        float ks[2] = {0.f, 0.f}, qs[2] = {0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int d = sl + i * NS;
+            if (d < D) {
+                S[i] = fmaf(-lost, S[i], S[i]);
+                ks[i & 1] = fmaf(row[D + d], S[i], ks[i & 1]);
+                qs[i & 1] = fmaf(row[d], S[i], qs[i & 1]);
+            }
+        }
+        red[tid] = ks[0] + ks[1];
+        red[STHREADS + tid] = qs[0] + qs[1];
+        __syncthreads();
+        float kS = 0.f, qS = 0.f;
+        for (int i = 0; i < NS; ++i) {
+            kS += red[i * EP + e];
+            qS += red[STHREADS + i * EP + e];
+        }
+        const float write = e < E ? beta * (row[2 * D + e] - fk * kS) : 0.f;
+        const float o = fmaf(dot, write, fq * qS), kw = fk * write;
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int d = sl + i * NS;
+            if (d < D) S[i] = fmaf(row[D + d], kw, S[i]);
+        }
+        if (sl == 0) {                        // whole warps: EP is a multiple of 32
+            const float ss = warp_sum(e < E ? o * o : 0.f);
+            if (lane == 0) scal[8 + warp] = ss;
+        }
+        __syncthreads();
+        if (sl == 0 && e < E) {
+            float ss = 0.f;
+            for (int i = 0; i < EP / 32; ++i) ss += scal[8 + i];
+            const float rinv = 1.0f / sqrtf(ss / (float)E + sp.norm_eps);
+            static_cast<T*>(sp.y)[(size_t)(q_beg + j) * sp.y_ld + (size_t)h * E + e] =
+                from_float<T>(o * rinv * sp.norm_gain[e] * (gate * sigmoidf_(gate)));
+        }
+    }
+    if (st) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int d = sl + i * NS;
+            if (d < D && e < E) st[(size_t)d * E] = S[i];
+        }
+    }
+    if (cst) {
+        const int from = h % R == 0 ? 0 : 2 * D;          // the key head's channels are its first head's to write
+        for (int idx = tid; idx < (K - 1) * (Ch - from); idx += STHREADS) {
+            const int i = idx / (Ch - from), c = from + idx % (Ch - from);
+            cst[(size_t)i * C + channel(c)] = hist[i * Ch + c];
+        }
+    }
+}
+
+// Rows of the state a thread holds; 0: the kernel does not take these sizes.
+static int step_rows(int H, int G, int D, int E) {
+    if (D <= 0 || E <= 0 || E > 256 || G <= 0 || H % G != 0 || H / G > 8) return 0;
+    int ep = 32;
+    while (ep < E) ep *= 2;
+    const int nr = ceil_div(D, STHREADS / ep);
+    return nr > 64 ? 0 : nr;
+}
+LLMK_EXPORT int llmk_head_delta_step_usable(int H, int G, int D, int E) { return step_rows(H, G, D, E) > 0 ? 1 : 0; }
+
+template <typename T>
+static cudaError_t launch_step(const StepParams& p, size_t smem, int rows, cudaStream_t s) {
+    const dim3 grid(p.prep.H, p.prep.n_seqs), block(STHREADS), cluster(p.prep.H / p.prep.G, 1, 1);
+#define HEAD_DELTA_STEP(NR)                                                                                                        \
+    do {                                                                                                                           \
+        if (smem > 48 * 1024) {                                                                                                    \
+            cudaError_t e = cudaFuncSetAttribute(head_delta_step_kernel<T, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return e;                                                                                        \
+        }                                                                                                                          \
+        return llmk_launch_clusters(head_delta_step_kernel<T, NR>, grid, block, smem, s, true, cluster, p);                        \
+    } while (0)
+    if (rows <= 4) HEAD_DELTA_STEP(4);
+    if (rows <= 8) HEAD_DELTA_STEP(8);
+    if (rows <= 16) HEAD_DELTA_STEP(16);
+    if (rows <= 32) HEAD_DELTA_STEP(32);
+    HEAD_DELTA_STEP(64);
+#undef HEAD_DELTA_STEP
+}
+
+// y [n_tokens, y_ld] of the storage dtype: RMSNorm(o) * norm_gain * silu(gate) per head.  state: slot 0's S; the convolution's part of the
+// row begins behind it at conv_state.  Everything else as for head_delta_prep.
+LLMK_EXPORT int llmk_head_delta_step(void* y, long long y_ld, const void* x, long long x_ld, int beta_off, int decay_off, int gate_off,
+                                     const float* taps, const float* dt_bias, const float* a_log, const float* norm_gain, float norm_eps,
+                                     float* state, float* conv_state, long long state_ld, const int* cu_q, const int* state_slots, int n_seqs,
+                                     int n_tokens, int H, int G, int D, int E, int K, float unit_eps, float q_scale, int dtype, void* stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return LLMK_OK;
+    const int rows = step_rows(H, G, D, E);
+    if (rows == 0) LLMK_FAIL("head_delta_step: heads %d on %d, widths %d and %d are not taken", H, G, D, E);
+    if (K < 1 || K > MAX_TAPS) LLMK_FAIL("head_delta_step: %d taps (1 to %d are built)", K, MAX_TAPS);
+    if (!y || !x || !taps || !dt_bias || !a_log || !norm_gain || !state || (!conv_state && K > 1) || !cu_q || !state_slots) LLMK_FAIL("head_delta_step: bad arguments");
+    if (n_seqs > 65535) LLMK_FAIL("head_delta_step: %d sequences", n_seqs);
+    StepParams p;
+    p.y = y; p.y_ld = y_ld;
+    p.prep = {nullptr, nullptr, x, x_ld, beta_off, decay_off, taps, dt_bias, a_log, conv_state, state_ld, cu_q, state_slots,
+              n_seqs, n_tokens, H, G, D, E, K, unit_eps, q_scale};
+    p.gate_off = gate_off; p.norm_gain = norm_gain; p.norm_eps = norm_eps; p.state = state;
+    p.EP = 32;
+    while (p.EP < E) p.EP *= 2;
+    const size_t smem = ((size_t)K * (2 * D + E) + 2 * STHREADS + 16) * sizeof(float);
+    cudaError_t e;
+    if (dtype == LLMK_F32) e = launch_step<float>(p, smem, rows, (cudaStream_t)stream);
+    else if (dtype == LLMK_BF16) e = launch_step<bf16>(p, smem, rows, (cudaStream_t)stream);
+    else LLMK_FAIL("head_delta_step: unknown dtype %d", dtype);
+    LLMK_CHECK_LAUNCH_RC("head_delta_step", e);
     return LLMK_OK;
 }

@@ -576,7 +576,7 @@ struct DeltaParams {
     const float* qkv;        // [n_tokens, ld]: q at column 0, k at G * D, v at 2 * G * D, prepared
     long long qkv_ld;
     const float* beta;       // [n_tokens, H + G]: beta of every head, then q . k of every key head
-    const float* decay;      // [n_tokens, H * D]: 1 - g (null: one decay per head, `beta` is then [n_tokens, 2 H + G]: beta, 1 - g, q . k)
+    const float* decay;      // [n_tokens, H * D]: 1 - g (null: one decay per head, `beta` is then [n_tokens, 2 H + G]: beta, log g, q . k)
     float* state;            // [slots, state_ld]: S [H][D][E]
     long long state_ld;
     const int* cu_q;
@@ -644,7 +644,7 @@ __device__ __forceinline__ void delta_load_chunk(const DeltaParams& p, float* bu
         const float* row = p.beta + (size_t)(t_first + threadIdx.x) * ((HEAD ? 2 : 1) * p.H + p.G);
         bs[threadIdx.x] = row[h];
         bs[DELTA_CHUNK + threadIdx.x] = row[(HEAD ? 2 : 1) * p.H + kvh];
-        if (HEAD) bs[2 * DELTA_CHUNK + threadIdx.x] = row[p.H + h];
+        if (HEAD) bs[2 * DELTA_CHUNK + threadIdx.x] = -expm1f(row[p.H + h]);
     }
 }
 
@@ -794,7 +794,7 @@ LLMK_EXPORT int llmk_delta_scan(float* out, float* qkv, long long qkv_ld, const 
 }
 
 // The same walk with one decay per head over rows that are already prepared (csrc/head_delta.cu): qkv float32 with q and k as unit
-// vectors (q scaled), gates float32 [n_tokens, 2 H + G]: beta, 1 - g, q . k of every key head.
+// vectors (q scaled), gates float32 [n_tokens, 2 H + G]: beta, log g, q . k of every key head.
 LLMK_EXPORT int llmk_delta_scan_heads(float* out, const float* qkv, long long qkv_ld, const float* gates, float* state, long long state_ld,
                                       const int* cu_q, const int* state_slots, int n_seqs, int n_tokens, int H, int G, int D, int E,
                                       void* stream) {

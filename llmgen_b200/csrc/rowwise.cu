@@ -13,7 +13,8 @@
 //   act_rows        relu(x)^2, tanh(x), gelu_tanh(x), the clamped gated unit  g' s(alpha g') (u' + 1)  with g' = min(g, L), u' = clamp(u, -L, L),
 //                   or the gated units gelu_tanh(g) u and silu(g) u
 //   gated_rmsnorm   out[r, :] = rmsnorm(o[r, :]) * w * sigmoid(g[r, :])   (or, without gains, o * sigmoid(g)); the gate may
-//                   pass silu instead, or enter as it is; the gains may differ between `w_rows` consecutive rows (heads)
+//                   pass silu instead, or enter as it is; the gains may differ between `w_rows` consecutive rows (heads);
+//                   a token's heads lie side by side, tokens `ldo` values apart
 //   add_bias        y[r, :] += b, y an array of T or of float32, or the float32 slices of a product (the first slice takes it)
 //   concat_stream   out[r, :] = [ (T)(resid[r, :] + delta[r, :]) | (T) x0[r, :] ]: the operand of a product that mixes the
 //                   residual stream with the embedding's output
@@ -50,7 +51,7 @@ __global__ void norm_add_kernel(float* __restrict__ resid, const void* __restric
     float ss = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float v = load_sum<T>(y, r * H + i, splits, split_stride);
-        if (y2) v = a * v + b * load_sum<T>(y2, r * H + i, splits2, split_stride2);
+        v = y2 ? a * v + b * load_sum<T>(y2, r * H + i, splits2, split_stride2) : a * v;
         srow[i] = v;
         ss += v * v;
     }
@@ -77,7 +78,7 @@ __global__ void norm_add_kernel(float* __restrict__ resid, const void* __restric
     for (int i = threadIdx.x; i < H; i += blockDim.x) copy[r * H + i] = from_float<T>(srow[i] * rinv2 * w_next[i]);
 }
 
-// y2 (with its own slices) null: resid += rmsnorm(y) w.  Else resid += rmsnorm(a y + b y2) w.  w_next non-null: `copy`
+// y2 (with its own slices) null: resid += rmsnorm(a y) w.  Else resid += rmsnorm(a y + b y2) w.  w_next non-null: `copy`
 // receives rmsnorm(new row) * w_next (eps_next inside the root) instead of the new row.
 LLMK_EXPORT int llmk_norm_add2(float* resid, const void* y, const float* w, void* copy, int n_rows, int H, float eps,
                                int splits, long long split_stride, const void* y2, int splits2, long long split_stride2,
@@ -477,7 +478,7 @@ enum { GATE_SIGMOID = 0, GATE_SILU = 1, GATE_PLAIN = 2 };
 template <typename T>
 __global__ void gated_rmsnorm_kernel(T* __restrict__ out, const float* __restrict__ o, const T* __restrict__ g,
                                      const float* __restrict__ w, int H, long long ldg, float eps, int gate_act, int w_rows,
-                                     int heads) {
+                                     int heads, long long ldo) {
     __shared__ float scratch[33];
     const size_t r = blockIdx.x;
     pdl_launch_dependents();
@@ -495,11 +496,12 @@ __global__ void gated_rmsnorm_kernel(T* __restrict__ out, const float* __restric
     const size_t head = r % (size_t)heads;
     const float* wr = w ? w + (head % (size_t)w_rows) * H : nullptr;
     const T* gr = g + (r / (size_t)heads) * ldg + head * H;
+    T* dst = out + (r / (size_t)heads) * ldo + head * H;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         const float gv = to_float(gr[i]);
         const float sg = 1.0f / (1.0f + expf(-gv));
         const float gate = gate_act == GATE_SIGMOID ? sg : gate_act == GATE_SILU ? gv * sg : gv;
-        out[r * H + i] = from_float<T>(o[r * H + i] * rinv * (wr ? wr[i] : 1.f) * gate);
+        dst[i] = from_float<T>(o[r * H + i] * rinv * (wr ? wr[i] : 1.f) * gate);
     }
 }
 
@@ -507,7 +509,7 @@ __global__ void gated_rmsnorm_kernel(T* __restrict__ out, const float* __restric
 template <typename T>
 __global__ void __launch_bounds__(256) gated_rmsnorm_warp_kernel(T* __restrict__ out, const float* __restrict__ o, const T* __restrict__ g,
                                                                  const float* __restrict__ w, int n_rows, int H, long long ldg, float eps,
-                                                                 int gate_act, int w_rows, int heads) {
+                                                                 int gate_act, int w_rows, int heads, long long ldo) {
     const size_t r = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     pdl_launch_dependents();
@@ -526,16 +528,17 @@ __global__ void __launch_bounds__(256) gated_rmsnorm_warp_kernel(T* __restrict__
     const size_t head = r % (size_t)heads;
     const float* wr = w ? w + (head % (size_t)w_rows) * H : nullptr;
     const T* gr = g + (r / (size_t)heads) * ldg + head * H;
+    T* dst = out + (r / (size_t)heads) * ldo + head * H;
     for (int i = lane; i < H; i += 32) {
         const float gv = to_float(gr[i]);
         const float sg = 1.0f / (1.0f + expf(-gv));
         const float gate = gate_act == GATE_SIGMOID ? sg : gate_act == GATE_SILU ? gv * sg : gv;
-        out[r * H + i] = from_float<T>(o[r * H + i] * rinv * (wr ? wr[i] : 1.f) * gate);
+        dst[i] = from_float<T>(o[r * H + i] * rinv * (wr ? wr[i] : 1.f) * gate);
     }
 }
 
 LLMK_EXPORT int llmk_gated_rmsnorm(void* out, const float* o, const void* g, const float* w, int n_rows, int H, long long ldg,
-                                   float eps, int gate_act, int w_rows, int heads, int dtype, void* stream) {
+                                   float eps, int gate_act, int w_rows, int heads, long long ldo, int dtype, void* stream) {
     if (n_rows <= 0 || H <= 0) return LLMK_OK;
     if (gate_act < GATE_SIGMOID || gate_act > GATE_PLAIN || heads < 1 || (w_rows != 1 && w_rows != heads))
         LLMK_FAIL("gated_rmsnorm: gate form %d, %d heads a token, %d rows of gains", gate_act, heads, w_rows);
@@ -545,16 +548,16 @@ LLMK_EXPORT int llmk_gated_rmsnorm(void* out, const float* o, const void* g, con
     if (H <= 256 && n_rows >= 64 && (dtype == LLMK_F32 || dtype == LLMK_BF16)) {
         const dim3 grid((unsigned)ceil_div(n_rows, 8));
         if (dtype == LLMK_F32)
-            e = llmk_launch(gated_rmsnorm_warp_kernel<float>, grid, dim3(256), 0, s, true, (float*)out, o, (const float*)g, w, n_rows, H, ldg, eps, gate_act, w_rows, heads);
+            e = llmk_launch(gated_rmsnorm_warp_kernel<float>, grid, dim3(256), 0, s, true, (float*)out, o, (const float*)g, w, n_rows, H, ldg, eps, gate_act, w_rows, heads, ldo);
         else
-            e = llmk_launch(gated_rmsnorm_warp_kernel<bf16>, grid, dim3(256), 0, s, true, (bf16*)out, o, (const bf16*)g, w, n_rows, H, ldg, eps, gate_act, w_rows, heads);
+            e = llmk_launch(gated_rmsnorm_warp_kernel<bf16>, grid, dim3(256), 0, s, true, (bf16*)out, o, (const bf16*)g, w, n_rows, H, ldg, eps, gate_act, w_rows, heads, ldo);
         LLMK_CHECK_LAUNCH_RC("gated_rmsnorm", e);
         return LLMK_OK;
     }
     if (dtype == LLMK_F32)
-        e = llmk_launch(gated_rmsnorm_kernel<float>, dim3(n_rows), dim3(threads), 0, s, true, (float*)out, o, (const float*)g, w, H, ldg, eps, gate_act, w_rows, heads);
+        e = llmk_launch(gated_rmsnorm_kernel<float>, dim3(n_rows), dim3(threads), 0, s, true, (float*)out, o, (const float*)g, w, H, ldg, eps, gate_act, w_rows, heads, ldo);
     else if (dtype == LLMK_BF16)
-        e = llmk_launch(gated_rmsnorm_kernel<bf16>, dim3(n_rows), dim3(threads), 0, s, true, (bf16*)out, o, (const bf16*)g, w, H, ldg, eps, gate_act, w_rows, heads);
+        e = llmk_launch(gated_rmsnorm_kernel<bf16>, dim3(n_rows), dim3(threads), 0, s, true, (bf16*)out, o, (const bf16*)g, w, H, ldg, eps, gate_act, w_rows, heads, ldo);
     else
         LLMK_FAIL("gated_rmsnorm: unknown dtype %d", dtype);
     LLMK_CHECK_LAUNCH_RC("gated_rmsnorm", e);
@@ -624,7 +627,7 @@ LLMK_EXPORT int llmk_concat_stream(void* out, const float* resid, const void* de
 }
 
 // ------------------------------------------------------------------------------------------------ several residual streams
-// streams [n, S, H] float32.  With y (an array of T, float32 slices, or a y + b y2): every stream is rewritten from all the old
+// streams [n, S, H] float32.  With y (an array of T or float32 slices, times a, or a y + b y2): every stream is rewritten from all the old
 // ones, x_t <- sum_s mix[s * S + t] x_s + out_coef[t] y.  With next_in: normed[r, :] = rmsnorm(sum_t next_in[t] x_t) * next_gain
 // (the new streams), the input of the sublayer that follows.  Either half may be absent.  A block per token row.
 constexpr int MAX_STREAMS = 16;
@@ -660,7 +663,7 @@ __global__ void __launch_bounds__(512) stream_step_kernel(float* __restrict__ st
         float u = 0.f;
         if (y) {
             float v = load_sum<T>(y, r * H + i, splits, split_stride);
-            if (y2) v = a * v + b * load_sum<T>(y2, r * H + i, splits2, split_stride2);
+            v = y2 ? a * v + b * load_sum<T>(y2, r * H + i, splits2, split_stride2) : a * v;
             // every new stream from the old ones (x stays as it was read); the next sublayer's sum is taken on the way
 #pragma unroll(MS <= 8 ? MS : 1)
             for (int t = 0; t < MS; ++t) {

@@ -197,6 +197,11 @@ class ModelCost:
                 n_mm += mixer.hidden_size * (2 * kd + 3 * vd + 2 * mixer.num_heads)
                 token_flops += 6 * mixer.num_heads * mixer.key_dim * mixer.value_dim       # read-out and update over the memory
                 state_bytes += 4 * (mixer.num_heads * mixer.key_dim * (mixer.value_dim + 1) + mixer.num_heads)
+            elif kind == "head_decay_delta":
+                kd, vd = mixer.num_kv_heads * mixer.key_dim, mixer.num_heads * mixer.value_dim
+                n_mm += mixer.hidden_size * (2 * kd + 3 * vd + 2 * mixer.num_heads)
+                token_flops += 7 * mixer.num_heads * mixer.key_dim * mixer.value_dim + 2 * mixer.conv.taps * mixer.conv.channels
+                state_bytes += 4 * (mixer.num_heads * mixer.key_dim * mixer.value_dim + (mixer.conv.taps - 1) * mixer.conv.channels)
             elif kind == "general_delta":
                 hd = mixer.num_heads * mixer.head_dim
                 n_mm += mixer.hidden_size * (6 * hd + mixer.decay_rank) + mixer.decay_rank * hd
@@ -218,7 +223,7 @@ class ModelCost:
             elif getattr(ffn, "kind", None) == "routed_mlp":
                 # what one token uses: the router, its chosen experts and the shared one
                 matrices = 3 if getattr(ffn.experts[0], "gate_proj", None) else 2
-                n_mm += ffn.hidden_size * (len(ffn.experts) + matrices * ffn.top_k * ffn.experts[0].intermediate_size)
+                n_mm += ffn.hidden_size * (len(ffn.experts) + ffn.identity_outputs + (1 if ffn.shared_gate else 0) + matrices * ffn.top_k * ffn.experts[0].intermediate_size)
                 if ffn.shared is not None:
                     n_mm += 3 * ffn.hidden_size * ffn.shared.intermediate_size
             elif ffn is not None:
@@ -406,6 +411,26 @@ def _cost_delta_scan(a, info: PassInfo) -> Tuple[int, int]:
     return flops, bytes_
 
 
+def _cost_head_delta_prep(a, info: PassInfo) -> Tuple[int, int]:
+    n, C = a["qkv"].shape
+    H, K = int(a["heads"]), int(a["taps"].shape[1])
+    return n * C * (2 * K + 8), n * (C + 2 * H) * a["packed"].element_size() + _nbytes(a["qkv"]) + _nbytes(a["gates"])
+
+
+def _cost_head_delta(a, info: PassInfo) -> Tuple[int, int]:
+    H, D, E = int(a["heads"]), int(a["dim"]), int(a["vdim"])
+    n = a["out"].shape[0]
+    flops = n * H * 7 * D * E                              # decay, two dot products and the update over the state, a token
+    return flops, _nbytes(a["qkv"]) + _nbytes(a["gates"]) + _nbytes(a["out"]) + 2 * len(info.q_lens) * H * D * E * 4
+
+
+def _cost_head_delta_step(a, info: PassInfo) -> Tuple[int, int]:
+    H, D, E = int(a["heads"]), int(a["dim"]), int(a["vdim"])
+    n, (C, K) = a["y"].shape[0], a["taps"].shape
+    moved = n * (C + H * (E + 2)) * a["packed"].element_size() + _nbytes(a["y"]) + _nbytes(a["taps"])
+    return n * (H * 7 * D * E + C * (2 * K + 8)), moved + 8 * len(info.q_lens) * (H * D * E + (K - 1) * C)
+
+
 def _cost_decay_scan(a, info: PassInfo) -> Tuple[int, int]:
     H, D, E = int(a["heads"]), int(a["dim"]), int(a["vdim"])
     n = a["out"].shape[0]
@@ -558,7 +583,8 @@ OP_COSTS: Dict[str, Callable] = {
     "attn_prep": _cost_attn_prep, "gemm_simt": _cost_product, "gemv_bf16": _cost_product, "gemm_tc": _cost_product,
     "gemm_skinny": _cost_product, "gemm_rows8": _cost_product, "gemm_rows8_gated": _cost_product, "paged_attention": _cost_attention, "attention_decode": _cost_attention,
     "attention_tc": _cost_attention, "attention_mma": _cost_attention, "attention_mma_parts": _cost_attention, "sample": _cost_all_operands,
-    "short_conv": _cost_short_conv, "rglru": _cost_rglru, "delta_scan": _cost_delta_scan, "add_bias": _cost_all_operands,
+    "short_conv": _cost_short_conv, "rglru": _cost_rglru, "delta_scan": _cost_delta_scan, "delta_scan_heads": _cost_head_delta, "head_delta_prep": _cost_head_delta_prep,
+    "head_delta_chunks": _cost_head_delta, "head_delta_step": _cost_head_delta_step, "add_bias": _cost_all_operands,
     "concat_stream": _cost_all_operands, "logit_cap": _cost_all_operands,
     "decay_scan": _cost_decay_scan, "token_shift_mix": _cost_token_shift, "scaled_sum": _cost_scaled_sum,
     "stream_step": _cost_stream_step, "stream_spread": _cost_in_place, "attn_prep_rows": _cost_attn_prep_rows,

@@ -814,7 +814,7 @@ def norm_add(resid: torch.Tensor, y, weight: torch.Tensor, eps: float, copy: Opt
 
 class WeightedPair:
     """a * first + b * second, not yet added up: what a mixer made of two mixers side by side returns.  Each of the two
-    is an array of the storage dtype or a `Partials`.  `norm_add` takes it as it is; `scaled_sum` adds it up for
+    is an array of the storage dtype or a `Partials`; without a second (None) it is a * first.  `norm_add` takes it as it is; `scaled_sum` adds it up for
     consumers that take one array."""
 
     def __init__(self, first, a: float, second, b: float):
@@ -836,9 +836,9 @@ def scaled_sum(out: torch.Tensor, pair: WeightedPair, dtype: torch.dtype) -> Par
             or out.shape[2] != pair.cols:
         raise KernelError("scaled_sum: the sum goes to a contiguous float32 [1, rows, cols] array")
     src, splits, stride = _delta_args(pair.first, dtype)
-    src2, splits2, stride2 = _delta_args(pair.second, dtype)
+    src2, splits2, stride2 = _delta_args(pair.second if pair.second is not None else pair.first, dtype)
     _check(lib, lib.llmk_scaled_sum(_ptr(out), _ptr(src), c_int(splits), c_longlong(stride), _ptr(src2), c_int(splits2),
-                                    c_longlong(stride2), c_float(pair.a), c_float(pair.b), c_longlong(pair.rows * pair.cols),
+                                    c_longlong(stride2), c_float(pair.a), c_float(pair.b if pair.second is not None else 0.0), c_longlong(pair.rows * pair.cols),
                                     c_int(dtype_code(dtype)), _stream()))
     return Partials(out)
 
@@ -938,9 +938,12 @@ def gated_rmsnorm(out: torch.Tensor, o: torch.Tensor, gate: torch.Tensor, weight
     o float32 [n, H] contiguous, gate of the storage dtype with any row stride.  Without `weight`: o * f(gate).
     `heads` > 1: every row of out and o is one head of a token (row = token * heads + head) and the gate is
     [n / heads, heads * H] with any row stride; `weight` is then [H], shared by the heads, or, with `gains_per_head`,
-    [heads, H]."""
+    [heads, H].  `out` may then also be given as [n / heads, heads * H] with any row stride."""
     lib = build.load("rowwise")
-    n, H = out.shape
+    n, H = o.shape
+    if tuple(out.shape) not in ((n, H), (n // heads, heads * H)) or (out.shape[0] == n and not out.is_contiguous()):
+        raise KernelError("gated_rmsnorm: out is [n, H] or [n / heads, heads * H]")
+    ldo = heads * H if out.shape[0] == n else _row_stride(out)
     if o.dtype != torch.float32 or not o.is_contiguous() or gate.dtype != out.dtype or n % heads != 0:
         raise KernelError("gated_rmsnorm: o must be contiguous float32 and the gate of the storage dtype")
     w_rows = heads if gains_per_head else 1
@@ -950,7 +953,7 @@ def gated_rmsnorm(out: torch.Tensor, o: torch.Tensor, gate: torch.Tensor, weight
         raise KernelError("gated_rmsnorm: the gate is [tokens, heads * H]")
     _check(lib, lib.llmk_gated_rmsnorm(_ptr(out), _ptr(o), _ptr(gate), _ptr(weight), c_int(n), c_int(H), c_longlong(_row_stride(gate)),
                                        c_float(eps), c_int(GATE_FORMS[gate_form]), c_int(w_rows), c_int(heads),
-                                       c_int(dtype_code(out.dtype)), _stream()))
+                                       c_longlong(ldo), c_int(dtype_code(out.dtype)), _stream()))
 
 
 def add_bias(y, bias: torch.Tensor) -> None:
@@ -1254,7 +1257,7 @@ def head_delta_prep(qkv: torch.Tensor, gates: torch.Tensor, packed: torch.Tensor
     """What precedes the gated delta rule with one decay per head (csrc/head_delta.cu).  `packed` [n, ...] (storage dtype, any row
     stride): the projections of q, k, v at column 0, of beta and of the decays at `beta_off` and `decay_off`.  qkv float32
     [n, 2 kv_heads dim + heads vdim] = short convolution (`taps` float32 [channels, K]) and silu, q and k as unit vectors per head, q
-    times dim^-1/2; gates float32 [n, 2 heads + kv_heads] = beta, 1 - decay, q . k.  `conv_state` (K > 1): the columns of the state
+    times dim^-1/2; gates float32 [n, 2 heads + kv_heads] = beta, log of the decay, q . k.  `conv_state` (K > 1): the columns of the state
     array from the convolution's inputs on, [slots, >= (K - 1) channels], read and left with the last K - 1 inputs."""
     lib = build.load("head_delta")
     n, C = qkv.shape
@@ -1292,6 +1295,53 @@ def delta_scan_heads(out: torch.Tensor, qkv: torch.Tensor, gates: torch.Tensor, 
     _check(lib, lib.llmk_delta_scan_heads(_ptr(out), _ptr(qkv), c_longlong(_row_stride(qkv)), _ptr(gates), _ptr(state), c_longlong(_row_stride(state)),
                                           _ptr(cu_q), _ptr(state_slots), c_int(n_seqs), c_int(out.shape[0]), c_int(heads), c_int(kv_heads),
                                           c_int(dim), c_int(vdim), _stream()))
+
+
+def head_delta_chunk_floats(n_tokens: int, n_seqs: int, heads: int, kv_heads: int, dim: int, vdim: int) -> int:
+    """Floats of scratch `head_delta_chunks` needs for a step of this shape; 0: it does not take these widths."""
+    fn = build.load("head_delta").llmk_head_delta_chunk_floats
+    fn.restype = c_longlong
+    return int(fn(c_int(n_tokens), c_int(n_seqs), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim)))
+
+
+def head_delta_chunks(out: torch.Tensor, qkv: torch.Tensor, gates: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor,
+                      state_slots: torch.Tensor, scratch: torch.Tensor, n_seqs: int, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
+    """The same result as `delta_scan_heads`, chunks of 64 tokens at a time (csrc/head_delta.cu); key widths up to 128; `scratch`:
+    `head_delta_chunk_floats` float32."""
+    lib = build.load("head_delta")
+    _check_head_delta("head_delta_chunks", out, qkv, gates, state, heads, kv_heads, dim, vdim)
+    if scratch.dtype != torch.float32 or scratch.numel() < head_delta_chunk_floats(out.shape[0], n_seqs, heads, kv_heads, dim, vdim):
+        raise KernelError("head_delta_chunks: the scratch is too small")
+    _check(lib, lib.llmk_head_delta_chunks(_ptr(out), _ptr(qkv), _ptr(gates), _ptr(state), c_longlong(_row_stride(state)), _ptr(cu_q),
+                                           _ptr(state_slots), _ptr(scratch), c_int(n_seqs), c_int(out.shape[0]), c_int(heads), c_int(kv_heads),
+                                           c_int(dim), c_int(vdim), _stream()), 2)
+
+
+def head_delta_step_usable(heads: int, kv_heads: int, dim: int, vdim: int) -> bool:
+    return bool(build.load("head_delta").llmk_head_delta_step_usable(c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim)))
+
+
+def head_delta_step(y: torch.Tensor, packed: torch.Tensor, beta_off: int, decay_off: int, gate_off: int, taps: torch.Tensor,
+                    dt_bias: torch.Tensor, a_log: torch.Tensor, norm_gain: torch.Tensor, norm_eps: float, state: torch.Tensor,
+                    cu_q: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, heads: int, kv_heads: int, dim: int, vdim: int,
+                    unit_eps: float) -> None:
+    """A few tokens of every sequence through the gated delta rule with one decay per head in one launch (csrc/head_delta.cu): what
+    `head_delta_prep` and `delta_scan_heads` do, each head's RMSNorm (`norm_gain` float32 [vdim]) and the gate silu(packed[:, gate_off
+    ..]).  y [n, heads vdim] (the dtype of `packed`, any row stride); state [slots, heads dim vdim + (taps - 1) channels] float32."""
+    lib = build.load("head_delta")
+    n = y.shape[0]
+    C, K = taps.shape
+    size = heads * dim * vdim
+    if y.dtype != packed.dtype or y.shape[1] != heads * vdim or packed.shape[0] != n or C != 2 * kv_heads * dim + heads * vdim \
+            or state.dtype != torch.float32 or state.shape[1] < size + (K - 1) * C or taps.dtype != torch.float32 or not taps.is_contiguous() \
+            or norm_gain.dtype != torch.float32 or norm_gain.numel() != vdim:
+        raise KernelError("head_delta_step: shapes or dtypes do not fit")
+    conv_state = state[:, size:] if K > 1 else None
+    _check(lib, lib.llmk_head_delta_step(_ptr(y), c_longlong(_row_stride(y)), _ptr(packed), c_longlong(_row_stride(packed)), c_int(beta_off),
+                                         c_int(decay_off), c_int(gate_off), _ptr(taps), _ptr(dt_bias), _ptr(a_log), _ptr(norm_gain), c_float(norm_eps),
+                                         _ptr(state), _ptr(conv_state), c_longlong(_row_stride(state)), _ptr(cu_q), _ptr(state_slots), c_int(n_seqs),
+                                         c_int(n), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(K), c_float(unit_eps),
+                                         c_float(float(dim) ** -0.5), c_int(dtype_code(packed.dtype)), _stream()))
 
 
 DECAY_FORMS = {"sigmoid_pow": 0, "exp_exp": 1}

@@ -5,7 +5,7 @@ import torch
 
 from ..cache.manager import FULL, WINDOW
 from ..kernels import ops
-from .base import KVRequest, LayerCache, Mixer, StateRequest
+from .base import KVRequest, LayerCache, Mixer, SharedProjections, StateRequest
 from .linear import GEMM_MODULES, linear, linear_sliced
 from .registry import build_position, norm_class, register_mixer
 from .spec import INIT_ONE_PLUS_NORMAL, VECTOR, AttentionSpec, RopeSpec, WeightDecl
@@ -131,6 +131,7 @@ class GQAAttention(Mixer):
         # packed on the device: each matrix goes up through the loader's pinned stage as the file holds it
         names = [spec.q_proj, spec.k_proj] + ([] if spec.values_from_keys else [spec.v_proj]) + ([spec.gate_proj] if spec.gate_proj else [])
         self.w_qkv = torch.cat([weights.device_tensor(n, dtype, device, keep=False) for n in names], dim=0).contiguous()
+        self.packed_columns = self.w_qkv.shape[0]
         self.w_q = self.w_qkv[: self.nq * self.hd]
         self.gate_off = (self.nq + self.nkv) * self.hd + self.nkv * self.vd if spec.gate_proj else -1
         # a run item that reads another item's cache projects q (and the gate) only
@@ -278,7 +279,7 @@ class GQAAttention(Mixer):
         """Bytes of activations this part keeps in the step's workspace for `tokens` rows: the packed projection
         (and the float32 slices of two products cut along K), q, the attention's output and the output projection."""
         elem = 2 if self.dtype == torch.bfloat16 else 4
-        packed = self.w_qkv.shape[0]
+        packed = self.packed_columns
         return tokens * (packed + 2 * self.nq * max(self.hd, self.vd) + self.spec.hidden_size) * elem + 2 * ops.SLICED_PRODUCT_BYTES
 
     def forward(self, ctx, x, cache: LayerCache):
@@ -348,6 +349,30 @@ class GQAAttention(Mixer):
             return self._forward_row_norms(ctx, x, cache, group, cos, sin, rot)
         w = self.w_qkv if cache.writes else self.w_q_gate
         packed = linear(x, w, ws.buffer("attn_qkvg" if cache.writes else "attn_qg", T, w.shape[0], self.dtype))
+        o = ws.buffer("attn_o", T, self.nq * self.vd, self.dtype)
+        self.forward_inner(ctx, packed, cache, o)
+        out = linear_sliced(ws, "mixer_out", o, self.w_o, self.dtype)
+        if self.o_bias is not None:
+            ops.add_bias(out, self.o_bias)
+        return out
+
+    # -- what a parallel mixer asks that multiplies with several branches' matrices at once (see `parts.parallel`)
+    def shared_projections(self):
+        spec = self.spec
+        if not self.is_varied or spec.values_from_keys or self.row_norms or self.o_bias is not None:
+            return None
+        return SharedProjections(self.w_qkv, self.w_o)
+
+    def drop_projections(self) -> None:
+        self.w_qkv = self.w_q = self.w_q_gate = self.w_o = None
+
+    def forward_inner(self, ctx, packed, cache, o) -> None:
+        """From the packed projection [q | k | v | gate] (q and the gate alone where another item wrote the cache) to the heads' rows."""
+        T, ws = ctx.n_tokens, ctx.workspace
+        group = ctx.groups[cache.group]
+        nk = self.nkv if cache.writes else 0
+        cos, sin = self.position.tables() if self.position is not None else (None, None)
+        rot = self.position.rotary_dim if self.position is not None else 0
         gate = None
         if self.gate_off >= 0:
             gate = packed[:, self.gate_off:] if cache.writes else packed[:, self.nq * self.hd:]
@@ -356,7 +381,6 @@ class GQAAttention(Mixer):
         ops.attn_prep(packed, cache.k, cache.v, ctx.positions, group.slots, cos, sin, self.q_gain, self.k_gain,
                       self.nq, nk, self.hd, rot, cache.page_size, self.norm_eps, self.q_off, self.k_off, q_out=q,
                       pairing=self.pairing, head_norm=self.head_norm, bias=bias, vd=self.vd)
-        o = ws.buffer("attn_o", T, self.nq * self.vd, self.dtype)
         mma_bq = 0 if ctx.pure_decode else self.mma_tile_queries()
         if mma_bq and ctx.has_array(f"attention_tiles_bq{mma_bq}_seq"):
             # portions of prompts in bfloat16: the products on the tensor cores, the weights float32 (three terms)
@@ -365,14 +389,17 @@ class GQAAttention(Mixer):
                               ctx.array(f"attention_tiles_bq{mma_bq}_q0"), tile_seq.numel(), self.nq, self.nkv, self.hd, self.vd,
                               cache.page_size, self.window, float(self.spec.scale), softcap=self.softcap, sink=self.sink, gate=gate,
                               chunk=self.chunk)
-            out = linear_sliced(ws, "mixer_out", o, self.w_o, self.dtype)
-            if self.o_bias is not None:
-                ops.add_bias(out, self.o_bias)
-            return out
-        tile_seq = ctx.array(self.tiles_name + "_seq")
-        tile_q0 = ctx.array(self.tiles_name + "_q0")
+            return
         # single decoded tokens: the keys in parts that are merged afterwards (the sink enters once, in the merge)
         parts, part_size = self._split(ctx)
+        if ctx.pure_decode and gate is None and self.mma_tile_queries():
+            # in bfloat16 without a gate: the parts of a token's keys are the blocks of a cluster
+            ops.attention_mma_parts(o, q, cache.k, cache.v, group.block_tables, group.max_blocks, ctx.ctx_len, ctx.cu_q, ctx.n_seqs, self.nq,
+                                    self.nkv, self.hd, self.vd, cache.page_size, self.window, float(self.spec.scale),
+                                    min(parts, ops.ATTENTION_MMA_MAX_PARTS), softcap=self.softcap, sink=self.sink, chunk=self.chunk)
+            return
+        tile_seq = ctx.array(self.tiles_name + "_seq")
+        tile_q0 = ctx.array(self.tiles_name + "_q0")
         scratch = None
         if parts > 1:
             scratch = ws.flat("attn_split", ops.attention_scratch_floats(T, self.nq, self.vd, parts), torch.float32)
@@ -380,10 +407,6 @@ class GQAAttention(Mixer):
                             ctx.ctx_len, ctx.cu_q, tile_seq, tile_q0, tile_seq.numel(), T, self.nq, self.nkv,
                             self.hd, cache.page_size, self.window, float(self.spec.scale), parts, part_size, scratch,
                             vd=self.vd, softcap=self.softcap, sink=self.sink, gate=gate, chunk=self.chunk)
-        out = linear_sliced(ws, "mixer_out", o, self.w_o, self.dtype)
-        if self.o_bias is not None:
-            ops.add_bias(out, self.o_bias)
-        return out
 
     def _forward_row_norms(self, ctx, x, cache, group, cos, sin, rot):
         """A layer whose q and k are normed over their whole projections: the packed projection [q | k | v | gate], the short

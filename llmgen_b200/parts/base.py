@@ -36,6 +36,8 @@ Mixer:
     forward(ctx, x, cache) -> [T, H]          x is the normed input; `cache` is this run
                                               item's `LayerCache`; returns an array or a
                                               `Partials` (see `parts.linear.linear_sliced`)
+    shared_projections() -> SharedProjections | None
+                                              optional: see that class
 Feed-forward:
     forward(ctx, x) -> [T, H]                 an array or a `Partials`
 Any part, optional:
@@ -94,6 +96,16 @@ class StateRequest:
     """One array of `shape` and `dtype` per request, zero when the request starts."""
     shape: Tuple[int, ...]
     dtype: torch.dtype = torch.float32
+
+
+@dataclass(frozen=True)
+class SharedProjections:
+    """What a mixer offers that a parallel mixer may run between projections of its own: its packed input matrix [columns, hidden] and its
+    output matrix [hidden, inner].  The mixer then has `forward_inner(ctx, packed, cache, out)`: `packed` is the input's product with
+    the first (any row stride), `out` takes the rows that the second multiplies (any row stride); and, unless it is the first
+    branch, `scale_output(factor)`: every such row times a constant, folded into what makes it.  `drop_projections()` lets go of both."""
+    w_in: torch.Tensor
+    w_out: torch.Tensor
 
 
 @dataclass

@@ -5,7 +5,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import LayerCache, Mixer, StateRequest
+from .base import LayerCache, Mixer, SharedProjections, StateRequest
 from .linear import GEMM_MODULES, linear, linear_sliced
 from .registry import norm_class, register_mixer
 from .spec import VECTOR, GatedDeltaSpec, HeadDecayDeltaSpec, WeightDecl
@@ -99,8 +99,10 @@ class GatedDelta(Mixer):
 
 class HeadDecayDelta(Mixer):
     """One packed projection [q | k | v | gate | beta | decay] -> one pass over the tokens: the short convolution and silu of q, k, v, unit
-    vectors, beta's sigmoid and the decays (`head_delta_prep`, float32 out) -> the recurrence over each sequence's new tokens
-    (`delta_scan_heads`) -> RMSNorm of each head's output times silu(gate), one kernel -> output projection.
+    vectors, beta's sigmoid and the decays (`head_delta_prep`, float32 out) -> the recurrence over each sequence's new tokens, for
+    steps of `CHUNKED_ROWS` rows and more chunk by chunk (`head_delta_chunks`), else token by token (`delta_scan_heads`) -> RMSNorm of
+    each head's output times silu(gate), one kernel -> output projection.  Single tokens, and steps of up to `STEP_ROWS` rows, do all
+    between the two projections in one launch (`head_delta_step`).
 
     State of a request, one float32 row of the cache manager's slots: [S (heads x key_dim x value_dim) | the
     convolution's last taps - 1 inputs over the channels of q, k, v side by side, oldest first].  Lengths and slots
@@ -108,6 +110,8 @@ class HeadDecayDelta(Mixer):
 
     step_arrays_follow_shapes = True
     replay_any_step = True
+    CHUNKED_ROWS = 256
+    STEP_ROWS = 16
 
     @staticmethod
     def weight_decls(spec: HeadDecayDeltaSpec):
@@ -148,6 +152,7 @@ class HeadDecayDelta(Mixer):
         self.norm_gain = weights.device_tensor(spec.out_norm.weight, dtype, device)
         self.norm_eps = float(spec.out_norm.eps)
         self.s_size = H * D * E
+        self.step_usable = ops.head_delta_step_usable(H, G, D, E)
 
     def state_request(self) -> StateRequest:
         return StateRequest((self.s_size + (self.spec.conv.taps - 1) * self.qkv,), torch.float32)
@@ -155,24 +160,49 @@ class HeadDecayDelta(Mixer):
     def workspace_bytes(self, tokens: int) -> int:
         elem = 2 if self.dtype == torch.bfloat16 else 4
         he = self.H * self.E
-        return tokens * (self.w_in.shape[0] * elem + self.qkv * 4 + (2 * self.H + self.G) * 4 + he * (4 + elem)
+        chunks = 4 * ops.head_delta_chunk_floats(tokens, 1, self.H, self.G, self.D, self.E)
+        return chunks + tokens * ((self.decay_off + self.H) * elem + self.qkv * 4 + (2 * self.H + self.G) * 4 + he * (4 + elem)
                          + self.spec.hidden_size * elem) + ops.SLICED_PRODUCT_BYTES
+
+    # -- what a parallel mixer asks that multiplies with several branches' matrices at once (see `parts.parallel`)
+    def shared_projections(self):
+        return SharedProjections(self.w_in, self.w_o)
+
+    def drop_projections(self) -> None:
+        self.w_in = self.w_o = None
+
+    def scale_output(self, factor: float) -> None:
+        self.norm_gain = self.norm_gain * factor
 
     def forward(self, ctx, x, cache: LayerCache):
         T, ws = ctx.n_tokens, ctx.workspace
-        H, G, D, E = self.H, self.G, self.D, self.E
         packed = linear(x, self.w_in, ws.buffer("hdelta_in", T, self.w_in.shape[0], self.dtype))
+        y = ws.buffer("hdelta_y", T, self.H * self.E, self.dtype)
+        self.forward_inner(ctx, packed, cache, y)
+        return linear_sliced(ws, "hdelta_out", y, self.w_o, self.dtype)
+
+    def forward_inner(self, ctx, packed, cache: LayerCache, y) -> None:
+        """From the packed projection to the rows that the output matrix takes."""
+        T, ws = ctx.n_tokens, ctx.workspace
+        H, G, D, E = self.H, self.G, self.D, self.E
+        if (ctx.pure_decode or T <= self.STEP_ROWS) and self.step_usable:
+            ops.head_delta_step(y, packed, self.beta_off, self.decay_off, self.gate_off, self.conv_w, self.dt_bias, self.a_log, self.norm_gain,
+                                self.norm_eps, cache.state, ctx.cu_q, ctx.state_slots, ctx.n_seqs, H, G, D, E, float(self.spec.unit_eps))
+            return
         qkv = ws.buffer("hdelta_qkv", T, self.qkv, torch.float32)
         gates = ws.buffer("hdelta_gates", T, 2 * H + G, torch.float32)
         ops.head_delta_prep(qkv, gates, packed, self.beta_off, self.decay_off, self.conv_w, self.dt_bias, self.a_log,
                             cache.state[:, self.s_size:] if self.spec.conv.taps > 1 else None, ctx.cu_q, ctx.state_slots, ctx.n_seqs,
                             H, G, D, E, float(self.spec.unit_eps))
         o = ws.buffer("hdelta_o", T, H * E, torch.float32)
-        ops.delta_scan_heads(o, qkv, gates, cache.state, ctx.cu_q, ctx.state_slots, ctx.n_seqs, H, G, D, E)
-        y = ws.buffer("hdelta_y", T, H * E, self.dtype)
-        ops.gated_rmsnorm(y.view(T * H, E), o.view(T * H, E), packed[:, self.gate_off:self.beta_off], self.norm_gain, self.norm_eps,
+        floats = ops.head_delta_chunk_floats(T, ctx.n_seqs, H, G, D, E) if T >= self.CHUNKED_ROWS else 0
+        if floats:
+            scratch = ws.flat("hdelta_chunks", floats, torch.float32)
+            ops.head_delta_chunks(o, qkv, gates, cache.state, ctx.cu_q, ctx.state_slots, scratch, ctx.n_seqs, H, G, D, E)
+        else:
+            ops.delta_scan_heads(o, qkv, gates, cache.state, ctx.cu_q, ctx.state_slots, ctx.n_seqs, H, G, D, E)
+        ops.gated_rmsnorm(y, o.view(T * H, E), packed[:, self.gate_off:self.beta_off], self.norm_gain, self.norm_eps,
                           gate_form="silu", heads=H)
-        return linear_sliced(ws, "hdelta_out", y, self.w_o, self.dtype)
 
 
 register_mixer("gated_delta", GatedDelta)

@@ -5,6 +5,7 @@ import torch
 
 from ..kernels import ops
 from .base import LayerCache, Mixer, StateRequest
+from .linear import GEMM_MODULES, linear, linear_sliced
 from .registry import build_mixer, mixer_class, register_mixer
 from .spec import ParallelMixerSpec
 
@@ -24,7 +25,12 @@ class ParallelMixer(Mixer):
     Cache: the one branch that keeps paged keys and values (at most one may) receives the run item's pages; the
     branches that keep a per-request state share the item's state row, each its own stretch of it, in branch order.
     With two branches the result is handed on as an `ops.WeightedPair`, which the kernel that norms a sublayer's output
-    adds up on the way (`norm_add`); more branches are added up pair by pair into a float32 buffer."""
+    adds up on the way (`norm_add`, `stream_step`); more branches are added up pair by pair into a float32 buffer.
+
+    Branches that all offer `shared_projections` run between two products of the whole mixer: one with their input matrices stacked,
+    and one with their output matrices side by side over their inner rows side by side, which is the sum over the branches.  The
+    first branch's scale stays with the result (a `WeightedPair` without a second), the others' scales relative to it are folded into
+    what makes their inner rows."""
 
     @staticmethod
     def weight_decls(spec: ParallelMixerSpec):
@@ -32,7 +38,7 @@ class ParallelMixer(Mixer):
 
     @staticmethod
     def kernel_modules(spec):
-        return ("rowwise",) + tuple(m for b in spec.branches for m in mixer_class(b).kernel_modules(b))
+        return ("rowwise",) + GEMM_MODULES + tuple(m for b in spec.branches for m in mixer_class(b).kernel_modules(b))
 
     def __init__(self, spec: ParallelMixerSpec, weights, dtype, device):
         if len(spec.branches) < 2 or len(spec.branches) != len(spec.scales):
@@ -57,10 +63,31 @@ class ParallelMixer(Mixer):
             self.state_ranges.append((at, at + n, tuple(req.shape)))
             at += n
         self.state_size = at
+        self._share_projections(dtype)
         self.replay_any_step = all(getattr(b, "replay_any_step", False) for b in self.branches)
         self.step_arrays_follow_shapes = all(getattr(b, "step_arrays_follow_shapes", False) or not hasattr(b, "prepare_step")
                                              for b in self.branches)
         self.capturable = all(getattr(b, "capturable", True) for b in self.branches)
+
+    def _share_projections(self, dtype) -> None:
+        self.w_in = self.w_out = None
+        offers = [b.shared_projections() if hasattr(b, "shared_projections") else None for b in self.branches]
+        if any(o is None for o in offers) or self.scales[0] == 0.0 or any(not hasattr(b, "scale_output") for b in self.branches[1:]):
+            return
+        # every branch's columns and inner rows begin on 16 bytes
+        if any(o.w_in.shape[0] % 8 for o in offers[:-1]) or any(o.w_out.shape[1] % 8 for o in offers):
+            return
+        self.w_in = torch.cat([o.w_in for o in offers], dim=0).contiguous()
+        self.w_out = torch.cat([o.w_out for o in offers], dim=1).contiguous()
+        for b, s in zip(self.branches[1:], self.scales[1:]):
+            b.scale_output(s / self.scales[0])
+        self.in_ranges, self.inner_ranges = [], []
+        at = inner = 0
+        for b, o in zip(self.branches, offers):
+            self.in_ranges.append((at, at + o.w_in.shape[0]))
+            self.inner_ranges.append((inner, inner + o.w_out.shape[1]))
+            at, inner = at + o.w_in.shape[0], inner + o.w_out.shape[1]
+            b.drop_projections()           # the stacked matrices took their place
 
     # -- what the engine asks
     def cache_request(self):
@@ -88,7 +115,8 @@ class ParallelMixer(Mixer):
 
     def workspace_bytes(self, tokens: int) -> int:
         asks = [getattr(b, "workspace_bytes", None) for b in self.branches]
-        return sum(f(tokens) for f in asks if f is not None) + tokens * self.cols_hint() * 4
+        shared = tokens * (self.w_in.shape[0] + self.w_out.shape[1]) * self.w_in.element_size() if self.w_in is not None else 0
+        return sum(f(tokens) for f in asks if f is not None) + tokens * self.cols_hint() * 4 + shared
 
     def cols_hint(self) -> int:
         return int(getattr(self.spec.branches[0], "hidden_size", 0))
@@ -106,6 +134,16 @@ class ParallelMixer(Mixer):
                           page_size=cache.page_size, writes=cache.writes, state=state)
 
     def forward(self, ctx, x, cache: LayerCache):
+        if self.w_in is not None:
+            if not cache.writes:
+                raise ValueError("parallel mixer: branches between shared projections write their own cache")
+            T, ws = ctx.n_tokens, ctx.workspace
+            packed = linear(x, self.w_in, ws.buffer("parallel_in", T, self.w_in.shape[0], self.dtype))
+            inner = ws.buffer("parallel_inner", T, self.w_out.shape[1], self.dtype)
+            for i, b in enumerate(self.branches):
+                (lo, hi), (to, end) = self.in_ranges[i], self.inner_ranges[i]
+                b.forward_inner(ctx, packed[:, lo:hi], self._branch_cache(i, cache), inner[:, to:end])
+            return ops.WeightedPair(linear_sliced(ws, "parallel_out", inner, self.w_out, self.dtype), self.scales[0], None, 0.0)
         outs = [b.forward(ctx, x, self._branch_cache(i, cache)) for i, b in enumerate(self.branches)]
         pair = ops.WeightedPair(outs[0], self.scales[0], outs[1], self.scales[1])
         for y, s in zip(outs[2:], self.scales[2:]):
