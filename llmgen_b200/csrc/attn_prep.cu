@@ -490,6 +490,113 @@ static bool launch_vec(const void* qkv, long long row_stride, void* q_out, long 
     return true;
 }
 
+// The general kernel's arithmetic with 16-byte accesses for pairs (2i, 2i + 1): a pair never leaves its lane's vector, so any
+// rotary width, biases and values of their own width are taken, where all of them are whole vectors.  `LPR` lanes share one
+// (token, head) row.
+template <typename T, int LPR>
+__global__ void __launch_bounds__(256)
+attn_prep_pairs_kernel(const T* __restrict__ qkv, long long row_stride, T* __restrict__ q_out, long long q_stride, T* __restrict__ kcache,
+                       T* __restrict__ vcache, const int* __restrict__ positions, const int* __restrict__ slots,
+                       const float* __restrict__ cos_tab, const float* __restrict__ sin_tab, const float* __restrict__ q_gain,
+                       const float* __restrict__ k_gain, int n_tokens, int nq, int nk, int nkv_cache, int hd, int rot, int page_size,
+                       float eps, float q_off, float k_off, const float* __restrict__ bias, int vd) {
+    constexpr int EPL = Vec16<T>::N;
+    const unsigned heads = (unsigned)(nq + 2 * nk);
+    const unsigned row = (blockIdx.x * blockDim.x + threadIdx.x) / LPR;
+    const int at = (int)(threadIdx.x % LPR) * EPL;
+    pdl_launch_dependents();
+    pdl_wait();
+    const bool live = row < (unsigned)n_tokens * heads;
+    const int t = live ? (int)(row / heads) : 0;
+    const int h = live ? (int)(row - (unsigned)t * heads) : 0;
+    const bool is_q = h < nq, is_v = h >= nq + nk;
+    const int width = is_v ? vd : hd;
+    const bool on = live && at < width;
+    const size_t col0 = is_v ? (size_t)(nq + nk) * hd + (size_t)(h - nq - nk) * vd : (size_t)h * hd;
+    const int slot = slots ? slots[t] : -1;
+    const int pos = cos_tab ? positions[t] : 0;
+    float f[EPL];
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) f[i] = 0.f;
+    if (on) {
+        Vec16<T> x;
+        x.raw = *reinterpret_cast<const decltype(x.raw)*>(qkv + (size_t)t * row_stride + col0 + at);
+        x.unpack(f);
+        if (bias) {
+#pragma unroll
+            for (int i = 0; i < EPL; i += 4) {
+                const float4 b = *reinterpret_cast<const float4*>(bias + col0 + at + i);
+                f[i] += b.x; f[i + 1] += b.y; f[i + 2] += b.z; f[i + 3] += b.w;
+            }
+        }
+    }
+    const float* gain = is_v ? nullptr : is_q ? q_gain : k_gain;
+    const float goff = is_q ? q_off : k_off;
+    float ss = 0.f;                           // every lane takes part in the shuffles
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) ss = fmaf(f[i], f[i], ss);
+#pragma unroll
+    for (int o = LPR / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!on) return;
+    if (gain) {
+        const float rinv = 1.0f / sqrtf(ss / (float)hd + eps);
+#pragma unroll
+        for (int i = 0; i < EPL; i += 4) {
+            const float4 g = *reinterpret_cast<const float4*>(gain + at + i);
+            f[i] *= rinv * (g.x + goff); f[i + 1] *= rinv * (g.y + goff); f[i + 2] *= rinv * (g.z + goff); f[i + 3] *= rinv * (g.w + goff);
+        }
+    }
+    if (!is_v && cos_tab && at < rot) {
+        const float* c = cos_tab + (size_t)pos * (rot / 2) + at / 2;
+        const float* s = sin_tab + (size_t)pos * (rot / 2) + at / 2;
+#pragma unroll
+        for (int i = 0; i < EPL; i += 4) {
+            const float2 cv = *reinterpret_cast<const float2*>(c + i / 2), sv = *reinterpret_cast<const float2*>(s + i / 2);
+            const float a0 = f[i], b0 = f[i + 1], a1 = f[i + 2], b1 = f[i + 3];
+            f[i] = a0 * cv.x - b0 * sv.x;
+            f[i + 1] = b0 * cv.x + a0 * sv.x;
+            f[i + 2] = a1 * cv.y - b1 * sv.y;
+            f[i + 3] = b1 * cv.y + a1 * sv.y;
+        }
+    }
+    T* dst = nullptr;
+    if (is_q) {
+        dst = q_out + (size_t)t * q_stride + (size_t)h * hd;
+    } else if (slot >= 0) {
+        T* cache = is_v ? vcache : kcache;
+        const int kvh = is_v ? h - nq - nk : h - nq, page = slot / page_size;
+        if (cache) dst = cache + (((size_t)page * nkv_cache + kvh) * page_size + (slot - page * page_size)) * width;
+    }
+    if (!dst) return;
+    Vec16<T> y;
+    y.pack(f);
+    *reinterpret_cast<decltype(y.raw)*>(dst + at) = y.raw;
+}
+
+template <typename T>
+static bool launch_pairs(const void* qkv, long long row_stride, void* q_out, long long q_stride, void* kcache, void* vcache, const int* positions,
+                         const int* slots, const float* cos_tab, const float* sin_tab, const float* q_gain, const float* k_gain, int n_tokens,
+                         int nq, int nk, int nkv_cache, int hd, int rot, int page_size, float eps, float q_off, float k_off,
+                         const float* bias, int vd, cudaStream_t s, cudaError_t* e) {
+    constexpr int EPL = Vec16<T>::N;
+    const int most = (nk > 0 && vd > hd ? vd : hd) / EPL;
+    if (hd % EPL || vd % EPL || rot % EPL || row_stride % EPL || q_stride % EPL || most > 32 || !host_aligned16(qkv) || !host_aligned16(q_out) ||
+        !host_aligned16(kcache) || !host_aligned16(vcache) || !host_aligned16(cos_tab) || !host_aligned16(sin_tab) || !host_aligned16(bias) ||
+        !host_aligned16(q_gain) || !host_aligned16(k_gain) || (long long)n_tokens * (nq + 2 * nk) * 32 > 2000000000LL)
+        return false;
+    const long long rows = (long long)n_tokens * (nq + 2 * nk);
+#define ATTN_PREP_PAIRS(LPR)                                                                                                            \
+    *e = llmk_launch(attn_prep_pairs_kernel<T, LPR>, dim3((unsigned)((rows * LPR + 255) / 256)), dim3(256), 0, s, true, (const T*)qkv,  \
+                     row_stride, (T*)q_out, q_stride, (T*)kcache, (T*)vcache, positions, slots, cos_tab, sin_tab, q_gain, k_gain,       \
+                     n_tokens, nq, nk, nkv_cache, hd, rot, page_size, eps, q_off, k_off, bias, vd)
+    if (most <= 4) ATTN_PREP_PAIRS(4);
+    else if (most <= 8) ATTN_PREP_PAIRS(8);
+    else if (most <= 16) ATTN_PREP_PAIRS(16);
+    else ATTN_PREP_PAIRS(32);
+#undef ATTN_PREP_PAIRS
+    return true;
+}
+
 // nk = number of k (and v) heads present in the packed rows: num_kv_heads for a layer that
 // writes its cache, 0 for a layer that only reads another layer's cache.
 LLMK_EXPORT int llmk_attn_prep(const void* qkv, long long row_stride, int splits, long long split_stride, void* q_out,
@@ -532,6 +639,19 @@ LLMK_EXPORT int llmk_attn_prep(const void* qkv, long long row_stride, int splits
         else if (dtype == LLMK_BF16)
             taken = launch_vec<bf16>(qkv, row_stride, q_out, q_stride, kcache, vcache, positions, slots, cos_tab, sin_tab,
                                      q_gain, k_gain, n_tokens, nq, nk, nkv_cache, hd, rot, page_size, eps, q_off, k_off, s, &e);
+        if (taken) {
+            LLMK_CHECK_LAUNCH_RC("attn_prep", e);
+            return LLMK_OK;
+        }
+    }
+    if (splits == 0 && interleaved && !norm_after) {
+        bool taken = false;
+        if (dtype == LLMK_F32)
+            taken = launch_pairs<float>(qkv, row_stride, q_out, q_stride, kcache, vcache, positions, slots, cos_tab, sin_tab, q_gain, k_gain,
+                                        n_tokens, nq, nk, nkv_cache, hd, rot, page_size, eps, q_off, k_off, bias, vd, s, &e);
+        else if (dtype == LLMK_BF16)
+            taken = launch_pairs<bf16>(qkv, row_stride, q_out, q_stride, kcache, vcache, positions, slots, cos_tab, sin_tab, q_gain, k_gain,
+                                       n_tokens, nq, nk, nkv_cache, hd, rot, page_size, eps, q_off, k_off, bias, vd, s, &e);
         if (taken) {
             LLMK_CHECK_LAUNCH_RC("attn_prep", e);
             return LLMK_OK;

@@ -145,6 +145,165 @@ __global__ void __launch_bounds__(256) head_delta_prep_kernel(PrepParams p) {
     }
 }
 
+// The same where rows of q, k and v are whole vectors of four channels and a key head has at most 128 * NB of them: a warp takes one key
+// head (q and k) or one value head over WTB token rows, four channels a lane (NB times), with the last KT - 1 inputs and the taps in
+// registers; a convolution of fewer taps has zeros in front.
+constexpr int WTB = 8;
+
+template <typename T>
+__device__ __forceinline__ float4 load_four(const T* p) {
+    if constexpr (sizeof(T) == 4) return *reinterpret_cast<const float4*>(p);
+    else {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        return make_float4(a.x, a.y, b.x, b.y);
+    }
+}
+
+template <int KT>
+struct ConvLane {                 // four channels of one lane
+    float tp[KT][4], w[KT - 1][4];
+    __device__ __forceinline__ void taps(const float* src, int K) {
+#pragma unroll
+        for (int i = 0; i < KT; ++i)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) tp[i][c] = i >= KT - K ? src[(size_t)c * K + i - (KT - K)] : 0.f;
+    }
+    template <typename T>
+    __device__ __forceinline__ void history(const T* x, long long x_ld, int q_beg, int j, const float* st, int C, int K, size_t gc) {
+#pragma unroll
+        for (int i = 0; i < KT - 1; ++i) {
+            const int r = j - (KT - 1) + i;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (r >= 0) v = load_four(x + (size_t)(q_beg + r) * x_ld + gc);
+            else if (st && r >= -(K - 1)) {
+                const float* p = st + (size_t)(K - 1 + r) * C + gc;
+                v = make_float4(p[0], p[1], p[2], p[3]);
+            }
+            w[i][0] = v.x; w[i][1] = v.y; w[i][2] = v.z; w[i][3] = v.w;
+        }
+    }
+    __device__ __forceinline__ void next(const float4& v, float (&out)[4]) {
+        const float in[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            float acc = 0.f;
+#pragma unroll
+            for (int i = 0; i < KT - 1; ++i) acc = fmaf(tp[i][c], w[i][c], acc);
+            acc = fmaf(tp[KT - 1][c], in[c], acc);
+            out[c] = acc / (1.0f + expf(-acc));
+#pragma unroll
+            for (int i = 0; i < KT - 1; ++i) w[i][c] = i + 1 < KT - 1 ? w[i + 1][c] : in[c];
+        }
+    }
+};
+
+template <typename T, int KT, int NB>
+__global__ void __launch_bounds__(128) head_delta_prep_warp_kernel(PrepParams p, int tiles) {
+    const int lane = threadIdx.x & 31;
+    const int items = p.G + p.H + 1;
+    const int id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int item = id % items, t0 = id / items * WTB;
+    if (id >= tiles * items) return;
+    const int D = p.D, E = p.E, K = p.K, GD = p.G * D, C = 2 * GD + p.H * E, width = 2 * p.H + p.G;
+    const T* x = static_cast<const T*>(p.x);
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t1 = min(t0 + WTB, min(p.n_tokens, p.cu_q[p.n_seqs]));
+    if (item == p.G + p.H) {                  // beta and the decays
+        for (int idx = lane; idx < (t1 - t0) * p.H; idx += 32) {
+            const int t = t0 + idx / p.H, h = idx % p.H;
+            const T* row = x + (size_t)t * p.x_ld;
+            float* out = p.gates + (size_t)t * width;
+            out[h] = sigmoidf_(to_float(row[p.beta_off + h]));
+            out[p.H + h] = -expf(p.a_log[h]) * softplusf_(to_float(row[p.decay_off + h]) + p.dt_bias[h]);
+        }
+        return;
+    }
+    int held = -1, s = t0 < t1 ? seq_of_row(p.cu_q, p.n_seqs, t0) : 0;
+    if (item < p.G) {
+        ConvLane<KT> cq[NB], ck[NB];
+#pragma unroll
+        for (int b = 0; b < NB; ++b) {
+            const int d = b * 128 + lane * 4;
+            if (d < D) {
+                cq[b].taps(p.taps + (size_t)(item * D + d) * K, K);
+                ck[b].taps(p.taps + (size_t)(GD + item * D + d) * K, K);
+            }
+        }
+        for (int t = t0; t < t1; ++t) {
+            while (t >= p.cu_q[s + 1]) ++s;
+            if (s != held) {
+                const int slot = p.state_slots[s], q_beg = p.cu_q[s];
+                const float* st = slot >= 0 && K > 1 ? p.state + (size_t)slot * p.state_ld : nullptr;
+#pragma unroll
+                for (int b = 0; b < NB; ++b) {
+                    const int d = b * 128 + lane * 4;
+                    if (d < D) {
+                        cq[b].history(x, p.x_ld, q_beg, t - q_beg, st, C, K, (size_t)item * D + d);
+                        ck[b].history(x, p.x_ld, q_beg, t - q_beg, st, C, K, (size_t)GD + item * D + d);
+                    }
+                }
+                held = s;
+            }
+            float q[NB][4], k[NB][4];
+            float sq = 0.f, sk = 0.f, qk = 0.f;
+#pragma unroll
+            for (int b = 0; b < NB; ++b) {
+                const int d = b * 128 + lane * 4;
+                if (d < D) {
+                    const T* row = x + (size_t)t * p.x_ld + (size_t)item * D + d;
+                    cq[b].next(load_four(row), q[b]);
+                    ck[b].next(load_four(row + GD), k[b]);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) {
+                        sq = fmaf(q[b][c], q[b][c], sq);
+                        sk = fmaf(k[b][c], k[b][c], sk);
+                        qk = fmaf(q[b][c], k[b][c], qk);
+                    }
+                }
+            }
+            sq = warp_sum(sq);
+            sk = warp_sum(sk);
+            qk = warp_sum(qk);
+            const float fq = p.q_scale / sqrtf(sq + p.unit_eps), fk = 1.0f / sqrtf(sk + p.unit_eps);
+            float* out = p.qkv + (size_t)t * C + (size_t)item * D;
+#pragma unroll
+            for (int b = 0; b < NB; ++b) {
+                const int d = b * 128 + lane * 4;
+                if (d < D) {
+                    *reinterpret_cast<float4*>(out + d) = make_float4(q[b][0] * fq, q[b][1] * fq, q[b][2] * fq, q[b][3] * fq);
+                    *reinterpret_cast<float4*>(out + GD + d) = make_float4(k[b][0] * fk, k[b][1] * fk, k[b][2] * fk, k[b][3] * fk);
+                }
+            }
+            if (lane == 0) p.gates[(size_t)t * width + 2 * p.H + item] = fq * fk * qk;
+        }
+        return;
+    }
+    const size_t v0 = (size_t)2 * GD + (size_t)(item - p.G) * E;
+    const int s_first = s;
+    for (int e0 = 0; e0 < E; e0 += 128) {      // a value head's columns need not be held together
+        const int e = e0 + lane * 4;
+        if (e >= E) continue;
+        ConvLane<KT> cv;
+        cv.taps(p.taps + (v0 + e) * K, K);
+        held = -1;
+        s = s_first;
+        for (int t = t0; t < t1; ++t) {
+            while (t >= p.cu_q[s + 1]) ++s;
+            if (s != held) {
+                const int slot = p.state_slots[s], q_beg = p.cu_q[s];
+                cv.history(x, p.x_ld, q_beg, t - q_beg, slot >= 0 && K > 1 ? p.state + (size_t)slot * p.state_ld : nullptr, C, K, v0 + e);
+                held = s;
+            }
+            float v[4];
+            cv.next(load_four(x + (size_t)t * p.x_ld + v0 + e), v);
+            *reinterpret_cast<float4*>(p.qkv + (size_t)t * C + v0 + e) = make_float4(v[0], v[1], v[2], v[3]);
+        }
+    }
+}
+
 // The last K - 1 inputs of every sequence into its state, behind the preparation that read the old ones.
 template <typename T>
 __global__ void conv_tail_kernel(PrepParams p) {
@@ -183,7 +342,14 @@ static cudaError_t launch_prep(const PrepParams& p, cudaStream_t s) {
         cudaError_t e = cudaFuncSetAttribute(head_delta_prep_kernel<T, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
-    cudaError_t e = llmk_launch(head_delta_prep_kernel<T, TB>, dim3(ceil_div(p.n_tokens, TB)), dim3(256), smem, s, true, p);
+    cudaError_t e;
+    const bool vec = p.D % 4 == 0 && p.E % 4 == 0 && p.x_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(p.x) & (4 * sizeof(T) - 1)) == 0 && host_aligned16(p.qkv);
+    const int tiles = ceil_div(p.n_tokens, WTB);
+    const dim3 wgrid(ceil_div(tiles * (p.G + p.H + 1), 4));
+    if (vec && p.D <= 128 && p.K <= 4) e = llmk_launch(head_delta_prep_warp_kernel<T, 4, 1>, wgrid, dim3(128), 0, s, true, p, tiles);
+    else if (vec && p.D <= 128) e = llmk_launch(head_delta_prep_warp_kernel<T, 8, 1>, wgrid, dim3(128), 0, s, true, p, tiles);
+    else if (vec && p.D <= 256 && p.K <= 4) e = llmk_launch(head_delta_prep_warp_kernel<T, 4, 2>, wgrid, dim3(128), 0, s, true, p, tiles);
+    else e = llmk_launch(head_delta_prep_kernel<T, TB>, dim3(ceil_div(p.n_tokens, TB)), dim3(256), smem, s, true, p);
     if (e == cudaSuccess && p.K > 1)
         e = llmk_launch(conv_tail_kernel<T>, dim3(ceil_div(C, 128), p.n_seqs), dim3(128), 0, s, true, p);
     return e;
@@ -224,7 +390,7 @@ struct ChunkParams {
     const int* cu_q;
     const int* state_slots;
     float* qs;               // [places][G][CHUNK][DP]
-    float* ks;               // [places][G][CHUNK][DP]
+    float* ks;               // [places][G][CHUNK * DP], in the order the walk's threads read it: see `key_place`
     float* w;                // [places][H][CHUNK][DP]
     float* uv;               // [places][H][CHUNK][EP]
     float* p;                // [places][H][CHUNK][CHUNK]
@@ -232,16 +398,51 @@ struct ChunkParams {
     int n_seqs, n_tokens, H, G, D, E, EP, vec_ok;
 };
 
+// Where four key channels d .. d + 3 of token i lie in a chunk's keys: the walk's thread (d / 4) * TS + i % TS reads its i / TS-th
+// vector there, so a warp reads 512 bytes side by side.
+template <int DP>
+__device__ __forceinline__ int key_place(int i, int d) {
+    constexpr int TS = CTHREADS / (DP / 4);
+    return (((i / TS) * (DP / 4) + d / 4) * TS + i % TS) * 4;
+}
+
+__device__ __forceinline__ unsigned long long pack2(float a, float b) {
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 unpack2(unsigned long long v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+// two float32 multiply-adds at a time
+__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+
+constexpr int CHUNK_VALUES = 128;          // columns of v that a block holds in shared memory
+
+__device__ __forceinline__ void cp_async16(float* smem_dst, const float* src) {
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(smem_dst);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
 // Everything of one (chunk, head) that does not need the state.
 template <int DP>
 __global__ void __launch_bounds__(CTHREADS, 2) chunk_prep_kernel(ChunkParams p) {
-    constexpr int LD = DP + 4, MLD = CHUNK + 4;
+    constexpr int MLD = CHUNK, TILES = CHUNK / 4, LOWER = TILES * (TILES + 1) / 2;
     extern __shared__ __align__(16) float csm[];
-    float* Ks = csm;                        // [CHUNK][LD]
-    float* Qs = Ks + CHUNK * LD;            // [CHUNK][LD]
-    float* M = Qs + CHUNK * LD;             // [CHUNK][MLD]
+    float* Ks = csm;                        // [CHUNK][DP], vectors of four swizzled by the row's tile
+    float* Qs = Ks + CHUNK * DP;            // the same
+    float* M = Qs + CHUNK * DP;             // [CHUNK][MLD]: minus the lower triangle, zeros from the diagonal on
     float* bet = M + CHUNK * MLD;           // [CHUNK]
     float* L = bet + CHUNK;                 // [CHUNK]
+    float* bel = L + CHUNK;                 // [CHUNK] beta e^L
+    float* Vs = bel + CHUNK;                // [CHUNK][VC] the first columns of v
     const int place = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int kvh = h / (p.H / p.G);
     const bool writes_qk = h % (p.H / p.G) == 0;
@@ -258,29 +459,40 @@ __global__ void __launch_bounds__(CTHREADS, 2) chunk_prep_kernel(ChunkParams p) 
     if (n <= 0) return;
     const int t0 = q_beg + first;
     const int D = p.D, E = p.E, GD = p.G * D, C = 2 * GD + p.H * E;
-#pragma unroll 4
+    auto at = [](int i, int d) { return i * DP + ((((d >> 2) ^ (i >> 2)) & (DP / 4 < 8 ? DP / 4 - 1 : 7)) | ((d >> 2) & ~7)) * 4 + (d & 3); };
+    float* kout = p.ks + (size_t)(place * p.G + kvh) * CHUNK * DP;
+    float* qout = p.qs + (size_t)(place * p.G + kvh) * CHUNK * DP;
+    const int VC = min(p.EP, CHUNK_VALUES);
+    const float* vsrc = p.qkv + (size_t)t0 * C + 2 * GD + (size_t)h * E;
     for (int idx = tid; idx < CHUNK * DP / 4; idx += CTHREADS) {
         const int i = idx / (DP / 4), d = idx % (DP / 4) * 4;
+        const float* row = p.qkv + (size_t)(t0 + i) * C + (size_t)kvh * D + d;
         float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv;
         if (i < n && d < D) {
-            const float* row = p.qkv + (size_t)(t0 + i) * C + (size_t)kvh * D + d;
             if (p.vec_ok) {
-                qv = *reinterpret_cast<const float4*>(row);
-                kv = *reinterpret_cast<const float4*>(row + GD);
-            } else {
-                qv.x = row[0]; kv.x = row[GD];
-                if (d + 1 < D) { qv.y = row[1]; kv.y = row[GD + 1]; }
-                if (d + 2 < D) { qv.z = row[2]; kv.z = row[GD + 2]; }
-                if (d + 3 < D) { qv.w = row[3]; kv.w = row[GD + 3]; }
+                cp_async16(Ks + at(i, d), row + GD);
+                cp_async16(Qs + at(i, d), row);
+                continue;
             }
+            qv.x = row[0]; kv.x = row[GD];
+            if (d + 1 < D) { qv.y = row[1]; kv.y = row[GD + 1]; }
+            if (d + 2 < D) { qv.z = row[2]; kv.z = row[GD + 2]; }
+            if (d + 3 < D) { qv.w = row[3]; kv.w = row[GD + 3]; }
         }
-        *reinterpret_cast<float4*>(Ks + i * LD + d) = kv;
-        *reinterpret_cast<float4*>(Qs + i * LD + d) = qv;
-        if (writes_qk) {
-            const size_t at = ((size_t)(place * p.G + kvh) * CHUNK + i) * DP + d;
-            *reinterpret_cast<float4*>(p.ks + at) = kv;
-            *reinterpret_cast<float4*>(p.qs + at) = qv;
-        }
+        *reinterpret_cast<float4*>(Ks + at(i, d)) = kv;
+        *reinterpret_cast<float4*>(Qs + at(i, d)) = qv;
+    }
+    for (int idx = tid; idx < CHUNK * VC / 4; idx += CTHREADS) {
+        const int i = idx / (VC / 4), e = idx % (VC / 4) * 4;
+        if (p.vec_ok && i < n && e < E) cp_async16(Vs + i * VC + e, vsrc + (size_t)i * C + e);
+        else
+            for (int u = 0; u < 4; ++u) Vs[i * VC + e + u] = (i < n && e + u < E) ? vsrc[(size_t)i * C + e + u] : 0.f;
+    }
+    for (int idx = tid; idx < CHUNK * MLD; idx += CTHREADS) M[idx] = 0.f;
+    float* P = p.p + (size_t)(place * p.H + h) * CHUNK * CHUNK;
+    for (int idx = tid; idx < CHUNK * TILES; idx += CTHREADS) {      // the read-out's tiles above the diagonal
+        const int i = idx / TILES, tj = idx % TILES;
+        if (tj > i / 4) *reinterpret_cast<float4*>(P + i * CHUNK + tj * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
     }
     if (tid < 32) {           // running sums of log g, two rows a lane
         const float* g0 = p.gates + (size_t)t0 * (2 * p.H + p.G);
@@ -302,80 +514,105 @@ __global__ void __launch_bounds__(CTHREADS, 2) chunk_prep_kernel(ChunkParams p) 
         dec[b] = expf(sum);
         dec[CHUNK + a] = expf(all - (sum - lb));
         dec[CHUNK + b] = expf(all - sum);
+        bel[a] = bet[a] * expf(sum - lb);
+        bel[b] = bet[b] * expf(sum);
     }
+    cp_async_wait_all();
     __syncthreads();
-    {
-        // k_i . k_j and q_i . k_j, a thread a tile of 4 x 4; tiles above the diagonal are zero
-        const int ti = tid >> 4, tj = tid & 15;
-        float kk[4][4], qk[4][4];
+    if (writes_qk) {
+        for (int idx = tid; idx < CHUNK * DP / 4; idx += CTHREADS) {
+            const int i = idx / (DP / 4), d = idx % (DP / 4) * 4;
+            *reinterpret_cast<float4*>(kout + key_place<DP>(i, d)) = *reinterpret_cast<const float4*>(Ks + at(i, d));
+            *reinterpret_cast<float4*>(qout + i * DP + d) = *reinterpret_cast<const float4*>(Qs + at(i, d));
+        }
+    }
+    // k_i . k_j, then q_i . k_j: the tiles of 4 x 4 on and below the diagonal, a thread a tile
+    for (int idx = tid; idx < 2 * LOWER; idx += CTHREADS) {
+        const bool read = idx >= LOWER;
+        const int tile = read ? idx - LOWER : idx;
+        int ti = (int)((sqrtf(8.f * tile + 1.f) - 1.f) * 0.5f);
+        ti += (ti + 1) * (ti + 2) / 2 <= tile ? 1 : 0;
+        ti -= ti * (ti + 1) / 2 > tile ? 1 : 0;
+        const int tj = tile - ti * (ti + 1) / 2;
+        const float* A = read ? Qs : Ks;
+        unsigned long long acc[4][4];
 #pragma unroll
         for (int a = 0; a < 4; ++a)
 #pragma unroll
-            for (int b = 0; b < 4; ++b) kk[a][b] = qk[a][b] = 0.f;
-        if (tj <= ti) {
+            for (int b = 0; b < 4; ++b) acc[a][b] = 0ull;
 #pragma unroll 2
-            for (int d = 0; d < DP; d += 4) {
-                float4 ka[4], qa[4], kb[4];
+        for (int d = 0; d < DP; d += 4) {
+            ulonglong2 av[4], bv[4];
 #pragma unroll
-                for (int a = 0; a < 4; ++a) {
-                    ka[a] = *reinterpret_cast<const float4*>(Ks + (ti * 4 + a) * LD + d);
-                    qa[a] = *reinterpret_cast<const float4*>(Qs + (ti * 4 + a) * LD + d);
-                    kb[a] = *reinterpret_cast<const float4*>(Ks + (tj * 4 + a) * LD + d);
-                }
-#pragma unroll
-                for (int a = 0; a < 4; ++a)
-#pragma unroll
-                    for (int b = 0; b < 4; ++b) {
-                        kk[a][b] = fmaf(ka[a].x, kb[b].x, kk[a][b]); qk[a][b] = fmaf(qa[a].x, kb[b].x, qk[a][b]);
-                        kk[a][b] = fmaf(ka[a].y, kb[b].y, kk[a][b]); qk[a][b] = fmaf(qa[a].y, kb[b].y, qk[a][b]);
-                        kk[a][b] = fmaf(ka[a].z, kb[b].z, kk[a][b]); qk[a][b] = fmaf(qa[a].z, kb[b].z, qk[a][b]);
-                        kk[a][b] = fmaf(ka[a].w, kb[b].w, kk[a][b]); qk[a][b] = fmaf(qa[a].w, kb[b].w, qk[a][b]);
-                    }
+            for (int a = 0; a < 4; ++a) {
+                av[a] = *reinterpret_cast<const ulonglong2*>(A + at(ti * 4 + a, d));
+                bv[a] = *reinterpret_cast<const ulonglong2*>(Ks + at(tj * 4 + a, d));
             }
+#pragma unroll
+            for (int a = 0; a < 4; ++a)
+#pragma unroll
+                for (int b = 0; b < 4; ++b) acc[a][b] = fma2(av[a].y, bv[b].y, fma2(av[a].x, bv[b].x, acc[a][b]));
         }
-        float* P = p.p + (size_t)(place * p.H + h) * CHUNK * CHUNK;
 #pragma unroll
         for (int a = 0; a < 4; ++a) {
             const int i = ti * 4 + a;
-            float pr[4];
+            float r[4];
 #pragma unroll
             for (int b = 0; b < 4; ++b) {
                 const int j = tj * 4 + b;
-                const float e = j <= i ? expf(L[i] - L[j]) : 0.f;
-                pr[b] = e * qk[a][b];
-                M[i * MLD + j] = j < i ? bet[i] * e * kk[a][b] : 0.f;
+                const float2 two = unpack2(acc[a][b]);
+                r[b] = (read ? j <= i : j < i) ? (two.x + two.y) * expf(L[i] - L[j]) : 0.f;
+                if (!read) r[b] *= -bet[i];
             }
-            *reinterpret_cast<float4*>(P + i * CHUNK + tj * 4) = make_float4(pr[0], pr[1], pr[2], pr[3]);
+            *reinterpret_cast<float4*>((read ? P + i * CHUNK : M + i * MLD) + tj * 4) = make_float4(r[0], r[1], r[2], r[3]);
         }
     }
     __syncthreads();
-    // (I + M) x = b, a column a thread: the columns of diag(beta e^L) K, then those of diag(beta) V
+    // (I + M) x = b, a column a thread, two rows of it in a register pair: the columns of diag(beta e^L) K, then those of diag(beta) V
     float* W = p.w + (size_t)(place * p.H + h) * CHUNK * DP;
     float* U = p.uv + (size_t)(place * p.H + h) * CHUNK * p.EP;
     for (int c = tid; c < DP + p.EP; c += CTHREADS) {
         const bool key = c < DP;
         const int e = c - DP;
-        const float* v = p.qkv + (size_t)t0 * C + 2 * GD + (size_t)h * E + e;
-        float x[CHUNK];
+        float* dst = key ? W + c : U + e;
+        const int ld = key ? DP : p.EP;
+        unsigned long long x[CHUNK / 2];
 #pragma unroll
-        for (int i = 0; i < CHUNK; ++i) {
-            if (key) x[i] = bet[i] * expf(L[i]) * Ks[i * LD + c];
-            else x[i] = (i < n && e < E) ? bet[i] * v[(size_t)i * C] : 0.f;
+        for (int i = 0; i < CHUNK; i += 2) {
+            float b0, b1;
+            if (key) {
+                b0 = bel[i] * Ks[at(i, c)];
+                b1 = bel[i + 1] * Ks[at(i + 1, c)];
+            } else if (e < VC) {
+                b0 = bet[i] * Vs[i * VC + e];
+                b1 = bet[i + 1] * Vs[(i + 1) * VC + e];
+            } else {
+                b0 = (i < n && e < E) ? bet[i] * vsrc[(size_t)i * C + e] : 0.f;
+                b1 = (i + 1 < n && e < E) ? bet[i + 1] * vsrc[(size_t)(i + 1) * C + e] : 0.f;
+            }
+            x[i / 2] = pack2(b0, b1);
         }
 #pragma unroll
-        for (int i = 0; i < CHUNK; ++i) {
-            float part[4] = {x[i], 0.f, 0.f, 0.f};
+        for (int i = 0; i < CHUNK; i += 2) {
+            // rows i and i + 1; what lies right of the diagonal in M is zero, so whole groups of four are added
+            unsigned long long p0 = 0ull, p1 = 0ull, r0 = 0ull, r1 = 0ull;
 #pragma unroll
             for (int j = 0; j < i; j += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(M + i * MLD + j);
-                part[0] = fmaf(-m.x, x[j], part[0]);
-                if (j + 1 < i) part[1] = fmaf(-m.y, x[j + 1], part[1]);
-                if (j + 2 < i) part[2] = fmaf(-m.z, x[j + 2], part[2]);
-                if (j + 3 < i) part[3] = fmaf(-m.w, x[j + 3], part[3]);
+                const ulonglong2 m0 = *reinterpret_cast<const ulonglong2*>(M + i * MLD + j);
+                const ulonglong2 m1 = *reinterpret_cast<const ulonglong2*>(M + (i + 1) * MLD + j);
+                p0 = fma2(m0.x, x[j / 2], p0);
+                r0 = fma2(m1.x, x[j / 2], r0);
+                if (j + 2 < i) {
+                    p1 = fma2(m0.y, x[j / 2 + 1], p1);
+                    r1 = fma2(m1.y, x[j / 2 + 1], r1);
+                }
             }
-            x[i] = (part[0] + part[1]) + (part[2] + part[3]);
-            if (key) W[i * DP + c] = x[i];
-            else U[i * p.EP + e] = x[i];
+            const float2 b = unpack2(x[i / 2]), a0 = unpack2(p0), a1 = unpack2(p1), c0 = unpack2(r0), c1 = unpack2(r1);
+            const float x0 = b.x + ((a0.x + a1.x) + (a0.y + a1.y));
+            const float x1 = fmaf(M[(i + 1) * MLD + i], x0, b.y + ((c0.x + c1.x) + (c0.y + c1.y)));
+            x[i / 2] = pack2(x0, x1);
+            dst[(size_t)i * ld] = x0;
+            dst[(size_t)(i + 1) * ld] = x1;
         }
     }
 }
@@ -443,9 +680,9 @@ __global__ void __launch_bounds__(CTHREADS) chunk_scan_kernel(ChunkParams p) {
             for (int i = 0; i < KR; ++i) a4[r][i] = *reinterpret_cast<const float4*>(src + r * DP + i * 32 + ks * 4);
     };
     auto load_keys = [&](int c) {
-        const float* src = p.ks + ((size_t)(place0 + c) * p.G + kvh) * CHUNK * DP + d0;
+        const float* src = p.ks + ((size_t)(place0 + c) * p.G + kvh) * CHUNK * DP + tid * 4;
 #pragma unroll
-        for (int j = 0; j < TR; ++j) k4[j] = *reinterpret_cast<const float4*>(src + (j * TS + ts) * DP);
+        for (int j = 0; j < TR; ++j) k4[j] = *reinterpret_cast<const float4*>(src + j * CTHREADS * 4);
     };
     load_rows(0);
     load_keys(0);
@@ -601,10 +838,11 @@ LLMK_EXPORT long long llmk_head_delta_chunk_floats(int n_tokens, int n_seqs, int
 
 template <int DP>
 static cudaError_t launch_chunks(const ChunkParams& p, int places, cudaStream_t s) {
-    const size_t smem = ((size_t)2 * CHUNK * (DP + 4) + CHUNK * (CHUNK + 4) + 2 * CHUNK) * sizeof(float);
+    const size_t smem = ((size_t)2 * CHUNK * DP + CHUNK * CHUNK + 3 * CHUNK + (size_t)CHUNK * std::min(p.EP, CHUNK_VALUES)) * sizeof(float);
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(chunk_prep_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(chunk_prep_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                             (2 * CHUNK * DP + CHUNK * CHUNK + 3 * CHUNK + CHUNK * CHUNK_VALUES) * (int)sizeof(float));
         if (e != cudaSuccess) return e;
         configured = true;
     }
@@ -636,7 +874,7 @@ LLMK_EXPORT int llmk_head_delta_chunks(float* out, const float* qkv, const float
     p.p = p.uv + rows * H * ep;
     p.dec = p.p + rows * H * CHUNK;
     p.n_seqs = n_seqs; p.n_tokens = n_tokens; p.H = H; p.G = G; p.D = D; p.E = E; p.EP = (int)ep;
-    p.vec_ok = (D % 4 == 0 && (2 * G * D + H * E) % 4 == 0 && host_aligned16(qkv)) ? 1 : 0;
+    p.vec_ok = (D % 4 == 0 && E % 4 == 0 && (2 * G * D + H * E) % 4 == 0 && host_aligned16(qkv)) ? 1 : 0;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e = dp == 32 ? launch_chunks<32>(p, places, s) : dp == 64 ? launch_chunks<64>(p, places, s) : launch_chunks<128>(p, places, s);
     LLMK_CHECK_LAUNCH_RC("head_delta_chunks", e);
