@@ -35,6 +35,18 @@ __device__ __forceinline__ int seq_of_row(const int* __restrict__ cu_q, int n_se
 }
 
 __device__ __forceinline__ float sigmoidf_(float x) { return 1.0f / (1.0f + expf(-x)); }
+// The activation behind the short convolution, and the inverse lengths of q and k: with rows of bfloat16 through the special-function unit (a few units in the last place of
+// a float32, far below the rounding of what went in).
+template <typename T>
+__device__ __forceinline__ float inverse_root(float x) {
+    if constexpr (sizeof(T) == 2) return rsqrtf(x);
+    else return 1.0f / sqrtf(x);
+}
+template <typename T>
+__device__ __forceinline__ float conv_silu(float x) {
+    if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-x));
+    else return x / (1.0f + expf(-x));
+}
 __device__ __forceinline__ float softplusf_(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
 struct PrepParams {
@@ -99,7 +111,7 @@ __global__ void __launch_bounds__(256) head_delta_prep_kernel(PrepParams p) {
                 if (i < K - 1) acc = fmaf(tp[i], w[i], acc);
                 else if (i == K - 1) acc = fmaf(tp[i], v, acc);
             }
-            rows[tt * C + c] = acc / (1.0f + expf(-acc));
+            rows[tt * C + c] = conv_silu<T>(acc);
 #pragma unroll
             for (int i = 0; i < MAX_TAPS - 1; ++i)
                 if (i < K - 1) w[i] = i + 1 < K - 1 ? w[i + 1] : v;
@@ -165,6 +177,14 @@ template <int KT>
 struct ConvLane {                 // four channels of one lane
     float tp[KT][4], w[KT - 1][4];
     __device__ __forceinline__ void taps(const float* src, int K) {
+        if (KT == 4 && K == 4 && aligned16(src)) {
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const float4 v = *reinterpret_cast<const float4*>(src + c * 4);
+                tp[0][c] = v.x; tp[1][c] = v.y; tp[KT - 2][c] = v.z; tp[KT - 1][c] = v.w;
+            }
+            return;
+        }
 #pragma unroll
         for (int i = 0; i < KT; ++i)
 #pragma unroll
@@ -184,6 +204,7 @@ struct ConvLane {                 // four channels of one lane
             w[i][0] = v.x; w[i][1] = v.y; w[i][2] = v.z; w[i][3] = v.w;
         }
     }
+    template <typename T>
     __device__ __forceinline__ void next(const float4& v, float (&out)[4]) {
         const float in[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
@@ -192,7 +213,7 @@ struct ConvLane {                 // four channels of one lane
 #pragma unroll
             for (int i = 0; i < KT - 1; ++i) acc = fmaf(tp[i][c], w[i][c], acc);
             acc = fmaf(tp[KT - 1][c], in[c], acc);
-            out[c] = acc / (1.0f + expf(-acc));
+            out[c] = conv_silu<T>(acc);
 #pragma unroll
             for (int i = 0; i < KT - 1; ++i) w[i][c] = i + 1 < KT - 1 ? w[i + 1][c] : in[c];
         }
@@ -200,7 +221,7 @@ struct ConvLane {                 // four channels of one lane
 };
 
 template <typename T, int KT, int NB>
-__global__ void __launch_bounds__(128) head_delta_prep_warp_kernel(PrepParams p, int tiles) {
+__global__ void __launch_bounds__(128, NB == 1 && KT == 4 ? 4 : 2) head_delta_prep_warp_kernel(PrepParams p, int tiles) {
     const int lane = threadIdx.x & 31;
     const int items = p.G + p.H + 1;
     const int id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -232,30 +253,26 @@ __global__ void __launch_bounds__(128) head_delta_prep_warp_kernel(PrepParams p,
                 ck[b].taps(p.taps + (size_t)(GD + item * D + d) * K, K);
             }
         }
-        for (int t = t0; t < t1; ++t) {
-            while (t >= p.cu_q[s + 1]) ++s;
-            if (s != held) {
-                const int slot = p.state_slots[s], q_beg = p.cu_q[s];
-                const float* st = slot >= 0 && K > 1 ? p.state + (size_t)slot * p.state_ld : nullptr;
-#pragma unroll
-                for (int b = 0; b < NB; ++b) {
-                    const int d = b * 128 + lane * 4;
-                    if (d < D) {
-                        cq[b].history(x, p.x_ld, q_beg, t - q_beg, st, C, K, (size_t)item * D + d);
-                        ck[b].history(x, p.x_ld, q_beg, t - q_beg, st, C, K, (size_t)GD + item * D + d);
-                    }
-                }
-                held = s;
-            }
-            float q[NB][4], k[NB][4];
-            float sq = 0.f, sk = 0.f, qk = 0.f;
+        auto begin = [&](int t) {             // the history of token t's sequence
+            const int slot = p.state_slots[s], q_beg = p.cu_q[s];
+            const float* st = slot >= 0 && K > 1 ? p.state + (size_t)slot * p.state_ld : nullptr;
 #pragma unroll
             for (int b = 0; b < NB; ++b) {
                 const int d = b * 128 + lane * 4;
                 if (d < D) {
-                    const T* row = x + (size_t)t * p.x_ld + (size_t)item * D + d;
-                    cq[b].next(load_four(row), q[b]);
-                    ck[b].next(load_four(row + GD), k[b]);
+                    cq[b].history(x, p.x_ld, q_beg, t - q_beg, st, C, K, (size_t)item * D + d);
+                    ck[b].history(x, p.x_ld, q_beg, t - q_beg, st, C, K, (size_t)GD + item * D + d);
+                }
+            }
+        };
+        auto token = [&](int t, const float4 (&xq)[NB], const float4 (&xk)[NB]) {
+            float q[NB][4], k[NB][4];
+            float sq = 0.f, sk = 0.f, qk = 0.f;
+#pragma unroll
+            for (int b = 0; b < NB; ++b) {
+                if (b * 128 + lane * 4 < D) {
+                    cq[b].template next<T>(xq[b], q[b]);
+                    ck[b].template next<T>(xk[b], k[b]);
 #pragma unroll
                     for (int c = 0; c < 4; ++c) {
                         sq = fmaf(q[b][c], q[b][c], sq);
@@ -267,7 +284,7 @@ __global__ void __launch_bounds__(128) head_delta_prep_warp_kernel(PrepParams p,
             sq = warp_sum(sq);
             sk = warp_sum(sk);
             qk = warp_sum(qk);
-            const float fq = p.q_scale / sqrtf(sq + p.unit_eps), fk = 1.0f / sqrtf(sk + p.unit_eps);
+            const float fq = p.q_scale * inverse_root<T>(sq + p.unit_eps), fk = inverse_root<T>(sk + p.unit_eps);
             float* out = p.qkv + (size_t)t * C + (size_t)item * D;
 #pragma unroll
             for (int b = 0; b < NB; ++b) {
@@ -278,6 +295,34 @@ __global__ void __launch_bounds__(128) head_delta_prep_warp_kernel(PrepParams p,
                 }
             }
             if (lane == 0) p.gates[(size_t)t * width + 2 * p.H + item] = fq * fk * qk;
+        };
+        auto load = [&](int t, float4 (&xq)[NB], float4 (&xk)[NB]) {
+#pragma unroll
+            for (int b = 0; b < NB; ++b) {
+                const int d = b * 128 + lane * 4;
+                if (d < D) {
+                    const T* row = x + (size_t)t * p.x_ld + (size_t)item * D + d;
+                    xq[b] = load_four(row);
+                    xk[b] = load_four(row + GD);
+                }
+            }
+        };
+        if (t0 + WTB <= p.cu_q[s + 1] && t1 == t0 + WTB) {     // one sequence: all rows asked for at once
+            float4 xq[WTB][NB], xk[WTB][NB];
+#pragma unroll
+            for (int i = 0; i < WTB; ++i) load(t0 + i, xq[i], xk[i]);
+            begin(t0);
+#pragma unroll
+            for (int i = 0; i < WTB; ++i) token(t0 + i, xq[i], xk[i]);
+            return;
+        }
+        for (int t = t0; t < t1; ++t) {
+            while (t >= p.cu_q[s + 1]) ++s;
+            if (s != held) begin(t);
+            held = s;
+            float4 xq[NB], xk[NB];
+            load(t, xq, xk);
+            token(t, xq, xk);
         }
         return;
     }
@@ -288,18 +333,31 @@ __global__ void __launch_bounds__(128) head_delta_prep_warp_kernel(PrepParams p,
         if (e >= E) continue;
         ConvLane<KT> cv;
         cv.taps(p.taps + (v0 + e) * K, K);
-        held = -1;
         s = s_first;
+        auto begin = [&](int t) {
+            const int slot = p.state_slots[s], q_beg = p.cu_q[s];
+            cv.history(x, p.x_ld, q_beg, t - q_beg, slot >= 0 && K > 1 ? p.state + (size_t)slot * p.state_ld : nullptr, C, K, v0 + e);
+        };
+        auto token = [&](int t, const float4& in) {
+            float v[4];
+            cv.template next<T>(in, v);
+            *reinterpret_cast<float4*>(p.qkv + (size_t)t * C + v0 + e) = make_float4(v[0], v[1], v[2], v[3]);
+        };
+        if (t0 + WTB <= p.cu_q[s + 1] && t1 == t0 + WTB) {
+            float4 in[WTB];
+#pragma unroll
+            for (int i = 0; i < WTB; ++i) in[i] = load_four(x + (size_t)(t0 + i) * p.x_ld + v0 + e);
+            begin(t0);
+#pragma unroll
+            for (int i = 0; i < WTB; ++i) token(t0 + i, in[i]);
+            continue;
+        }
+        held = -1;
         for (int t = t0; t < t1; ++t) {
             while (t >= p.cu_q[s + 1]) ++s;
-            if (s != held) {
-                const int slot = p.state_slots[s], q_beg = p.cu_q[s];
-                cv.history(x, p.x_ld, q_beg, t - q_beg, slot >= 0 && K > 1 ? p.state + (size_t)slot * p.state_ld : nullptr, C, K, v0 + e);
-                held = s;
-            }
-            float v[4];
-            cv.next(load_four(x + (size_t)t * p.x_ld + v0 + e), v);
-            *reinterpret_cast<float4*>(p.qkv + (size_t)t * C + v0 + e) = make_float4(v[0], v[1], v[2], v[3]);
+            if (s != held) begin(t);
+            held = s;
+            token(t, load_four(x + (size_t)t * p.x_ld + v0 + e));
         }
     }
 }
@@ -883,7 +941,7 @@ LLMK_EXPORT int llmk_head_delta_chunks(float* out, const float* qkv, const float
 
 // ------------------------------------------------------------------------------------------------ a few tokens
 // Block (head, sequence), the heads of one key head a cluster: they all read the key head's history of the convolution, and only then
-// does the first of them write it anew.  The state stays in registers: thread (e, slice) holds column e's rows slice, slice + NS, ...
+// does the first of them write it anew.  The state stays in registers: thread (e, slice) holds NR rows of column e.
 constexpr int STHREADS = 512;
 
 struct StepParams {
@@ -903,92 +961,106 @@ __global__ void __launch_bounds__(STHREADS) head_delta_step_kernel(StepParams sp
     const PrepParams& p = sp.prep;
     const int D = p.D, E = p.E, K = p.K, GD = p.G * D, C = 2 * GD + p.H * E, Ch = 2 * D + E, EP = sp.EP, NS = STHREADS / EP;
     float* hist = ssm;                        // [K - 1][Ch]
-    float* row = hist + (K - 1) * Ch;         // [Ch] after the convolution
-    float* red = row + Ch;                    // [2][STHREADS]
-    float* scal = red + 2 * STHREADS;         // fq, fk, dot, beta, 1 - g, the norm's warp sums [8]
+    float* tap = hist + (K - 1) * Ch;         // [K][Ch]
+    const int DR = NR * NS;                   // key channels with those that pad them (zeros)
+    float* row = tap + K * Ch;                // [DR] q, [DR] k, [EP] v after the convolution
+    row += (4 - ((2 * K - 1) * Ch & 3)) & 3;  // on 16 bytes
+    float* red = row + 2 * DR + EP;           // [2][STHREADS]
+    float* scal = red + 2 * STHREADS;         // |q|^2, |k|^2, q . k, beta, 1 - g, the norm's warp sums [8]
     const int h = blockIdx.x, s = blockIdx.y, R = p.H / p.G, kvh = h / R;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int e = tid & (EP - 1), sl = tid / EP;
     const T* x = static_cast<const T*>(p.x);
+    auto channel = [&](int c) { return c < D ? kvh * D + c : c < 2 * D ? GD + kvh * D + c - D : 2 * GD + h * E + c - 2 * D; };
+    auto place = [&](int c) { return c < D ? c : c < 2 * D ? DR + c - D : 2 * DR + c - 2 * D; };
     pdl_launch_dependents();
+    for (int i = tid; i < 2 * DR + EP; i += STHREADS) row[i] = 0.f;
+    // weights, before the wait for the kernel that makes x
+    for (int c = tid; c < Ch; c += STHREADS) {
+        const float* src = p.taps + (size_t)channel(c) * K;
+        for (int i = 0; i < K; ++i) tap[i * Ch + c] = src[i];
+    }
+    const float gain = e < E ? sp.norm_gain[e] : 0.f, rate = -expf(p.a_log[h]), dt = p.dt_bias[h];
     pdl_wait();
-    const int q_beg = p.cu_q[s], n = p.cu_q[s + 1] - q_beg;
+    const int q_beg = p.cu_q[s], n = p.cu_q[s + 1] - q_beg, slot = p.state_slots[s];
     if (n <= 0) return;                       // the whole cluster
-    const int slot = p.state_slots[s];
     float* st = slot >= 0 ? sp.state + (size_t)slot * p.state_ld + (size_t)h * D * E + e : nullptr;
     float* cst = slot >= 0 && K > 1 ? p.state + (size_t)slot * p.state_ld : nullptr;
-    float S[NR];
-#pragma unroll
-    for (int i = 0; i < NR; ++i) {
-        const int d = sl + i * NS;
-        S[i] = (st && d < D && e < E) ? st[(size_t)d * E] : 0.f;
+    for (int c = tid; c < Ch; c += STHREADS) {
+        const int gc = channel(c);
+        for (int i = 0; i < K - 1; ++i) hist[i * Ch + c] = cst ? cst[(size_t)i * C + gc] : 0.f;
     }
-    auto channel = [&](int c) { return c < D ? kvh * D + c : c < 2 * D ? GD + kvh * D + c - D : 2 * GD + h * E + c - 2 * D; };
-    for (int idx = tid; idx < (K - 1) * Ch; idx += STHREADS) hist[idx] = cst ? cst[(size_t)(idx / Ch) * C + channel(idx % Ch)] : 0.f;
-    if (R > 1) cluster_sync_all();
+    float S[NR];
+    const int d0 = sl * NR, live = e < E ? min(NR, D - d0) : 0;       // rows that exist
+    float* own = st ? st + (size_t)d0 * E : nullptr;
+    if (own && live == NR) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) S[i] = own[i * E];
+    } else {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) S[i] = (own && i < live) ? own[i * E] : 0.f;
+    }
+    if (R > 1) cluster_sync_all();            // every head of the key head has read its history
     else __syncthreads();
     for (int j = 0; j < n; ++j) {
         const T* xr = x + (size_t)(q_beg + j) * p.x_ld;
         const float gate = (sl == 0 && e < E) ? to_float(xr[sp.gate_off + h * E + e]) : 0.f;
+#pragma unroll 1
         for (int c = tid; c < Ch; c += STHREADS) {
-            const int gc = channel(c);
-            const float v = to_float(xr[gc]);
+            const float v = to_float(xr[channel(c)]);
             float acc = 0.f;
+#pragma unroll 1
             for (int i = 0; i < K - 1; ++i) {
-                acc = fmaf(p.taps[(size_t)gc * K + i], hist[i * Ch + c], acc);
+                acc = fmaf(tap[i * Ch + c], hist[i * Ch + c], acc);
                 hist[i * Ch + c] = i + 1 < K - 1 ? hist[(i + 1) * Ch + c] : v;
             }
-            acc = fmaf(p.taps[(size_t)gc * K + K - 1], v, acc);
-            row[c] = acc / (1.0f + expf(-acc));
+            acc = fmaf(tap[(K - 1) * Ch + c], v, acc);
+            row[place(c)] = conv_silu<T>(acc);
         }
-        __syncthreads();
-        if (warp == 0) {
-            float sq = 0.f, sk = 0.f, qk = 0.f;
-            for (int d = lane; d < D; d += 32) {
-                const float qv = row[d], kv = row[D + d];
-                sq = fmaf(qv, qv, sq);
-                sk = fmaf(kv, kv, sk);
-                qk = fmaf(qv, kv, qk);
-            }
-            sq = warp_sum(sq);
-            sk = warp_sum(sk);
-            qk = warp_sum(qk);
-            if (lane == 0) {
-                const float fq = p.q_scale / sqrtf(sq + p.unit_eps), fk = 1.0f / sqrtf(sk + p.unit_eps);
-                scal[0] = fq;
-                scal[1] = fk;
-                scal[2] = fq * fk * qk;
-            }
-        } else if (warp == 1 && lane == 0) {
+        if (warp == 3 && lane == 0) {
             scal[3] = sigmoidf_(to_float(xr[p.beta_off + h]));
-            scal[4] = -expm1f(-expf(p.a_log[h]) * softplusf_(to_float(xr[p.decay_off + h]) + p.dt_bias[h]));
+            scal[4] = -expm1f(rate * softplusf_(to_float(xr[p.decay_off + h]) + dt));
         }
         __syncthreads();
-        const float fq = scal[0], fk = scal[1], dot = scal[2], beta = scal[3], lost = scal[4];
-        float ks[2] = {0.f, 0.f}, qs[2] = {0.f, 0.f};
+        if (warp < 3) {                       // |q|^2, |k|^2, q . k
+            const float* a = warp == 1 ? row + DR : row;
+            const float* b = warp == 0 ? row : row + DR;
+            float sum = 0.f;
+            for (int d = lane; d < D; d += 32) sum = fmaf(a[d], b[d], sum);
+            sum = warp_sum(sum);
+            if (lane == 0) scal[warp] = sum;
+        }
+        const float lost = scal[4];
+        float ks[4] = {0.f, 0.f, 0.f, 0.f}, qs[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int d = sl + i * NS;
-            if (d < D) {
-                S[i] = fmaf(-lost, S[i], S[i]);
-                ks[i & 1] = fmaf(row[D + d], S[i], ks[i & 1]);
-                qs[i & 1] = fmaf(row[d], S[i], qs[i & 1]);
+        for (int i = 0; i < NR; i += 4) {
+            const float4 k4 = *reinterpret_cast<const float4*>(row + DR + d0 + i), q4 = *reinterpret_cast<const float4*>(row + d0 + i);
+            const float kv[4] = {k4.x, k4.y, k4.z, k4.w}, qv[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                S[i + u] = fmaf(-lost, S[i + u], S[i + u]);
+                ks[u] = fmaf(kv[u], S[i + u], ks[u]);
+                qs[u] = fmaf(qv[u], S[i + u], qs[u]);
             }
         }
-        red[tid] = ks[0] + ks[1];
-        red[STHREADS + tid] = qs[0] + qs[1];
+        red[tid] = (ks[0] + ks[1]) + (ks[2] + ks[3]);
+        red[STHREADS + tid] = (qs[0] + qs[1]) + (qs[2] + qs[3]);
         __syncthreads();
+        const float fq = p.q_scale * inverse_root<T>(scal[0] + p.unit_eps), fk = inverse_root<T>(scal[1] + p.unit_eps), dot = fq * fk * scal[2], beta = scal[3];
         float kS = 0.f, qS = 0.f;
         for (int i = 0; i < NS; ++i) {
             kS += red[i * EP + e];
             qS += red[STHREADS + i * EP + e];
         }
-        const float write = e < E ? beta * (row[2 * D + e] - fk * kS) : 0.f;
+        const float write = beta * (row[2 * DR + e] - fk * kS);      // columns beyond E: zero
         const float o = fmaf(dot, write, fq * qS), kw = fk * write;
 #pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int d = sl + i * NS;
-            if (d < D) S[i] = fmaf(row[D + d], kw, S[i]);
+        for (int i = 0; i < NR; i += 4) {
+            const float4 k4 = *reinterpret_cast<const float4*>(row + DR + d0 + i);
+            S[i] = fmaf(k4.x, kw, S[i]);
+            S[i + 1] = fmaf(k4.y, kw, S[i + 1]);
+            S[i + 2] = fmaf(k4.z, kw, S[i + 2]);
+            S[i + 3] = fmaf(k4.w, kw, S[i + 3]);
         }
         if (sl == 0) {                        // whole warps: EP is a multiple of 32
             const float ss = warp_sum(e < E ? o * o : 0.f);
@@ -1000,21 +1072,22 @@ __global__ void __launch_bounds__(STHREADS) head_delta_step_kernel(StepParams sp
             for (int i = 0; i < EP / 32; ++i) ss += scal[8 + i];
             const float rinv = 1.0f / sqrtf(ss / (float)E + sp.norm_eps);
             static_cast<T*>(sp.y)[(size_t)(q_beg + j) * sp.y_ld + (size_t)h * E + e] =
-                from_float<T>(o * rinv * sp.norm_gain[e] * (gate * sigmoidf_(gate)));
+                from_float<T>(o * rinv * gain * (gate * sigmoidf_(gate)));
         }
     }
-    if (st) {
+    if (own && live == NR) {
 #pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int d = sl + i * NS;
-            if (d < D && e < E) st[(size_t)d * E] = S[i];
-        }
+        for (int i = 0; i < NR; ++i) own[i * E] = S[i];
+    } else if (own) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i)
+            if (i < live) own[i * E] = S[i];
     }
     if (cst) {
         const int from = h % R == 0 ? 0 : 2 * D;          // the key head's channels are its first head's to write
-        for (int idx = tid; idx < (K - 1) * (Ch - from); idx += STHREADS) {
-            const int i = idx / (Ch - from), c = from + idx % (Ch - from);
-            cst[(size_t)i * C + channel(c)] = hist[i * Ch + c];
+        for (int c = from + tid; c < Ch; c += STHREADS) {
+            const int gc = channel(c);
+            for (int i = 0; i < K - 1; ++i) cst[(size_t)i * C + gc] = hist[i * Ch + c];
         }
     }
 }
@@ -1067,7 +1140,8 @@ LLMK_EXPORT int llmk_head_delta_step(void* y, long long y_ld, const void* x, lon
     p.gate_off = gate_off; p.norm_gain = norm_gain; p.norm_eps = norm_eps; p.state = state;
     p.EP = 32;
     while (p.EP < E) p.EP *= 2;
-    const size_t smem = ((size_t)K * (2 * D + E) + 2 * STHREADS + 16) * sizeof(float);
+    const int held = rows <= 4 ? 4 : rows <= 8 ? 8 : rows <= 16 ? 16 : rows <= 32 ? 32 : 64;
+    const size_t smem = ((size_t)(2 * K - 1) * (2 * D + E) + 4 + 2 * held * (STHREADS / p.EP) + p.EP + 2 * STHREADS + 16) * sizeof(float);
     cudaError_t e;
     if (dtype == LLMK_F32) e = launch_step<float>(p, smem, rows, (cudaStream_t)stream);
     else if (dtype == LLMK_BF16) e = launch_step<bf16>(p, smem, rows, (cudaStream_t)stream);
