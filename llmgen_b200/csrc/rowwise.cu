@@ -692,6 +692,113 @@ __global__ void __launch_bounds__(512) stream_step_kernel(float* __restrict__ st
     for (int i = threadIdx.x; i < H; i += blockDim.x) normed[r * H + i] = from_float<T>(srow[i] * rinv * next_gain[i]);
 }
 
+template <typename T>
+__device__ __forceinline__ float4 load_sum4(const void* y, size_t at, int splits, long long split_stride) {
+    if (splits == 0) {
+        if constexpr (sizeof(T) == 4) return *reinterpret_cast<const float4*>(static_cast<const float*>(y) + at);
+        else {
+            const uint2 raw = *reinterpret_cast<const uint2*>(static_cast<const T*>(y) + at);
+            const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+            const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+            return make_float4(a.x, a.y, b.x, b.y);
+        }
+    }
+    const float* p = static_cast<const float*>(y) + at;
+    float4 acc = *reinterpret_cast<const float4*>(p);
+    for (int s = 1; s < splits; ++s) {
+        const float4 v = *reinterpret_cast<const float4*>(p + (size_t)s * split_stride);
+        acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
+    }
+    return acc;
+}
+
+// The same with four neighbouring values a thread, which holds them from the streams to the normed row: rows of up to 4,096
+// values, a multiple of four, on 16-byte boundaries; up to 8 streams.
+template <typename T, int MS>
+__global__ void __launch_bounds__(1024) stream_step_vec_kernel(float* __restrict__ streams, const void* __restrict__ y, int splits, long long split_stride,
+                                   const void* __restrict__ y2, int splits2, long long split_stride2, float a, float b,
+                                   const float* __restrict__ mix, const float* __restrict__ out_coef,
+                                   const float* __restrict__ next_in, const float* __restrict__ next_gain, float eps,
+                                   T* __restrict__ normed, int S, int H) {
+    __shared__ float scratch[33];
+    __shared__ float coef[MS * MS + 2 * MS];      // mix [S, S], out [S], in [S]
+    const size_t r = blockIdx.x;
+    for (int i = threadIdx.x; i < S * S + 2 * S; i += blockDim.x) {
+        float c = 0.f;
+        if (i < S * S) c = mix ? mix[i] : 0.f;
+        else if (i < S * S + S) c = out_coef ? out_coef[i - S * S] : 0.f;
+        else c = next_in ? next_in[i - S * S - S] : 0.f;
+        coef[i] = c;
+    }
+    const int i = threadIdx.x * 4;
+    const bool on = i < H;
+    float4 g = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (on && next_in) g = *reinterpret_cast<const float4*>(next_gain + i);
+    pdl_launch_dependents();
+    pdl_wait();
+    __syncthreads();
+    float u[4] = {0.f, 0.f, 0.f, 0.f};
+    if (on) {
+        float* xs = streams + r * S * H + i;
+        float x[MS][4];
+#pragma unroll
+        for (int s = 0; s < MS; ++s) {
+            if (s < S) {
+                const float4 v = *reinterpret_cast<const float4*>(xs + (size_t)s * H);
+                x[s][0] = v.x; x[s][1] = v.y; x[s][2] = v.z; x[s][3] = v.w;
+            }
+        }
+        if (y) {
+            float4 v = load_sum4<T>(y, r * H + i, splits, split_stride);
+            v.x *= a; v.y *= a; v.z *= a; v.w *= a;
+            if (y2) {
+                const float4 w = load_sum4<T>(y2, r * H + i, splits2, split_stride2);
+                v.x += b * w.x; v.y += b * w.y; v.z += b * w.z; v.w += b * w.w;
+            }
+#pragma unroll
+            for (int t = 0; t < MS; ++t) {
+                if (t < S) {
+                    const float o = coef[S * S + t], in = coef[S * S + S + t];
+                    float acc[4] = {o * v.x, o * v.y, o * v.z, o * v.w};
+#pragma unroll
+                    for (int s = 0; s < MS; ++s) {
+                        if (s < S) {
+                            const float m = coef[s * S + t];
+#pragma unroll
+                            for (int c = 0; c < 4; ++c) acc[c] = fmaf(m, x[s][c], acc[c]);
+                        }
+                    }
+                    *reinterpret_cast<float4*>(xs + (size_t)t * H) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) u[c] = fmaf(in, acc[c], u[c]);
+                }
+            }
+        } else {
+#pragma unroll
+            for (int t = 0; t < MS; ++t)
+                if (t < S) {
+                    const float in = coef[S * S + S + t];
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) u[c] = fmaf(in, x[t][c], u[c]);
+                }
+        }
+    }
+    if (!next_in) return;
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < 4; ++c) ss = fmaf(u[c], u[c], ss);
+    ss = block_sum(ss, scratch);
+    if (!on) return;
+    const float rinv = 1.0f / sqrtf(ss / (float)H + eps);
+    T* dst = normed + r * H + i;
+    const float n0 = u[0] * rinv * g.x, n1 = u[1] * rinv * g.y, n2 = u[2] * rinv * g.z, n3 = u[3] * rinv * g.w;
+    if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = make_float4(n0, n1, n2, n3);
+    else {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(n0, n1), hi = __floats2bfloat162_rn(n2, n3);
+        *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+    }
+}
+
 LLMK_EXPORT int llmk_stream_step(float* streams, const void* y, int splits, long long split_stride, const void* y2, int splits2,
                                  long long split_stride2, float a, float b, const float* mix, const float* out_coef,
                                  const float* next_in, const float* next_gain, float eps, void* normed, int n_rows, int S, int H,
@@ -705,6 +812,23 @@ LLMK_EXPORT int llmk_stream_step(float* streams, const void* y, int splits, long
     const int threads = H >= 2048 ? 512 : H >= 512 ? 256 : 128;
     cudaStream_t st = (cudaStream_t)stream;
     cudaError_t e;
+    const size_t vec = dtype == LLMK_F32 ? 16 : 8;
+    if (S <= 8 && H % 4 == 0 && H <= 4096 && (dtype == LLMK_F32 || dtype == LLMK_BF16) && host_aligned16(streams) && host_aligned16(next_gain) &&
+        (reinterpret_cast<uintptr_t>(y) & (splits ? 15 : vec - 1)) == 0 && (reinterpret_cast<uintptr_t>(y2) & (splits2 ? 15 : vec - 1)) == 0 &&
+        split_stride % 4 == 0 && split_stride2 % 4 == 0 && (reinterpret_cast<uintptr_t>(normed) & (vec - 1)) == 0) {
+        const dim3 block(ceil_div(H / 4, 32) * 32);
+#define STREAM_STEP_VEC(TYPE, MS)                                                                                                     \
+    e = llmk_launch(stream_step_vec_kernel<TYPE, MS>, dim3(n_rows), block, 0, st, true, streams, y, splits, split_stride, y2, splits2, \
+                    split_stride2, a, b, mix, out_coef, next_in, next_gain, eps, (TYPE*)normed, S, H)
+        if (dtype == LLMK_F32) {
+            if (S <= 4) STREAM_STEP_VEC(float, 4); else STREAM_STEP_VEC(float, 8);
+        } else {
+            if (S <= 4) STREAM_STEP_VEC(bf16, 4); else STREAM_STEP_VEC(bf16, 8);
+        }
+#undef STREAM_STEP_VEC
+        LLMK_CHECK_LAUNCH_RC("stream_step", e);
+        return LLMK_OK;
+    }
 #define STREAM_STEP_LAUNCH(TYPE, MS)                                                                                                   \
     do {                                                                                                                               \
         if (smem > 48 * 1024) cudaFuncSetAttribute(stream_step_kernel<TYPE, MS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
