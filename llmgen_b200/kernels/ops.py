@@ -941,9 +941,12 @@ def gated_rmsnorm(out: torch.Tensor, o: torch.Tensor, gate: torch.Tensor, weight
     [heads, H].  `out` may then also be given as [n / heads, heads * H] with any row stride."""
     lib = build.load("rowwise")
     n, H = o.shape
-    if tuple(out.shape) not in ((n, H), (n // heads, heads * H)) or (out.shape[0] == n and not out.is_contiguous()):
-        raise KernelError("gated_rmsnorm: out is [n, H] or [n / heads, heads * H]")
-    ldo = heads * H if out.shape[0] == n else _row_stride(out)
+    if tuple(out.shape) == (n // heads, heads * H):
+        ldo = _row_stride(out)
+    elif tuple(out.shape) == (n, H) and out.is_contiguous():
+        ldo = heads * H
+    else:
+        raise KernelError("gated_rmsnorm: out is [n / heads, heads * H], or [n, H] and contiguous")
     if o.dtype != torch.float32 or not o.is_contiguous() or gate.dtype != out.dtype or n % heads != 0:
         raise KernelError("gated_rmsnorm: o must be contiguous float32 and the gate of the storage dtype")
     w_rows = heads if gains_per_head else 1
