@@ -160,7 +160,7 @@ class HeadDecayDelta(Mixer):
     def workspace_bytes(self, tokens: int) -> int:
         elem = 2 if self.dtype == torch.bfloat16 else 4
         he = self.H * self.E
-        chunks = 4 * ops.head_delta_chunk_floats(tokens, 1, self.H, self.G, self.D, self.E)
+        chunks = 4 * ops.head_delta_chunk_floats(tokens, max(1, tokens // 32), self.H, self.G, self.D, self.E)
         return chunks + tokens * ((self.decay_off + self.H) * elem + self.qkv * 4 + (2 * self.H + self.G) * 4 + he * (4 + elem)
                          + self.spec.hidden_size * elem) + ops.SLICED_PRODUCT_BYTES
 
